@@ -508,6 +508,11 @@ int lb_qkv_rotary_store(int dtype, const float* proj, int64_t ld, int q_off, int
                         void* q_out, int64_t ldq, void* cache, const int32_t* slot_mapping, int n_tokens, int n_head, int n_kv_head, int dim, int vdim,
                         int padded, int page_size, int norm_mode, float eps, const int32_t* positions, const float* freq, int rot_dims,
                         const float* v_first_in, float* v_first_out, int64_t ldv, const float* lambda, void* stream);
+/* lb_qkv_rotary_store with the rotation's pairing as an argument: interleaved 1 pairs value 2i with 2i + 1. */
+int lb_qkv_rotary_store_layout(int dtype, const float* proj, int64_t ld, int q_off, int k_off, int v_off, const float* q_weight, const float* k_weight,
+                               void* q_out, int64_t ldq, void* cache, const int32_t* slot_mapping, int n_tokens, int n_head, int n_kv_head, int dim, int vdim,
+                               int padded, int page_size, int norm_mode, float eps, const int32_t* positions, const float* freq, int rot_dims,
+                               const float* v_first_in, float* v_first_out, int64_t ldv, const float* lambda, int interleaved, void* stream);
 /* out[r, c] = o[r, c] / sqrt(mean(o[r, :]^2) + eps) * gain[c] * act(g[r, c]); gain and g may be null; act 0 sigmoid, 1 silu. */
 int lb_row_norm_gate(int out_dtype, const float* o, int64_t ldo, const float* g, int64_t ldg, const float* gain, void* out, int64_t ld_out, int n_rows,
                      int width, int act, float eps, void* stream);
@@ -515,6 +520,106 @@ int lb_row_norm_gate(int out_dtype, const float* o, int64_t ldo, const float* g,
 int lb_activate_columns(float* x, int64_t ld, int n_rows, int cols, int act, void* stream);
 /* ids[r, j] = table[tokens[r], j] and weights[r, j] = 1 / top: a row's experts looked up by its token id (table int32 [vocab, top]). */
 int lb_router_table(const int32_t* tokens, const int32_t* table, int32_t* ids, float* weights, int n_rows, int top, int n_experts, int vocab, void* stream);
+
+/* A sublayer's output as the launch after it reads it: the sum of up to four rows, each times a number, and, with `pairs`, of the routed experts'
+ * results of row t: for k < top, weights[t top + k] * (ids[t top + k] < n_real ? pairs[place ? place[t top + k] : t top + k] : self[t]).
+ * self: rows of the element type the call names, lds elements apart. */
+typedef struct lb_output_terms {
+    int n_rows;
+    const float* y[4];
+    int64_t ldy[4];
+    float scale[4];
+    const float* pairs;
+    int64_t ldp;
+    const int32_t* place;
+    const int32_t* ids;
+    const float* weights;
+    int top, n_real;
+    const void* self;
+    int64_t lds;
+} lb_output_terms;
+/* A router whose choice is corrected and restricted to the best groups (see streams.cu); matrix [n_experts, width] of the call's element type,
+ * ids and weights [rows, top]. */
+typedef struct lb_router {
+    const void* matrix;
+    const float* bias;
+    const float* correction;
+    int n_experts, top, groups, keep, softmax, renormalise;
+    float scale;
+    int32_t* ids;
+    float* weights;
+} lb_router;
+/* The streams x [rows, n_streams * width] between two sublayers (see streams.cu).  mix [n_streams, n_streams] indexed [from, to], to [n_streams],
+ * scale [width] or null: of the sublayer that ends; next_in [n_streams] (null: ones), alpha [1] (null: no norm), gain, offset [width]: of the one
+ * that begins, whose input goes to h (rows ldh elements apart; null: none begins).  fresh: rows that every stream starts as.  rows: the rows of x
+ * to read (nothing is written back). */
+typedef struct lb_streams_args {
+    float* x;
+    int64_t ldx;
+    const float* fresh;
+    int64_t ldf;
+    const int32_t* rows;
+    int n_streams, width;
+    const float* mix;
+    const float* to;
+    const float* scale;
+    const float* next_in;
+    const float* alpha;
+    const float* gain;
+    const float* offset;
+    void* h;
+    int64_t ldh;
+} lb_streams_args;
+int lb_streams_join(int dtype, const lb_streams_args* args, const lb_output_terms* terms, const lb_router* router, int n_rows, void* stream);
+int lb_router_choice(int dtype, const lb_router* router, const void* h, int64_t ldh, int n_rows, int width, void* stream);
+int lb_terms_sum(int dtype, const lb_output_terms* terms, float* x, int64_t ldx, int n_rows, int width, int overwrite, void* stream);
+/* lb_expert_product_kind without a plan, for a few pairs (bfloat16): pair p = (row p / top, choice p % top) goes to expert ids[p]; a pair whose
+ * expert is n_experts or more is left alone.  The first half reads a[p / top] and writes out[p], the second reads a[p].  Supported: see
+ * lb_expert_product_direct_supports. */
+int lb_expert_product_direct_supports(int dtype, const void* a, int64_t lda, const void* w, int64_t expert_stride, int n_pairs, int k);
+int lb_expert_product_direct(int dtype, int gated, const void* a, int64_t lda, const void* w, int64_t expert_stride, const int32_t* ids, const float* weights,
+                             void* out, int64_t ldo, int n_pairs, int n_experts, int n, int k, int top, int act, float alpha, float limit, void* stream);
+
+/* A memory per head with a decay per key channel (see channel_memory.cu).  The projection's float rows hold [q (kv_head dim) | k (kv_head dim) |
+ * v (n_head vdim)] first; a_off: the input of the decays' low-rank map (rank columns), g_off: the gate's pre-activations (n_head vdim columns) or,
+ * with g2, the input of its map (gate_rank columns), b_off: the delta rule's rates before their sigmoid (n_head columns).  a2 [n_head dim, rank] and
+ * g2 [n_head vdim, gate_rank] are of the call's element type, everything else float.  conv [channels, taps] or null; a_log [n_head] or null
+ * (then tau); z_bias [n_head dim] or null; norm [vdim]. */
+typedef struct lb_channel_memory {
+    int n_head, kv_head, dim, vdim;
+    int delta, taps, unit, rank, gate_rank, gate_act;
+    int a_off, g_off, b_off;
+    const float* conv;
+    const void* a2;
+    const void* g2;
+    const float* z_bias;
+    const float* a_log;
+    const float* norm;
+    float tau, q_scale, unit_eps, eps;
+    int64_t slot_stride;
+} lb_channel_memory;
+/* A step's rows: the projection, the layout (tok_seq [T], positions [T], q_start [S + 1], slots [S]), the state, and where the heads go: `heads` of the
+ * call's element type after norm and gate, and, where `o` is given, the float heads before them. */
+typedef struct lb_channel_step {
+    const float* proj;
+    int64_t ld;
+    const int32_t* positions;
+    const int32_t* tok_seq;
+    const int32_t* q_start;
+    const int32_t* slots;
+    float* state;
+    float* o;
+    int64_t ldo;
+    void* heads;
+    int64_t ldh;
+} lb_channel_step;
+/* Row by row; decode_only: every request brings one row (the convolution's inputs then enter the state in the same launch). */
+int lb_channel_memory_rows(int dtype, const lb_channel_memory* memory, const lb_channel_step* step, int n_seq, int decode_only, void* stream);
+/* In pieces of 32 rows.  Scratch: rows [T, channels] (with a convolution or unit vectors), log_decay [T, n_head dim], gate [T, n_head vdim] (with g2) and
+ * lb_channel_memory_pieces_floats(..) floats. */
+int64_t lb_channel_memory_pieces_floats(int n_tokens, int n_seq, int n_head, int dim, int vdim, int delta);
+int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memory, const lb_channel_step* step, float* rows, float* log_decay, float* gate,
+                             float* scratch, int n_tokens, int n_seq, void* stream);
 
 #ifdef __cplusplus
 }

@@ -89,7 +89,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, c
 #pragma unroll
         for (int i = 0; i < 8; ++i) qf[g][i] *= scale * kLog2e;
     }
-    // The heads' pairs (r1, r2) of the penalty by distance; in the scores' base-2 scale a key d positions back loses r1 log2(1 + r2 d).
+    // The heads' pairs (r1, r2) of the penalty by distance; in the scores' base-2 scale a key d positions back loses r1 log2(1 + r2 d) (or r1 d log2 e).
     float r1[G], r2[G];
 #pragma unroll
     for (int g = 0; g < G; ++g) {
@@ -140,7 +140,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, c
 #pragma unroll
                 for (int o = TPK / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
                 if (live) {
-                    if (distance != nullptr) s = fmaf(-r1[g], __log2f(fmaf(r2[g], (float)(pos - j), 1.0f)), s);
+                    if (distance != nullptr) s -= lb_distance_penalty_log2(r1[g], r2[g], pos - j);
                     const float m_new = fmaxf(m[g], s);
                     const float corr = exp2f(m[g] - m_new);
                     const float p = exp2f(s - m_new);

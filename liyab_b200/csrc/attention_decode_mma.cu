@@ -166,7 +166,7 @@ decode_attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, int kv_r
     float m_lo = -CUDART_INF_F, m_hi = -CUDART_INF_F, l_lo = 0.0f, l_hi = 0.0f;
     const float sc = scale * kLog2e;
     // The pairs (r1, r2) of the penalty by distance of this thread's two rows (query heads kvh G + g and + 8); in the scores' base-2
-    // scale a key d positions back loses r1 log2(1 + r2 d).  Weights: read before the wait for the kernel before this one.
+    // scale a key d positions back loses r1 log2(1 + r2 d) (or r1 d log2 e).  Weights: read before the wait for the kernel before this one.
     const bool biased = distance != nullptr;
     const float r1_lo = biased && g < G ? distance[kvh * G + g] : 0.0f, r2_lo = biased && g < G ? distance[n_head + kvh * G + g] : 0.0f;
     const float r1_hi = biased && g + 8 < G ? distance[kvh * G + g + 8] : 0.0f, r2_hi = biased && g + 8 < G ? distance[n_head + kvh * G + g + 8] : 0.0f;
@@ -244,7 +244,7 @@ decode_attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, int kv_r
             for (int e = 0; e < 4; ++e) {
                 const int j = j0 + nt * 8 + 2 * t + (e & 1);
                 float v = s[nt][e] * sc;
-                if (biased) v = fmaf(-(e >= 2 ? r1_hi : r1_lo), __log2f(fmaf(e >= 2 ? r2_hi : r2_lo, (float)max(pos - j, 0), 1.0f)), v);
+                if (biased) v -= lb_distance_penalty_log2(e >= 2 ? r1_hi : r1_lo, e >= 2 ? r2_hi : r2_lo, max(pos - j, 0));
                 s[nt][e] = (j >= begin && j < end) ? v : -CUDART_INF_F;
             }
             mx_lo = fmaxf(mx_lo, fmaxf(s[nt][0], s[nt][1]));

@@ -143,7 +143,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, 
     for (int i = 0; i < OT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     float m_lo = -CUDART_INF_F, m_hi = -CUDART_INF_F, l_lo = 0.0f, l_hi = 0.0f;
     const float sc = scale * kLog2e;
-    // The head's pair (r1, r2) of the penalty by distance; in the scores' base-2 scale a key d positions back loses r1 log2(1 + r2 d).
+    // The head's pair (r1, r2) of the penalty by distance; in the scores' base-2 scale a key d positions back loses r1 log2(1 + r2 d) (or r1 d log2 e).
     const float r1 = distance != nullptr ? distance[head] : 0.0f, r2 = distance != nullptr ? distance[n_head + head] : 0.0f;
 
     for (int tile = 0; tile < n_tiles; ++tile) {
@@ -187,7 +187,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, 
                 float v = s[nt][e] * sc;
                 if (distance != nullptr) {
                     const int d = (e >= 2 ? pos_hi : pos_lo) - (j0 + nt * 8 + 2 * t + (e & 1));
-                    v = fmaf(-r1, __log2f(fmaf(r2, (float)max(d, 0), 1.0f)), v);
+                    v -= lb_distance_penalty_log2(r1, r2, max(d, 0));
                 }
                 if (need_mask) {
                     const int j = j0 + nt * 8 + 2 * t + (e & 1);

@@ -256,9 +256,9 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int first = lb_first_visible(pos, window);
         const float sc = scale * kLog2e;
         // The head's penalty by distance in the units of the raw scores (which are multiplied by sc later): a key d positions
-        // back loses r1 ln(1 + r2 d) / scale = pen log2(1 + r2 d).
-        const float pen = distance != nullptr ? distance[head] * 0.6931471805599453f / scale : 0.0f;
+        // back loses r1 ln(1 + r2 d) / scale = pen log2(1 + r2 d), or, with r2 < 0, r1 d / scale = pen d.
         const float r2 = distance != nullptr ? distance[n_head + head] : 0.0f;
+        const float pen = distance != nullptr ? distance[head] * (r2 < 0.0f ? 1.0f : 0.6931471805599453f) / scale : 0.0f;
         const uint32_t swz = (uint32_t)(r & 7);
         uint8_t* p_row = p_s + (size_t)r * 128;
         float m = -CUDART_INF_F, l = 0.0f;                              // l: this thread's part of the row's sum
@@ -277,7 +277,12 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             if (ok) {
                 tmem_ld32(s_row, v);
                 tmem_ld_wait();
-                if (distance != nullptr) {
+                if (distance != nullptr && r2 < 0.0f) {
+                    // pen (pos - j0 - i) = b0 - pen i.
+                    const float b0 = pen * (float)(pos - j0);
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) - fmaf(-pen, (float)i, b0));
+                } else if (distance != nullptr) {
                     // 1 + r2 (pos - j0 - i) = a0 - r2 i; keys after the query (masked below) are kept from an argument below zero.
                     const float a0 = fmaf(r2, (float)(pos - j0), 1.0f);
 #pragma unroll

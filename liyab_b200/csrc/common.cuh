@@ -111,8 +111,14 @@ __host__ __device__ __forceinline__ int lb_first_visible(int pos, int window) {
     return 0;
 }
 
-// What a score loses by the distance between query and key, for heads that carry the pair (r1, r2): r1 ln(1 + r2 distance).
-__device__ __forceinline__ float lb_distance_penalty(float r1, float r2, int distance) { return r1 * logf(fmaf(r2, (float)distance, 1.0f)); }
+// What a score loses by the distance between query and key, for heads that carry the pair (r1, r2): r1 ln(1 + r2 distance), or, where r2 is
+// negative (which has no logarithm), a straight line: r1 distance.  The second form is in the scale of base-2 exponentials.
+__device__ __forceinline__ float lb_distance_penalty(float r1, float r2, int distance) {
+    return r2 < 0.0f ? r1 * (float)distance : r1 * logf(fmaf(r2, (float)distance, 1.0f));
+}
+__device__ __forceinline__ float lb_distance_penalty_log2(float r1, float r2, int distance) {
+    return r2 < 0.0f ? r1 * (1.4426950408889634f * (float)distance) : r1 * __log2f(fmaf(r2, (float)distance, 1.0f));
+}
 
 // A head's sink joins a finished softmax state: exp(sink) is added to the divisor, with no key and no value.  `m` is the state's running
 // maximum and `sink` the head's number, both in the scale of the kernel's exponentials (base 2: sink * log2(e)); `l` becomes the new divisor

@@ -14,8 +14,8 @@ __device__ __forceinline__ float rr_sigmoid(float z) { return 1.0f / (1.0f + exp
 // A block per token.  From the float row [.. q (H x D) .. k (G x D) .. v (G x E) ..]:
 //   norm_mode 0: queries and keys as they are; 1: every head over its own root mean square, gains [D] shared by the heads;
 //   2: all of q (and all of k) over one root mean square, gains [H x D] and [G x D];
-//   then the first rot_dims values of every query and key head are rotated, value i with value i + rot_dims / 2, by the
-//   angle position * freq[i];
+//   then the first rot_dims values of every query and key head are rotated, value i with value i + rot_dims / 2 (`interleaved`:
+//   value 2i with 2i + 1), by the angle position * freq[i];
 //   values: with v_first_in, v = (1 - lambda) v + lambda v_first_in[t]; with v_first_out, the row's own values are left there.
 // Queries go to q_out [H x P] (P >= D, E; the rest zeros), keys and values into the cache [page][K|V][G][slot][P].
 template <typename T>
@@ -23,7 +23,8 @@ __global__ void qkv_rotary_store_kernel(const float* __restrict__ proj, int64_t 
                                         const float* __restrict__ kw, T* __restrict__ q_out, int64_t ldq, T* __restrict__ cache,
                                         const int32_t* __restrict__ slot_mapping, int H, int G, int D, int E, int P, int page_size, int norm_mode, float eps,
                                         const int32_t* __restrict__ positions, const float* __restrict__ freq, int rot_dims,
-                                        const float* __restrict__ v_first_in, float* __restrict__ v_first_out, int64_t ldv, const float* __restrict__ lambda) {
+                                        const float* __restrict__ v_first_in, float* __restrict__ v_first_out, int64_t ldv, const float* __restrict__ lambda,
+                                        int interleaved) {
     __shared__ float red[2][32];
     extern __shared__ float turn[];            // [rot_dims]: cosine then sine of every pair's angle, made once for all heads of the token
     lb_wait_for_predecessor();
@@ -103,10 +104,11 @@ __global__ void qkv_rotary_store_kernel(const float* __restrict__ proj, int64_t 
             float v = 0.0f;
             if (d < D) {
                 if (d < rot_dims) {
-                    const int i = d < half ? d : d - half;
+                    const bool first = interleaved ? (d & 1) == 0 : d < half;
+                    const int i = interleaved ? d >> 1 : first ? d : d - half;
                     const float cs = turn[i], sn = turn[half + i];
-                    const float lo = normed(i), hi = normed(i + half);
-                    v = d < half ? lo * cs - hi * sn : hi * cs + lo * sn;
+                    const float lo = normed(interleaved ? 2 * i : i), hi = normed(interleaved ? 2 * i + 1 : i + half);
+                    v = first ? lo * cs - hi * sn : hi * cs + lo * sn;
                 } else {
                     v = normed(d);
                 }
@@ -270,6 +272,15 @@ extern "C" int lb_qkv_rotary_store(int dtype, const float* proj, int64_t ld, int
                                    void* q_out, int64_t ldq, void* cache, const int32_t* slot_mapping, int n_tokens, int n_head, int n_kv_head, int dim,
                                    int vdim, int padded, int page_size, int norm_mode, float eps, const int32_t* positions, const float* freq, int rot_dims,
                                    const float* v_first_in, float* v_first_out, int64_t ldv, const float* lambda, void* stream) {
+    return lb_qkv_rotary_store_layout(dtype, proj, ld, q_off, k_off, v_off, q_weight, k_weight, q_out, ldq, cache, slot_mapping, n_tokens, n_head, n_kv_head, dim,
+                                      vdim, padded, page_size, norm_mode, eps, positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda, 0, stream);
+}
+
+extern "C" int lb_qkv_rotary_store_layout(int dtype, const float* proj, int64_t ld, int q_off, int k_off, int v_off, const float* q_weight,
+                                          const float* k_weight, void* q_out, int64_t ldq, void* cache, const int32_t* slot_mapping, int n_tokens, int n_head,
+                                          int n_kv_head, int dim, int vdim, int padded, int page_size, int norm_mode, float eps, const int32_t* positions,
+                                          const float* freq, int rot_dims, const float* v_first_in, float* v_first_out, int64_t ldv, const float* lambda,
+                                          int interleaved, void* stream) {
     LB_CHECK_ARG(n_tokens >= 0 && n_head > 0 && n_kv_head > 0 && dim > 0 && vdim > 0 && padded >= dim && padded >= vdim && page_size > 0,
                  "qkv_rotary_store: bad sizes heads=%d/%d dim=%d vdim=%d padded=%d", n_head, n_kv_head, dim, vdim, padded);
     LB_CHECK_ARG(norm_mode >= 0 && norm_mode <= 2, "qkv_rotary_store: norm mode %d (0 none, 1 a head, 2 the whole projection)", norm_mode);
@@ -284,11 +295,11 @@ extern "C" int lb_qkv_rotary_store(int dtype, const float* proj, int64_t ld, int
     if (dtype == LB_F32)
         LB_CHECK_CUDA(lb_launch_overlapped(qkv_rotary_store_kernel<float>, dim3(n_tokens), dim3(threads), smem, s, proj, ld, q_off, k_off, v_off, q_weight, k_weight,
                                            (float*)q_out, ldq, (float*)cache, slot_mapping, n_head, n_kv_head, dim, vdim, padded, page_size, norm_mode, eps,
-                                           positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda));
+                                           positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda, interleaved));
     else if (dtype == LB_BF16)
         LB_CHECK_CUDA(lb_launch_overlapped(qkv_rotary_store_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), smem, s, proj, ld, q_off, k_off, v_off, q_weight,
                                            k_weight, (__nv_bfloat16*)q_out, ldq, (__nv_bfloat16*)cache, slot_mapping, n_head, n_kv_head, dim, vdim, padded,
-                                           page_size, norm_mode, eps, positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda));
+                                           page_size, norm_mode, eps, positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda, interleaved));
     else return lb_fail(LB_ERR_INVALID_ARGUMENT, "qkv_rotary_store: unknown dtype %d", dtype);
     return LB_OK;
 }

@@ -146,6 +146,7 @@ struct ProductArgs {
     int64_t ldo;
     int E, N, K, top, act;
     float alpha, limit;        // the capped gate's two numbers
+    const int32_t* ids;        // [pairs]: every pair's expert, where no plan was made (the form for a few pairs); else null
 };
 
 constexpr int kBN = 64, kBK = 16;
@@ -433,13 +434,19 @@ __global__ void __launch_bounds__(128) expert_product_rows_kernel(ProductArgs p)
     const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int n0 = (blockIdx.y * 4 + warp) * F;
     if (n0 >= p.N) return;
-    // The expert whose rows hold r: as many experts after the first start at or before r.
-    int e = 0;
-    for (int base = 1; base < p.E; base += 32) {
-        const bool at_or_before = base + lane < p.E && p.offsets[base + lane] <= r;
-        e += __popc(__ballot_sync(0xffffffffu, at_or_before));
+    int e = 0, pair = r;
+    if (p.ids != nullptr) {                     // without a plan: pairs in their own order
+        e = p.ids[r];
+        if (e < 0 || e >= p.E) return;          // not one of the experts with matrices
+    } else {
+        if (r >= p.offsets[p.E]) return;        // pairs without an expert are not in the plan
+        // The expert whose rows hold r: as many experts after the first start at or before r.
+        for (int base = 1; base < p.E; base += 32) {
+            const bool at_or_before = base + lane < p.E && p.offsets[base + lane] <= r;
+            e += __popc(__ballot_sync(0xffffffffu, at_or_before));
+        }
+        pair = p.pair_at[r];
     }
-    const int pair = p.pair_at[r];
     const uint4* a_row = reinterpret_cast<const uint4*>(static_cast<const B16*>(p.a) + (size_t)(GATED ? pair / p.top : r) * p.lda);
     const B16* W = static_cast<const B16*>(p.w) + (size_t)e * p.expert_stride;
     const int k8 = p.K / 8;
@@ -605,7 +612,7 @@ extern "C" int lb_expert_product_kind(int dtype, int gated, const void* a, int64
                                       int act, float alpha, float limit, void* stream) {
     LB_CHECK_ARG(n_pairs >= 0 && n_experts > 0 && n > 0 && k > 0 && top > 0 && act >= 0 && act <= LB_GATE_CAPPED, "expert product: bad sizes");
     if (n_pairs == 0) return LB_OK;
-    ProductArgs p{a, lda, w, expert_stride, offsets, pair_at, weights, out, ldo, n_experts, n, k, top, act, alpha, limit};
+    ProductArgs p{a, lda, w, expert_stride, offsets, pair_at, weights, out, ldo, n_experts, n, k, top, act, alpha, limit, nullptr};
     auto s = static_cast<cudaStream_t>(stream);
     if (dtype == LB_F32) return gated ? launch_product<float, true>(p, n_pairs, s) : launch_product<float, false>(p, n_pairs, s);
     if (dtype == LB_BF16 && mma_takes(p) && !lb_expert_product_plain_only && n_pairs <= kFewPairs)
@@ -614,6 +621,23 @@ extern "C" int lb_expert_product_kind(int dtype, int gated, const void* a, int64
         return gated ? launch_product_mma<true>(p, n_pairs, s) : launch_product_mma<false>(p, n_pairs, s);
     if (dtype == LB_BF16) return gated ? launch_product<__nv_bfloat16, true>(p, n_pairs, s) : launch_product<__nv_bfloat16, false>(p, n_pairs, s);
     return lb_fail(LB_ERR_INVALID_ARGUMENT, "expert product: unknown dtype %d", dtype);
+}
+
+extern "C" int lb_expert_product_direct_supports(int dtype, const void* a, int64_t lda, const void* w, int64_t expert_stride, int n_pairs, int k) {
+    ProductArgs p{};
+    p.a = a; p.lda = lda; p.w = w; p.expert_stride = expert_stride; p.K = k;
+    return dtype == LB_BF16 && n_pairs <= kFewPairs && mma_takes(p) && !lb_expert_product_plain_only ? 1 : 0;
+}
+
+extern "C" int lb_expert_product_direct(int dtype, int gated, const void* a, int64_t lda, const void* w, int64_t expert_stride, const int32_t* ids,
+                                        const float* weights, void* out, int64_t ldo, int n_pairs, int n_experts, int n, int k, int top, int act, float alpha,
+                                        float limit, void* stream) {
+    LB_CHECK_ARG(n_pairs >= 0 && n_experts > 0 && n > 0 && k > 0 && top > 0 && act >= 0 && act <= LB_GATE_CAPPED && ids != nullptr, "expert product: bad sizes");
+    LB_CHECK_ARG(lb_expert_product_direct_supports(dtype, a, lda, w, expert_stride, n_pairs, k), "expert product without a plan: %d pairs, K = %d are not taken", n_pairs, k);
+    if (n_pairs == 0) return LB_OK;
+    ProductArgs p{a, lda, w, expert_stride, nullptr, nullptr, weights, out, ldo, n_experts, n, k, top, act, alpha, limit, ids};
+    auto s = static_cast<cudaStream_t>(stream);
+    return gated ? launch_product_rows<true>(p, n_pairs, s) : launch_product_rows<false>(p, n_pairs, s);
 }
 
 extern "C" int lb_expert_combine(float* x, int64_t ldx, const float* y, int64_t ldy, const int32_t* place, int n_rows, int width, int top, void* stream) {

@@ -1,0 +1,428 @@
+// Blocks around several residual streams, and routers with corrected choices.
+//
+//   lb_streams_join     one launch between two sublayers.  The stream is a row of S parts of W values.  With y the sublayer's output (the sum of up
+//                       to four terms, each a row times a number, or a row gathered from routed experts' results),
+//                           X'[t] = sum_s M[s, t] X[s] + c[t] (scale * y)            (all t from the old X),
+//                       then the next sublayer's input from the new parts, h = tanh(alpha sum_s a[s] X'[s]) gain + bias, and, where the next
+//                       sublayer routes its rows to experts, the router on h.  Every step is optional: with `fresh` all parts start equal to
+//                       a row of it; without a sublayer's output the parts stay as they are; with `rows` rows are gathered and nothing is written back.
+//   lb_router_choice    the router by itself: z = R h (+ bias) in 32-bit, scores s = softmax(z) or sigmoid(z); the experts are chosen by
+//                       s + correction among the `keep` best of `groups` equal groups of neighbours (a group counts as its best expert);
+//                       weights = s of the chosen, times a factor, optionally over their sum.  Ties go to the lower index.
+//   lb_terms_sum        x (+)= the sum of such terms, for arrangements with one stream.
+//
+// An expert's number of n_real or more stands for the identity: its result is the row `self` (the sublayer's input).
+#include "api.h"
+#include "common.cuh"
+
+#include <math_constants.h>
+
+namespace {
+
+constexpr int kMaxStreams = 16;
+
+template <typename T>
+__device__ __forceinline__ float4 load4(const T* p);
+template <>
+__device__ __forceinline__ float4 load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <>
+__device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// V values at a time: V = 4 (16-byte pieces) or 1.
+template <int V>
+struct Vals {
+    float v[V];
+};
+template <int V, typename T>
+__device__ __forceinline__ Vals<V> load_vals(const T* p) {
+    Vals<V> r;
+    if constexpr (V == 4) {
+        const float4 f = load4<T>(p);
+        r.v[0] = f.x; r.v[1] = f.y; r.v[2] = f.z; r.v[3] = f.w;
+    } else {
+        r.v[0] = lb_to_float(*p);
+    }
+    return r;
+}
+template <int V>
+__device__ __forceinline__ void store_vals(float* p, const Vals<V>& r) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+    else *p = r.v[0];
+}
+template <int V>
+__device__ __forceinline__ void store_vals(__nv_bfloat16* p, const Vals<V>& r) {
+    if constexpr (V == 4) {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(r.v[0], r.v[1]), hi = __floats2bfloat162_rn(r.v[2], r.v[3]);
+        uint2 u;
+        u.x = *reinterpret_cast<const uint32_t*>(&lo);
+        u.y = *reinterpret_cast<const uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(p) = u;
+    } else {
+        *p = __float2bfloat16_rn(r.v[0]);
+    }
+}
+
+// Columns c .. c + V - 1 of row t of the terms' sum.
+template <int V, typename T>
+__device__ __forceinline__ Vals<V> terms_at(const lb_output_terms& o, int t, int c) {
+    Vals<V> sum;
+#pragma unroll
+    for (int i = 0; i < V; ++i) sum.v[i] = 0.0f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        if (k >= o.n_rows) break;
+        const Vals<V> y = load_vals<V>(o.y[k] + (size_t)t * o.ldy[k] + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) sum.v[i] = fmaf(o.scale[k], y.v[i], sum.v[i]);
+    }
+    if (o.pairs != nullptr) {
+        for (int k = 0; k < o.top; ++k) {
+            const int p = t * o.top + k, e = o.ids[p];
+            const float w = o.weights != nullptr ? o.weights[p] : 1.0f;
+            const Vals<V> y = e < o.n_real ? load_vals<V>(o.pairs + (size_t)(o.place != nullptr ? o.place[p] : p) * o.ldp + c)
+                                           : load_vals<V>(static_cast<const T*>(o.self) + (size_t)t * o.lds + c);
+#pragma unroll
+            for (int i = 0; i < V; ++i) sum.v[i] = fmaf(w, y.v[i], sum.v[i]);
+        }
+    }
+    return sum;
+}
+
+template <int V, typename T>
+__global__ void __launch_bounds__(256) terms_sum_kernel(lb_output_terms o, float* __restrict__ x, int64_t ldx, int n_rows, int width, int overwrite) {
+    lb_wait_for_predecessor();
+    lb_dependents_may_launch();
+    const long per_row = width / V, total = (long)n_rows * per_row;
+    for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long)gridDim.x * blockDim.x) {
+        const int t = (int)(i / per_row), c = V * (int)(i - (long)t * per_row);
+        Vals<V> s = terms_at<V, T>(o, t, c);
+        float* dst = x + (size_t)t * ldx + c;
+        if (!overwrite) {
+            const Vals<V> old = load_vals<V>(dst);
+#pragma unroll
+            for (int k = 0; k < V; ++k) s.v[k] += old.v[k];
+        }
+        store_vals<V>(dst, s);
+    }
+}
+
+// ---------------------------------------------------------------- router
+// Row t's experts from its input h (in shared memory) by the whole block: a warp per expert for the sums, then warp 0 chooses.
+// smem: z [n], c [n], best [groups], taken [groups] (int).
+template <typename T>
+__device__ __forceinline__ void route_row(const lb_router& r, const float* h, int width, int t, float* smem) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5, n = r.n_experts;
+    float* z = smem;
+    float* c = z + n;
+    float* best = c + n;
+    int* taken = reinterpret_cast<int*>(best + r.groups);
+    const T* R = static_cast<const T*>(r.matrix);
+    for (int e = warp; e < n; e += n_warps) {
+        const T* w = R + (size_t)e * width;
+        float acc = 0.0f;
+        if (width % 4 == 0 && (reinterpret_cast<uintptr_t>(R) & 15) == 0) {        // four values a lane and load, four loads in flight
+            for (int k0 = 4 * lane; k0 < width; k0 += 4 * 128) {
+                float4 a[4], b[4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    const int k = k0 + 128 * u;
+                    const bool in = k < width;
+                    b[u] = in ? load4<T>(w + k) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                    a[u] = in ? load4<float>(h + k) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                }
+#pragma unroll
+                for (int u = 0; u < 4; ++u) acc = fmaf(a[u].x, b[u].x, fmaf(a[u].y, b[u].y, fmaf(a[u].z, b[u].z, fmaf(a[u].w, b[u].w, acc))));
+            }
+        } else {
+            for (int k = lane; k < width; k += 32) acc = fmaf(h[k], lb_to_float(w[k]), acc);
+        }
+        acc = lb_warp_sum(acc);
+        if (lane == 0) z[e] = r.bias != nullptr ? acc + r.bias[e] : acc;
+    }
+    __syncthreads();
+    if (warp != 0) return;
+    float top_z = -CUDART_INF_F, sum = 0.0f;
+    if (r.softmax) {
+        for (int e = lane; e < n; e += 32) top_z = fmaxf(top_z, z[e]);
+        top_z = lb_warp_max(top_z);
+        for (int e = lane; e < n; e += 32) sum += expf(z[e] - top_z);
+        sum = lb_warp_sum(sum);
+    }
+    for (int e = lane; e < n; e += 32) {
+        const float s = r.softmax ? expf(z[e] - top_z) / sum : 1.0f / (1.0f + expf(-z[e]));
+        z[e] = s;
+        c[e] = r.correction != nullptr ? s + r.correction[e] : s;
+    }
+    __syncwarp();
+    // The largest of v[0 .. count), the lowest index among equals; every lane gets the index.
+    auto argmax = [&](const float* v, int count) {
+        float m = -CUDART_INF_F;
+        int at = 0x7fffffff;
+        for (int i = lane; i < count; i += 32)
+            if (at == 0x7fffffff || v[i] > m) { m = v[i]; at = i; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float m2 = __shfl_xor_sync(0xffffffffu, m, o);
+            const int at2 = __shfl_xor_sync(0xffffffffu, at, o);
+            if (at == 0x7fffffff || (at2 != 0x7fffffff && (m2 > m || (m2 == m && at2 < at)))) { m = m2; at = at2; }
+        }
+        return min(at, count - 1);
+    };
+    if (r.groups > 1 && r.keep < r.groups) {
+        const int size = n / r.groups;
+        for (int g = lane; g < r.groups; g += 32) {
+            float m = -CUDART_INF_F;
+            for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, c[e]);
+            best[g] = m;
+            taken[g] = 0;
+        }
+        __syncwarp();
+        for (int k = 0; k < r.keep; ++k) {
+            const int g = argmax(best, r.groups);
+            __syncwarp();
+            if (lane == 0) { taken[g] = 1; best[g] = -CUDART_INF_F; }
+            __syncwarp();
+        }
+        for (int e = lane; e < n; e += 32)
+            if (!taken[e / size]) c[e] = -CUDART_INF_F;
+        __syncwarp();
+    }
+    float total = 0.0f;
+    for (int k = 0; k < r.top; ++k) {
+        const int e = argmax(c, n);
+        const float s = z[e];
+        total += s;
+        __syncwarp();
+        if (lane == 0) c[e] = -CUDART_INF_F;
+        __syncwarp();
+        if (lane == 0) {
+            r.ids[(size_t)t * r.top + k] = e;
+            r.weights[(size_t)t * r.top + k] = r.renormalise != 0 ? s : s * r.scale;
+        }
+    }
+    if (r.renormalise != 0 && lane == 0)
+        for (int k = 0; k < r.top; ++k) r.weights[(size_t)t * r.top + k] *= r.scale / total;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(512) router_choice_kernel(lb_router r, const T* __restrict__ h, int64_t ldh, int width) {
+    extern __shared__ __align__(16) float smem[];
+    lb_wait_for_predecessor();
+    lb_dependents_may_launch();
+    const int t = blockIdx.x;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) smem[c] = lb_to_float(h[(size_t)t * ldh + c]);
+    __syncthreads();
+    route_row<T>(r, smem, width, t, smem + (width + 3) / 4 * 4);
+}
+
+// ---------------------------------------------------------------- the streams between two sublayers
+// A block per row.  MAXS: as many streams as a thread keeps (EXACT: S is MAXS).
+template <int V, int MAXS, bool EXACT, typename T>
+__global__ void __launch_bounds__(512) streams_join_kernel(lb_streams_args a, lb_output_terms o, lb_router r) {
+    extern __shared__ __align__(16) float smem[];       // with a router: the row h, then the router's scratch
+    __shared__ float hc[kMaxStreams * kMaxStreams + 2 * kMaxStreams];
+    const int S = EXACT ? MAXS : a.n_streams, W = a.width;
+    float* mix = hc;
+    float* to = hc + S * S;
+    float* next = to + S;
+    // Weights: read before the wait for the kernel before this one.
+    const bool moves = o.n_rows > 0 || o.pairs != nullptr, goes_on = a.h != nullptr;
+    if (moves)
+        for (int i = threadIdx.x; i < S * S + S; i += blockDim.x) hc[i] = i < S * S ? a.mix[i] : a.to[i - S * S];
+    if (goes_on)
+        for (int i = threadIdx.x; i < S; i += blockDim.x) next[i] = a.next_in != nullptr ? a.next_in[i] : 1.0f;
+    const float alpha = a.alpha != nullptr ? a.alpha[0] : 1.0f;
+    lb_wait_for_predecessor();
+    lb_dependents_may_launch();
+    __syncthreads();
+    const int t = blockIdx.x;
+    float* xrow = a.x + (size_t)(a.rows != nullptr ? a.rows[t] : t) * a.ldx;
+    for (int c = V * threadIdx.x; c < W; c += V * blockDim.x) {
+        Vals<V> x[MAXS];
+        if (a.fresh != nullptr) {
+            x[0] = load_vals<V>(a.fresh + (size_t)t * a.ldf + c);
+#pragma unroll
+            for (int s = 1; s < MAXS; ++s) x[s] = x[0];
+        } else {
+#pragma unroll
+            for (int s = 0; s < MAXS; ++s)
+                if (EXACT || s < S) x[s] = load_vals<V>(xrow + (size_t)s * W + c);
+        }
+        Vals<V> u;
+#pragma unroll
+        for (int i = 0; i < V; ++i) u.v[i] = 0.0f;
+        if (moves) {
+            Vals<V> y = terms_at<V, T>(o, t, c);
+            if (a.scale != nullptr) {
+                const Vals<V> g = load_vals<V>(a.scale + c);
+#pragma unroll
+                for (int i = 0; i < V; ++i) y.v[i] *= g.v[i];
+            }
+#pragma unroll(EXACT ? MAXS : 1)
+            for (int q = 0; q < S; ++q) {
+                Vals<V> z;
+#pragma unroll
+                for (int i = 0; i < V; ++i) z.v[i] = to[q] * y.v[i];
+#pragma unroll
+                for (int s = 0; s < MAXS; ++s) {
+                    if (!EXACT && s >= S) break;
+                    const float m = mix[s * S + q];
+#pragma unroll
+                    for (int i = 0; i < V; ++i) z.v[i] = fmaf(m, x[s].v[i], z.v[i]);
+                }
+                store_vals<V>(xrow + (size_t)q * W + c, z);
+                if (goes_on) {
+                    const float n = next[q];
+#pragma unroll
+                    for (int i = 0; i < V; ++i) u.v[i] = fmaf(n, z.v[i], u.v[i]);
+                }
+            }
+        } else {
+#pragma unroll
+            for (int q = 0; q < MAXS; ++q) {
+                if (!EXACT && q >= S) break;
+                if (a.fresh != nullptr) store_vals<V>(xrow + (size_t)q * W + c, x[q]);
+                if (goes_on) {
+                    const float n = next[q];
+#pragma unroll
+                    for (int i = 0; i < V; ++i) u.v[i] = fmaf(n, x[q].v[i], u.v[i]);
+                }
+            }
+        }
+        if (!goes_on) continue;
+        if (a.alpha != nullptr) {
+            const Vals<V> g = load_vals<V>(a.gain + c), b = load_vals<V>(a.offset + c);
+#pragma unroll
+            for (int i = 0; i < V; ++i) u.v[i] = fmaf(tanhf(alpha * u.v[i]), g.v[i], b.v[i]);
+        }
+        store_vals<V>(static_cast<T*>(a.h) + (size_t)t * a.ldh + c, u);
+        if (r.matrix != nullptr) {
+#pragma unroll
+            for (int i = 0; i < V; ++i) smem[c + i] = lb_to_float(lb_from_float<T>(u.v[i]));        // the router reads what the experts read
+        }
+    }
+    if (r.matrix == nullptr) return;
+    __syncthreads();
+    route_row<T>(r, smem, W, t, smem + (W + 3) / 4 * 4);
+}
+
+size_t router_floats(const lb_router& r) { return 2 * (size_t)r.n_experts + 2 * (size_t)r.groups; }
+
+int check_router(const lb_router& r) {
+    LB_CHECK_ARG(r.n_experts > 0 && r.n_experts <= 4096 && r.top > 0 && r.ids != nullptr && r.weights != nullptr && r.groups >= 1 && r.keep >= 1 &&
+                     r.keep <= r.groups && r.n_experts % r.groups == 0 && r.top <= r.n_experts / r.groups * r.keep,
+                 "router: top %d of %d experts, %d of %d groups", r.top, r.n_experts, r.keep, r.groups);
+    return LB_OK;
+}
+
+bool on16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+bool terms_on16(const lb_output_terms& o) {
+    for (int k = 0; k < o.n_rows; ++k)
+        if (o.ldy[k] % 4 != 0 || !on16(o.y[k])) return false;
+    return o.pairs == nullptr || (o.ldp % 4 == 0 && on16(o.pairs) && (o.self == nullptr || (o.lds % 4 == 0 && on16(o.self))));
+}
+int check_terms(const lb_output_terms& o) {
+    LB_CHECK_ARG(o.n_rows >= 0 && o.n_rows <= 4, "output terms: %d rows", o.n_rows);
+    LB_CHECK_ARG(o.pairs == nullptr || (o.top > 0 && o.ids != nullptr), "output terms: gathered results need their experts");
+    return LB_OK;
+}
+
+template <int V, typename T>
+int launch_join(const lb_streams_args& a, const lb_output_terms& o, const lb_router& r, int n_rows, cudaStream_t s) {
+    const int pieces = a.width / V;
+    int threads = min(512, max(32, (pieces + 31) / 32 * 32));
+    if (r.matrix != nullptr) threads = max(threads, 32 * min(8, r.n_experts));
+    const size_t smem = r.matrix != nullptr ? ((size_t)(a.width + 3) / 4 * 4 + router_floats(r)) * sizeof(float) : 0;
+    LB_CHECK_ARG(smem <= 200 * 1024, "streams: rows of %d values with a router do not fit shared memory", a.width);
+#define LB_JOIN(MAXS, EXACT)                                                                                                                    \
+    do {                                                                                                                                        \
+        auto kernel = streams_join_kernel<V, MAXS, EXACT, T>;                                                                                   \
+        if (smem > 40 * 1024) LB_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));             \
+        LB_CHECK_CUDA(lb_launch_overlapped(kernel, dim3(n_rows), dim3(threads), smem, s, a, o, r));                                            \
+        return LB_OK;                                                                                                                           \
+    } while (0)
+    if constexpr (V == 1) {
+        if (a.n_streams <= 4) LB_JOIN(4, false);
+        LB_JOIN(kMaxStreams, false);
+    } else {
+        switch (a.n_streams) {
+            case 1: LB_JOIN(1, true);
+            case 2: LB_JOIN(2, true);
+            case 3: LB_JOIN(3, true);
+            case 4: LB_JOIN(4, true);
+            default:
+                if (a.n_streams <= 8) LB_JOIN(8, false);
+                LB_JOIN(kMaxStreams, false);
+        }
+    }
+#undef LB_JOIN
+}
+
+}  // namespace
+
+extern "C" int lb_streams_join(int dtype, const lb_streams_args* args, const lb_output_terms* terms, const lb_router* router, int n_rows, void* stream) {
+    LB_CHECK_ARG(args != nullptr && args->n_streams >= 1 && args->n_streams <= kMaxStreams && args->width > 0 && n_rows >= 0 && args->x != nullptr,
+                 "streams: %d streams (1 to %d)", args == nullptr ? 0 : args->n_streams, kMaxStreams);
+    LB_CHECK_ARG(dtype == LB_F32 || dtype == LB_BF16, "streams: unknown dtype %d", dtype);
+    const lb_streams_args a = *args;
+    lb_output_terms o{};
+    lb_router r{};
+    if (terms != nullptr) o = *terms;
+    if (router != nullptr) r = *router;
+    r.groups = r.matrix != nullptr ? r.groups : 1;
+    if (int rc = check_terms(o)) return rc;
+    const bool moves = o.n_rows > 0 || o.pairs != nullptr;
+    LB_CHECK_ARG(!moves || (a.mix != nullptr && a.to != nullptr && a.rows == nullptr && a.fresh == nullptr), "streams: a sublayer's output needs its mixing weights and every row in place");
+    LB_CHECK_ARG(a.alpha == nullptr || (a.gain != nullptr && a.offset != nullptr), "streams: the norm needs gain and offset");
+    LB_CHECK_ARG(r.matrix == nullptr || a.h != nullptr, "streams: a router reads the next sublayer's input");
+    if (r.matrix != nullptr)
+        if (int rc = check_router(r)) return rc;
+    if (n_rows == 0) return LB_OK;
+    auto s = static_cast<cudaStream_t>(stream);
+    const bool vec = a.width % 4 == 0 && a.ldx % 4 == 0 && on16(a.x) && (a.fresh == nullptr || (a.ldf % 4 == 0 && on16(a.fresh))) && on16(a.scale) && on16(a.gain) &&
+                     on16(a.offset) && (a.h == nullptr || (a.ldh % 4 == 0 && on16(a.h))) && terms_on16(o);
+    if (dtype == LB_F32) return vec ? launch_join<4, float>(a, o, r, n_rows, s) : launch_join<1, float>(a, o, r, n_rows, s);
+    return vec ? launch_join<4, __nv_bfloat16>(a, o, r, n_rows, s) : launch_join<1, __nv_bfloat16>(a, o, r, n_rows, s);
+}
+
+extern "C" int lb_router_choice(int dtype, const lb_router* router, const void* h, int64_t ldh, int n_rows, int width, void* stream) {
+    LB_CHECK_ARG(router != nullptr && router->matrix != nullptr && n_rows >= 0 && width > 0, "router: bad sizes");
+    if (int rc = check_router(*router)) return rc;
+    if (n_rows == 0) return LB_OK;
+    auto s = static_cast<cudaStream_t>(stream);
+    const int threads = 32 * max(1, min(16, router->n_experts));
+    const size_t smem = ((size_t)(width + 3) / 4 * 4 + router_floats(*router)) * sizeof(float);
+    LB_CHECK_ARG(smem <= 200 * 1024, "router: rows of %d values do not fit shared memory", width);
+    auto launch = [&](auto kernel, auto* rows) -> int {
+        if (smem > 48 * 1024) LB_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        LB_CHECK_CUDA(lb_launch_overlapped(kernel, dim3(n_rows), dim3(threads), smem, s, *router, rows, ldh, width));
+        return LB_OK;
+    };
+    if (dtype == LB_F32) return launch(router_choice_kernel<float>, static_cast<const float*>(h));
+    if (dtype == LB_BF16) return launch(router_choice_kernel<__nv_bfloat16>, static_cast<const __nv_bfloat16*>(h));
+    return lb_fail(LB_ERR_INVALID_ARGUMENT, "router: unknown dtype %d", dtype);
+}
+
+extern "C" int lb_terms_sum(int dtype, const lb_output_terms* terms, float* x, int64_t ldx, int n_rows, int width, int overwrite, void* stream) {
+    LB_CHECK_ARG(terms != nullptr && n_rows >= 0 && width > 0, "sum of output terms: bad sizes");
+    LB_CHECK_ARG(dtype == LB_F32 || dtype == LB_BF16, "sum of output terms: unknown dtype %d", dtype);
+    if (int rc = check_terms(*terms)) return rc;
+    if (n_rows == 0) return LB_OK;
+    const lb_output_terms o = *terms;
+    auto s = static_cast<cudaStream_t>(stream);
+    const bool vec = width % 4 == 0 && ldx % 4 == 0 && on16(x) && terms_on16(o);
+    const long total = (long)n_rows * (width / (vec ? 4 : 1));
+    const dim3 grid((unsigned)min((total + 255) / 256, (long)148 * 16));
+    if (dtype == LB_F32) {
+        if (vec) LB_CHECK_CUDA(lb_launch_overlapped(terms_sum_kernel<4, float>, grid, dim3(256), 0, s, o, x, ldx, n_rows, width, overwrite));
+        else LB_CHECK_CUDA(lb_launch_overlapped(terms_sum_kernel<1, float>, grid, dim3(256), 0, s, o, x, ldx, n_rows, width, overwrite));
+    } else {
+        if (vec) LB_CHECK_CUDA(lb_launch_overlapped(terms_sum_kernel<4, __nv_bfloat16>, grid, dim3(256), 0, s, o, x, ldx, n_rows, width, overwrite));
+        else LB_CHECK_CUDA(lb_launch_overlapped(terms_sum_kernel<1, __nv_bfloat16>, grid, dim3(256), 0, s, o, x, ldx, n_rows, width, overwrite));
+    }
+    return LB_OK;
+}

@@ -9,6 +9,7 @@
 
 #include "decoder.h"
 #include "parts.h"
+#include "safetensors.h"
 
 namespace liyab {
 namespace {
@@ -58,6 +59,7 @@ void register_puzutar();   // puzutar.cpp
 void register_vosurax();   // vosurax.cpp
 void register_viresun();   // viresun.cpp
 void register_revudra();   // revudra.cpp
+void register_mokisun();   // mokisun.cpp
 
 void register_architecture(Architecture arch) { table()[arch.name] = std::move(arch); }
 
@@ -69,6 +71,7 @@ void register_builtin_architectures() {
         register_vosurax();
         register_viresun();
         register_revudra();
+        register_mokisun();
         register_architecture({"liyab_spec", {}, [](const Json& raw) { return std::make_unique<SpecConfig>(raw); }});
     });
     // Plug-ins named by the environment (paths separated by ':') are loaded once, so that the programs can run
@@ -143,7 +146,17 @@ std::unique_ptr<ArchitectureConfig> read_config(const std::string& model_dir) {
         throw invalid_model("{}", e.message());
     }
     if (!raw.is_object()) throw invalid_model("{} does not hold a JSON object", path);
-    return parse_config(raw);
+    std::unique_ptr<ArchitectureConfig> config = parse_config(raw);
+    // A folder without weights (or with broken ones, which loading will report) keeps the sizes of config.json.
+    try {
+        const ModelFiles files(model_dir);
+        config->read_shapes([&](const std::string& name) -> const std::vector<int64_t>* {
+            const TensorEntry* e = files.find(name);
+            return e != nullptr ? &e->shape : nullptr;
+        });
+    } catch (const Error&) {
+    }
+    return config;
 }
 
 }  // namespace liyab

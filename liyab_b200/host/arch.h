@@ -28,6 +28,10 @@ public:
     virtual CheckpointMap checkpoint_map() const = 0;
     // Regular expressions of tensors a file may hold that carry no weights.
     virtual std::vector<std::string> ignored_tensors() const { return {}; }
+    // Sizes that only the model file's tensors tell: `shape_of` gives a tensor's shape in the file (null: no such tensor).  Called before the
+    // specification is asked for, where the model folder holds weights.
+    using ShapeOf = std::function<const std::vector<int64_t>*(const std::string& name)>;
+    virtual void read_shapes(const ShapeOf& shape_of) {}
     // Prefixes a file may put before every tensor name.
     virtual std::vector<std::string> name_prefixes() const { return {""}; }
 };

@@ -2,6 +2,7 @@
 #include "parallel_parts.h"
 #include "gated_parts.h"
 #include "state_parts.h"
+#include "stream_parts.h"
 
 #include <mutex>
 
@@ -59,6 +60,18 @@ void register_builtin_parts() {
         mixers().add("state_space", {StateSpaceMixer::parameters, [](const PartSpec& s, const Params& p, const Runtime&) {
                                          return std::make_shared<StateSpaceMixer>(s, p);
                                      }});
+        norms().add("dynamic_tanh", {TanhNorm::parameters, [](const PartSpec& s, const Params& p, const Runtime&) {
+                                         return std::make_shared<TanhNorm>(s, p);
+                                     }});
+        joins().add("hyper", {HyperJoin::parameters, [](const PartSpec& s, const Params& p, const Runtime&) {
+                                  return std::make_shared<HyperJoin>(s, p);
+                              }});
+        mixers().add("channel_memory", {ChannelMemory::parameters, [](const PartSpec& s, const Params& p, const Runtime&) {
+                                            return std::make_shared<ChannelMemory>(s, p);
+                                        }});
+        arrangements().add("streams", {[](const LayerSpec& l, const LayerParts& parts, const Runtime&) {
+                               return std::make_shared<StreamsBlock>(l, parts);
+                           }});
         arrangements().add("parallel", {[](const LayerSpec& l, const LayerParts& parts, const Runtime&) {
                                return std::make_shared<ParallelBlock>(l, parts);
                            }});

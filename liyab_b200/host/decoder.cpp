@@ -18,6 +18,7 @@ std::vector<ParamDecl> slot_parameters(const SlotSpec& s) {
         case Role::FeedForward: return feed_forwards().get(s.part.kind).parameters(s.part);
         case Role::Shift: return shifts().get(s.part.kind).parameters(s.part);
         case Role::TokenInput: return token_inputs().get(s.part.kind).parameters(s.part);
+        case Role::Join: return joins().get(s.part.kind).parameters(s.part);
     }
     return {};
 }
@@ -29,6 +30,7 @@ std::shared_ptr<Part> build_slot(const SlotSpec& s, const Params& p, const Runti
         case Role::FeedForward: return feed_forwards().get(s.part.kind).build(s.part, p, rt);
         case Role::Shift: return shifts().get(s.part.kind).build(s.part, p, rt);
         case Role::TokenInput: return token_inputs().get(s.part.kind).build(s.part, p, rt);
+        case Role::Join: return joins().get(s.part.kind).build(s.part, p, rt);
     }
     return nullptr;
 }
@@ -69,8 +71,12 @@ DecoderModel::DecoderModel(ModelSpec spec_, const Params& params, Runtime runtim
         const Params lp = params_.sub(std::format("layers.{}.", i));
         for (const auto& slot : spec.layers[i].slots) layer.parts.by_name[slot.name] = build_slot(slot, lp.sub(slot.name + "."), runtime);
         layer.block = arrangements().get(spec.layers[i].arrangement).build(spec.layers[i], layer.parts, runtime);
+        if (layer.block->streams() != spec.streams)
+            throw invalid_model("layer {} is arranged for {} residual streams, the model has {}", i, layer.block->streams(), spec.streams);
         layers.push_back(std::move(layer));
     }
+    for (const auto& e : spec.run_order)
+        if (e.offset_row >= 0 && spec.streams > 1) throw unsupported("pass offsets go with one residual stream");
     final_norm = norms().get(spec.final_norm.kind).build(spec.final_norm, params_.sub("final_norm."), runtime);
     head_weight = spec.head.tied ? embedding : params_.at("head.weight");
     if (spec.head.bias) head_bias = static_cast<const float*>(params_.at("head.bias").data);
@@ -158,6 +164,8 @@ Rows DecoderModel::forward(StepContext& ctx) {
     ctx.stream_rounded_entry = -1;
     position->embed(ctx, embedding, static_cast<float>(spec.embedding.scale), x);
     ctx.tap("embed", x);
+    ctx.next_input_entry = -1;
+    if (spec.streams > 1) return forward_streams(ctx, x);
     for (size_t i = 0; i < spec.run_order.size(); ++i) {
         const RunEntry& e = spec.run_order[i];
         if (e.offset_row >= 0) {
@@ -168,12 +176,57 @@ Rows DecoderModel::forward(StepContext& ctx) {
         layers[static_cast<size_t>(e.layer)].block->forward(ctx, x, CacheUnit{e.cache, e.cache == static_cast<int>(i), static_cast<int>(i)});
     }
     const int R = ctx.n_logit_rows;
-    if (R == 0) return Rows{nullptr, DType::F32, 0, spec.vocab_size(), spec.vocab_size()};
+    if (R == 0) return no_logits();
     // The head's buffers are sized by the rows whose logits are wanted, not by the step's tokens.
     ctx.phase(Phase::Head);
     const Rows y = ws.get("head.normed", R, width, runtime.dtype, false);
     final_norm->forward(ctx, x, y, R, ctx.logit_rows);
     ctx.tap("final_norm", y);
+    return head(ctx, y);
+}
+
+Rows DecoderModel::no_logits() const { return Rows{nullptr, DType::F32, 0, spec.vocab_size(), spec.vocab_size()}; }
+
+Rows DecoderModel::forward_streams(StepContext& ctx, const Rows& embedded) {
+    const int T = ctx.n_tokens, S = static_cast<int>(spec.streams);
+    const int64_t width = spec.hidden();
+    Workspace& ws = *ctx.workspace;
+    const Rows x = ws.get("streams", T, width * S, DType::F32);
+    auto reader_of = [&](size_t run) { return layers[static_cast<size_t>(spec.run_order[run].layer)].block->reader(); };
+    // All streams start as the embedded row; the same launch makes the first sublayer's input.
+    const std::optional<StreamReader> first = reader_of(0);
+    const Rows h = ws.get("block.normed", T, width, runtime.dtype);
+    kernels::streams_open(ctx.stream(), runtime.dtype, embedded, x, S, T, first ? &*first : nullptr, first ? &h : nullptr);
+    if (first) {
+        ctx.next_input = h;
+        ctx.next_input_entry = 0;
+    }
+    for (size_t i = 0; i < spec.run_order.size(); ++i) {
+        const RunEntry& e = spec.run_order[i];
+        const std::optional<StreamReader> next = i + 1 < spec.run_order.size() ? reader_of(i + 1) : std::nullopt;
+        ctx.next_reader = next ? &*next : nullptr;
+        layers[static_cast<size_t>(e.layer)].block->forward(ctx, x, CacheUnit{e.cache, e.cache == static_cast<int>(i), static_cast<int>(i)});
+    }
+    ctx.next_reader = nullptr;
+    ctx.next_input_entry = -1;
+    const int R = ctx.n_logit_rows;
+    if (R == 0) return no_logits();
+    ctx.phase(Phase::Head);
+    const Rows y = ws.get("head.normed", R, width, runtime.dtype, false);
+    if (const auto recipe = final_norm->tanh_recipe()) {
+        kernels::streams_read(ctx.stream(), runtime.dtype, x, S, ctx.logit_rows, R, *recipe, y);      // the sum of the streams and its norm in one launch
+    } else {
+        const Rows sum = ws.get("head.streams_sum", R, width, DType::F32, false);
+        kernels::streams_read(ctx.stream(), DType::F32, x, S, ctx.logit_rows, R, StreamReader{}, sum);
+        final_norm->forward(ctx, sum, y, R, nullptr);
+    }
+    ctx.tap("final_norm", y);
+    return head(ctx, y);
+}
+
+Rows DecoderModel::head(StepContext& ctx, const Rows& y) {
+    const int R = ctx.n_logit_rows;
+    Workspace& ws = *ctx.workspace;
     const Rows logits = ws.get("logits", R, spec.vocab_size(), DType::F32, false);
     kernels::linear(runtime, &ws, y, head_weight, head_bias, logits, R, kernels::kNone, nullptr);
     if (spec.head.logit_scale != 1.0 || spec.head.soft_cap > 0.0)

@@ -51,6 +51,10 @@ public:
     Rows forward(StepContext& ctx);
 
 private:
+    // The layers over several residual streams, from the embedded rows on; the head's product; what a step without wanted rows returns.
+    Rows forward_streams(StepContext& ctx, const Rows& embedded);
+    Rows head(StepContext& ctx, const Rows& normed);
+    Rows no_logits() const;
     Mixer* mixer_of(const RunEntry& e) const;
     Params params_;
 };

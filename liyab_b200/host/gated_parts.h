@@ -74,6 +74,9 @@ inline std::vector<float> rotation_frequencies(int dims, double base) {
 // joins the divisor of the head's softmax; it has no key and no value and is not scaled.  `value_blend`: "source" leaves the step's values
 // (as projected) where later layers of the model find them; "blend" replaces its own by (1 - b) v + b v_source with the learned number `blend`
 // before they are cached.  The source is the model's first layer that says so; all such layers have n_kv_head x vdim values alike.
+// `rot_layout` "interleaved": the rotation pairs value 2i with 2i + 1.  `values` "keys": the values are the keys as projected (no rows for v in the
+// projection; vdim = dim, and no rotation or norm may come between).  `slopes`: the score of the key d positions back loses
+// slope_h d with slope_h = 2^(-8 (h + 1) / n_head) for head h counted from 0.  `unit_sink`: one is added to every softmax's divisor.
 
 class GatedAttention final : public Mixer {
 public:
@@ -114,20 +117,41 @@ public:
         if (rot_dims < 0 || rot_dims > D || rot_dims % 2 != 0) throw invalid_model("gated_attention: {} of {} values cannot be rotated in pairs", rot_dims, D);
         freq.host = rotation_frequencies(rot_dims, s.options.get_number("rot_base", 10000.0));
         if (s.options.get_bool("sink", false)) shape.sink = f32_or_null(&p.at("sink"));
+        const std::string layout = s.options.get_string("rot_layout", "half");
+        if (layout != "half" && layout != "interleaved") throw unsupported("gated_attention: rot_layout '{}' is not supported; supported: half, interleaved", layout);
+        interleaved = layout == "interleaved";
+        values_are_keys = values_from_keys(s);
+        if (values_are_keys && (E != D || qk_norm || rot_dims > 0))
+            throw unsupported("gated_attention: values that are the keys as projected take vdim = dim, no norm of the keys and no rotation");
+        if (s.options.get_bool("slopes", false)) {
+            if (shape.distance != nullptr) throw unsupported("gated_attention: slopes or a learned penalty by distance, not both");
+            for (int h = 0; h < H; ++h) slopes.host.push_back(static_cast<float>(std::exp2(-8.0 * (h + 1) / H)));
+            for (int h = 0; h < H; ++h) slopes.host.push_back(-1.0f);        // a negative second number: a straight line
+        }
+        if (s.options.get_bool("unit_sink", false)) {
+            if (shape.sink != nullptr) throw unsupported("gated_attention: learned sinks or one in every divisor, not both");
+            unit_sinks.host.assign(static_cast<size_t>(H), 0.0f);
+        }
         const std::string vb = s.options.get_string("value_blend", "none");
         if (vb != "none" && vb != "source" && vb != "blend") throw unsupported("gated_attention: value_blend '{}' is not supported; supported: none, source, blend", vb);
         blend_source = vb == "source";
         if (vb == "blend") blend = f32_or_null(&p.at("blend"));
+        if (values_are_keys && vb != "none") throw unsupported("gated_attention: values that are the keys do not blend with others");
         rotary_store = norm_projection || rot_dims > 0 || vb != "none";
         if (rotary_store && temp_every > 0) throw unsupported("gated_attention: a temperature on the queries goes with neither rotation, norm over the projection nor blended values");
     }
+    static bool values_from_keys(const PartSpec& s) {
+        const std::string v = s.options.get_string("values", "own");
+        if (v != "own" && v != "keys") throw unsupported("gated_attention: values '{}' are not supported; supported: own, keys", v);
+        return v == "keys";
+    }
     static std::vector<ParamDecl> parameters(const PartSpec& s) {
         const int64_t hidden = need_int(s, "hidden"), H = need_int(s, "n_head"), G = s.options.get_int("n_kv_head", H), D = need_int(s, "dim");
-        const int64_t E = s.options.get_int("vdim", D);
+        const int64_t E = s.options.get_int("vdim", D), VE = values_from_keys(s) ? 0 : E;
         const bool gated = s.options.get_string("gate", "none") != "none";
         std::vector<ParamDecl> out;
-        Linear::declare(out, "proj.", H * D + G * D + G * E + (gated ? H * E : 0), hidden, false);
-        if (s.options.get_bool("bias", false)) out.push_back({"qkv_bias", {H * D + G * D + G * E}, ParamKind::Vector});
+        Linear::declare(out, "proj.", H * D + G * D + G * VE + (gated ? H * E : 0), hidden, false);
+        if (s.options.get_bool("bias", false)) out.push_back({"qkv_bias", {H * D + G * D + G * VE}, ParamKind::Vector});
         if (s.options.get_bool("qk_norm", false) && s.options.get_bool("qk_gain", true)) {
             const bool whole = s.options.get_string("qk_norm_over", "head") == "projection";
             out.push_back({"q_norm.weight", {whole ? H * D : D}, ParamKind::Vector});
@@ -168,7 +192,7 @@ public:
     kernels::AttentionShape shape;
     int64_t hidden = 0;
     int H = 0, G = 0, D = 0, E = 0, gate = -1;
-    bool qk_norm = false, norm_projection = false, blend_source = false, rotary_store = false;
+    bool qk_norm = false, norm_projection = false, blend_source = false, rotary_store = false, interleaved = false, values_are_keys = false;
     int rot_dims = 0;
     const float* blend = nullptr;
     float eps = 1e-6f, temp_coef = 0.0f;
@@ -178,7 +202,7 @@ public:
     const float* k_gain = nullptr;
 
 private:
-    int64_t qkv_cols() const { return static_cast<int64_t>(H) * D + static_cast<int64_t>(G) * (D + E); }
+    int64_t qkv_cols() const { return static_cast<int64_t>(H) * D + static_cast<int64_t>(G) * (D + (values_are_keys ? 0 : E)); }
     // Either the normalised rows h, or the stream's rows x_in with the recipe of the norm before the mixer.
     void run(StepContext& ctx, const Rows* h, const Rows* x_in, const NormRecipe* norm, const Rows& y, const Rows* residual, CacheUnit unit) {
         const int T = ctx.n_tokens, P = shape.head_dim;
@@ -193,15 +217,17 @@ private:
         void* cache = ctx.kv(unit.read, &view);
         kernels::AttentionShape a = shape;
         a.page_size = view->group->page_size;
+        if (!slopes.host.empty()) a.distance = slopes.get(s);
+        if (!unit_sinks.host.empty()) a.sink = unit_sinks.get(s);
         const Rows q = ws.get("gated_attention.q", T, static_cast<int64_t>(H) * P, dt);
-        const kernels::QkvColumns cols{0, H * D, H * D + G * D, H, G, D, E, P, a.page_size};
+        const kernels::QkvColumns cols{0, H * D, values_are_keys ? H * D : H * D + G * D, H, G, D, E, P, a.page_size};
         if (rotary_store) {
             // The values that layers blend with travel from the source layer to the others in a buffer of the step.
             Rows shared;
             if (blend_source || blend != nullptr) shared = ws.get("gated_attention.value_source", T, static_cast<int64_t>(G) * E, DType::F32);
             kernels::qkv_rotary_store(s, pr, cols, q_gain, k_gain, q, unit.write ? cache : nullptr, view->slot_mapping, T, !qk_norm ? 0 : norm_projection ? 2 : 1, eps,
                                       ctx.positions, rot_dims > 0 ? freq.get(s) : nullptr, rot_dims, blend != nullptr ? &shared : nullptr,
-                                      blend_source ? &shared : nullptr, blend);
+                                      blend_source ? &shared : nullptr, blend, interleaved);
         } else {
             kernels::qk_norm_store(s, pr, cols, q_gain, k_gain, q, unit.write ? cache : nullptr, view->slot_mapping, T, qk_norm, eps, ctx.positions, temp_coef,
                                    temp_every);
@@ -221,7 +247,7 @@ private:
         kernels::linear(ctx.runtime, &ws, heads, out.weight, nullptr, y, T, kernels::kNone, residual);
     }
     PartialBias bias;
-    DeviceFloats freq;
+    DeviceFloats freq, slopes, unit_sinks;
 };
 
 // ---- a matrix memory per head ----------------------------------------------------------------------------------
@@ -361,16 +387,19 @@ private:
 // x += scale * sum_b rms(mixer_b(h)) * gain_b: every branch reads the same input, its output is divided by its root mean square
 // over the width and multiplied by its gain.  Options: `branches` [{"name", "part": {kind, options}}], `scale`, `eps`, `size`.
 // At most one branch may keep keys and values and at most one a state: both live under the block's one cache unit.
+// `norm` false: the branches' outputs as they are, each times its own number (`scale` of the branch, default 1), no gains: x += scale * sum_b scale_b mixer_b(h).
 
 class BranchSum final : public Mixer {
 public:
     BranchSum(const PartSpec& s, const Params& p, const Runtime& rt) : size(need_int(s, "size")), scale(static_cast<float>(s.options.get_number("scale", 1.0))),
-                                                                       eps(static_cast<float>(s.options.get_number("eps", 1e-6))) {
+                                                                       eps(static_cast<float>(s.options.get_number("eps", 1e-6))),
+                                                                       normed(s.options.get_bool("norm", true)) {
         for (const auto& [name, part] : branch_specs(s)) {
             names.push_back(name);
             branches.push_back(mixers().get(part.kind).build(part, p.sub(name + "."), rt));
-            gains.push_back(f32_or_null(&p.at(name + "_out.weight")));
+            if (normed) gains.push_back(f32_or_null(&p.at(name + "_out.weight")));
         }
+        for (const auto& b : s.options.find("branches")->items()) branch_scale.push_back(scale * static_cast<float>(b.get_number("scale", 1.0)));
         int kv = 0, st = 0;
         for (const auto& b : branches) {
             kv += b->kv_need().has_value();
@@ -389,7 +418,7 @@ public:
         std::vector<ParamDecl> out;
         for (const auto& [name, part] : branch_specs(s)) {
             for (const auto& d : mixers().get(part.kind).parameters(part)) out.push_back({name + "." + d.name, d.shape, d.kind});
-            out.push_back({name + "_out.weight", {need_int(s, "size")}, ParamKind::Vector});
+            if (s.options.get_bool("norm", true)) out.push_back({name + "_out.weight", {need_int(s, "size")}, ParamKind::Vector});
         }
         return out;
     }
@@ -409,6 +438,15 @@ public:
         return std::nullopt;
     }
     void forward(StepContext& ctx, const Rows& h, const Rows& x, CacheUnit unit) override { run(ctx, &h, nullptr, nullptr, x, unit); }
+    void forward_into(StepContext& ctx, const Rows& h, const Rows& y, CacheUnit unit) override {
+        if (normed) return Mixer::forward_into(ctx, h, y, unit);
+        kernels::terms_sum(ctx.stream(), ctx.runtime.dtype, terms(outputs(ctx, &h, nullptr, nullptr, unit)), y, ctx.n_tokens, true);
+    }
+    // Branches without norms leave their sum to the launch that joins it to the streams.
+    OutputTerms forward_terms(StepContext& ctx, const Rows& h, const Rows& y, CacheUnit unit) override {
+        if (normed) return Mixer::forward_terms(ctx, h, y, unit);
+        return terms(outputs(ctx, &h, nullptr, nullptr, unit));
+    }
     // Where every branch can normalise the rows itself for this step, the norm before the mixer is not launched.
     bool normalises(const StepContext& ctx, const Rows& x_in) const override {
         for (const auto& b : branches)
@@ -422,18 +460,34 @@ public:
     }
     int64_t size;
     float scale, eps;
+    bool normed;
+    std::vector<float> branch_scale;
     std::vector<std::string> names;
     std::vector<std::shared_ptr<Mixer>> branches;
     std::vector<const float*> gains;
 
 private:
-    void run(StepContext& ctx, const Rows* h, const Rows* x_in, const NormRecipe* norm, const Rows& x, CacheUnit unit) {
+    OutputTerms terms(std::vector<Rows> ys) const {
+        OutputTerms t;
+        t.rows = std::move(ys);
+        t.scale = branch_scale;
+        return t;
+    }
+    std::vector<Rows> outputs(StepContext& ctx, const Rows* h, const Rows* x_in, const NormRecipe* norm, CacheUnit unit) {
         std::vector<Rows> ys;
         for (size_t i = 0; i < branches.size(); ++i) {
             ys.push_back(ctx.workspace->get(std::format("branch_sum.{}", i), ctx.n_tokens, size, DType::F32));
             if (h != nullptr) branches[i]->forward_into(ctx, *h, ys.back(), unit);
             else branches[i]->forward_from_into(ctx, *x_in, *norm, ys.back(), unit);
             ctx.tap("branch." + names[i], ys.back());
+        }
+        return ys;
+    }
+    void run(StepContext& ctx, const Rows* h, const Rows* x_in, const NormRecipe* norm, const Rows& x, CacheUnit unit) {
+        std::vector<Rows> ys = outputs(ctx, h, x_in, norm, unit);
+        if (!normed) {
+            kernels::terms_sum(ctx.stream(), ctx.runtime.dtype, terms(std::move(ys)), x, ctx.n_tokens, false);
+            return;
         }
         kernels::rms_sum_add(ctx.stream(), x, ys, gains, ctx.n_tokens, scale, eps);
     }
@@ -507,6 +561,10 @@ private:
 // gate_up [experts x 2 inner, hidden] (per expert its gate rows, then its up rows) and down [experts x hidden, inner].
 // `route` "table": no router; the parameter `table` (int32 [vocab, top], a row's entries all different) names the experts of every token id,
 // each with the weight 1 / top.
+// Further options of the router.  `identity` n: the last n of the router's experts + n outputs are experts without matrices whose result is the
+// input itself (times the weight; with weight_on output).  `correction`: a learned number an expert that is added to its score for the choice only.
+// `groups` g and `keep_groups` k: the outputs form g equal groups of neighbours, a group counts as its best choice score, and only experts of
+// the k best groups can be chosen.  `route_scale`: a factor on the weights.
 
 class RoutedExperts final : public FeedForward {
 public:
@@ -514,7 +572,7 @@ public:
         : hidden(need_int(s, "hidden")), inner(need_int(s, "inner")), experts(static_cast<int>(need_int(s, "experts"))), top(static_cast<int>(need_int(s, "top"))),
           gate(kernels::gate_from_name(s.options.get_string("activation", "silu"))), renormalise(s.options.get_bool("renormalise", false)),
           alpha(static_cast<float>(s.options.get_number("gate_alpha", 1.0))), limit(static_cast<float>(s.options.get_number("gate_limit", 0.0))) {
-        if (top > experts) throw invalid_model("routed: top {} of {} experts", top, experts);
+        if (top > experts + s.options.get_int("identity", 0)) throw invalid_model("routed: top {} of {} experts", top, experts);
         const std::string score = s.options.get_string("score", "sigmoid");
         if (score != "sigmoid" && score != "softmax") throw unsupported("routed: score '{}' is not supported; supported: sigmoid, softmax", score);
         softmax = score == "softmax";
@@ -527,6 +585,16 @@ public:
         if (by_table) table = p.at("table");
         else router = p.at("router.weight");
         if (!by_table && s.options.get_bool("router_bias", false)) router_bias = f32_or_null(&p.at("router.bias"));
+        identity = static_cast<int>(s.options.get_int("identity", 0));
+        groups = static_cast<int>(s.options.get_int("groups", 1));
+        keep_groups = static_cast<int>(s.options.get_int("keep_groups", groups));
+        route_scale = static_cast<float>(s.options.get_number("route_scale", 1.0));
+        if (s.options.get_bool("correction", false)) correction = f32_or_null(&p.at("router.correction"));
+        corrected = identity > 0 || groups > 1 || correction != nullptr || route_scale != 1.0f;
+        if (corrected && by_table) throw unsupported("routed: a table of experts has no router to correct");
+        if (identity < 0 || groups < 1 || (experts + identity) % groups != 0 || keep_groups < 1 || keep_groups > groups || top > (experts + identity) / groups * keep_groups)
+            throw invalid_model("routed: top {} of {} experts and {} identities in {} groups of which {} count", top, experts, identity, groups, keep_groups);
+        if (identity > 0 && !weight_on_output) throw unsupported("routed: identity experts take the weight on the output");
         gate_up = p.at("experts.gate_up.weight");
         down = p.at("experts.down.weight");
         if (s.options.get_int("shared_inner", 0) > 0) shared = std::make_unique<GatedFeedForward>(shared_spec(s), p.sub("shared."));
@@ -541,8 +609,10 @@ public:
         if (s.options.get_string("route", "scores") == "table") {
             out.push_back({"table", {need_int(s, "vocab"), need_int(s, "top")}, ParamKind::Index});
         } else {
-            out.push_back({"router.weight", {E, hidden}, ParamKind::Matrix});
-            if (s.options.get_bool("router_bias", false)) out.push_back({"router.bias", {E}, ParamKind::Vector});
+            const int64_t N = E + s.options.get_int("identity", 0);
+            out.push_back({"router.weight", {N, hidden}, ParamKind::Matrix});
+            if (s.options.get_bool("router_bias", false)) out.push_back({"router.bias", {N}, ParamKind::Vector});
+            if (s.options.get_bool("correction", false)) out.push_back({"router.correction", {N}, ParamKind::Vector});
         }
         for (ParamDecl d : std::vector<ParamDecl>{{"experts.gate_up.weight", {E * 2 * inner, hidden}, ParamKind::Matrix},
                                    {"experts.down.weight", {E * hidden, inner}, ParamKind::Matrix}})
@@ -555,7 +625,72 @@ public:
     void forward(StepContext& ctx, const Rows& h, const Rows& x) override { run(ctx, h, x, false); }
     // The rows' sums are written instead of added, so nothing has to be cleared first (a shared expert then adds to them).
     void forward_into(StepContext& ctx, const Rows& h, const Rows& y) override { run(ctx, h, y, true); }
+    // The rows' sums are left to the launch that joins them to the streams; the experts may have been chosen by the launch that made h.
+    OutputTerms forward_terms(StepContext& ctx, const Rows& h, const Rows& y, bool routed) override {
+        if (!corrected) return FeedForward::forward_terms(ctx, h, y, routed);
+        const int T = ctx.n_tokens, pairs = T * top;
+        Workspace& ws = *ctx.workspace;
+        cudaStream_t s = ctx.stream();
+        const RowRouter r = *row_router(ctx);
+        if (!routed) kernels::router_choice(s, h, r, T);
+        Rows mid = ws.get("routed.inner", T, static_cast<int64_t>(top) * inner, ctx.runtime.dtype);
+        mid = Rows{mid.data, mid.dtype, static_cast<int64_t>(pairs), inner, inner};
+        Rows out = ws.get("routed.out", T, static_cast<int64_t>(top) * hidden, DType::F32);
+        out = Rows{out.data, out.dtype, static_cast<int64_t>(pairs), hidden, hidden};
+        const float* on_input = weight_on_output ? nullptr : r.weights;
+        OutputTerms t;
+        const int N1 = static_cast<int>(inner), N2 = static_cast<int>(hidden);
+        if (kernels::expert_product_direct_supports(h, gate_up, pairs, N1, N2, true) && kernels::expert_product_direct_supports(mid, down, pairs, N2, N1, false)) {
+            // A few pairs: every pair finds its expert by itself, no plan.
+            kernels::expert_product_direct(s, true, h, gate_up, experts, r.ids, on_input, mid, pairs, N1, N2, top, gate, alpha, limit);
+            kernels::expert_product_direct(s, false, mid, down, experts, r.ids, nullptr, out, pairs, N2, N1, top, gate);
+        } else {
+            int32_t* place = static_cast<int32_t*>(ws.get("routed.place", T, top, DType::I32).data);
+            int32_t* pair_at = static_cast<int32_t*>(ws.get("routed.pair_at", T, top, DType::I32).data);
+            int32_t* offsets = static_cast<int32_t*>(ws.flat("routed.offsets", experts + 1, DType::I32));
+            kernels::expert_plan(s, r.ids, pairs, experts, offsets, place, pair_at);
+            kernels::expert_product(s, true, h, gate_up, experts, offsets, pair_at, on_input, mid, pairs, N1, N2, top, gate, alpha, limit);
+            kernels::expert_product(s, false, mid, down, experts, offsets, pair_at, nullptr, out, pairs, N2, N1, top, gate);
+            t.place = place;
+        }
+        t.pairs = out;
+        t.self = h;
+        t.ids = r.ids;
+        t.weights = weight_on_output ? r.weights : nullptr;
+        t.top = top;
+        t.n_real = experts;
+        if (shared) {
+            shared->forward_into(ctx, h, y);
+            t.rows = {y};
+            t.scale = {1.0f};
+        }
+        return t;
+    }
+    std::optional<RowRouter> row_router(StepContext& ctx) override {
+        if (!corrected) return std::nullopt;
+        const int T = ctx.n_tokens;
+        RowRouter r;
+        r.matrix = router.data;
+        r.bias = router_bias;
+        r.correction = correction;
+        r.n_experts = experts + identity;
+        r.top = top;
+        r.groups = groups;
+        r.keep = keep_groups;
+        r.softmax = softmax;
+        r.renormalise = renormalise;
+        r.scale = route_scale;
+        r.ids = static_cast<int32_t*>(ctx.workspace->get("routed.ids", T, top, DType::I32).data);
+        r.weights = ctx.workspace->get("routed.weights", T, top, DType::F32).f32();
+        return r;
+    }
     void run(StepContext& ctx, const Rows& h, const Rows& x, bool overwrite) {
+        if (corrected) {
+            const Rows y = ctx.workspace->get("routed.shared", ctx.n_tokens, hidden, DType::F32);
+            kernels::terms_sum(ctx.stream(), ctx.runtime.dtype, forward_terms(ctx, h, y, false), x, ctx.n_tokens, overwrite);
+            ctx.tap("routed", x);
+            return;
+        }
         const int T = ctx.n_tokens, pairs = T * top;
         Workspace& ws = *ctx.workspace;
         cudaStream_t s = ctx.stream();
@@ -590,7 +725,10 @@ public:
     static constexpr int kLookupInPlan = 1024;
     int64_t hidden, inner;
     int experts, top, gate;
-    bool renormalise, softmax = false, weight_on_output = false, by_table = false;
+    bool renormalise, softmax = false, weight_on_output = false, by_table = false, corrected = false;
+    int identity = 0, groups = 1, keep_groups = 1;
+    float route_scale = 1.0f;
+    const float* correction = nullptr;
     float alpha, limit;
     const float* router_bias = nullptr;
     Tensor router, table, gate_up, down;

@@ -360,16 +360,16 @@ void gated_act(cudaStream_t s, const Rows& gu, const Rows& mid, int n_rows, int 
 
 void qkv_rotary_store(cudaStream_t s, const Rows& proj, const QkvColumns& c, const float* q_weight, const float* k_weight, const Rows& q_out, void* cache,
                       const int32_t* slot_mapping, int n_tokens, int norm_mode, float eps, const int32_t* positions, const float* freq, int rot_dims,
-                      const Rows* v_first_in, const Rows* v_first_out, const float* lambda) {
+                      const Rows* v_first_in, const Rows* v_first_out, const float* lambda, bool interleaved) {
     if (proj.dtype != DType::F32 || q_out.cols != static_cast<int64_t>(c.n_head) * c.padded) throw invalid_argument("qkv_rotary_store: buffers do not fit");
     const int64_t vcols = static_cast<int64_t>(c.n_kv_head) * c.vdim;
     const Rows* shared = v_first_in != nullptr ? v_first_in : v_first_out;
     if (shared != nullptr && (shared->dtype != DType::F32 || shared->cols != vcols || shared->rows < n_tokens))
         throw invalid_argument("qkv_rotary_store: the shared values are float32 [tokens, {}]", vcols);
-    check(lb_qkv_rotary_store(code(q_out.dtype, "q_out"), proj.f32(), proj.stride, c.q_off, c.k_off, c.v_off, q_weight, k_weight, q_out.data, q_out.stride, cache,
+    check(lb_qkv_rotary_store_layout(code(q_out.dtype, "q_out"), proj.f32(), proj.stride, c.q_off, c.k_off, c.v_off, q_weight, k_weight, q_out.data, q_out.stride, cache,
                               slot_mapping, n_tokens, c.n_head, c.n_kv_head, c.dim, c.vdim, c.padded, c.page_size, norm_mode, eps, positions, freq, rot_dims,
                               v_first_in != nullptr ? v_first_in->f32() : nullptr, v_first_out != nullptr ? v_first_out->f32() : nullptr,
-                              shared != nullptr ? shared->stride : 0, lambda, s), "qkv_rotary_store");
+                              shared != nullptr ? shared->stride : 0, lambda, interleaved ? 1 : 0, s), "qkv_rotary_store");
 }
 
 void row_norm_gate(cudaStream_t s, const Rows& o, const Rows& g, const float* gain, const Rows& out, int n_rows, int gate, float eps) {
@@ -604,6 +604,149 @@ void latent_attention(cudaStream_t s, DType cache_dtype, const Rows& wide, const
     const lb_latent_extras x = latent_extras(a, gate);
     check(lb_latent_attention_ext(code(cache_dtype, "cache"), wide.f32(), wide.stride, cache, tok_seq, positions, block_table, table_width, out.f32(),
                                   out.stride, n_tokens, a.n_head, a.rank, a.rot, a.page_size, a.scale, a.window, &x, s), "latent_attention");
+}
+
+namespace {
+lb_output_terms terms_of(const OutputTerms& t, DType dtype, int64_t width) {
+    lb_output_terms o{};
+    if (t.rows.size() > 4 || t.rows.size() != t.scale.size()) throw invalid_argument("output terms: at most four rows, each with its number");
+    for (size_t i = 0; i < t.rows.size(); ++i) {
+        if (t.rows[i].dtype != DType::F32 || t.rows[i].cols != width) throw invalid_argument("output terms: float32 rows of the stream's width");
+        o.y[i] = t.rows[i].f32();
+        o.ldy[i] = t.rows[i].stride;
+        o.scale[i] = t.scale[i];
+    }
+    o.n_rows = static_cast<int>(t.rows.size());
+    if (t.pairs.data != nullptr) {
+        if (t.pairs.dtype != DType::F32 || t.pairs.cols != width || (t.self.data != nullptr && (t.self.dtype != dtype || t.self.cols != width)))
+            throw invalid_argument("output terms: the experts' results do not fit the stream");
+        o.pairs = t.pairs.f32();
+        o.ldp = t.pairs.stride;
+        o.place = t.place;
+        o.ids = t.ids;
+        o.weights = t.weights;
+        o.top = t.top;
+        o.n_real = t.n_real;
+        o.self = t.self.data;
+        o.lds = t.self.stride;
+    }
+    return o;
+}
+lb_router router_of(const RowRouter& r) {
+    return lb_router{r.matrix, r.bias, r.correction, r.n_experts, r.top, r.groups, r.keep, r.softmax ? 1 : 0, r.renormalise ? 1 : 0, r.scale, r.ids, r.weights};
+}
+lb_streams_args streams_of(const Rows& x, int n_streams, const StreamReader* reader, const Rows* h, DType dtype) {
+    if (x.dtype != DType::F32 || n_streams < 1 || x.cols % n_streams != 0) throw invalid_argument("streams: float32 rows of {} equal parts", n_streams);
+    lb_streams_args a{};
+    a.x = x.f32();
+    a.ldx = x.stride;
+    a.n_streams = n_streams;
+    a.width = static_cast<int>(x.cols / n_streams);
+    if (reader != nullptr) {
+        if (h == nullptr || h->dtype != dtype || h->cols != a.width) throw invalid_argument("streams: the next input does not fit");
+        a.next_in = reader->in;
+        a.alpha = reader->alpha;
+        a.gain = reader->gain;
+        a.offset = reader->offset;
+        a.h = h->data;
+        a.ldh = h->stride;
+    }
+    return a;
+}
+}  // namespace
+
+void streams_open(cudaStream_t s, DType dtype, const Rows& embedded, const Rows& x, int n_streams, int n_rows, const StreamReader* reader, const Rows* h) {
+    lb_streams_args a = streams_of(x, n_streams, reader, h, dtype);
+    if (embedded.dtype != DType::F32 || embedded.cols != a.width) throw invalid_argument("streams: the embedded rows do not fit");
+    a.fresh = embedded.f32();
+    a.ldf = embedded.stride;
+    check(lb_streams_join(code(dtype, "h"), &a, nullptr, nullptr, n_rows, s), "streams_open");
+}
+
+void streams_read(cudaStream_t s, DType dtype, const Rows& x, int n_streams, const int32_t* rows, int n_rows, const StreamReader& reader, const Rows& out) {
+    lb_streams_args a = streams_of(x, n_streams, &reader, &out, dtype);
+    a.rows = rows;
+    check(lb_streams_join(code(dtype, "out"), &a, nullptr, nullptr, n_rows, s), "streams_read");
+}
+
+void streams_join(cudaStream_t s, DType dtype, const Rows& x, const Join& join, const OutputTerms& terms, int n_rows, const StreamReader* reader, const Rows* h,
+                  const RowRouter* router) {
+    lb_streams_args a = streams_of(x, join.streams(), reader, h, dtype);
+    a.mix = join.mix();
+    a.to = join.out();
+    a.scale = join.scale();
+    const lb_output_terms o = terms_of(terms, dtype, a.width);
+    lb_router r{};
+    if (router != nullptr) r = router_of(*router);
+    check(lb_streams_join(code(dtype, "h"), &a, &o, router != nullptr ? &r : nullptr, n_rows, s), "streams_join");
+}
+
+void router_choice(cudaStream_t s, const Rows& h, const RowRouter& router, int n_rows) {
+    const lb_router r = router_of(router);
+    check(lb_router_choice(code(h.dtype, "h"), &r, h.data, h.stride, n_rows, static_cast<int>(h.cols), s), "router_choice");
+}
+
+void terms_sum(cudaStream_t s, DType dtype, const OutputTerms& terms, const Rows& x, int n_rows, bool overwrite) {
+    if (x.dtype != DType::F32) throw invalid_argument("sum of output terms: into float32 rows");
+    const lb_output_terms o = terms_of(terms, dtype, x.cols);
+    check(lb_terms_sum(code(dtype, "self"), &o, x.f32(), x.stride, n_rows, static_cast<int>(x.cols), overwrite ? 1 : 0, s), "terms_sum");
+}
+
+bool expert_product_direct_supports(const Rows& a, const Tensor& w, int n_pairs, int n, int k, bool gated) {
+    return a.dtype == w.dtype && lb_expert_product_direct_supports(code(a.dtype, "a"), a.data, a.stride, w.data, static_cast<int64_t>(gated ? 2 : 1) * n * k, n_pairs, k) != 0;
+}
+
+void expert_product_direct(cudaStream_t s, bool gated, const Rows& a, const Tensor& w, int n_experts, const int32_t* ids, const float* weights, const Rows& out,
+                           int n_pairs, int n, int k, int top, int gate, float alpha, float limit) {
+    if (a.dtype != w.dtype || w.numel() != static_cast<int64_t>(n_experts) * (gated ? 2 : 1) * n * k || a.cols != k || out.cols != n)
+        throw invalid_argument("expert product: shapes do not fit");
+    if (out.dtype != (gated ? a.dtype : DType::F32)) throw invalid_argument("expert product: the output has the wrong type");
+    check(lb_expert_product_direct(code(a.dtype, "a"), gated ? 1 : 0, a.data, a.stride, w.data, static_cast<int64_t>(gated ? 2 : 1) * n * k, ids, weights, out.data,
+                                   out.stride, n_pairs, n_experts, n, k, top, gate, alpha, limit, s), "expert_product_direct");
+}
+
+namespace {
+lb_channel_memory channel_of(const ChannelMemoryShape& m) {
+    lb_channel_memory c{};
+    c.n_head = m.n_head; c.kv_head = m.kv_head; c.dim = m.dim; c.vdim = m.vdim;
+    c.delta = m.delta ? 1 : 0; c.taps = m.taps; c.unit = m.unit ? 1 : 0; c.rank = m.rank; c.gate_rank = m.gate_rank; c.gate_act = m.gate;
+    c.a_off = static_cast<int>(m.a_off()); c.g_off = static_cast<int>(m.g_off()); c.b_off = static_cast<int>(m.b_off());
+    c.conv = m.conv; c.a2 = m.a2.data; c.g2 = m.g2.data; c.z_bias = m.z_bias; c.a_log = m.a_log; c.norm = m.norm;
+    c.tau = m.tau; c.q_scale = m.q_scale; c.unit_eps = m.unit_eps; c.eps = m.eps;
+    c.slot_stride = m.slot_floats();
+    return c;
+}
+lb_channel_step channel_step_of(const ChannelMemoryShape& m, const ChannelStep& step, const Rows& proj, const Rows& o, const Rows& heads) {
+    if (proj.dtype != DType::F32 || proj.cols != m.cols() || heads.cols != static_cast<int64_t>(m.n_head) * m.vdim || m.a2.dtype != heads.dtype ||
+        (m.g2.data != nullptr && m.g2.dtype != heads.dtype) || (o.data != nullptr && (o.dtype != DType::F32 || o.cols != heads.cols)))
+        throw invalid_argument("channel memory: the rows do not fit the shape");
+    lb_channel_step c{};
+    c.proj = proj.f32(); c.ld = proj.stride;
+    c.positions = step.positions; c.tok_seq = step.tok_seq; c.q_start = step.q_start; c.slots = step.slots; c.state = step.state;
+    c.o = o.f32(); c.ldo = o.stride;
+    c.heads = heads.data; c.ldh = heads.stride;
+    return c;
+}
+}  // namespace
+
+void channel_memory_rows(cudaStream_t s, const ChannelMemoryShape& m, const ChannelStep& step, const Rows& proj, const Rows& o, const Rows& heads) {
+    const lb_channel_memory c = channel_of(m);
+    const lb_channel_step t = channel_step_of(m, step, proj, o, heads);
+    check(lb_channel_memory_rows(code(heads.dtype, "heads"), &c, &t, step.n_seq, step.decode_only ? 1 : 0, s), "channel_memory_rows");
+    if (m.conv != nullptr && !step.decode_only) launches.fetch_add(1, std::memory_order_relaxed);
+}
+
+void channel_memory_pieces(cudaStream_t s, Workspace* ws, const ChannelMemoryShape& m, const ChannelStep& step, const Rows& proj, const Rows& o, const Rows& heads) {
+    const lb_channel_memory c = channel_of(m);
+    const lb_channel_step t = channel_step_of(m, step, proj, o, heads);
+    const bool prepared = m.conv != nullptr || m.unit;
+    float* rows = prepared ? ws->get("channel_memory.rows", step.n_tokens, m.channels(), DType::F32).f32() : nullptr;
+    float* log_decay = ws->get("channel_memory.log_decay", step.n_tokens, static_cast<int64_t>(m.n_head) * m.dim, DType::F32).f32();
+    float* gate = m.g2.data != nullptr ? ws->get("channel_memory.gate", step.n_tokens, static_cast<int64_t>(m.n_head) * m.vdim, DType::F32).f32() : nullptr;
+    const int64_t floats = lb_channel_memory_pieces_floats(step.n_tokens, step.n_seq, m.n_head, m.dim, m.vdim, m.delta ? 1 : 0);
+    float* scratch = static_cast<float*>(ws->flat("channel_memory.pieces", floats, DType::F32));
+    check(lb_channel_memory_pieces(code(heads.dtype, "heads"), &c, &t, rows, log_decay, gate, scratch, step.n_tokens, step.n_seq, s), "channel_memory_pieces");
+    launches.fetch_add(3 + (m.g2.data != nullptr ? 1 : 0) + (prepared ? 1 : 0) + (m.conv != nullptr ? 1 : 0), std::memory_order_relaxed);
 }
 
 void sample(cudaStream_t s, const float* logits, int64_t row_stride, int n_rows, int vocab, const float* temperature,

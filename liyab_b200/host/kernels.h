@@ -14,6 +14,7 @@
 #include <vector>
 
 #include "device.h"
+#include "parts.h"
 #include "spec.h"
 
 namespace liyab::kernels {
@@ -190,11 +191,11 @@ void qk_norm_store(cudaStream_t s, const Rows& proj, const QkvColumns& c, const 
                    int temp_every = 0);
 // The same for queries and keys that are normed over the whole projection and rotated, and for values that blend with an earlier layer's:
 // norm_mode 0 none, 1 a head (gains [dim]), 2 all of q and all of k each over one root mean square (gains [n_head * dim], [n_kv_head * dim]);
-// the first rot_dims values of a head rotated in pairs (i, i + rot_dims / 2) by positions[t] * freq[i]; with v_first_in the values become
+// the first rot_dims values of a head rotated in pairs (i, i + rot_dims / 2), or, `interleaved`, (2i, 2i + 1), by positions[t] * freq[i]; with v_first_in the values become
 // (1 - lambda) v + lambda v_first_in[t], with v_first_out the row's own values are left there (float [T, n_kv_head * vdim]).
 void qkv_rotary_store(cudaStream_t s, const Rows& proj, const QkvColumns& c, const float* q_weight, const float* k_weight, const Rows& q_out, void* cache,
                       const int32_t* slot_mapping, int n_tokens, int norm_mode, float eps, const int32_t* positions, const float* freq, int rot_dims,
-                      const Rows* v_first_in, const Rows* v_first_out, const float* lambda);
+                      const Rows* v_first_in, const Rows* v_first_out, const float* lambda, bool interleaved = false);
 // out = o over the root mean square of the whole row, times gain (or null), times gate(g) (rows g without data: no gate).
 void row_norm_gate(cudaStream_t s, const Rows& o, const Rows& g, const float* gain, const Rows& out, int n_rows, int gate, float eps);
 // In place over the float rows x[:n_rows]: sigmoid, silu, gelu_tanh or relu (a Gate code).
@@ -265,6 +266,57 @@ void ssm_prepare(cudaStream_t s, const Rows& proj, const float* taps, const floa
 // out = (o + skip_gain[head] * skip) * silu(z) in `groups` equal parts, each over its root mean square, times weight.
 void gated_group_norm(cudaStream_t s, const Rows& o, const Rows* skip, const float* skip_gain, int head, const Rows* z, const float* weight, const Rows& out,
                       int n_rows, int groups, float eps);
+
+// ---- several residual streams ----
+// x: float rows of n_streams parts.  All parts start as the embedded rows; with `reader` the first sublayer's input goes to h (rows of the type `dtype`).
+void streams_open(cudaStream_t s, DType dtype, const Rows& embedded, const Rows& x, int n_streams, int n_rows, const StreamReader* reader, const Rows* h);
+// out[r] = what `reader` makes of the streams of row rows[r] (rows null: of row r).
+void streams_read(cudaStream_t s, DType dtype, const Rows& x, int n_streams, const int32_t* rows, int n_rows, const StreamReader& reader, const Rows& out);
+// The streams take a sublayer's output; with `reader` the next sublayer's input goes to h, and with `router` its rows are routed.
+void streams_join(cudaStream_t s, DType dtype, const Rows& x, const Join& join, const OutputTerms& terms, int n_rows, const StreamReader* reader, const Rows* h,
+                  const RowRouter* router);
+void router_choice(cudaStream_t s, const Rows& h, const RowRouter& router, int n_rows);
+// x (+)= the terms' sum; `dtype`: the type of the terms' own rows (`self`).
+void terms_sum(cudaStream_t s, DType dtype, const OutputTerms& terms, const Rows& x, int n_rows, bool overwrite);
+// The experts' products of a few pairs without a plan (pairs in their own order; a pair whose expert has no matrix is left alone).
+bool expert_product_direct_supports(const Rows& a, const Tensor& w, int n_pairs, int n, int k, bool gated);
+void expert_product_direct(cudaStream_t s, bool gated, const Rows& a, const Tensor& w, int n_experts, const int32_t* ids, const float* weights, const Rows& out,
+                           int n_pairs, int n, int k, int top, int gate, float alpha = 0.0f, float limit = 0.0f);
+
+// ---- a matrix memory per head with a decay per key channel (gated linear attention; the delta rule) ----
+struct ChannelMemoryShape {
+    int n_head = 0, kv_head = 0, dim = 0, vdim = 0, taps = 0, rank = 0, gate_rank = 0, gate = 0;
+    bool delta = false, unit = false;
+    float tau = 0.0f, q_scale = 1.0f, unit_eps = 1e-6f, eps = 1e-6f;
+    const float* conv = nullptr;     // [channels, taps]
+    const float* z_bias = nullptr;   // [n_head dim]
+    const float* a_log = nullptr;    // [n_head]
+    const float* norm = nullptr;     // [vdim]
+    Tensor a2, g2;                   // [n_head dim, rank], [n_head vdim, gate_rank] (g2 without data: the gate's pre-activations are columns)
+    int64_t channels() const { return 2 * static_cast<int64_t>(kv_head) * dim + static_cast<int64_t>(n_head) * vdim; }
+    int64_t memory_floats() const { return static_cast<int64_t>(n_head) * dim * vdim; }
+    int64_t ring_floats() const { return conv != nullptr || taps > 0 ? taps * channels() : 0; }
+    int64_t slot_floats() const { return memory_floats() + ring_floats(); }
+    // Columns of the projection: [q | k | v | the decays' rank | the gate (its rank, or n_head vdim) | the rates (delta)].
+    int64_t a_off() const { return channels(); }
+    int64_t g_off() const { return channels() + rank; }
+    int64_t gate_cols() const { return gate_rank > 0 ? gate_rank : static_cast<int64_t>(n_head) * vdim; }
+    int64_t b_off() const { return g_off() + gate_cols(); }
+    int64_t cols() const { return b_off() + (delta ? n_head : 0); }
+};
+struct ChannelStep {
+    const int32_t* positions = nullptr;
+    const int32_t* tok_seq = nullptr;
+    const int32_t* q_start = nullptr;
+    const int32_t* slots = nullptr;
+    float* state = nullptr;
+    int n_tokens = 0, n_seq = 0;
+    bool decode_only = false;
+};
+// From the float projection to the heads after norm and gate; `o` (float rows, or without data): the heads before them.
+void channel_memory_rows(cudaStream_t s, const ChannelMemoryShape& m, const ChannelStep& step, const Rows& proj, const Rows& o, const Rows& heads);
+// In pieces of 32 rows; `ws` lends the scratch.
+void channel_memory_pieces(cudaStream_t s, Workspace* ws, const ChannelMemoryShape& m, const ChannelStep& step, const Rows& proj, const Rows& o, const Rows& heads);
 
 void sample(cudaStream_t s, const float* logits, int64_t row_stride, int n_rows, int vocab, const float* temperature,
             const int32_t* top_k, const float* top_p, const double* uniform, int32_t* out_ids);

@@ -103,6 +103,10 @@ Registry<PartFactory<TokenInput>>& token_inputs() {
     static Registry<PartFactory<TokenInput>> r("token input");
     return r;
 }
+Registry<PartFactory<Join>>& joins() {
+    static Registry<PartFactory<Join>> r("join");
+    return r;
+}
 Registry<ArrangementFactory>& arrangements() {
     static Registry<ArrangementFactory> r("block arrangement");
     return r;

@@ -68,6 +68,41 @@ struct GroupView {
     const int32_t* slot_mapping = nullptr;       // device int32 [T]
 };
 
+// How a sublayer makes its input from the residual streams: u = sum_s in[s] x_s (in null: ones), then h = tanh(alpha u) * gain + offset where the
+// sublayer's norm is of that kind (alpha null: h = u).  Device pointers.
+struct StreamReader {
+    const float* in = nullptr;
+    const float* alpha = nullptr;
+    const float* gain = nullptr;
+    const float* offset = nullptr;
+};
+
+// A sublayer's output as terms to be summed by whoever joins it to the stream: rows times a number, and routed experts' results gathered row
+// by row (choice k of row t: weights[t top + k] times pairs[place[t top + k]] (place null: pairs[t top + k]), or times self[t] where its expert's
+// number is n_real or more).  At most four rows.
+struct OutputTerms {
+    std::vector<Rows> rows;
+    std::vector<float> scale;
+    Rows pairs, self;
+    const int32_t* place = nullptr;
+    const int32_t* ids = nullptr;
+    const float* weights = nullptr;
+    int top = 0, n_real = 0;
+};
+
+// A router that the launch which makes a feed-forward's input can run on every row: scores over n_experts, the choice by score + correction inside
+// the best groups (see csrc/streams.cu).  Pointers on the device; ids and weights [tokens, top] are its results.
+struct RowRouter {
+    const void* matrix = nullptr;
+    const float* bias = nullptr;
+    const float* correction = nullptr;
+    int n_experts = 0, top = 0, groups = 1, keep = 1;
+    bool softmax = false, renormalise = false;
+    float scale = 1.0f;
+    int32_t* ids = nullptr;
+    float* weights = nullptr;
+};
+
 using TapFn = std::function<void(std::string_view name, const Rows& rows)>;
 
 // Where a step's time goes, by phase, measured with events on the step's stream when asked for (the
@@ -118,6 +153,11 @@ struct StepContext {
     // else changes the stream.
     Rows stream_rounded;
     int stream_rounded_entry = -1;
+    // Models with several residual streams: what the run after this one makes its input from (null for the last run), and that input where the
+    // run before has made it already (for the run numbered `next_input_entry`; -1: nobody did), with the sublayer's last move of the streams.
+    const StreamReader* next_reader = nullptr;
+    Rows next_input;
+    int next_input_entry = -1;
 
     cudaStream_t stream() const { return runtime.stream; }
     // The unit's pages [page, K|V, kv_head, slot, head_dim] and its group's view.
@@ -159,6 +199,8 @@ public:
     // The recipe, where the norm is of that kind; an arrangement may then offer the un-normalised rows and the recipe
     // to the part after the norm (forward_from) and only runs the norm itself where that part declines.
     virtual std::optional<NormRecipe> recipe() const { return std::nullopt; }
+    // Where the norm acts on every value by itself, y = tanh(alpha x) * gain + offset: those three (`in` stays null).
+    virtual std::optional<StreamReader> tanh_recipe() const { return std::nullopt; }
 };
 
 class PositionEncoding : public Part {
@@ -188,6 +230,14 @@ public:
     virtual void forward_from_into(StepContext& ctx, const Rows& x_in, const NormRecipe& norm, const Rows& out, CacheUnit unit) {
         throw internal_error("this mixer does not normalise its input itself");
     }
+    // The mixer's output as terms for the launch that joins it to the streams (`y`: float32 [T, width] for the mixer's use).  By default one: forward_into.
+    virtual OutputTerms forward_terms(StepContext& ctx, const Rows& h, const Rows& y, CacheUnit unit) {
+        forward_into(ctx, h, y, unit);
+        OutputTerms t;
+        t.rows = {y};
+        t.scale = {1.0f};
+        return t;
+    }
 };
 
 class FeedForward : public Part {
@@ -198,6 +248,26 @@ public:
     virtual void forward_into(StepContext& ctx, const Rows& h, const Rows& out);
     // As Mixer::forward_from.
     virtual bool forward_from(StepContext& ctx, const Rows& x_in, const NormRecipe& norm, const Rows& x) { return false; }
+    // As Mixer::forward_terms.  `routed`: the rows' experts have been chosen already, by the launch that made h, with row_router's router.
+    virtual OutputTerms forward_terms(StepContext& ctx, const Rows& h, const Rows& y, bool routed) {
+        forward_into(ctx, h, y);
+        OutputTerms t;
+        t.rows = {y};
+        t.scale = {1.0f};
+        return t;
+    }
+    virtual std::optional<RowRouter> row_router(StepContext& ctx) { return std::nullopt; }
+};
+
+// How a sublayer of a model with several residual streams x_s reads them, u = sum_s in[s] x_s, and how its output y joins them, all at once:
+// x_t <- sum_s mix[s, t] x_s + out[t] * scale * y.  (One learned row of numbers a sublayer.)
+class Join : public Part {
+public:
+    virtual int streams() const = 0;
+    virtual const float* in() const = 0;             // [streams]
+    virtual const float* out() const = 0;            // [streams]
+    virtual const float* mix() const = 0;            // [streams, streams], indexed [from, to]
+    virtual const float* scale() const = 0;          // [width], or null
 };
 
 // A blend of every row of the mixer's input with the row before it in its sequence.  The last row a request brought
@@ -240,6 +310,10 @@ public:
     // State per request that the block keeps beside its mixer's (a token shift's last row); the k-th entry is
     // found at ctx.state(unit.extra_state(k)).
     virtual std::vector<StateNeed> extra_states() const { return {}; }
+    // How many residual streams the block works on; its `x` then holds them one after the other in a row.
+    virtual int streams() const { return 1; }
+    // What the block's first sublayer makes its input from, where the run before may do that for it.
+    virtual std::optional<StreamReader> reader() const { return std::nullopt; }
 };
 
 // -- registries ---------------------------------------------------------------------------------
@@ -286,6 +360,7 @@ Registry<PartFactory<Mixer>>& mixers();
 Registry<PartFactory<FeedForward>>& feed_forwards();
 Registry<PartFactory<Shift>>& shifts();
 Registry<PartFactory<TokenInput>>& token_inputs();
+Registry<PartFactory<Join>>& joins();
 Registry<ArrangementFactory>& arrangements();
 
 // Registers the library's own parts (idempotent; called before any model is built).

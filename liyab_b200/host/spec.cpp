@@ -26,6 +26,7 @@ const char* role_name(Role r) {
         case Role::FeedForward: return "feed_forward";
         case Role::Shift: return "shift";
         case Role::TokenInput: return "token_input";
+        case Role::Join: return "join";
     }
     return "?";
 }
@@ -36,7 +37,8 @@ Role role_from_name(const std::string& name) {
     if (name == "feed_forward") return Role::FeedForward;
     if (name == "shift") return Role::Shift;
     if (name == "token_input") return Role::TokenInput;
-    throw invalid_model("unknown slot role '{}' (norm, mixer, feed_forward, shift or token_input)", name);
+    if (name == "join") return Role::Join;
+    throw invalid_model("unknown slot role '{}' (norm, mixer, feed_forward, shift, token_input or join)", name);
 }
 
 const SlotSpec* LayerSpec::find(const std::string& name) const {
@@ -75,6 +77,7 @@ Json ModelSpec::to_json() const {
         ro.push(entry);
     }
     if (pass_offsets > 0) j.set("pass_offsets", pass_offsets);
+    if (streams != 1) j.set("streams", streams);
     j.set("run_order", ro);
     j.set("final_norm", final_norm.to_json());
     j.set("head", Json::object().set("vocab_size", head.vocab_size).set("size", head.size).set("tied", head.tied)
@@ -111,6 +114,7 @@ ModelSpec ModelSpec::from_json(const Json& j) {
         for (const auto& r : j.at("run_order").items())
             s.run_order.push_back({static_cast<int>(r.at("layer").as_int()), static_cast<int>(r.at("cache").as_int()), static_cast<int>(r.get_int("offset_row", -1))});
         s.pass_offsets = j.get_int("pass_offsets", 0);
+        s.streams = j.get_int("streams", 1);
         s.final_norm = PartSpec::from_json(j.at("final_norm"), "final_norm");
         const Json& h = j.at("head");
         s.head = {h.at("vocab_size").as_int(), h.at("size").as_int(), h.get_bool("tied", true), h.get_bool("bias", false),

@@ -34,8 +34,9 @@ struct PartSpec {
 };
 
 // Shift: a blend of the mixer's input with the row before it (state per request).  TokenInput: an addition to the
-// residual stream made from the step's token ids (a side table), after the block's other parts.
-enum class Role { Norm, Mixer, FeedForward, Shift, TokenInput };
+// residual stream made from the step's token ids (a side table), after the block's other parts.  Join: how a sublayer reads the
+// residual streams of a model that has several, and how its output joins them.
+enum class Role { Norm, Mixer, FeedForward, Shift, TokenInput, Join };
 const char* role_name(Role r);
 Role role_from_name(const std::string& name);
 
@@ -96,6 +97,7 @@ struct ModelSpec {
     PartSpec final_norm;
     HeadSpec head;
     int64_t max_positions = 0;
+    int64_t streams = 1;                 // residual streams of `embedding.size` values a token, all equal to the embedded row at the start, summed at the end
     int64_t pass_offsets = 0;            // rows of the parameter `pass_offsets.weight` (see RunEntry::offset_row); 0: none
     std::optional<int64_t> eos_token_id;
 
