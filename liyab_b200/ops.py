@@ -59,7 +59,7 @@ _SIGNATURES = {
     "lb_decode_attention_mma_sink": [_p, _l, _p, _i, _p, _p, _i, _p, _l, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _p],
     "lb_prefill_attention_sink": [_p, _l, _p, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p, _p],
     "lb_prefill_attention_tc_sink": [_p, _l, _i, _p, _i, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p, _p],
-    "lb_qkv_rotary_store": [_i, _p, _l, _i, _i, _i, _p, _p, _p, _l, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _p, _p, _l, _p, _p],
+    "lb_qkv_rotary_store_layout": [_i, _p, _l, _i, _i, _i, _p, _p, _p, _l, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _p, _p, _l, _p, _i, _p],
     "lb_row_norm_gate": [_i, _p, _l, _p, _l, _p, _p, _l, _i, _i, _i, _f, _p],
     "lb_activate_columns": [_p, _l, _i, _i, _i, _p],
     "lb_router_table": [_p, _p, _p, _p, _i, _i, _i, _i, _p],
@@ -858,16 +858,17 @@ def ssm_prepare(proj: torch.Tensor, xbc_off: int, dt_off: int, taps: torch.Tenso
 def qkv_rotary_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor],
                      q_out: torch.Tensor, cache: Optional[torch.Tensor], slot_mapping: torch.Tensor, n_head: int, n_kv_head: int, dim: int, vdim: int,
                      padded: int, page_size: int, norm_mode: int, eps: float, positions: torch.Tensor, freq: Optional[torch.Tensor], rot_dims: int,
-                     v_first_in: Optional[torch.Tensor] = None, v_first_out: Optional[torch.Tensor] = None, blend: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     v_first_in: Optional[torch.Tensor] = None, v_first_out: Optional[torch.Tensor] = None, blend: Optional[torch.Tensor] = None,
+                     interleaved: bool = False) -> torch.Tensor:
     """Queries, keys and values of a float projection on their way to attention: norm_mode 0 none, 1 a head, 2 the whole projection; the first
-    rot_dims values of every head rotated by positions[t] * freq[i]; values blended with v_first_in by blend[0], or left in v_first_out."""
+    rot_dims values of every head rotated by positions[t] * freq[i] (pairs (i, i + rot_dims / 2), or `interleaved` (2i, 2i + 1)); values blended with v_first_in by blend[0], or left in v_first_out."""
     shared = v_first_in if v_first_in is not None else v_first_out
-    check(lib().lb_qkv_rotary_store(_code(q_out.dtype, "q_out"), _dev(proj, "proj", torch.float32), proj.stride(0), q_off, k_off, v_off,
+    check(lib().lb_qkv_rotary_store_layout(_code(q_out.dtype, "q_out"), _dev(proj, "proj", torch.float32), proj.stride(0), q_off, k_off, v_off,
                                     _opt(q_weight, "q_weight", torch.float32), _opt(k_weight, "k_weight", torch.float32), _dev(q_out, "q_out"), q_out.stride(0),
                                     _opt(cache, "cache", q_out.dtype), _dev(slot_mapping, "slot_mapping", torch.int32), proj.shape[0], n_head, n_kv_head, dim, vdim,
                                     padded, page_size, norm_mode, float(eps), _dev(positions, "positions", torch.int32), _opt(freq, "freq", torch.float32), rot_dims,
                                     _opt(v_first_in, "v_first_in", torch.float32), _opt(v_first_out, "v_first_out", torch.float32),
-                                    shared.stride(0) if shared is not None else 0, _opt(blend, "blend", torch.float32), stream_ptr()), "qkv_rotary_store")
+                                    shared.stride(0) if shared is not None else 0, _opt(blend, "blend", torch.float32), int(interleaved), stream_ptr()), "qkv_rotary_store")
     return q_out
 
 
@@ -894,3 +895,126 @@ def router_table(tokens: torch.Tensor, table: torch.Tensor, n_experts: int):
     check(lib().lb_router_table(_dev(tokens, "tokens", torch.int32), _dev(table, "table", torch.int32), _dev(ids, "ids"), _dev(weights, "weights"), T, top,
                                 n_experts, table.shape[0], stream_ptr()), "router_table")
     return ids, weights
+
+
+# ------------------------------------------------------------------ several residual streams, corrected routers, memories with a decay per channel
+
+class OutputTerms(ctypes.Structure):
+    _fields_ = [("n_rows", _i), ("y", _p * 4), ("ldy", _l * 4), ("scale", _f * 4), ("pairs", _p), ("ldp", _l), ("place", _p), ("ids", _p), ("weights", _p),
+                ("top", _i), ("n_real", _i), ("self_rows", _p), ("lds", _l)]
+
+
+class Router(ctypes.Structure):
+    _fields_ = [("matrix", _p), ("bias", _p), ("correction", _p), ("n_experts", _i), ("top", _i), ("groups", _i), ("keep", _i), ("softmax", _i), ("renormalise", _i),
+                ("scale", _f), ("ids", _p), ("weights", _p)]
+
+
+class StreamsArgs(ctypes.Structure):
+    _fields_ = [("x", _p), ("ldx", _l), ("fresh", _p), ("ldf", _l), ("rows", _p), ("n_streams", _i), ("width", _i), ("mix", _p), ("to", _p), ("scale", _p),
+                ("next_in", _p), ("alpha", _p), ("gain", _p), ("offset", _p), ("h", _p), ("ldh", _l)]
+
+
+class ChannelMemoryArgs(ctypes.Structure):
+    _fields_ = [("n_head", _i), ("kv_head", _i), ("dim", _i), ("vdim", _i), ("delta", _i), ("taps", _i), ("unit", _i), ("rank", _i), ("gate_rank", _i),
+                ("gate_act", _i), ("a_off", _i), ("g_off", _i), ("b_off", _i), ("conv", _p), ("a2", _p), ("g2", _p), ("z_bias", _p), ("a_log", _p), ("norm", _p),
+                ("tau", _f), ("q_scale", _f), ("unit_eps", _f), ("eps", _f), ("slot_stride", _l)]
+
+
+class ChannelStepArgs(ctypes.Structure):
+    _fields_ = [("proj", _p), ("ld", _l), ("positions", _p), ("tok_seq", _p), ("q_start", _p), ("slots", _p), ("state", _p), ("o", _p), ("ldo", _l), ("heads", _p),
+                ("ldh", _l)]
+
+
+declare("lb_streams_join", [_i, _p, _p, _p, _i, _p])
+declare("lb_router_choice", [_i, _p, _p, _l, _i, _i, _p])
+declare("lb_terms_sum", [_i, _p, _p, _l, _i, _i, _i, _p])
+declare("lb_expert_product_direct", [_i, _i, _p, _l, _p, _l, _p, _p, _p, _l, _i, _i, _i, _i, _i, _i, _f, _f, _p])
+declare("lb_channel_memory_rows", [_i, _p, _p, _i, _i, _p])
+declare("lb_channel_memory_pieces", [_i, _p, _p, _p, _p, _p, _p, _i, _i, _p])
+
+
+def output_terms(rows=(), scale=(), pairs: Optional[torch.Tensor] = None, place: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
+                 weights: Optional[torch.Tensor] = None, n_real: int = 0, self_rows: Optional[torch.Tensor] = None) -> OutputTerms:
+    """A sublayer's output as the launch that joins it reads it: rows times numbers, and routed experts' results gathered row by row."""
+    o = OutputTerms()
+    o.n_rows = len(rows)
+    for k, (y, s) in enumerate(zip(rows, scale)):
+        o.y[k], o.ldy[k], o.scale[k] = _dev(y, "y", torch.float32), y.stride(0), float(s)
+    if pairs is not None:
+        o.pairs, o.ldp, o.place, o.ids = _dev(pairs, "pairs", torch.float32), pairs.stride(0), _opt(place, "place", torch.int32), _dev(ids, "ids", torch.int32)
+        o.weights, o.top, o.n_real = _opt(weights, "weights", torch.float32), ids.shape[1], n_real
+        if self_rows is not None:
+            o.self_rows, o.lds = _dev(self_rows, "self_rows"), self_rows.stride(0)
+    return o
+
+
+def router_args(matrix: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.Tensor, bias: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None,
+           groups: int = 1, keep: int = 1, softmax: bool = True, renormalise: bool = False, scale: float = 1.0) -> Router:
+    return Router(_dev(matrix, "matrix"), _opt(bias, "bias", torch.float32), _opt(correction, "correction", torch.float32), matrix.shape[0], top, groups, keep,
+                  int(softmax), int(renormalise), float(scale), _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32))
+
+
+def streams_join(x: torch.Tensor, n_streams: int, n_rows: int, terms: Optional[OutputTerms] = None, mix: Optional[torch.Tensor] = None,
+                 to: Optional[torch.Tensor] = None, scale: Optional[torch.Tensor] = None, fresh: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+                 next_in: Optional[torch.Tensor] = None, norm=None, h: Optional[torch.Tensor] = None, router: Optional[Router] = None) -> None:
+    """The streams x [rows, n_streams * width] between two sublayers (csrc/streams.cu); norm: (alpha, gain, offset) of the sublayer that begins."""
+    f32 = torch.float32
+    alpha, gain, offset = norm if norm is not None else (None, None, None)
+    a = StreamsArgs(_dev(x, "x", f32), x.stride(0), _opt(fresh, "fresh", f32), fresh.stride(0) if fresh is not None else 0, _opt(rows, "rows", torch.int32), n_streams,
+                    x.shape[1] // n_streams, _opt(mix, "mix", f32), _opt(to, "to", f32), _opt(scale, "scale", f32), _opt(next_in, "next_in", f32),
+                    _opt(alpha, "alpha", f32), _opt(gain, "gain", f32), _opt(offset, "offset", f32), _opt(h, "h"), h.stride(0) if h is not None else 0)
+    check(lib().lb_streams_join(_code(h.dtype, "h") if h is not None else F32, _c.byref(a), _c.byref(terms) if terms is not None else None,
+                                _c.byref(router) if router is not None else None, n_rows, stream_ptr()), "streams_join")
+
+
+def router_choice(r: Router, h: torch.Tensor) -> None:
+    check(lib().lb_router_choice(_code(h.dtype, "h"), _c.byref(r), _dev(h, "h"), h.stride(0), h.shape[0], h.shape[1], stream_ptr()), "router_choice")
+
+
+def terms_sum(terms: OutputTerms, x: torch.Tensor, dtype: torch.dtype, overwrite: bool) -> torch.Tensor:
+    check(lib().lb_terms_sum(_code(dtype, "self"), _c.byref(terms), _dev(x, "x", torch.float32), x.stride(0), x.shape[0], x.shape[1], int(overwrite), stream_ptr()),
+          "terms_sum")
+    return x
+
+
+def experts_direct(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, gate: str = "silu") -> torch.Tensor:
+    """Every pair's result [T * top, width] without a plan (a few pairs, bfloat16); gate_up [E, 2 F, width], down [E, width, F].  Pairs whose expert is not
+    one of the E stay NaN."""
+    T, top = ids.shape
+    E, F2, width = gate_up.shape
+    mid = torch.full((T * top, F2 // 2), float("nan"), dtype=h.dtype, device=h.device)
+    out = torch.full((T * top, width), float("nan"), dtype=torch.float32, device=h.device)
+    for gated, a, w, o, n, k in ((1, h, gate_up, mid, F2 // 2, width), (0, mid, down, out, width, F2 // 2)):
+        check(lib().lb_expert_product_direct(_code(h.dtype, "h"), gated, _dev(a, "a"), a.stride(0), _dev(w, "w", h.dtype), w.stride(0), _dev(ids, "ids", torch.int32), None,
+                                             _dev(o, "o"), o.stride(0), T * top, E, n, k, top, GATE_KINDS[gate], 0.0, 0.0, stream_ptr()), "expert_product_direct")
+    return out
+
+
+def channel_memory(m: dict, proj: torch.Tensor, positions: torch.Tensor, tok_seq: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, state: torch.Tensor,
+                   heads: torch.Tensor, o: Optional[torch.Tensor], pieces: bool, decode_only: bool = False) -> torch.Tensor:
+    """A memory per head with a decay per channel (csrc/channel_memory.cu) over the float projection rows [q | k | v | decays' rank | gate | rates].  m: n_head,
+    kv_head, dim, vdim, delta, taps, unit, gate ("silu", "sigmoid"), a2, g2 (or None), conv (or None), z_bias, a_log (or None), tau, norm, q_scale, eps."""
+    f32 = torch.float32
+    H, G, D, E = m["n_head"], m["kv_head"], m["dim"], m["vdim"]
+    rank, gate_rank = m["a2"].shape[1], m["g2"].shape[1] if m["g2"] is not None else 0
+    channels = 2 * G * D + H * E
+    g_off = channels + rank
+    b_off = g_off + (gate_rank if gate_rank else H * E)
+    a = ChannelMemoryArgs(H, G, D, E, int(m["delta"]), m["taps"], int(m["unit"]), rank, gate_rank, {"sigmoid": 0, "silu": 1}[m["gate"]], channels, g_off, b_off,
+                          _opt(m["conv"], "conv", f32), _dev(m["a2"], "a2", heads.dtype), _opt(m["g2"], "g2", heads.dtype), _opt(m["z_bias"], "z_bias", f32),
+                          _opt(m["a_log"], "a_log", f32), _dev(m["norm"], "norm", f32), float(m["tau"]), float(m["q_scale"]), 1e-6, float(m["eps"]), state.stride(0))
+    i32 = torch.int32
+    s = ChannelStepArgs(_dev(proj, "proj", f32), proj.stride(0), _dev(positions, "positions", i32), _dev(tok_seq, "tok_seq", i32), _dev(q_start, "q_start", i32),
+                        _dev(slots, "slots", i32), _dev(state, "state", f32), _opt(o, "o", f32), o.stride(0) if o is not None else 0, _dev(heads, "heads"),
+                        heads.stride(0))
+    T, S, code = proj.shape[0], q_start.numel() - 1, _code(heads.dtype, "heads")
+    if not pieces:
+        check(lib().lb_channel_memory_rows(code, _c.byref(a), _c.byref(s), S, int(decode_only), stream_ptr()), "channel_memory_rows")
+        return heads
+    fn = lib().lb_channel_memory_pieces_floats
+    fn.argtypes, fn.restype = [_i, _i, _i, _i, _i, _i], _l
+    scratch = torch.full((fn(T, S, H, D, E, int(m["delta"])),), float("nan"), device=proj.device)
+    rows, decay, gate = (torch.full((T, n), float("nan"), device=proj.device) for n in (channels, H * D, H * E))
+    check(lib().lb_channel_memory_pieces(code, _c.byref(a), _c.byref(s), _dev(rows, "rows"), _dev(decay, "decay"), _dev(gate, "gate"), _dev(scratch, "scratch"), T, S,
+                                         stream_ptr()), "channel_memory_pieces")
+    return heads
