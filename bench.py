@@ -7,6 +7,7 @@
     python bench.py --design vosurax [--size small]   # Vosurax likewise (see vosurax_line)
     python bench.py --design viresun [--size small]   # Viresun beside Vosurax and GPT-2 (see viresun_line)
     python bench.py --design revudra [--size small]   # Revudra beside Vosurax and GPT-2 (see revudra_line)
+    python bench.py --design mokisun [--size small]   # Mokisun beside Vosurax and GPT-2 (see mokisun_line)
 
 A step is one decode step of the whole batch.  The default run has the layer
 sizes of GPT-2 small (12 layers, width 768, 12 heads) with random weights, a batch of
@@ -601,6 +602,92 @@ def revudra_line(args) -> int:
     return 0
 
 
+def mokisun_config(size, layers=0):
+    """Mokisun with the width, depth, head count, inner width and vocabulary of a GPT-2 size.  Of every four blocks the first is gated linear
+    attention (heads of 64 x 64), the second attention under a window of 512 (heads of 64, a quarter as many key/value heads, half of a head rotated), the
+    others a pair: attention over keys alone under a window of 512 (heads of 64, a quarter as many key/value heads) beside a gated delta rule (half as many
+    heads, 64 / 128 values, four taps); 16 experts of a quarter of the inner width and two identities in two groups, two a token of the better group; two
+    streams."""
+    g = SIZES[size]
+    L, W, H = max(4, layers or g["n_layer"]), g["n_embd"], g["n_head"]
+    kv, half = max(1, H // 4), max(1, H // 2)
+    gla = dict(heads=H, dim=64, vdim=64, tau=16.0, a_rank=16)
+    attn = dict(heads=H, kv_heads=kv, dim=64, vdim=64, scale=0.125, mask=dict(size=512), rot=dict(base=1e5, dims=32))
+    pair = dict(left=dict(heads=H, kv_heads=kv, dim=64, vdim=64, scale=0.125, mask=dict(size=512)),
+                right=dict(heads=half, kv_heads=half, dim=64, vdim=128, conv=4, a_rank=32, g_rank=32), left_scale=1.0, right_scale=1.0)
+    moe = dict(kind="moe", expert=dict(ff=g["n_inner"] // 4), router=dict(experts=16, top=2, identity=2, scale=2.0, groups=dict(count=2, keep=1)))
+    kinds = [("gla", gla), ("attention", attn), ("parallel", pair), ("parallel", pair)]
+    return dict(architecture="Mokisun", vocab=g["vocab_size"], width=W, streams=2, norm=dict(eps=1e-5), max_positions=g["n_positions"],
+                layers=[dict(type=kinds[i % 4][0], mixer=kinds[i % 4][1], mlp=moe) for i in range(L)])
+
+
+def mokisun_bytes_and_flops(cfg, dtype_bytes, batch):
+    """Bytes a decode step of `batch` requests must read (weights its rows touch, memories read and written, visible cache rows) and the FLOPs of a
+    prefill (products with the weights a token uses, attention inside its window, the memories' updates and reads: 4 D E a token and head, and 2 D E more for
+    what the delta rule reads before it writes).  An even router sends top / 18 of the pairs to each of the 16 experts and two identities."""
+    W, V = cfg["width"], cfg["vocab"]
+    step_bytes, token_flops, attn, mem = 2 * V * W * dtype_bytes, 2 * V * W, [], []
+    for l in cfg["layers"]:
+        m, mlp = l["mixer"], l["mlp"]
+        mats = 0
+        if l["type"] == "gla":
+            H, D, E = m["heads"], m["dim"], m["vdim"]
+            mats = W * (2 * H * D + 2 * H * E + m["a_rank"]) + m["a_rank"] * H * D + W * H * E
+            mem.append((H, D, E, 4, 0))
+        else:
+            a = m if l["type"] == "attention" else m["left"]
+            H, G, D, E = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            mats = W * (H * D + G * (D + (E if l["type"] == "attention" else 0))) + W * H * E
+            attn.append((H, G, D, E, a["mask"]["size"], 2 if l["type"] == "attention" else 1))
+            if l["type"] == "parallel":
+                r = m["right"]
+                H, G, D, E = r["heads"], r["kv_heads"], r["dim"], r["vdim"]
+                mats += W * (2 * G * D + H * E + r["a_rank"] + r["g_rank"] + H) + r["a_rank"] * H * D + r["g_rank"] * H * E + W * H * E
+                mem.append((H, D, E, 6, r["conv"] * (2 * G * D + H * E)))
+        router, F = mlp["router"], mlp["expert"]["ff"]
+        X, N, top = router["experts"], router["experts"] + router["identity"], router["top"]
+        token_flops += 2 * (mats + N * W + 3 * W * F * top * X / N)
+        step_bytes += (mats + N * W + 3 * W * F * X * (1.0 - (1.0 - top / N) ** batch)) * dtype_bytes      # the experts a batch is expected to touch
+    state_bytes = sum(2 * 4 * H * D * E + 4 * ring for H, D, E, _, ring in mem)
+    cache_row_bytes = [dtype_bytes * planes * G * max(D, E) for _, G, D, E, _, planes in attn]
+
+    def decode_bytes(mean_context):
+        return step_bytes + batch * (state_bytes + sum(b * min(mean_context, a[4]) for b, a in zip(cache_row_bytes, attn)))
+
+    def prefill_flops(seq_lens, rows):
+        total = sum(seq_lens) * (token_flops - 2 * V * W) + 2 * rows * V * W
+        for H, G, D, E, c, _ in attn:
+            total += sum(2 * H * (D + E) * sum(min(i + 1, c) for i in range(s)) for s in seq_lens)
+        for H, D, E, f, _ in mem:
+            total += sum(seq_lens) * f * H * D * E
+        return total
+
+    return decode_bytes, prefill_flops
+
+
+def mokisun_line(args) -> int:
+    """--design mokisun: decode (batch 1 / 8 / 64, 512-token prompts) and prefill (2 x 1024 tokens) of Mokisun at the layer sizes of GPT-2 `--size`, and the
+    same four figures of Vosurax (the engine's closest design: attention under a mask beside a matrix memory per head with gates, routed experts) and of GPT-2 at
+    that size."""
+    from liyab_b200.weights import write_random_model
+    pk = peaks()
+    dtype_bytes = 2 if args.dtype == "bfloat16" else 4
+    cfg = mokisun_config(args.size, args.layers)
+    steps = min(args.steps, 128)
+    out = {"design": "mokisun", "size": args.size, "dtype": args.dtype, "peaks": pk["source"],
+           "config": {k: cfg[k] for k in ("width", "vocab", "streams")} | {"layers": len(cfg["layers"])} | {l["type"]: l["mixer"] for l in cfg["layers"]} |
+                     {"experts": cfg["layers"][0]["mlp"]}}
+    with tempfile.TemporaryDirectory(prefix="liyab_b200_bench_") as tmp:
+        folder = write_random_model(os.path.join(tmp, "mokisun"), cfg, seed=0, dtype=args.dtype)
+        out["mokisun"] = design_block(folder, args.dtype, steps, pk, lambda b: mokisun_bytes_and_flops(cfg, dtype_bytes, b))
+        other = vosurax_config(args.size, args.layers + 2 if args.layers else 0)
+        folder = write_random_model(os.path.join(tmp, "vosurax"), other, seed=0, dtype=args.dtype)
+        out["vosurax"] = design_block(folder, args.dtype, steps, pk, lambda b: vosurax_bytes_and_flops(other, dtype_bytes, b))
+        if not args.layers:
+            out["gpt2"], _ = size_block(tmp, args.size, args.dtype, steps, pk)
+    print(json.dumps(out))
+    return 0
+
 
 def reference_arm(args) -> int:
     from baseline.reference_arm import run
@@ -619,8 +706,8 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-points", action="store_true", help="the headline figure only")
     ap.add_argument("--no-extra", action="store_true", help="skip the 32-bit engine, the other sizes and the mixed workload")
-    ap.add_argument("--design", default="gpt2", choices=["gpt2", "puzutar", "vosurax", "viresun", "revudra"],
-                    help="puzutar, vosurax, viresun, revudra: that design at the layer sizes of GPT-2 --size beside GPT-2 itself (its own JSON line; the default run is unchanged)")
+    ap.add_argument("--design", default="gpt2", choices=["gpt2", "puzutar", "vosurax", "viresun", "revudra", "mokisun"],
+                    help="puzutar, vosurax, viresun, revudra, mokisun: that design at the layer sizes of GPT-2 --size beside GPT-2 itself (its own JSON line; the default run is unchanged)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
@@ -632,6 +719,8 @@ def main() -> int:
         return viresun_line(args)
     if args.design == "revudra":
         return revudra_line(args)
+    if args.design == "mokisun":
+        return mokisun_line(args)
     if args.gpus != 1:
         print(f"bench.py measures a single-GPU engine; --gpus {args.gpus} is not supported (run with --gpus 1)")
         return 2
