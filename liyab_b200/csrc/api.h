@@ -615,11 +615,9 @@ typedef struct lb_channel_step {
 } lb_channel_step;
 /* Row by row; decode_only: every request brings one row (the convolution's inputs then enter the state in the same launch). */
 int lb_channel_memory_rows(int dtype, const lb_channel_memory* memory, const lb_channel_step* step, int n_seq, int decode_only, void* stream);
-/* In pieces of 32 rows.  Scratch: rows [T, channels] (with a convolution or unit vectors), log_decay [T, n_head dim], gate [T, n_head vdim] (with g2) and
- * lb_channel_memory_pieces_floats(..) floats. */
+/* In pieces of 32 rows; scratch: lb_channel_memory_pieces_floats(..) floats. */
 int64_t lb_channel_memory_pieces_floats(int n_tokens, int n_seq, int n_head, int dim, int vdim, int delta);
-int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memory, const lb_channel_step* step, float* rows, float* log_decay, float* gate,
-                             float* scratch, int n_tokens, int n_seq, void* stream);
+int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memory, const lb_channel_step* step, float* scratch, int n_tokens, int n_seq, void* stream);
 
 #ifdef __cplusplus
 }

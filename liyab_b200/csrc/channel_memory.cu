@@ -22,7 +22,8 @@
 //     so U = M V - (M K~) S0 with M = (I + diag(beta) A)^-1 diag(beta), a triangular solve of the piece alone;
 //     o_t = S0^T (exp(b_t) q_t) + sum_{j <= t} P(t, j) u_j,      S1 = diag(exp(b_n)) S0 + sum_j (exp(b_n - b_j) k_j) u_j^T.
 // Every exponent is at most 0 (the pairs' exponentials are made pair by pair), so a strong decay underflows to zero and nothing overflows.
-// Launches: the low-rank maps, the convolution, the pieces' own matrices, the scan over a request's pieces, the outputs with norm and gate.
+// Pairs of a row of a piece's second half with a key of its first meet at the border between them (two factors, each at most 1).
+// Launches: the pieces' own matrices (convolution, unit vectors and decays included), the scan over a request's pieces, the outputs with norm and gate.
 #include "api.h"
 #include "common.cuh"
 
@@ -231,83 +232,6 @@ __global__ void __launch_bounds__(256) channel_ring_kernel(lb_channel_memory m, 
     for (int row = max(row0, row1 - m.taps); row < row1; ++row) ring[(size_t)(a.positions[row] % m.taps) * channels + c] = a.proj[(size_t)row * a.ld + c];
 }
 
-// ---------------------------------------------------------------- a low-rank map over many rows
-// out[t, c] = f(sum_r x[t, r] w[c, r] + bias[c]): the decays' logarithms (base 2), or the map alone (a gate's pre-activations).  32 rows x 64 columns
-// a block, a thread 2 x 4 of them.
-template <typename T, bool DECAY>
-__global__ void __launch_bounds__(256) low_rank_kernel(lb_channel_memory m, const float* __restrict__ x, int64_t ldx, const T* __restrict__ w, int rank,
-                                                       float* __restrict__ out, int64_t ldo, int n_rows, int n_cols) {
-    __shared__ float xs[32][33];
-    __shared__ float ws[32][65];
-    const int t0 = blockIdx.y * 32, c0 = blockIdx.x * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-    lb_wait_for_predecessor();
-    lb_dependents_may_launch();
-    float acc[2][4] = {};
-    for (int r0 = 0; r0 < rank; r0 += 32) {
-        for (int i = threadIdx.x; i < 32 * 32; i += 256) {
-            const int t = i >> 5, r = i & 31;
-            xs[t][r] = t0 + t < n_rows && r0 + r < rank ? x[(size_t)(t0 + t) * ldx + r0 + r] : 0.0f;
-        }
-        for (int i = threadIdx.x; i < 64 * 32; i += 256) {
-            const int c = i >> 5, r = i & 31;
-            ws[r][c] = c0 + c < n_cols && r0 + r < rank ? lb_to_float(w[(size_t)(c0 + c) * rank + r0 + r]) : 0.0f;
-        }
-        __syncthreads();
-        const int n = min(32, rank - r0);
-        for (int r = 0; r < n; ++r) {
-            const float a0 = xs[ty][r], a1 = xs[ty + 16][r];
-#pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const float b = ws[r][tx + 16 * j];
-                acc[0][j] = fmaf(a0, b, acc[0][j]);
-                acc[1][j] = fmaf(a1, b, acc[1][j]);
-            }
-        }
-        __syncthreads();
-    }
-#pragma unroll
-    for (int i = 0; i < 2; ++i)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const int t = t0 + ty + 16 * i, c = c0 + tx + 16 * j;
-            if (t >= n_rows || c >= n_cols) continue;
-            float z = acc[i][j];
-            if (DECAY) {
-                if (m.z_bias != nullptr) z += m.z_bias[c];
-                z = cm_log2_decay(m, z, c / m.dim);
-            }
-            out[(size_t)t * ldo + c] = z;
-        }
-}
-
-// ---------------------------------------------------------------- convolution, SiLU and unit vectors over many rows
-// A block per row, a warp per query, key or value head: [q | k | v] as the recurrence reads them (queries without their factor).
-__global__ void __launch_bounds__(256) channel_prepare_kernel(lb_channel_memory m, StepArgs a, float* __restrict__ out, int64_t ldo) {
-    lb_wait_for_predecessor();
-    lb_dependents_may_launch();
-    const int row = blockIdx.x, seq = a.tok_seq[row], row0 = a.q_start[seq], pos = a.positions[row], channels = channels_of(m);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
-    const float* ring = a.state + (size_t)a.slots[seq] * m.slot_stride + (size_t)m.n_head * m.dim * m.vdim;
-    for (int job = blockIdx.y * n_warps + warp; job < 2 * m.kv_head + m.n_head; job += gridDim.y * n_warps) {
-        const bool is_v = job >= 2 * m.kv_head;
-        const int size = is_v ? m.vdim : m.dim, first = is_v ? 2 * m.kv_head * m.dim + (job - 2 * m.kv_head) * m.vdim : job * m.dim;
-        float held[8];
-        float ss = 0.0f;
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int c = lane + 32 * i;
-            held[i] = c < size ? conv_channel(m, a, ring, first + c, row, row0, pos, channels) : 0.0f;
-            ss = fmaf(held[i], held[i], ss);
-        }
-        const float f = m.unit && !is_v ? 1.0f / sqrtf(lb_warp_sum(ss) + m.unit_eps) : 1.0f;
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int c = lane + 32 * i;
-            if (c < size) out[(size_t)row * ldo + first + c] = held[i] * f;
-        }
-    }
-}
-
 // ---------------------------------------------------------------- pieces of 32 rows
 struct PieceLayout {
     int64_t p, q, keep, b, w, u, s, total;      // floats from the start of a (piece, head)'s scratch
@@ -321,8 +245,8 @@ __host__ __device__ inline PieceLayout piece_layout(int D, int E, int delta) {
     l.q = take(kPiece * D);                     // exp(b_t) q_t
     l.keep = take(D);                           // exp(b_n)
     l.b = take(delta ? kPiece * D : 0);         // exp(b_n - b_j) k_j
-    l.w = take(delta ? kPiece * D : 0);         // M K~
-    l.u = take(delta ? kPiece * E : 0);         // M V; after the scan U
+    l.w = take(delta ? kPiece * D : 0);         // M K~, transposed: [D][32]
+    l.u = take(kPiece * E);                     // V, or under the delta rule M V and after the scan U
     l.s = take((int64_t)D * E);                 // without the delta rule the piece's own sum; after the scan the state before the piece
     l.total = at;
     return l;
@@ -342,18 +266,6 @@ __device__ __forceinline__ bool find_piece(const int32_t* q_start, int n_seq, in
     return false;
 }
 
-struct PieceArgs {
-    const float* q;            // [T, ldq] query, key and value rows (column blocks of one buffer)
-    const float* k;
-    const float* v;
-    int64_t ldq;
-    const float* log_decay;    // [T, ldd] base 2
-    int64_t ldd;
-    const float* gate;         // [T, ldg] the gate's pre-activations
-    int64_t ldg;
-    float* scratch;            // [pieces][heads][piece_layout.total]
-};
-
 // y[t][x] = sum_j m[t][j] v[j][x] for 8 rows t0 .. t0 + 7 of one column (m [32][36] lower triangular, v column x at stride ldv).
 __device__ __forceinline__ void tri_product(float (&y)[8], const float* m, const float* v, int ldv, int t0) {
 #pragma unroll
@@ -368,46 +280,132 @@ __device__ __forceinline__ void tri_product(float (&y)[8], const float* m, const
     }
 }
 
-template <bool DELTA>
-__global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m, StepArgs a, PieceArgs w, int n_seq) {
+// z[t][x] for eight rows t0 .. of column x: sum over a chunk of up to 32 of the rank; xT [32 r][36] holds the rows' inputs, w the column's weights.
+__device__ __forceinline__ void rank_chunk(float (&z)[8], const float* xT, const float* w, int t0, int n) {
+    for (int r = 0; r < n; ++r) {
+        const float4 lo = *reinterpret_cast<const float4*>(xT + r * 36 + t0), hi = *reinterpret_cast<const float4*>(xT + r * 36 + t0 + 4);
+        const float v = w[r];
+        z[0] = fmaf(v, lo.x, z[0]); z[1] = fmaf(v, lo.y, z[1]); z[2] = fmaf(v, lo.z, z[2]); z[3] = fmaf(v, lo.w, z[3]);
+        z[4] = fmaf(v, hi.x, z[4]); z[5] = fmaf(v, hi.y, z[5]); z[6] = fmaf(v, hi.z, z[6]); z[7] = fmaf(v, hi.w, z[7]);
+    }
+}
+// A chunk of a low-rank map's operands: xT[r][t] = x[row0 + t][r0 + r] (zeros past the piece), w[c][r] = map[c][r0 + r] at stride 33.
+template <typename T>
+__device__ __forceinline__ void load_rank_chunk(float* xT, float* ws, const float* __restrict__ x, int64_t ldx, const T* __restrict__ map, int rank, int r0, int n_rows,
+                                                int n_cols) {
+    const int n = min(32, rank - r0);
+    for (int i = threadIdx.x; i < 32 * 32; i += blockDim.x) {
+        const int t = i >> 5, r = i & 31;
+        xT[r * 36 + t] = t < n_rows && r < n ? x[(size_t)t * ldx + r0 + r] : 0.0f;
+    }
+    for (int i = threadIdx.x; i < n_cols * 32; i += blockDim.x) {
+        const int c = i >> 5, r = i & 31;
+        if (r < n) ws[c * 33 + r] = lb_to_float(map[(size_t)c * rank + r0 + r]);
+    }
+}
+
+__device__ __forceinline__ float fast_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// A piece's own matrices, from the projection's rows on: convolution, unit vectors and decays, the pairs' products, the triangle's solution.
+template <typename T, bool DELTA>
+__global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m, StepArgs a, float* __restrict__ scratch, int n_seq) {
     extern __shared__ __align__(16) float smem[];
     lb_wait_for_predecessor();
     lb_dependents_may_launch();
     int seq, piece;
     if (!find_piece(a.q_start, n_seq, blockIdx.x, &seq, &piece)) return;
-    const int h = blockIdx.y, D = m.dim, E = m.vdim, LD = D + 1, LE = E + 1, g = h / (m.n_head / m.kv_head);
-    const int row0 = a.q_start[seq] + piece * kPiece, n = min(kPiece, a.q_start[seq + 1] - row0);
+    const int h = blockIdx.y, D = m.dim, E = m.vdim, LD = D + 1, LE = E + 1, g = h / (m.n_head / m.kv_head), channels = channels_of(m);
+    const int first = a.q_start[seq], row0 = first + piece * kPiece, n = min(kPiece, a.q_start[seq + 1] - row0), pos0 = a.positions[row0];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    float* Am = smem;                          // [32][36]
+    float* Am = smem;                          // [32][36]; before the pairs the decays' inputs [32 r][36]
     float* M = Am + kPiece * 36;               // [32][36]
     float* beta = M + kPiece * 36;             // [32]
     float* qs = beta + kPiece;                 // [32][LD]
     float* ks = qs + kPiece * LD;              // [32][LD]
     float* bs = ks + kPiece * LD;              // [32][LD] log decays, then their running sums
     float* vs = bs + kPiece * LD;              // [32][LE]
+    float* fs = vs + kPiece * LE;              // [48][LD] rows with one half of a pair's exponential; before that the decays' map [D][33]
     const PieceLayout l = piece_layout(D, E, DELTA);
-    float* out = w.scratch + ((size_t)blockIdx.x * m.n_head + h) * l.total;
-    for (int t = warp; t < kPiece; t += 8) {
-        const bool in = t < n;
-        const size_t row = (size_t)(row0 + (in ? t : 0));
-        for (int d = lane; d < D; d += 32) {
-            if (in) {
-                cm_cp_async4(qs + t * LD + d, w.q + row * w.ldq + g * D + d);
-                cm_cp_async4(ks + t * LD + d, w.k + row * w.ldq + g * D + d);
-                cm_cp_async4(bs + t * LD + d, w.log_decay + row * w.ldd + h * D + d);
-            } else {
-                qs[t * LD + d] = ks[t * LD + d] = bs[t * LD + d] = 0.0f;
+    float* out = scratch + ((size_t)blockIdx.x * m.n_head + h) * l.total;
+    const float* slot = a.state + (size_t)a.slots[seq] * m.slot_stride;
+    const float* ring = slot + (size_t)m.n_head * D * E;
+    // Queries, keys and values: eight rows of a channel an item, the convolution's earlier inputs in registers.
+    for (int i = threadIdx.x; i < 4 * (2 * D + E); i += blockDim.x) {
+        const int part = i / (2 * D + E), x = i - part * (2 * D + E), t0 = 8 * part;
+        const int c = x < D ? g * D + x : x < 2 * D ? (m.kv_head + g) * D + (x - D) : 2 * m.kv_head * D + h * E + (x - 2 * D);
+        float* dst = x < D ? qs + x : x < 2 * D ? ks + (x - D) : vs + (x - 2 * D);
+        const int ld = x < 2 * D ? LD : LE;
+        const float* col = a.proj + (size_t)row0 * a.ld + c;
+        auto input = [&](int t) -> float {     // the channel's input at row row0 + t: of this step, of an earlier one, or before the start
+            if (row0 + t >= first) return t < n ? col[(int64_t)t * a.ld] : 0.0f;
+            const int p = pos0 + t;
+            return p >= 0 ? ring[(size_t)(p % m.taps) * channels + c] : 0.0f;
+        };
+        if (m.conv == nullptr) {
+            float u[8];
+#pragma unroll
+            for (int k = 0; k < 8; ++k) u[k] = input(t0 + k);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) dst[(t0 + k) * ld] = u[k];
+        } else if (m.taps <= 4) {
+            float u[11], w[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) w[k] = k < m.taps ? m.conv[(size_t)c * m.taps + m.taps - 1 - k] : 0.0f;      // w[k]: of the input k tokens ago
+#pragma unroll
+            for (int k = 0; k < 11; ++k) u[k] = k >= 4 - m.taps ? input(t0 + k - 3) : 0.0f;
+#pragma unroll
+            for (int k = 0; k < 8; ++k) {
+                const float z = fmaf(w[3], u[k], fmaf(w[2], u[k + 1], fmaf(w[1], u[k + 2], w[0] * u[k + 3])));
+                dst[(t0 + k) * ld] = t0 + k < n ? z * cm_sigmoid(z) : 0.0f;
+            }
+        } else {
+            for (int k = 0; k < 8; ++k) {
+                float z = 0.0f;
+                for (int j = 0; j < m.taps; ++j) z = fmaf(m.conv[(size_t)c * m.taps + j], input(t0 + k - (m.taps - 1) + j), z);
+                dst[(t0 + k) * ld] = t0 + k < n ? z * cm_sigmoid(z) : 0.0f;
             }
         }
-        for (int x = lane; x < E; x += 32) {
-            if (in) cm_cp_async4(vs + t * LE + x, w.v + row * w.ldq + h * E + x);
-            else vs[t * LE + x] = 0.0f;
-        }
-        if (DELTA && lane == 0) beta[t] = in ? cm_sigmoid(a.proj[row * a.ld + m.b_off + h]) : 0.0f;
     }
-    cm_cp_commit();
-    cm_cp_wait_all();
+    if (DELTA && threadIdx.x < kPiece) beta[threadIdx.x] = threadIdx.x < n ? cm_sigmoid(a.proj[(size_t)(row0 + threadIdx.x) * a.ld + m.b_off + h]) : 0.0f;
+    // The decays: the low-rank map in chunks of 32 of its rank, eight rows of a channel an item.
+    const float a_exp = m.a_log != nullptr ? expf(m.a_log[h]) * kLbLog2e : kLbLog2e / m.tau;
+    for (int r0 = 0; r0 < m.rank; r0 += 32) {
+        if (r0 > 0) __syncthreads();
+        load_rank_chunk(Am, fs, a.proj + (size_t)row0 * a.ld + m.a_off, a.ld, static_cast<const T*>(m.a2) + (size_t)h * D * m.rank, m.rank, r0, n, D);
+        __syncthreads();
+        for (int i = threadIdx.x; i < 4 * D; i += blockDim.x) {
+            const int part = i / D, d = i - part * D, t0 = 8 * part;
+            float z[8];
+#pragma unroll
+            for (int k = 0; k < 8; ++k) z[k] = r0 > 0 ? bs[(t0 + k) * LD + d] : m.z_bias != nullptr ? m.z_bias[h * D + d] : 0.0f;
+            rank_chunk(z, Am, fs + d * 33, t0, min(32, m.rank - r0));
+            if (r0 + 32 >= m.rank) {
+#pragma unroll
+                for (int k = 0; k < 8; ++k) z[k] = t0 + k < n ? -a_exp * (m.a_log != nullptr ? lb_softplus(z[k]) : lb_softplus(-z[k])) : 0.0f;
+            }
+#pragma unroll
+            for (int k = 0; k < 8; ++k) bs[(t0 + k) * LD + d] = z[k];
+        }
+    }
     __syncthreads();
+    if (m.unit) {
+        for (int t = warp; t < n; t += 8) {
+            float sq = 0.0f, sk = 0.0f;
+            for (int d = lane; d < D; d += 32) {
+                sq = fmaf(qs[t * LD + d], qs[t * LD + d], sq);
+                sk = fmaf(ks[t * LD + d], ks[t * LD + d], sk);
+            }
+            const float iq = 1.0f / sqrtf(lb_warp_sum(sq) + m.unit_eps), ik = 1.0f / sqrtf(lb_warp_sum(sk) + m.unit_eps);
+            for (int d = lane; d < D; d += 32) {
+                qs[t * LD + d] *= iq;
+                ks[t * LD + d] *= ik;
+            }
+        }
+    }
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
         float b = 0.0f;
 #pragma unroll
@@ -417,20 +415,56 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
         }
     }
     __syncthreads();
-    // The pairs: a warp per row t, lane j.
-    for (int t = warp; t < kPiece; t += 8) {
+    // The pairs.  Rows of the second half meet keys of the first through the border between them: exp(b_t - b_j) = exp(b_t - b_15) exp(b_15 - b_j), both
+    // exponents at most 0, so those 256 pairs are plain products; pairs inside a half make their exponentials one by one.
+    constexpr int kHalf = kPiece / 2;
+    for (int i = threadIdx.x; i < kHalf * D; i += blockDim.x) {
+        const int t = i / D, d = i - t * D;
+        const float border = bs[(kHalf - 1) * LD + d], e = fast_exp2(bs[(kHalf + t) * LD + d] - border);
+        fs[t * LD + d] = qs[(kHalf + t) * LD + d] * e;
+        if (DELTA) fs[(kHalf + t) * LD + d] = ks[(kHalf + t) * LD + d] * e;
+        fs[(2 * kHalf + t) * LD + d] = ks[t * LD + d] * fast_exp2(border - bs[t * LD + d]);
+    }
+    __syncthreads();
+    {
+        const int t = threadIdx.x >> 4, j = threadIdx.x & 15;
+        const float *qt = fs + t * LD, *kt = fs + (kHalf + t) * LD, *kj = fs + (2 * kHalf + j) * LD;
+        float p0 = 0.0f, p1 = 0.0f, a0 = 0.0f, a1 = 0.0f;
+        int d = 0;
+#pragma unroll 4
+        for (; d + 1 < D; d += 2) {
+            p0 = fmaf(qt[d], kj[d], p0);
+            p1 = fmaf(qt[d + 1], kj[d + 1], p1);
+            if (DELTA) {
+                a0 = fmaf(kt[d], kj[d], a0);
+                a1 = fmaf(kt[d + 1], kj[d + 1], a1);
+            }
+        }
+        if (d < D) {
+            p0 = fmaf(qt[d], kj[d], p0);
+            if (DELTA) a0 = fmaf(kt[d], kj[d], a0);
+        }
+        out[l.p + (kHalf + t) * kPiece + j] = (p0 + p1) * m.q_scale;
+        out[l.p + t * kPiece + kHalf + j] = 0.0f;
+        if (DELTA) {
+            Am[(kHalf + t) * 36 + j] = a0 + a1;
+            Am[t * 36 + kHalf + j] = 0.0f;
+        }
+    }
+    for (int r = warp; r < kHalf; r += 8) {    // a warp: row r of the first half and row r of the second, a half of the lanes each
+        const int half = lane >> 4 << 4, t = half + r, j = half + (lane & 15);
         float p = 0.0f, av = 0.0f;
-        if (lane <= t && t < n) {
-            const float *qt = qs + t * LD, *kt = ks + t * LD, *bt = bs + t * LD, *kj = ks + lane * LD, *bj = bs + lane * LD;
+        if (j <= t && t < n) {
+            const float *qt = qs + t * LD, *kt = ks + t * LD, *bt = bs + t * LD, *kj = ks + j * LD, *bj = bs + j * LD;
 #pragma unroll 4
             for (int d = 0; d < D; ++d) {
-                const float e = exp2f(bt[d] - bj[d]) * kj[d];
+                const float e = fast_exp2(bt[d] - bj[d]) * kj[d];
                 p = fmaf(qt[d], e, p);
                 if (DELTA) av = fmaf(kt[d], e, av);
             }
         }
-        out[l.p + t * kPiece + lane] = p * m.q_scale;
-        if (DELTA) Am[t * 36 + lane] = lane < t ? av : 0.0f;
+        out[l.p + t * kPiece + j] = p * m.q_scale;
+        if (DELTA) Am[t * 36 + j] = j < t ? av : 0.0f;
     }
     __syncthreads();
     // Warp 0 solves the triangle, a column a lane; the others turn the rows into what the scan and the outputs read.
@@ -448,10 +482,10 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
             M[t * 36 + lane] = x[t];
         }
     } else {
-        const int first = DELTA ? threadIdx.x - 32 : threadIdx.x, step = DELTA ? blockDim.x - 32 : blockDim.x;
-        for (int i = first; i < kPiece * D; i += step) {
+        const int first_i = DELTA ? threadIdx.x - 32 : threadIdx.x, step = DELTA ? blockDim.x - 32 : blockDim.x;
+        for (int i = first_i; i < kPiece * D; i += step) {
             const int t = i / D, d = i - t * D;
-            const float b = bs[t * LD + d], b_last = bs[(kPiece - 1) * LD + d], k = ks[t * LD + d], e = exp2f(b), kb = exp2f(b_last - b) * k;
+            const float b = bs[t * LD + d], b_last = bs[(kPiece - 1) * LD + d], k = ks[t * LD + d], e = fast_exp2(b), kb = fast_exp2(b_last - b) * k;
             out[l.q + i] = qs[t * LD + d] * m.q_scale * e;
             if (DELTA) {
                 out[l.b + i] = kb;
@@ -459,7 +493,7 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
             } else {
                 ks[t * LD + d] = kb;
             }
-            if (t == 0) out[l.keep + d] = exp2f(b_last);
+            if (t == 0) out[l.keep + d] = fast_exp2(b_last);
         }
     }
     __syncthreads();
@@ -470,13 +504,17 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
             float y[8];
             if (x < D) tri_product(y, M, ks + x, LD, t0);
             else tri_product(y, M, vs + (x - D), LE, t0);
+            if (x < D) {
+                float4* dst = reinterpret_cast<float4*>(out + l.w + x * kPiece + t0);
+                dst[0] = make_float4(y[0], y[1], y[2], y[3]);
+                dst[1] = make_float4(y[4], y[5], y[6], y[7]);
+            } else {
 #pragma unroll
-            for (int k = 0; k < 8; ++k) {
-                if (x < D) out[l.w + (t0 + k) * D + x] = y[k];
-                else out[l.u + (t0 + k) * E + (x - D)] = y[k];
+                for (int k = 0; k < 8; ++k) out[l.u + (t0 + k) * E + (x - D)] = y[k];
             }
         }
     } else {
+        for (int i = threadIdx.x; i < kPiece * E; i += blockDim.x) out[l.u + i] = vs[i / E * LE + i % E];
         // The piece's own sum: thread (column, eight channels).
         const int parts = (D + 7) / 8;
         for (int i = threadIdx.x; i < parts * E; i += blockDim.x) {
@@ -496,7 +534,7 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
 
 // The scan without the delta rule: every element of S by itself, S <- exp(b_n)[d] S + sum, the state before every piece left in the sum's place.
 constexpr int kAhead = 8;
-__global__ void __launch_bounds__(256) channel_scan_kernel(lb_channel_memory m, StepArgs a, PieceArgs w) {
+__global__ void __launch_bounds__(256) channel_scan_kernel(lb_channel_memory m, StepArgs a, float* __restrict__ scratch) {
     lb_wait_for_predecessor();
     lb_dependents_may_launch();
     const int seq = blockIdx.x, h = blockIdx.y, D = m.dim, E = m.vdim, i = blockIdx.z * blockDim.x + threadIdx.x;
@@ -507,7 +545,7 @@ __global__ void __launch_bounds__(256) channel_scan_kernel(lb_channel_memory m, 
     const PieceLayout l = piece_layout(D, E, 0);
     float* st = a.state + (size_t)a.slots[seq] * m.slot_stride + (size_t)h * D * E + i;
     const size_t stride = (size_t)m.n_head * l.total;
-    float* first = w.scratch + ((size_t)g0 * m.n_head + h) * l.total;
+    float* first = scratch + ((size_t)g0 * m.n_head + h) * l.total;
     const int d = i / E;
     float S = *st;
     for (int p0 = 0; p0 < pieces; p0 += kAhead) {
@@ -529,9 +567,11 @@ __global__ void __launch_bounds__(256) channel_scan_kernel(lb_channel_memory m, 
 }
 
 // The scan under the delta rule: a block per (request, head, VT value columns) walks the request's pieces, U = M V - (M K~) S, then
-// S <- exp(b_n) S + sum_j (exp(b_n - b_j) k_j) u_j^T; the next piece's matrices travel while this one is added.
+// S <- exp(b_n) S + sum_j (exp(b_n - b_j) k_j) u_j^T; the next piece's matrices travel while this one is added.  U: the eight warps share the channels,
+// a lane 4 x 4 results, the shares meet in shared memory in the warps' order.
 template <int VT>
-__global__ void __launch_bounds__(256) delta_scan_kernel(lb_channel_memory m, StepArgs a, PieceArgs w) {
+__global__ void __launch_bounds__(256) delta_scan_kernel(lb_channel_memory m, StepArgs a, float* __restrict__ scratch) {
+    static_assert(VT == 16, "a warp's lanes are 8 x 4 tiles of 4 rows x 4 columns");
     extern __shared__ __align__(16) float smem[];
     lb_wait_for_predecessor();
     lb_dependents_may_launch();
@@ -541,113 +581,117 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(lb_channel_memory m, St
     int g0 = 0;
     for (int s = 0; s < seq; ++s) g0 += (a.q_start[s + 1] - a.q_start[s] + kPiece - 1) / kPiece;
     const PieceLayout l = piece_layout(D, E, 1);
-    const int LS = VT;
-    const int matrix = (kPiece * D + 3) / 4 * 4, d4 = (D + 3) / 4 * 4;
+    const int matrix = kPiece * D, d4 = (D + 3) / 4 * 4;
     float* S = smem;                           // [d4][VT]
-    float* U = S + d4 * LS;                    // [32][VT]
-    float* buf = U + kPiece * VT;              // [2][W | B | keep | M V's columns]
+    float* U = S + d4 * VT;                    // [32][VT]
+    float* red = U + kPiece * VT;              // [8][32][VT]
+    float* buf = red + 8 * kPiece * VT;        // [2][W^T | B | keep | M V's columns]
     const int buf_floats = 2 * matrix + d4 + kPiece * VT;
     const size_t stride = (size_t)m.n_head * l.total;
-    float* first = w.scratch + ((size_t)g0 * m.n_head + h) * l.total;
+    float* first = scratch + ((size_t)g0 * m.n_head + h) * l.total;
     float* st = a.state + (size_t)a.slots[seq] * m.slot_stride + (size_t)h * D * E;
+    const bool whole = (E & 3) == 0 && c0 + VT <= E;      // the tile's columns travel in 16-byte pieces
     auto ask = [&](int p) {
         const float* src = first + (size_t)p * stride;
         float* dst = buf + (p & 1) * buf_floats;
-        cm_fetch(dst, src + l.w, kPiece * D);
-        cm_fetch(dst + matrix, src + l.b, kPiece * D);
+        cm_fetch(dst, src + l.w, matrix);
+        cm_fetch(dst + matrix, src + l.b, matrix);
         cm_fetch(dst + 2 * matrix, src + l.keep, D);
-        for (int i = threadIdx.x; i < kPiece * VT; i += blockDim.x) {
-            const int t = i / VT, x = i - t * VT;
-            if (c0 + x < E) cm_cp_async4(dst + 2 * matrix + d4 + i, src + l.u + t * E + c0 + x);
-            else dst[2 * matrix + d4 + i] = 0.0f;
+        float* mv = dst + 2 * matrix + d4;
+        if (whole) {
+            for (int i = threadIdx.x; i < kPiece * VT / 4; i += blockDim.x) cm_cp_async16(mv + 4 * i, src + l.u + (i / (VT / 4)) * E + c0 + 4 * (i % (VT / 4)));
+        } else {
+            for (int i = threadIdx.x; i < kPiece * VT; i += blockDim.x) {
+                const int t = i / VT, x = i - t * VT;
+                if (c0 + x < E) cm_cp_async4(mv + i, src + l.u + t * E + c0 + x);
+                else mv[i] = 0.0f;
+            }
         }
         cm_cp_commit();
     };
     ask(0);
     for (int i = threadIdx.x; i < d4 * VT; i += blockDim.x) {
         const int d = i / VT, x = i - d * VT;
-        S[d * LS + x] = d < D && c0 + x < E ? st[(size_t)d * E + c0 + x] : 0.0f;
+        S[i] = d < D && c0 + x < E ? st[(size_t)d * E + c0 + x] : 0.0f;
     }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lt = 4 * (lane >> 2), lc = 4 * (lane & 3);
     const int c = threadIdx.x % VT, tr = threadIdx.x / VT;
     constexpr int TR = 256 / VT;               // thread rows
     for (int p = 0; p < pieces; ++p) {
         cm_cp_wait_all();
         __syncthreads();                       // the piece has arrived; S is whole; the other buffer is free
         if (p + 1 < pieces) ask(p + 1);
-        const float* W = buf + (p & 1) * buf_floats;
+        const float* W = buf + (p & 1) * buf_floats;       // [D][32]
         const float* B = W + matrix;
         const float* keep = B + matrix;
         const float* MV = keep + d4;
         float* at = first + (size_t)p * stride;
         for (int i = threadIdx.x; i < D * VT; i += blockDim.x) {
             const int d = i / VT, x = i - d * VT;
-            if (c0 + x < E) at[l.s + (size_t)d * E + c0 + x] = S[d * LS + x];
+            if (c0 + x < E) at[l.s + (size_t)d * E + c0 + x] = S[i];
         }
-        constexpr int R = kPiece / TR > 0 ? kPiece / TR : 1;
-        if (tr < kPiece) {
-            float y[R];
+        float y[4][4] = {};
+#pragma unroll 4
+        for (int d = warp; d < D; d += 8) {
+            const float4 w = *reinterpret_cast<const float4*>(W + d * kPiece + lt), s = *reinterpret_cast<const float4*>(S + d * VT + lc);
+            const float wv[4] = {w.x, w.y, w.z, w.w}, sv[4] = {s.x, s.y, s.z, s.w};
 #pragma unroll
-            for (int i = 0; i < R; ++i) y[i] = MV[(tr + i * TR) * VT + c];
-            if ((D & 3) == 0) {
-                for (int d = 0; d < D; d += 4) {
-                    const float s0 = S[d * LS + c], s1 = S[(d + 1) * LS + c], s2 = S[(d + 2) * LS + c], s3 = S[(d + 3) * LS + c];
+            for (int i = 0; i < 4; ++i)
 #pragma unroll
-                    for (int i = 0; i < R; ++i) {
-                        const float4 r = *reinterpret_cast<const float4*>(W + (tr + i * TR) * D + d);
-                        y[i] = fmaf(-r.x, s0, fmaf(-r.y, s1, fmaf(-r.z, s2, fmaf(-r.w, s3, y[i]))));
-                    }
-                }
-            } else {
-                for (int d = 0; d < D; ++d) {
-                    const float s = S[d * LS + c];
+                for (int j = 0; j < 4; ++j) y[i][j] = fmaf(wv[i], sv[j], y[i][j]);
+        }
 #pragma unroll
-                    for (int i = 0; i < R; ++i) y[i] = fmaf(-W[(tr + i * TR) * D + d], s, y[i]);
-                }
-            }
+        for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(red + (warp * kPiece + lt + i) * VT + lc) = make_float4(y[i][0], y[i][1], y[i][2], y[i][3]);
+        __syncthreads();
 #pragma unroll
-            for (int i = 0; i < R; ++i) {
-                const int t = tr + i * TR;
-                U[t * VT + c] = y[i];
-                if (c0 + c < E) at[l.u + (size_t)t * E + c0 + c] = y[i];
-            }
+        for (int i = 0; i < 2; ++i) {
+            const int at_u = threadIdx.x + 256 * i;
+            float u = MV[at_u];
+#pragma unroll
+            for (int w = 0; w < 8; ++w) u -= red[w * kPiece * VT + at_u];
+            U[at_u] = u;
+            const int t = at_u / VT, x = at_u - t * VT;
+            if (c0 + x < E) at[l.u + (size_t)t * E + c0 + x] = u;
         }
         __syncthreads();
         // S: thread (column, four channels at a time).
         for (int d = 4 * tr; d < D; d += 4 * TR) {
-            float y[4] = {};
+            float z[4] = {};
             if ((D & 3) == 0) {
-#pragma unroll 8
+#pragma unroll 16
                 for (int t = 0; t < kPiece; ++t) {
                     const float u = U[t * VT + c];
                     const float4 r = *reinterpret_cast<const float4*>(B + t * D + d);
-                    y[0] = fmaf(r.x, u, y[0]);
-                    y[1] = fmaf(r.y, u, y[1]);
-                    y[2] = fmaf(r.z, u, y[2]);
-                    y[3] = fmaf(r.w, u, y[3]);
+                    z[0] = fmaf(r.x, u, z[0]);
+                    z[1] = fmaf(r.y, u, z[1]);
+                    z[2] = fmaf(r.z, u, z[2]);
+                    z[3] = fmaf(r.w, u, z[3]);
                 }
             } else {
                 for (int t = 0; t < kPiece; ++t) {
                     const float u = U[t * VT + c];
 #pragma unroll
-                    for (int k = 0; k < 4; ++k) y[k] = fmaf(B[t * D + min(d + k, D - 1)], u, y[k]);
+                    for (int k = 0; k < 4; ++k) z[k] = fmaf(B[t * D + min(d + k, D - 1)], u, z[k]);
                 }
             }
 #pragma unroll
             for (int k = 0; k < 4; ++k)
-                if (d + k < D) S[(d + k) * LS + c] = fmaf(keep[d + k], S[(d + k) * LS + c], y[k]);
+                if (d + k < D) S[(d + k) * VT + c] = fmaf(keep[d + k], S[(d + k) * VT + c], z[k]);
         }
     }
     __syncthreads();
     for (int i = threadIdx.x; i < D * VT; i += blockDim.x) {
         const int d = i / VT, x = i - d * VT;
-        if (c0 + x < E) st[(size_t)d * E + c0 + x] = S[d * LS + x];
+        if (c0 + x < E) st[(size_t)d * E + c0 + x] = S[i];
     }
 }
 
-// The outputs of a piece with the heads' norm and gate.  Thread (c, tg) owns column c for the R rows tg R .. tg R + R - 1.
-template <typename T, int R, bool DELTA>
-__global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory m, StepArgs a, PieceArgs w, int n_seq) {
+// The outputs of a piece with the heads' norm and gate.  Thread (c, tg) owns column c for the R rows tg R .. tg R + R - 1; the state before the piece
+// comes to shared memory (`staged`) while the gates are made.
+template <typename T, int R>
+__global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory m, StepArgs a, float* __restrict__ scratch, int n_seq, int staged) {
     extern __shared__ __align__(16) float smem[];
+    __shared__ float inv[kPiece];
     constexpr int EP = 8 * R;                  // threads across the columns: 256 / (32 / R)
     lb_wait_for_predecessor();
     lb_dependents_may_launch();
@@ -657,9 +701,12 @@ __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory 
     const int row0 = a.q_start[seq] + piece * kPiece, n = min(kPiece, a.q_start[seq + 1] - row0);
     float* P = smem;                           // [32][32]
     float* qs = P + kPiece * kPiece;           // [32][d4]
-    float* os = qs + kPiece * d4;              // [32][E + 1]
-    const PieceLayout l = piece_layout(D, E, DELTA);
-    const float* in = w.scratch + ((size_t)blockIdx.x * m.n_head + h) * l.total;
+    float* xT = qs + kPiece * d4;              // [32][36] the gates' inputs
+    float* gw = xT + 32 * 36;                  // [E][33] their map
+    float* os = gw;                            // [32][E + 1] afterwards
+    float* Ss = gw + ((E > 32 ? E : 32) * 33 + 35) / 4 * 4;      // [D][E]
+    const PieceLayout l = piece_layout(D, E, m.delta);
+    const float* in = scratch + ((size_t)blockIdx.x * m.n_head + h) * l.total;
     cm_fetch(P, in + l.p, kPiece * kPiece);
     if (D == d4) {
         cm_fetch(qs, in + l.q, kPiece * D);
@@ -670,15 +717,38 @@ __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory 
             else qs[i] = 0.0f;
         }
     }
+    if (staged) cm_fetch(Ss, in + l.s, D * E);
     cm_cp_commit();
+    const int c = threadIdx.x % EP, t0 = threadIdx.x / EP * R;
+    float gate[R];
+#pragma unroll
+    for (int i = 0; i < R; ++i) gate[i] = 0.0f;
+    if (m.g2 != nullptr) {
+        for (int r0 = 0; r0 < m.gate_rank; r0 += 32) {
+            if (r0 > 0) __syncthreads();
+            load_rank_chunk(xT, gw, a.proj + (size_t)row0 * a.ld + m.g_off, a.ld, static_cast<const T*>(m.g2) + (size_t)h * E * m.gate_rank, m.gate_rank, r0, n, E);
+            __syncthreads();
+            if (c < E) {
+                const int count = min(32, m.gate_rank - r0);
+                for (int r = 0; r < count; ++r) {
+                    const float w = gw[c * 33 + r];
+#pragma unroll
+                    for (int i = 0; i < R; ++i) gate[i] = fmaf(w, xT[r * 36 + t0 + i], gate[i]);
+                }
+            }
+        }
+    } else if (c < E) {
+#pragma unroll
+        for (int i = 0; i < R; ++i) gate[i] = t0 + i < n ? a.proj[(size_t)(row0 + t0 + i) * a.ld + m.g_off + h * E + c] : 0.0f;
+    }
     cm_cp_wait_all();
     __syncthreads();
-    const int c = threadIdx.x % EP, t0 = threadIdx.x / EP * R;
-    if (c < E) {
-        float y[R];
+    float y[R];
 #pragma unroll
-        for (int i = 0; i < R; ++i) y[i] = 0.0f;
-        const float* S = in + l.s + c;
+    for (int i = 0; i < R; ++i) y[i] = 0.0f;
+    if (c < E) {
+        const float* S = (staged ? Ss : in + l.s) + c;
+#pragma unroll 2
         for (int d = 0; d < D; d += 4) {
             float s[4];
 #pragma unroll
@@ -689,13 +759,13 @@ __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory 
                 y[i] = fmaf(q.x, s[0], fmaf(q.y, s[1], fmaf(q.z, s[2], fmaf(q.w, s[3], y[i]))));
             }
         }
-        const float* u = DELTA ? in + l.u + c : w.v + (size_t)row0 * w.ldq + h * E + c;
-        const size_t ldu = DELTA ? (size_t)E : (size_t)w.ldq;
+        const float* u = in + l.u + c;
         const int last = min(n, t0 + R);       // rows after the last of this thread's are not seen
+#pragma unroll 2
         for (int j = 0; j < last; j += 4) {
             float s[4];
 #pragma unroll
-            for (int k = 0; k < 4; ++k) s[k] = j + k < n ? u[(size_t)(j + k) * ldu] : 0.0f;
+            for (int k = 0; k < 4; ++k) s[k] = j + k < n ? u[(j + k) * E] : 0.0f;
 #pragma unroll
             for (int i = 0; i < R; ++i) {
                 const float4 p = *reinterpret_cast<const float4*>(P + (t0 + i) * kPiece + j);
@@ -711,12 +781,18 @@ __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory 
         const float* o = os + t * (E + 1);
         float ss = 0.0f;
         for (int x = lane; x < E; x += 32) ss = fmaf(o[x], o[x], ss);
-        const float inv = 1.0f / sqrtf(lb_warp_sum(ss) / (float)E + m.eps);
-        const size_t row = (size_t)(row0 + t);
-        for (int x = lane; x < E; x += 32) {
-            if (a.o != nullptr) a.o[row * a.ldo + h * E + x] = o[x];
-            static_cast<T*>(a.heads)[row * a.ldh + h * E + x] = lb_from_float<T>(o[x] * inv * m.norm[x] * cm_gate(w.gate[row * w.ldg + h * E + x], m.gate_act));
-        }
+        ss = lb_warp_sum(ss);
+        if (lane == 0) inv[t] = 1.0f / sqrtf(ss / (float)E + m.eps);
+    }
+    __syncthreads();
+    if (c >= E) return;
+    const float gain = m.norm[c];
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        if (t0 + i >= n) break;
+        const size_t row = (size_t)(row0 + t0 + i);
+        if (a.o != nullptr) a.o[row * a.ldo + h * E + c] = y[i];
+        static_cast<T*>(a.heads)[row * a.ldh + h * E + c] = lb_from_float<T>(y[i] * inv[t0 + i] * gain * cm_gate(gate[i], m.gate_act));
     }
 }
 
@@ -770,49 +846,15 @@ extern "C" int64_t lb_channel_memory_pieces_floats(int n_tokens, int n_seq, int 
     return ((int64_t)n_tokens / kPiece + n_seq) * n_head * piece_layout(dim, vdim, delta).total;
 }
 
-extern "C" int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memory, const lb_channel_step* step, float* rows, float* log_decay, float* gate,
-                                        float* scratch, int n_tokens, int n_seq, void* stream) {
+extern "C" int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memory, const lb_channel_step* step, float* scratch, int n_tokens, int n_seq,
+                                        void* stream) {
     if (int rc = check_shape(memory)) return rc;
     LB_CHECK_ARG(dtype == LB_F32 || dtype == LB_BF16, "channel memory: unknown dtype %d", dtype);
-    LB_CHECK_ARG(scratch != nullptr && log_decay != nullptr && ((memory->conv == nullptr && !memory->unit) || rows != nullptr) && (memory->g2 == nullptr || gate != nullptr),
-                 "channel memory in pieces: scratch is missing");
+    LB_CHECK_ARG(scratch != nullptr, "channel memory in pieces: scratch is missing");
     if (n_seq == 0 || n_tokens == 0) return LB_OK;
     const lb_channel_memory m = *memory;
     const StepArgs a = step_of(step);
     auto s = static_cast<cudaStream_t>(stream);
-    const int QD = m.kv_head * m.dim, HD = m.n_head * m.dim, HE = m.n_head * m.vdim, channels = 2 * QD + HE;
-    const dim3 tiles_d((HD + 63) / 64, (n_tokens + 31) / 32), tiles_e((HE + 63) / 64, (n_tokens + 31) / 32);
-    // The low-rank maps.
-    if (dtype == LB_F32) {
-        LB_CHECK_CUDA(lb_launch_overlapped(low_rank_kernel<float, true>, tiles_d, dim3(256), 0, s, m, a.proj + m.a_off, a.ld, (const float*)m.a2, m.rank, log_decay,
-                                           (int64_t)HD, n_tokens, HD));
-        if (m.g2 != nullptr)
-            LB_CHECK_CUDA(lb_launch_overlapped(low_rank_kernel<float, false>, tiles_e, dim3(256), 0, s, m, a.proj + m.g_off, a.ld, (const float*)m.g2, m.gate_rank,
-                                               gate, (int64_t)HE, n_tokens, HE));
-    } else {
-        LB_CHECK_CUDA(lb_launch_overlapped(low_rank_kernel<__nv_bfloat16, true>, tiles_d, dim3(256), 0, s, m, a.proj + m.a_off, a.ld, (const __nv_bfloat16*)m.a2,
-                                           m.rank, log_decay, (int64_t)HD, n_tokens, HD));
-        if (m.g2 != nullptr)
-            LB_CHECK_CUDA(lb_launch_overlapped(low_rank_kernel<__nv_bfloat16, false>, tiles_e, dim3(256), 0, s, m, a.proj + m.g_off, a.ld,
-                                               (const __nv_bfloat16*)m.g2, m.gate_rank, gate, (int64_t)HE, n_tokens, HE));
-    }
-    PieceArgs w{};
-    w.q = a.proj; w.ldq = a.ld;
-    if (m.conv != nullptr || m.unit) {
-        const int jobs = 2 * m.kv_head + m.n_head;
-        LB_CHECK_CUDA(lb_launch_overlapped(channel_prepare_kernel, dim3(n_tokens, (jobs + 7) / 8), dim3(256), 0, s, m, a, rows, (int64_t)channels));
-        w.q = rows;
-        w.ldq = channels;
-        if (m.conv != nullptr)
-            if (int rc = launch_ring(m, a, n_seq, s)) return rc;
-    }
-    w.k = w.q + QD;
-    w.v = w.q + 2 * QD;
-    w.log_decay = log_decay;
-    w.ldd = HD;
-    w.gate = m.g2 != nullptr ? gate : a.proj + m.g_off;
-    w.ldg = m.g2 != nullptr ? HE : a.ld;
-    w.scratch = scratch;
     const int pieces = n_tokens / kPiece + n_seq, D = m.dim, E = m.vdim, d4 = (D + 3) / 4 * 4;
     auto launch = [&](auto kernel, dim3 grid, size_t smem, auto... args) -> int {
         LB_CHECK_ARG(smem <= 220 * 1024, "channel memory in pieces: heads of %d x %d values do not fit shared memory", D, E);
@@ -820,26 +862,33 @@ extern "C" int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memo
         LB_CHECK_CUDA(lb_launch_overlapped(kernel, grid, dim3(256), smem, s, args...));
         return LB_OK;
     };
-    const size_t own = (2 * kPiece * 36 + kPiece + 3 * (size_t)kPiece * (D + 1) + (size_t)kPiece * (E + 1)) * sizeof(float);
+    const dim3 grid(pieces, m.n_head);
+    const size_t own = (2 * kPiece * 36 + kPiece + (3 * (size_t)kPiece + 48) * (D + 1) + (size_t)kPiece * (E + 1)) * sizeof(float);
     constexpr int VT = 16;
     if (m.delta) {
-        if (int rc = launch(channel_pieces_kernel<true>, dim3(pieces, m.n_head), own, m, a, w, n_seq)) return rc;
-        const size_t scan = ((size_t)d4 * VT + kPiece * VT + 2 * (2 * (size_t)kPiece * d4 + d4 + kPiece * VT)) * sizeof(float);
-        if (int rc = launch(delta_scan_kernel<VT>, dim3(n_seq, m.n_head, (E + VT - 1) / VT), scan, m, a, w)) return rc;
+        if (int rc = dtype == LB_F32 ? launch(channel_pieces_kernel<float, true>, grid, own, m, a, scratch, n_seq)
+                                     : launch(channel_pieces_kernel<__nv_bfloat16, true>, grid, own, m, a, scratch, n_seq)) return rc;
+        const size_t scan = ((size_t)d4 * VT + 9 * (size_t)kPiece * VT + 2 * (2 * (size_t)kPiece * D + d4 + kPiece * VT)) * sizeof(float);
+        if (int rc = launch(delta_scan_kernel<VT>, dim3(n_seq, m.n_head, (E + VT - 1) / VT), scan, m, a, scratch)) return rc;
     } else {
-        if (int rc = launch(channel_pieces_kernel<false>, dim3(pieces, m.n_head), own, m, a, w, n_seq)) return rc;
-        if (int rc = launch(channel_scan_kernel, dim3(n_seq, m.n_head, (D * E + 255) / 256), 0, m, a, w)) return rc;
+        if (int rc = dtype == LB_F32 ? launch(channel_pieces_kernel<float, false>, grid, own, m, a, scratch, n_seq)
+                                     : launch(channel_pieces_kernel<__nv_bfloat16, false>, grid, own, m, a, scratch, n_seq)) return rc;
+        if (int rc = launch(channel_scan_kernel, dim3(n_seq, m.n_head, (D * E + 255) / 256), 0, m, a, scratch)) return rc;
     }
-    const size_t outs = (kPiece * kPiece + (size_t)kPiece * d4 + (size_t)kPiece * (E + 1)) * sizeof(float);
-    const dim3 grid(pieces, m.n_head);
-#define LB_OUTPUTS(T, DELTA)                                                                             \
-    (E <= 8     ? launch(channel_outputs_kernel<T, 1, DELTA>, grid, outs, m, a, w, n_seq)                \
-     : E <= 16  ? launch(channel_outputs_kernel<T, 2, DELTA>, grid, outs, m, a, w, n_seq)                \
-     : E <= 32  ? launch(channel_outputs_kernel<T, 4, DELTA>, grid, outs, m, a, w, n_seq)                \
-     : E <= 64  ? launch(channel_outputs_kernel<T, 8, DELTA>, grid, outs, m, a, w, n_seq)                \
-     : E <= 128 ? launch(channel_outputs_kernel<T, 16, DELTA>, grid, outs, m, a, w, n_seq)               \
-                : launch(channel_outputs_kernel<T, 32, DELTA>, grid, outs, m, a, w, n_seq))
-    if (dtype == LB_F32) return m.delta ? LB_OUTPUTS(float, true) : LB_OUTPUTS(float, false);
-    return m.delta ? LB_OUTPUTS(__nv_bfloat16, true) : LB_OUTPUTS(__nv_bfloat16, false);
+    // The ring only after the pieces have read it.
+    if (m.conv != nullptr)
+        if (int rc = launch_ring(m, a, n_seq, s)) return rc;
+    const size_t base = (kPiece * kPiece + (size_t)kPiece * d4 + 32 * 36 + ((E > 32 ? E : 32) * 33 + 35) / 4 * 4) * sizeof(float);
+    const size_t with_state = base + (size_t)D * E * sizeof(float);
+    const int staged = with_state <= 110 * 1024 ? 1 : 0;
+    const size_t outs = staged ? with_state : base;
+#define LB_OUTPUTS(T)                                                                                 \
+    (E <= 8     ? launch(channel_outputs_kernel<T, 1>, grid, outs, m, a, scratch, n_seq, staged)      \
+     : E <= 16  ? launch(channel_outputs_kernel<T, 2>, grid, outs, m, a, scratch, n_seq, staged)      \
+     : E <= 32  ? launch(channel_outputs_kernel<T, 4>, grid, outs, m, a, scratch, n_seq, staged)      \
+     : E <= 64  ? launch(channel_outputs_kernel<T, 8>, grid, outs, m, a, scratch, n_seq, staged)      \
+     : E <= 128 ? launch(channel_outputs_kernel<T, 16>, grid, outs, m, a, scratch, n_seq, staged)     \
+                : launch(channel_outputs_kernel<T, 32>, grid, outs, m, a, scratch, n_seq, staged))
+    return dtype == LB_F32 ? LB_OUTPUTS(float) : LB_OUTPUTS(__nv_bfloat16);
 #undef LB_OUTPUTS
 }

@@ -133,6 +133,71 @@ __global__ void __launch_bounds__(1024) expert_plan_kernel(int32_t* __restrict__
     }
 }
 
+// The same plan for up to 256 experts and many pairs: every warp owns a stretch of pairs.  It counts its pairs by expert (lanes with one expert find
+// each other by a match), the warps' counts become places by a running sum over warps and experts, and a second walk over the stretch hands the places
+// out in the pairs' own order: three barriers, each pair read twice by one warp instead of twice by every expert's.
+__global__ void __launch_bounds__(1024) expert_plan_wide_kernel(const int32_t* __restrict__ ids, int n_pairs, int E, int32_t* __restrict__ offsets,
+                                                                int32_t* __restrict__ place, int32_t* __restrict__ pair_at) {
+    extern __shared__ int at[];        // [32 warps][E], then the experts' first places [E]
+    int* first = at + 32 * E;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int i = threadIdx.x; i < 32 * E; i += blockDim.x) at[i] = 0;
+    lb_wait_for_predecessor();
+    lb_dependents_may_launch();
+    __syncthreads();
+    const int steps = (n_pairs + 1023) / 1024, begin = warp * steps * 32;
+    int* mine = at + warp * E;
+    for (int i = 0; i < steps; ++i) {
+        const int p = begin + 32 * i + lane, e = p < n_pairs ? ids[p] : E;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        if (e >= 0 && e < E && (same & ((1u << lane) - 1u)) == 0) mine[e] += __popc(same);
+        __syncwarp();
+    }
+    __syncthreads();
+    // Expert e: the sum over the warps, every warp's count replaced by what the warps before it brought.
+    for (int e = threadIdx.x; e < E; e += blockDim.x) {
+        int sum = 0;
+        for (int w = 0; w < 32; ++w) {
+            const int n = at[w * E + e];
+            at[w * E + e] = sum;
+            sum += n;
+        }
+        first[e] = sum;
+    }
+    __syncthreads();
+    if (warp == 0) {                   // running sum over the experts, 32 at a time
+        int base = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int n = e0 + lane < E ? first[e0 + lane] : 0;
+            int sum = n;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int up = __shfl_up_sync(0xffffffffu, sum, o);
+                if (lane >= o) sum += up;
+            }
+            if (e0 + lane < E) {
+                first[e0 + lane] = base + sum - n;
+                offsets[e0 + lane] = base + sum - n;
+            }
+            base += __shfl_sync(0xffffffffu, sum, 31);
+        }
+        if (lane == 0) offsets[E] = base;
+    }
+    __syncthreads();
+    for (int i = 0; i < steps; ++i) {
+        const int p = begin + 32 * i + lane, e = p < n_pairs ? ids[p] : E;
+        const unsigned same = __match_any_sync(0xffffffffu, e), before = same & ((1u << lane) - 1u);
+        if (e >= 0 && e < E) {
+            const int where = first[e] + mine[e] + __popc(before);
+            place[p] = where;
+            pair_at[where] = p;
+        }
+        __syncwarp();
+        if (e >= 0 && e < E && before == 0) mine[e] += __popc(same);
+        __syncwarp();
+    }
+}
+
 // ---------------------------------------------------------------- the experts' products
 struct ProductArgs {
     const void* a;             // first half: the rows h [T, lda]; second half: mid [pairs, lda]
@@ -573,6 +638,11 @@ extern "C" int lb_router_topk_biased(int dtype, const void* h, int64_t ldh, cons
 
 extern "C" int lb_expert_plan(const int32_t* ids, int n_pairs, int n_experts, int32_t* offsets, int32_t* place, int32_t* pair_at, void* stream) {
     LB_CHECK_ARG(n_pairs >= 0 && n_experts > 0 && n_experts <= 4096, "expert plan: bad sizes");
+    if (n_experts <= 256 && n_pairs > 256) {
+        LB_CHECK_CUDA(lb_launch_overlapped(expert_plan_wide_kernel, dim3(1), dim3(1024), (size_t)33 * n_experts * sizeof(int), static_cast<cudaStream_t>(stream), ids,
+                                           n_pairs, n_experts, offsets, place, pair_at));
+        return LB_OK;
+    }
     const int threads = 32 * max(1, min(32, n_experts));
     const int staged = (size_t)(n_experts + 1 + n_pairs) * sizeof(int) <= 48 * 1024 ? 1 : 0;
     LB_CHECK_CUDA(lb_launch_overlapped(expert_plan_kernel, dim3(1), dim3(threads), (size_t)(n_experts + 1 + (staged ? n_pairs : 0)) * sizeof(int),

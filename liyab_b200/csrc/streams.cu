@@ -80,13 +80,28 @@ __device__ __forceinline__ Vals<V> terms_at(const lb_output_terms& o, int t, int
         for (int i = 0; i < V; ++i) sum.v[i] = fmaf(o.scale[k], y.v[i], sum.v[i]);
     }
     if (o.pairs != nullptr) {
-        for (int k = 0; k < o.top; ++k) {
-            const int p = t * o.top + k, e = o.ids[p];
-            const float w = o.weights != nullptr ? o.weights[p] : 1.0f;
-            const Vals<V> y = e < o.n_real ? load_vals<V>(o.pairs + (size_t)(o.place != nullptr ? o.place[p] : p) * o.ldp + c)
-                                           : load_vals<V>(static_cast<const T*>(o.self) + (size_t)t * o.lds + c);
+        // Two choices at a time: their experts, weights and places together, then their rows together.
+        for (int k0 = 0; k0 < o.top; k0 += 2) {
+            int e[2], at[2];
+            float w[2];
 #pragma unroll
-            for (int i = 0; i < V; ++i) sum.v[i] = fmaf(w, y.v[i], sum.v[i]);
+            for (int k = 0; k < 2; ++k) {
+                const int p = t * o.top + min(k0 + k, o.top - 1);
+                e[k] = o.ids[p];
+                w[k] = o.weights != nullptr ? o.weights[p] : 1.0f;
+                at[k] = o.place != nullptr ? o.place[p] : p;
+            }
+            Vals<V> y[2];
+#pragma unroll
+            for (int k = 0; k < 2; ++k)
+                if (k0 + k < o.top)
+                    y[k] = e[k] < o.n_real ? load_vals<V>(o.pairs + (size_t)at[k] * o.ldp + c) : load_vals<V>(static_cast<const T*>(o.self) + (size_t)t * o.lds + c);
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                if (k0 + k >= o.top) break;
+#pragma unroll
+                for (int i = 0; i < V; ++i) sum.v[i] = fmaf(w[k], y[k].v[i], sum.v[i]);
+            }
         }
     }
     return sum;
@@ -121,27 +136,40 @@ __device__ __forceinline__ void route_row(const lb_router& r, const float* h, in
     float* best = c + n;
     int* taken = reinterpret_cast<int*>(best + r.groups);
     const T* R = static_cast<const T*>(r.matrix);
-    for (int e = warp; e < n; e += n_warps) {
-        const T* w = R + (size_t)e * width;
-        float acc = 0.0f;
-        if (width % 4 == 0 && (reinterpret_cast<uintptr_t>(R) & 15) == 0) {        // four values a lane and load, four loads in flight
-            for (int k0 = 4 * lane; k0 < width; k0 += 4 * 128) {
-                float4 a[4], b[4];
+    // A warp takes three experts at once, so that a row of the matrix is not a round trip to memory by itself.
+    for (int e0 = warp; e0 < n; e0 += 3 * n_warps) {
+        float acc[3] = {0.0f, 0.0f, 0.0f};
+        const T* w[3];
 #pragma unroll
-                for (int u = 0; u < 4; ++u) {
+        for (int q = 0; q < 3; ++q) w[q] = R + (size_t)min(e0 + q * n_warps, n - 1) * width;
+        if (width % 4 == 0 && (reinterpret_cast<uintptr_t>(R) & 15) == 0) {        // four values a lane and load
+            for (int k0 = 4 * lane; k0 < width; k0 += 4 * 64) {
+                float4 a[2], b[3][2];
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
                     const int k = k0 + 128 * u;
                     const bool in = k < width;
-                    b[u] = in ? load4<T>(w + k) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
                     a[u] = in ? load4<float>(h + k) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+                    for (int q = 0; q < 3; ++q) b[q][u] = in ? load4<T>(w[q] + k) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
                 }
 #pragma unroll
-                for (int u = 0; u < 4; ++u) acc = fmaf(a[u].x, b[u].x, fmaf(a[u].y, b[u].y, fmaf(a[u].z, b[u].z, fmaf(a[u].w, b[u].w, acc))));
+                for (int q = 0; q < 3; ++q)
+#pragma unroll
+                    for (int u = 0; u < 2; ++u)
+                        acc[q] = fmaf(a[u].x, b[q][u].x, fmaf(a[u].y, b[q][u].y, fmaf(a[u].z, b[q][u].z, fmaf(a[u].w, b[q][u].w, acc[q]))));
             }
         } else {
-            for (int k = lane; k < width; k += 32) acc = fmaf(h[k], lb_to_float(w[k]), acc);
+            for (int k = lane; k < width; k += 32)
+#pragma unroll
+                for (int q = 0; q < 3; ++q) acc[q] = fmaf(h[k], lb_to_float(w[q][k]), acc[q]);
         }
-        acc = lb_warp_sum(acc);
-        if (lane == 0) z[e] = r.bias != nullptr ? acc + r.bias[e] : acc;
+#pragma unroll
+        for (int q = 0; q < 3; ++q) {
+            const int e = e0 + q * n_warps;
+            const float v = lb_warp_sum(acc[q]);
+            if (lane == 0 && e < n) z[e] = r.bias != nullptr ? v + r.bias[e] : v;
+        }
     }
     __syncthreads();
     if (warp != 0) return;
@@ -220,8 +248,8 @@ __global__ void __launch_bounds__(512) router_choice_kernel(lb_router r, const T
 }
 
 // ---------------------------------------------------------------- the streams between two sublayers
-// A block per row.  MAXS: as many streams as a thread keeps (EXACT: S is MAXS).
-template <int V, int MAXS, bool EXACT, typename T>
+// A block per row.  MAXS: as many streams as a thread keeps (EXACT: S is MAXS); ROUTES: with a router.
+template <int V, int MAXS, bool EXACT, bool ROUTES, typename T>
 __global__ void __launch_bounds__(512) streams_join_kernel(lb_streams_args a, lb_output_terms o, lb_router r) {
     extern __shared__ __align__(16) float smem[];       // with a router: the row h, then the router's scratch
     __shared__ float hc[kMaxStreams * kMaxStreams + 2 * kMaxStreams];
@@ -236,14 +264,35 @@ __global__ void __launch_bounds__(512) streams_join_kernel(lb_streams_args a, lb
     if (goes_on)
         for (int i = threadIdx.x; i < S; i += blockDim.x) next[i] = a.next_in != nullptr ? a.next_in[i] : 1.0f;
     const float alpha = a.alpha != nullptr ? a.alpha[0] : 1.0f;
+    const int t = blockIdx.x, c_first = V * threadIdx.x;
+    // The thread's first columns of the old streams too, where a sublayer's output joins them: the launch that wrote them lies before that sublayer's.
+    Vals<V> x_early[EXACT ? MAXS : 1], g_early, gain_early, offset_early;
+    const bool early = EXACT && moves && c_first < W;
+    if (early) {
+#pragma unroll
+        for (int s = 0; s < (EXACT ? MAXS : 1); ++s) x_early[s] = load_vals<V>(a.x + (size_t)t * a.ldx + (size_t)s * W + c_first);
+        if (a.scale != nullptr) g_early = load_vals<V>(a.scale + c_first);
+        if (goes_on && a.alpha != nullptr) {
+            gain_early = load_vals<V>(a.gain + c_first);
+            offset_early = load_vals<V>(a.offset + c_first);
+        }
+    }
+    if (ROUTES && gridDim.x <= 64) {      // a few rows: the router's matrix starts on its way
+        const char* R = static_cast<const char*>(r.matrix);
+        const size_t bytes = (size_t)r.n_experts * W * sizeof(T);
+        for (size_t i = (size_t)threadIdx.x * 128; i < bytes && i < 64 * 1024; i += (size_t)blockDim.x * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(R + i));
+    }
     lb_wait_for_predecessor();
     lb_dependents_may_launch();
     __syncthreads();
-    const int t = blockIdx.x;
     float* xrow = a.x + (size_t)(a.rows != nullptr ? a.rows[t] : t) * a.ldx;
-    for (int c = V * threadIdx.x; c < W; c += V * blockDim.x) {
+    for (int c = c_first; c < W; c += V * blockDim.x) {
         Vals<V> x[MAXS];
-        if (a.fresh != nullptr) {
+        const bool have = early && c == c_first;
+        if (have) {
+#pragma unroll
+            for (int s = 0; s < (EXACT ? MAXS : 1); ++s) x[s] = x_early[s];
+        } else if (a.fresh != nullptr) {
             x[0] = load_vals<V>(a.fresh + (size_t)t * a.ldf + c);
 #pragma unroll
             for (int s = 1; s < MAXS; ++s) x[s] = x[0];
@@ -258,7 +307,7 @@ __global__ void __launch_bounds__(512) streams_join_kernel(lb_streams_args a, lb
         if (moves) {
             Vals<V> y = terms_at<V, T>(o, t, c);
             if (a.scale != nullptr) {
-                const Vals<V> g = load_vals<V>(a.scale + c);
+                const Vals<V> g = have ? g_early : load_vals<V>(a.scale + c);
 #pragma unroll
                 for (int i = 0; i < V; ++i) y.v[i] *= g.v[i];
             }
@@ -295,19 +344,20 @@ __global__ void __launch_bounds__(512) streams_join_kernel(lb_streams_args a, lb
         }
         if (!goes_on) continue;
         if (a.alpha != nullptr) {
-            const Vals<V> g = load_vals<V>(a.gain + c), b = load_vals<V>(a.offset + c);
+            const Vals<V> g = have ? gain_early : load_vals<V>(a.gain + c), b = have ? offset_early : load_vals<V>(a.offset + c);
 #pragma unroll
             for (int i = 0; i < V; ++i) u.v[i] = fmaf(tanhf(alpha * u.v[i]), g.v[i], b.v[i]);
         }
         store_vals<V>(static_cast<T*>(a.h) + (size_t)t * a.ldh + c, u);
-        if (r.matrix != nullptr) {
+        if (ROUTES) {
 #pragma unroll
             for (int i = 0; i < V; ++i) smem[c + i] = lb_to_float(lb_from_float<T>(u.v[i]));        // the router reads what the experts read
         }
     }
-    if (r.matrix == nullptr) return;
-    __syncthreads();
-    route_row<T>(r, smem, W, t, smem + (W + 3) / 4 * 4);
+    if constexpr (ROUTES) {
+        __syncthreads();
+        route_row<T>(r, smem, W, t, smem + (W + 3) / 4 * 4);
+    }
 }
 
 size_t router_floats(const lb_router& r) { return 2 * (size_t)r.n_experts + 2 * (size_t)r.groups; }
@@ -335,16 +385,16 @@ template <int V, typename T>
 int launch_join(const lb_streams_args& a, const lb_output_terms& o, const lb_router& r, int n_rows, cudaStream_t s) {
     const int pieces = a.width / V;
     int threads = min(512, max(32, (pieces + 31) / 32 * 32));
-    if (r.matrix != nullptr) threads = max(threads, 32 * min(8, r.n_experts));
+    if (r.matrix != nullptr) threads = max(threads, 32 * min(n_rows <= 148 ? 16 : 8, r.n_experts));
     const size_t smem = r.matrix != nullptr ? ((size_t)(a.width + 3) / 4 * 4 + router_floats(r)) * sizeof(float) : 0;
     LB_CHECK_ARG(smem <= 200 * 1024, "streams: rows of %d values with a router do not fit shared memory", a.width);
-#define LB_JOIN(MAXS, EXACT)                                                                                                                    \
-    do {                                                                                                                                        \
-        auto kernel = streams_join_kernel<V, MAXS, EXACT, T>;                                                                                   \
-        if (smem > 40 * 1024) LB_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));             \
-        LB_CHECK_CUDA(lb_launch_overlapped(kernel, dim3(n_rows), dim3(threads), smem, s, a, o, r));                                            \
-        return LB_OK;                                                                                                                           \
-    } while (0)
+    auto launch = [&](auto kernel) -> int {
+        if (smem > 40 * 1024) LB_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        LB_CHECK_CUDA(lb_launch_overlapped(kernel, dim3(n_rows), dim3(threads), smem, s, a, o, r));
+        return LB_OK;
+    };
+#define LB_JOIN(MAXS, EXACT) \
+    return r.matrix != nullptr ? launch(streams_join_kernel<V, MAXS, EXACT, true, T>) : launch(streams_join_kernel<V, MAXS, EXACT, false, T>)
     if constexpr (V == 1) {
         if (a.n_streams <= 4) LB_JOIN(4, false);
         LB_JOIN(kMaxStreams, false);

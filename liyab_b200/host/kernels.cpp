@@ -739,14 +739,10 @@ void channel_memory_rows(cudaStream_t s, const ChannelMemoryShape& m, const Chan
 void channel_memory_pieces(cudaStream_t s, Workspace* ws, const ChannelMemoryShape& m, const ChannelStep& step, const Rows& proj, const Rows& o, const Rows& heads) {
     const lb_channel_memory c = channel_of(m);
     const lb_channel_step t = channel_step_of(m, step, proj, o, heads);
-    const bool prepared = m.conv != nullptr || m.unit;
-    float* rows = prepared ? ws->get("channel_memory.rows", step.n_tokens, m.channels(), DType::F32).f32() : nullptr;
-    float* log_decay = ws->get("channel_memory.log_decay", step.n_tokens, static_cast<int64_t>(m.n_head) * m.dim, DType::F32).f32();
-    float* gate = m.g2.data != nullptr ? ws->get("channel_memory.gate", step.n_tokens, static_cast<int64_t>(m.n_head) * m.vdim, DType::F32).f32() : nullptr;
     const int64_t floats = lb_channel_memory_pieces_floats(step.n_tokens, step.n_seq, m.n_head, m.dim, m.vdim, m.delta ? 1 : 0);
     float* scratch = static_cast<float*>(ws->flat("channel_memory.pieces", floats, DType::F32));
-    check(lb_channel_memory_pieces(code(heads.dtype, "heads"), &c, &t, rows, log_decay, gate, scratch, step.n_tokens, step.n_seq, s), "channel_memory_pieces");
-    launches.fetch_add(3 + (m.g2.data != nullptr ? 1 : 0) + (prepared ? 1 : 0) + (m.conv != nullptr ? 1 : 0), std::memory_order_relaxed);
+    check(lb_channel_memory_pieces(code(heads.dtype, "heads"), &c, &t, scratch, step.n_tokens, step.n_seq, s), "channel_memory_pieces");
+    launches.fetch_add(2 + (m.conv != nullptr ? 1 : 0), std::memory_order_relaxed);
 }
 
 void sample(cudaStream_t s, const float* logits, int64_t row_stride, int n_rows, int vocab, const float* temperature,

@@ -240,7 +240,8 @@ private:
         const int64_t HE = static_cast<int64_t>(m.n_head) * m.vdim;
         Workspace& ws = *ctx.workspace;
         cudaStream_t s = ctx.stream();
-        const Rows pr = ws.get("channel_memory.proj", T, m.cols(), DType::F32);
+        // Rows on 16-byte borders whatever the number of columns, so that the product may store them in large pieces.
+        const Rows pr = ws.get("channel_memory.proj", T, (m.cols() + 7) / 8 * 8, DType::F32).columns(0, m.cols());
         kernels::linear(ctx.runtime, &ws, h, proj.weight, nullptr, pr, T, kernels::kNone, nullptr);
         const Rows heads = ws.get("channel_memory.heads", T, HE, ctx.runtime.dtype);
         Rows o;

@@ -930,7 +930,7 @@ declare("lb_router_choice", [_i, _p, _p, _l, _i, _i, _p])
 declare("lb_terms_sum", [_i, _p, _p, _l, _i, _i, _i, _p])
 declare("lb_expert_product_direct", [_i, _i, _p, _l, _p, _l, _p, _p, _p, _l, _i, _i, _i, _i, _i, _i, _f, _f, _p])
 declare("lb_channel_memory_rows", [_i, _p, _p, _i, _i, _p])
-declare("lb_channel_memory_pieces", [_i, _p, _p, _p, _p, _p, _p, _i, _i, _p])
+declare("lb_channel_memory_pieces", [_i, _p, _p, _p, _i, _i, _p])
 
 
 def output_terms(rows=(), scale=(), pairs: Optional[torch.Tensor] = None, place: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
@@ -1014,7 +1014,5 @@ def channel_memory(m: dict, proj: torch.Tensor, positions: torch.Tensor, tok_seq
     fn = lib().lb_channel_memory_pieces_floats
     fn.argtypes, fn.restype = [_i, _i, _i, _i, _i, _i], _l
     scratch = torch.full((fn(T, S, H, D, E, int(m["delta"])),), float("nan"), device=proj.device)
-    rows, decay, gate = (torch.full((T, n), float("nan"), device=proj.device) for n in (channels, H * D, H * E))
-    check(lib().lb_channel_memory_pieces(code, _c.byref(a), _c.byref(s), _dev(rows, "rows"), _dev(decay, "decay"), _dev(gate, "gate"), _dev(scratch, "scratch"), T, S,
-                                         stream_ptr()), "channel_memory_pieces")
+    check(lib().lb_channel_memory_pieces(code, _c.byref(a), _c.byref(s), _dev(scratch, "scratch"), T, S, stream_ptr()), "channel_memory_pieces")
     return heads
