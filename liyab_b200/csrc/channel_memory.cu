@@ -266,16 +266,30 @@ __device__ __forceinline__ bool find_piece(const int32_t* q_start, int n_seq, in
     return false;
 }
 
-// y[t][x] = sum_j m[t][j] v[j][x] for 8 rows t0 .. t0 + 7 of one column (m [32][36] lower triangular, v column x at stride ldv).
-__device__ __forceinline__ void tri_product(float (&y)[8], const float* m, const float* v, int ldv, int t0) {
+// acc[i][j] += a_i b_j over 4 x 4 results.
+__device__ __forceinline__ void outer4(float (&acc)[4][4], const float4& a, const float4& b) {
+    const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
-    for (int i = 0; i < 8; ++i) y[i] = 0.0f;
-    for (int j = 0; j < t0 + 8; j += 4) {
-        const float v0 = v[(size_t)j * ldv], v1 = v[(size_t)(j + 1) * ldv], v2 = v[(size_t)(j + 2) * ldv], v3 = v[(size_t)(j + 3) * ldv];
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const float4 r = *reinterpret_cast<const float4*>(m + (t0 + i) * 36 + j);
-            y[i] = fmaf(r.x, v0, fmaf(r.y, v1, fmaf(r.z, v2, fmaf(r.w, v3, y[i]))));
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+}
+// y[t][x] = sum_j m[t][j] v[j][x] for 4 rows from t0 and 4 columns (m [32][36] lower triangular, v at stride ldv, both on 16-byte borders).
+__device__ __forceinline__ void tri_product(float (&y)[4][4], const float* m, const float* v, int ldv, int t0) {
+    for (int j = 0; j < t0 + 4; j += 4) {
+        float4 r[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) r[i] = *reinterpret_cast<const float4*>(m + (t0 + i) * 36 + j);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const float4 b = *reinterpret_cast<const float4*>(v + (size_t)(j + k) * ldv);
+            const float bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float rv = k == 0 ? r[i].x : k == 1 ? r[i].y : k == 2 ? r[i].z : r[i].w;
+#pragma unroll
+                for (int x = 0; x < 4; ++x) y[i][x] = fmaf(rv, bv[x], y[i][x]);
+            }
         }
     }
 }
@@ -294,13 +308,32 @@ template <typename T>
 __device__ __forceinline__ void load_rank_chunk(float* xT, float* ws, const float* __restrict__ x, int64_t ldx, const T* __restrict__ map, int rank, int r0, int n_rows,
                                                 int n_cols) {
     const int n = min(32, rank - r0);
-    for (int i = threadIdx.x; i < 32 * 32; i += blockDim.x) {
-        const int t = i >> 5, r = i & 31;
-        xT[r * 36 + t] = t < n_rows && r < n ? x[(size_t)t * ldx + r0 + r] : 0.0f;
+    constexpr int B = 4;               // loads a thread has in flight before it stores the first
+    for (int i0 = threadIdx.x; i0 < 32 * 32; i0 += B * blockDim.x) {
+        float v[B];
+#pragma unroll
+        for (int k = 0; k < B; ++k) {
+            const int i = i0 + k * blockDim.x, t = i >> 5, r = i & 31;
+            v[k] = i < 32 * 32 && t < n_rows && r < n ? x[(size_t)t * ldx + r0 + r] : 0.0f;
+        }
+#pragma unroll
+        for (int k = 0; k < B; ++k) {
+            const int i = i0 + k * blockDim.x;
+            if (i < 32 * 32) xT[(i & 31) * 36 + (i >> 5)] = v[k];
+        }
     }
-    for (int i = threadIdx.x; i < n_cols * 32; i += blockDim.x) {
-        const int c = i >> 5, r = i & 31;
-        if (r < n) ws[c * 33 + r] = lb_to_float(map[(size_t)c * rank + r0 + r]);
+    for (int i0 = threadIdx.x; i0 < n_cols * 32; i0 += 2 * B * blockDim.x) {
+        T v[2 * B];
+#pragma unroll
+        for (int k = 0; k < 2 * B; ++k) {
+            const int i = i0 + k * blockDim.x, c = i >> 5, r = i & 31;
+            v[k] = i < n_cols * 32 && r < n ? map[(size_t)c * rank + r0 + r] : lb_from_float<T>(0.0f);
+        }
+#pragma unroll
+        for (int k = 0; k < 2 * B; ++k) {
+            const int i = i0 + k * blockDim.x;
+            if (i < n_cols * 32) ws[(i >> 5) * 33 + (i & 31)] = lb_to_float(v[k]);
+        }
     }
 }
 
@@ -318,7 +351,7 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
     lb_dependents_may_launch();
     int seq, piece;
     if (!find_piece(a.q_start, n_seq, blockIdx.x, &seq, &piece)) return;
-    const int h = blockIdx.y, D = m.dim, E = m.vdim, LD = D + 1, LE = E + 1, g = h / (m.n_head / m.kv_head), channels = channels_of(m);
+    const int h = blockIdx.y, D = m.dim, E = m.vdim, D4 = (D + 3) / 4 * 4, E4 = (E + 3) / 4 * 4, LD = D4 + 4, LE = E4 + 4, g = h / (m.n_head / m.kv_head), channels = channels_of(m);
     const int first = a.q_start[seq], row0 = first + piece * kPiece, n = min(kPiece, a.q_start[seq + 1] - row0), pos0 = a.positions[row0];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     float* Am = smem;                          // [32][36]; before the pairs the decays' inputs [32 r][36]
@@ -329,6 +362,13 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
     float* bs = ks + kPiece * LD;              // [32][LD] log decays, then their running sums
     float* vs = bs + kPiece * LD;              // [32][LE]
     float* fs = vs + kPiece * LE;              // [48][LD] rows with one half of a pair's exponential; before that the decays' map [D][33]
+    // Rows start on 16-byte borders, columns up to the next multiple of four are zeros.
+    if (D4 > D || E4 > E) {
+        for (int t = warp; t < kPiece; t += 8) {
+            if (lane < D4 - D) qs[t * LD + D + lane] = ks[t * LD + D + lane] = bs[t * LD + D + lane] = 0.0f;
+            if (lane < E4 - E) vs[t * LE + E + lane] = 0.0f;
+        }
+    }
     const PieceLayout l = piece_layout(D, E, DELTA);
     float* out = scratch + ((size_t)blockIdx.x * m.n_head + h) * l.total;
     const float* slot = a.state + (size_t)a.slots[seq] * m.slot_stride;
@@ -418,36 +458,30 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
     // The pairs.  Rows of the second half meet keys of the first through the border between them: exp(b_t - b_j) = exp(b_t - b_15) exp(b_15 - b_j), both
     // exponents at most 0, so those 256 pairs are plain products; pairs inside a half make their exponentials one by one.
     constexpr int kHalf = kPiece / 2;
-    for (int i = threadIdx.x; i < kHalf * D; i += blockDim.x) {
-        const int t = i / D, d = i - t * D;
-        const float border = bs[(kHalf - 1) * LD + d], e = fast_exp2(bs[(kHalf + t) * LD + d] - border);
-        fs[t * LD + d] = qs[(kHalf + t) * LD + d] * e;
-        if (DELTA) fs[(kHalf + t) * LD + d] = ks[(kHalf + t) * LD + d] * e;
-        fs[(2 * kHalf + t) * LD + d] = ks[t * LD + d] * fast_exp2(border - bs[t * LD + d]);
-    }
+    for (int t = warp; t < kHalf; t += 8)
+        for (int d = lane; d < D4; d += 32) {
+            const float border = bs[(kHalf - 1) * LD + d], e = fast_exp2(bs[(kHalf + t) * LD + d] - border);
+            fs[t * LD + d] = qs[(kHalf + t) * LD + d] * e;
+            if (DELTA) fs[(kHalf + t) * LD + d] = ks[(kHalf + t) * LD + d] * e;
+            fs[(2 * kHalf + t) * LD + d] = ks[t * LD + d] * fast_exp2(border - bs[t * LD + d]);
+        }
     __syncthreads();
+    auto dot4 = [](const float4& x, const float4& y, float sum) { return fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, sum)))); };
     {
         const int t = threadIdx.x >> 4, j = threadIdx.x & 15;
-        const float *qt = fs + t * LD, *kt = fs + (kHalf + t) * LD, *kj = fs + (2 * kHalf + j) * LD;
-        float p0 = 0.0f, p1 = 0.0f, a0 = 0.0f, a1 = 0.0f;
-        int d = 0;
+        const float4 *qt = reinterpret_cast<const float4*>(fs + t * LD), *kt = reinterpret_cast<const float4*>(fs + (kHalf + t) * LD);
+        const float4* kj = reinterpret_cast<const float4*>(fs + (2 * kHalf + j) * LD);
+        float p = 0.0f, av = 0.0f;
 #pragma unroll 4
-        for (; d + 1 < D; d += 2) {
-            p0 = fmaf(qt[d], kj[d], p0);
-            p1 = fmaf(qt[d + 1], kj[d + 1], p1);
-            if (DELTA) {
-                a0 = fmaf(kt[d], kj[d], a0);
-                a1 = fmaf(kt[d + 1], kj[d + 1], a1);
-            }
+        for (int d = 0; d < D4 / 4; ++d) {
+            const float4 k = kj[d];
+            p = dot4(qt[d], k, p);
+            if (DELTA) av = dot4(kt[d], k, av);
         }
-        if (d < D) {
-            p0 = fmaf(qt[d], kj[d], p0);
-            if (DELTA) a0 = fmaf(kt[d], kj[d], a0);
-        }
-        out[l.p + (kHalf + t) * kPiece + j] = (p0 + p1) * m.q_scale;
+        out[l.p + (kHalf + t) * kPiece + j] = p * m.q_scale;
         out[l.p + t * kPiece + kHalf + j] = 0.0f;
         if (DELTA) {
-            Am[(kHalf + t) * 36 + j] = a0 + a1;
+            Am[(kHalf + t) * 36 + j] = av;
             Am[t * 36 + kHalf + j] = 0.0f;
         }
     }
@@ -455,12 +489,15 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
         const int half = lane >> 4 << 4, t = half + r, j = half + (lane & 15);
         float p = 0.0f, av = 0.0f;
         if (j <= t && t < n) {
-            const float *qt = qs + t * LD, *kt = ks + t * LD, *bt = bs + t * LD, *kj = ks + j * LD, *bj = bs + j * LD;
-#pragma unroll 4
-            for (int d = 0; d < D; ++d) {
-                const float e = fast_exp2(bt[d] - bj[d]) * kj[d];
-                p = fmaf(qt[d], e, p);
-                if (DELTA) av = fmaf(kt[d], e, av);
+            const float4 *qt = reinterpret_cast<const float4*>(qs + t * LD), *kt = reinterpret_cast<const float4*>(ks + t * LD);
+            const float4 *bt = reinterpret_cast<const float4*>(bs + t * LD), *kj = reinterpret_cast<const float4*>(ks + j * LD);
+            const float4* bj = reinterpret_cast<const float4*>(bs + j * LD);
+#pragma unroll 2
+            for (int d = 0; d < D4 / 4; ++d) {
+                const float4 x = bt[d], y = bj[d], k = kj[d];
+                const float4 e = make_float4(fast_exp2(x.x - y.x) * k.x, fast_exp2(x.y - y.y) * k.y, fast_exp2(x.z - y.z) * k.z, fast_exp2(x.w - y.w) * k.w);
+                p = dot4(qt[d], e, p);
+                if (DELTA) av = dot4(kt[d], e, av);
             }
         }
         out[l.p + t * kPiece + j] = p * m.q_scale;
@@ -482,52 +519,55 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
             M[t * 36 + lane] = x[t];
         }
     } else {
-        const int first_i = DELTA ? threadIdx.x - 32 : threadIdx.x, step = DELTA ? blockDim.x - 32 : blockDim.x;
-        for (int i = first_i; i < kPiece * D; i += step) {
-            const int t = i / D, d = i - t * D;
-            const float b = bs[t * LD + d], b_last = bs[(kPiece - 1) * LD + d], k = ks[t * LD + d], e = fast_exp2(b), kb = fast_exp2(b_last - b) * k;
-            out[l.q + i] = qs[t * LD + d] * m.q_scale * e;
-            if (DELTA) {
-                out[l.b + i] = kb;
-                ks[t * LD + d] = k * e;        // K~
-            } else {
-                ks[t * LD + d] = kb;
+        for (int t = DELTA ? warp - 1 : warp; t < kPiece; t += DELTA ? 7 : 8)
+            for (int d = lane; d < D; d += 32) {
+                const float b = bs[t * LD + d], b_last = bs[(kPiece - 1) * LD + d], k = ks[t * LD + d], e = fast_exp2(b), kb = fast_exp2(b_last - b) * k;
+                out[l.q + t * D + d] = qs[t * LD + d] * m.q_scale * e;
+                if (DELTA) {
+                    out[l.b + t * D + d] = kb;
+                    ks[t * LD + d] = k * e;        // K~
+                } else {
+                    ks[t * LD + d] = kb;
+                }
+                if (t == 0) out[l.keep + d] = fast_exp2(b_last);
             }
-            if (t == 0) out[l.keep + d] = fast_exp2(b_last);
-        }
     }
     __syncthreads();
     if (DELTA) {
-        // M K~ and M V: thread (column, eight rows).
-        for (int i = threadIdx.x; i < 4 * (D + E); i += blockDim.x) {
-            const int part = i / (D + E), x = i - part * (D + E), t0 = 8 * part;
-            float y[8];
-            if (x < D) tri_product(y, M, ks + x, LD, t0);
-            else tri_product(y, M, vs + (x - D), LE, t0);
-            if (x < D) {
-                float4* dst = reinterpret_cast<float4*>(out + l.w + x * kPiece + t0);
-                dst[0] = make_float4(y[0], y[1], y[2], y[3]);
-                dst[1] = make_float4(y[4], y[5], y[6], y[7]);
-            } else {
+        // M K~ and M V: thread (four rows, four columns).
+        const int tiles_d = D4 / 4, tiles = tiles_d + E4 / 4;
+        for (int i = threadIdx.x; i < 8 * tiles; i += blockDim.x) {
+            const int part = i / tiles, x = i - part * tiles, t0 = 4 * part;
+            float y[4][4] = {};
+            if (x < tiles_d) tri_product(y, M, ks + 4 * x, LD, t0);
+            else tri_product(y, M, vs + 4 * (x - tiles_d), LE, t0);
 #pragma unroll
-                for (int k = 0; k < 8; ++k) out[l.u + (t0 + k) * E + (x - D)] = y[k];
+            for (int k = 0; k < 4; ++k) {
+                if (x < tiles_d) {
+                    if (4 * x + k < D) *reinterpret_cast<float4*>(out + l.w + (4 * x + k) * kPiece + t0) = make_float4(y[0][k], y[1][k], y[2][k], y[3][k]);
+                } else {
+                    const int c = 4 * (x - tiles_d);
+#pragma unroll
+                    for (int v = 0; v < 4; ++v)
+                        if (c + v < E) out[l.u + (t0 + k) * E + c + v] = y[k][v];
+                }
             }
         }
     } else {
-        for (int i = threadIdx.x; i < kPiece * E; i += blockDim.x) out[l.u + i] = vs[i / E * LE + i % E];
-        // The piece's own sum: thread (column, eight channels).
-        const int parts = (D + 7) / 8;
-        for (int i = threadIdx.x; i < parts * E; i += blockDim.x) {
-            const int part = i / E, x = i - part * E, d0 = 8 * part;
-            float y[8] = {};
-            for (int j = 0; j < n; ++j) {
-                const float v = vs[j * LE + x];
+        for (int t = warp; t < kPiece; t += 8)
+            for (int x = lane; x < E; x += 32) out[l.u + t * E + x] = vs[t * LE + x];
+        // The piece's own sum: thread (four channels, four columns).
+        const int tiles_e = E4 / 4;
+        for (int i = threadIdx.x; i < D4 / 4 * tiles_e; i += blockDim.x) {
+            const int part = i / tiles_e, x = 4 * (i - part * tiles_e), d0 = 4 * part;
+            float y[4][4] = {};
+#pragma unroll 4
+            for (int j = 0; j < n; ++j) outer4(y, *reinterpret_cast<const float4*>(ks + j * LD + d0), *reinterpret_cast<const float4*>(vs + j * LE + x));
 #pragma unroll
-                for (int k = 0; k < 8; ++k) y[k] = fmaf(ks[j * LD + min(d0 + k, D - 1)], v, y[k]);
-            }
+            for (int k = 0; k < 4; ++k)
 #pragma unroll
-            for (int k = 0; k < 8; ++k)
-                if (d0 + k < D) out[l.s + (d0 + k) * E + x] = y[k];
+                for (int v = 0; v < 4; ++v)
+                    if (d0 + k < D && x + v < E) out[l.s + (d0 + k) * E + x + v] = y[k][v];
         }
     }
 }
@@ -687,7 +727,7 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(lb_channel_memory m, St
 }
 
 // The outputs of a piece with the heads' norm and gate.  Thread (c, tg) owns column c for the R rows tg R .. tg R + R - 1; the state before the piece
-// comes to shared memory (`staged`) while the gates are made.
+// and U come to shared memory (`staged`) while the gates are made.
 template <typename T, int R>
 __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory m, StepArgs a, float* __restrict__ scratch, int n_seq, int staged) {
     extern __shared__ __align__(16) float smem[];
@@ -717,7 +757,11 @@ __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory 
             else qs[i] = 0.0f;
         }
     }
-    if (staged) cm_fetch(Ss, in + l.s, D * E);
+    float* Us = Ss + (D * E + 3) / 4 * 4;      // [32][E]
+    if (staged) {
+        cm_fetch(Ss, in + l.s, D * E);
+        cm_fetch(Us, in + l.u, kPiece * E);
+    }
     cm_cp_commit();
     const int c = threadIdx.x % EP, t0 = threadIdx.x / EP * R;
     float gate[R];
@@ -732,8 +776,19 @@ __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory 
                 const int count = min(32, m.gate_rank - r0);
                 for (int r = 0; r < count; ++r) {
                     const float w = gw[c * 33 + r];
+                    if constexpr (R % 4 == 0) {
 #pragma unroll
-                    for (int i = 0; i < R; ++i) gate[i] = fmaf(w, xT[r * 36 + t0 + i], gate[i]);
+                        for (int i = 0; i < R; i += 4) {
+                            const float4 x = *reinterpret_cast<const float4*>(xT + r * 36 + t0 + i);
+                            gate[i] = fmaf(w, x.x, gate[i]);
+                            gate[i + 1] = fmaf(w, x.y, gate[i + 1]);
+                            gate[i + 2] = fmaf(w, x.z, gate[i + 2]);
+                            gate[i + 3] = fmaf(w, x.w, gate[i + 3]);
+                        }
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < R; ++i) gate[i] = fmaf(w, xT[r * 36 + t0 + i], gate[i]);
+                    }
                 }
             }
         }
@@ -759,7 +814,7 @@ __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory 
                 y[i] = fmaf(q.x, s[0], fmaf(q.y, s[1], fmaf(q.z, s[2], fmaf(q.w, s[3], y[i]))));
             }
         }
-        const float* u = in + l.u + c;
+        const float* u = (staged ? Us : in + l.u) + c;
         const int last = min(n, t0 + R);       // rows after the last of this thread's are not seen
 #pragma unroll 2
         for (int j = 0; j < last; j += 4) {
@@ -863,7 +918,7 @@ extern "C" int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memo
         return LB_OK;
     };
     const dim3 grid(pieces, m.n_head);
-    const size_t own = (2 * kPiece * 36 + kPiece + (3 * (size_t)kPiece + 48) * (D + 1) + (size_t)kPiece * (E + 1)) * sizeof(float);
+    const size_t own = (2 * kPiece * 36 + kPiece + (3 * (size_t)kPiece + 48) * (d4 + 4) + (size_t)kPiece * ((E + 3) / 4 * 4 + 4)) * sizeof(float);
     constexpr int VT = 16;
     if (m.delta) {
         if (int rc = dtype == LB_F32 ? launch(channel_pieces_kernel<float, true>, grid, own, m, a, scratch, n_seq)
@@ -879,7 +934,7 @@ extern "C" int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memo
     if (m.conv != nullptr)
         if (int rc = launch_ring(m, a, n_seq, s)) return rc;
     const size_t base = (kPiece * kPiece + (size_t)kPiece * d4 + 32 * 36 + ((E > 32 ? E : 32) * 33 + 35) / 4 * 4) * sizeof(float);
-    const size_t with_state = base + (size_t)D * E * sizeof(float);
+    const size_t with_state = base + ((size_t)(D * E + 3) / 4 * 4 + (size_t)kPiece * E) * sizeof(float);
     const int staged = with_state <= 110 * 1024 ? 1 : 0;
     const size_t outs = staged ? with_state : base;
 #define LB_OUTPUTS(T)                                                                                 \

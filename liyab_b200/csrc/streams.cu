@@ -126,53 +126,63 @@ __global__ void __launch_bounds__(256) terms_sum_kernel(lb_output_terms o, float
 }
 
 // ---------------------------------------------------------------- router
-// Row t's experts from its input h (in shared memory) by the whole block: a warp per expert for the sums, then warp 0 chooses.
-// smem: z [n], c [n], best [groups], taken [groups] (int).
-template <typename T>
-__device__ __forceinline__ void route_row(const lb_router& r, const float* h, int width, int t, float* smem) {
+// The experts of rows t0 .. t0 + ROWS - 1 from their inputs h (in shared memory, ldh floats apart) by the whole block: the sums with a warp per three
+// experts, all rows against every row of the matrix it reads, then a warp a row chooses.
+// smem, per row: z [n], c [n], best [groups], taken [groups] (int).
+template <int ROWS, typename T>
+__device__ __forceinline__ void route_rows(const lb_router& r, const float* h, int ldh, int width, int t0, int n_rows, float* smem) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5, n = r.n_experts;
-    float* z = smem;
-    float* c = z + n;
-    float* best = c + n;
-    int* taken = reinterpret_cast<int*>(best + r.groups);
+    const int per_row = 2 * n + 2 * r.groups;
     const T* R = static_cast<const T*>(r.matrix);
-    // A warp takes three experts at once, so that a row of the matrix is not a round trip to memory by itself.
     for (int e0 = warp; e0 < n; e0 += 3 * n_warps) {
-        float acc[3] = {0.0f, 0.0f, 0.0f};
+        float acc[3][ROWS];
         const T* w[3];
 #pragma unroll
-        for (int q = 0; q < 3; ++q) w[q] = R + (size_t)min(e0 + q * n_warps, n - 1) * width;
+        for (int q = 0; q < 3; ++q) {
+            w[q] = R + (size_t)min(e0 + q * n_warps, n - 1) * width;
+#pragma unroll
+            for (int i = 0; i < ROWS; ++i) acc[q][i] = 0.0f;
+        }
         if (width % 4 == 0 && (reinterpret_cast<uintptr_t>(R) & 15) == 0) {        // four values a lane and load
             for (int k0 = 4 * lane; k0 < width; k0 += 4 * 64) {
-                float4 a[2], b[3][2];
+                float4 b[3][2];
 #pragma unroll
-                for (int u = 0; u < 2; ++u) {
-                    const int k = k0 + 128 * u;
-                    const bool in = k < width;
-                    a[u] = in ? load4<float>(h + k) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                for (int u = 0; u < 2; ++u)
 #pragma unroll
-                    for (int q = 0; q < 3; ++q) b[q][u] = in ? load4<T>(w[q] + k) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                }
+                    for (int q = 0; q < 3; ++q) b[q][u] = k0 + 128 * u < width ? load4<T>(w[q] + k0 + 128 * u) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
-                for (int q = 0; q < 3; ++q)
+                for (int i = 0; i < ROWS; ++i)
 #pragma unroll
-                    for (int u = 0; u < 2; ++u)
-                        acc[q] = fmaf(a[u].x, b[q][u].x, fmaf(a[u].y, b[q][u].y, fmaf(a[u].z, b[q][u].z, fmaf(a[u].w, b[q][u].w, acc[q]))));
+                    for (int u = 0; u < 2; ++u) {
+                        if (k0 + 128 * u >= width) break;
+                        const float4 a = load4<float>(h + (size_t)i * ldh + k0 + 128 * u);
+#pragma unroll
+                        for (int q = 0; q < 3; ++q) acc[q][i] = fmaf(a.x, b[q][u].x, fmaf(a.y, b[q][u].y, fmaf(a.z, b[q][u].z, fmaf(a.w, b[q][u].w, acc[q][i]))));
+                    }
             }
         } else {
             for (int k = lane; k < width; k += 32)
 #pragma unroll
-                for (int q = 0; q < 3; ++q) acc[q] = fmaf(h[k], lb_to_float(w[q][k]), acc[q]);
+                for (int q = 0; q < 3; ++q)
+#pragma unroll
+                    for (int i = 0; i < ROWS; ++i) acc[q][i] = fmaf(h[(size_t)i * ldh + k], lb_to_float(w[q][k]), acc[q][i]);
         }
 #pragma unroll
-        for (int q = 0; q < 3; ++q) {
-            const int e = e0 + q * n_warps;
-            const float v = lb_warp_sum(acc[q]);
-            if (lane == 0 && e < n) z[e] = r.bias != nullptr ? v + r.bias[e] : v;
-        }
+        for (int q = 0; q < 3; ++q)
+#pragma unroll
+            for (int i = 0; i < ROWS; ++i) {
+                const int e = e0 + q * n_warps;
+                const float v = lb_warp_sum(acc[q][i]);
+                if (lane == 0 && e < n) smem[i * per_row + e] = r.bias != nullptr ? v + r.bias[e] : v;
+            }
     }
     __syncthreads();
-    if (warp != 0) return;
+    const int t = t0 + warp;
+    if (warp >= ROWS || t >= n_rows) return;
+    float* z = smem + warp * per_row;
+    float* c = z + n;
+    float* best = c + n;
+    int* taken = reinterpret_cast<int*>(best + r.groups);
     float top_z = -CUDART_INF_F, sum = 0.0f;
     if (r.softmax) {
         for (int e = lane; e < n; e += 32) top_z = fmaxf(top_z, z[e]);
@@ -244,14 +254,14 @@ __global__ void __launch_bounds__(512) router_choice_kernel(lb_router r, const T
     const int t = blockIdx.x;
     for (int c = threadIdx.x; c < width; c += blockDim.x) smem[c] = lb_to_float(h[(size_t)t * ldh + c]);
     __syncthreads();
-    route_row<T>(r, smem, width, t, smem + (width + 3) / 4 * 4);
+    route_rows<1, T>(r, smem, 0, width, t, t + 1, smem + (width + 3) / 4 * 4);
 }
 
 // ---------------------------------------------------------------- the streams between two sublayers
-// A block per row.  MAXS: as many streams as a thread keeps (EXACT: S is MAXS); ROUTES: with a router.
-template <int V, int MAXS, bool EXACT, bool ROUTES, typename T>
-__global__ void __launch_bounds__(512) streams_join_kernel(lb_streams_args a, lb_output_terms o, lb_router r) {
-    extern __shared__ __align__(16) float smem[];       // with a router: the row h, then the router's scratch
+// A block per ROWS rows.  MAXS: as many streams as a thread keeps (EXACT: S is MAXS); ROUTES: with a router.
+template <int V, int MAXS, bool EXACT, int ROWS, bool ROUTES, typename T>
+__global__ void __launch_bounds__(512) streams_join_kernel(lb_streams_args a, lb_output_terms o, lb_router r, int n_rows) {
+    extern __shared__ __align__(16) float smem[];       // with a router: the rows h, then the router's scratch
     __shared__ float hc[kMaxStreams * kMaxStreams + 2 * kMaxStreams];
     const int S = EXACT ? MAXS : a.n_streams, W = a.width;
     float* mix = hc;
@@ -264,13 +274,13 @@ __global__ void __launch_bounds__(512) streams_join_kernel(lb_streams_args a, lb
     if (goes_on)
         for (int i = threadIdx.x; i < S; i += blockDim.x) next[i] = a.next_in != nullptr ? a.next_in[i] : 1.0f;
     const float alpha = a.alpha != nullptr ? a.alpha[0] : 1.0f;
-    const int t = blockIdx.x, c_first = V * threadIdx.x;
+    const int t0 = blockIdx.x * ROWS, c_first = V * threadIdx.x;
     // The thread's first columns of the old streams too, where a sublayer's output joins them: the launch that wrote them lies before that sublayer's.
     Vals<V> x_early[EXACT ? MAXS : 1], g_early, gain_early, offset_early;
-    const bool early = EXACT && moves && c_first < W;
+    const bool early = EXACT && ROWS == 1 && moves && c_first < W;
     if (early) {
 #pragma unroll
-        for (int s = 0; s < (EXACT ? MAXS : 1); ++s) x_early[s] = load_vals<V>(a.x + (size_t)t * a.ldx + (size_t)s * W + c_first);
+        for (int s = 0; s < (EXACT ? MAXS : 1); ++s) x_early[s] = load_vals<V>(a.x + (size_t)t0 * a.ldx + (size_t)s * W + c_first);
         if (a.scale != nullptr) g_early = load_vals<V>(a.scale + c_first);
         if (goes_on && a.alpha != nullptr) {
             gain_early = load_vals<V>(a.gain + c_first);
@@ -285,78 +295,81 @@ __global__ void __launch_bounds__(512) streams_join_kernel(lb_streams_args a, lb
     lb_wait_for_predecessor();
     lb_dependents_may_launch();
     __syncthreads();
-    float* xrow = a.x + (size_t)(a.rows != nullptr ? a.rows[t] : t) * a.ldx;
-    for (int c = c_first; c < W; c += V * blockDim.x) {
-        Vals<V> x[MAXS];
-        const bool have = early && c == c_first;
-        if (have) {
+    const int W4 = (W + 3) / 4 * 4;
+    for (int t = t0; t < min(t0 + ROWS, n_rows); ++t) {
+        float* xrow = a.x + (size_t)(a.rows != nullptr ? a.rows[t] : t) * a.ldx;
+        for (int c = c_first; c < W; c += V * blockDim.x) {
+            Vals<V> x[MAXS];
+            const bool have = early && c == c_first;
+            if (have) {
 #pragma unroll
-            for (int s = 0; s < (EXACT ? MAXS : 1); ++s) x[s] = x_early[s];
-        } else if (a.fresh != nullptr) {
-            x[0] = load_vals<V>(a.fresh + (size_t)t * a.ldf + c);
+                for (int s = 0; s < (EXACT ? MAXS : 1); ++s) x[s] = x_early[s];
+            } else if (a.fresh != nullptr) {
+                x[0] = load_vals<V>(a.fresh + (size_t)t * a.ldf + c);
 #pragma unroll
-            for (int s = 1; s < MAXS; ++s) x[s] = x[0];
-        } else {
+                for (int s = 1; s < MAXS; ++s) x[s] = x[0];
+            } else {
 #pragma unroll
-            for (int s = 0; s < MAXS; ++s)
-                if (EXACT || s < S) x[s] = load_vals<V>(xrow + (size_t)s * W + c);
-        }
-        Vals<V> u;
-#pragma unroll
-        for (int i = 0; i < V; ++i) u.v[i] = 0.0f;
-        if (moves) {
-            Vals<V> y = terms_at<V, T>(o, t, c);
-            if (a.scale != nullptr) {
-                const Vals<V> g = have ? g_early : load_vals<V>(a.scale + c);
-#pragma unroll
-                for (int i = 0; i < V; ++i) y.v[i] *= g.v[i];
+                for (int s = 0; s < MAXS; ++s)
+                    if (EXACT || s < S) x[s] = load_vals<V>(xrow + (size_t)s * W + c);
             }
+            Vals<V> u;
+#pragma unroll
+            for (int i = 0; i < V; ++i) u.v[i] = 0.0f;
+            if (moves) {
+                Vals<V> y = terms_at<V, T>(o, t, c);
+                if (a.scale != nullptr) {
+                    const Vals<V> g = have ? g_early : load_vals<V>(a.scale + c);
+#pragma unroll
+                    for (int i = 0; i < V; ++i) y.v[i] *= g.v[i];
+                }
 #pragma unroll(EXACT ? MAXS : 1)
-            for (int q = 0; q < S; ++q) {
-                Vals<V> z;
+                for (int q = 0; q < S; ++q) {
+                    Vals<V> z;
 #pragma unroll
-                for (int i = 0; i < V; ++i) z.v[i] = to[q] * y.v[i];
+                    for (int i = 0; i < V; ++i) z.v[i] = to[q] * y.v[i];
 #pragma unroll
-                for (int s = 0; s < MAXS; ++s) {
-                    if (!EXACT && s >= S) break;
-                    const float m = mix[s * S + q];
+                    for (int s = 0; s < MAXS; ++s) {
+                        if (!EXACT && s >= S) break;
+                        const float m = mix[s * S + q];
 #pragma unroll
-                    for (int i = 0; i < V; ++i) z.v[i] = fmaf(m, x[s].v[i], z.v[i]);
+                        for (int i = 0; i < V; ++i) z.v[i] = fmaf(m, x[s].v[i], z.v[i]);
+                    }
+                    store_vals<V>(xrow + (size_t)q * W + c, z);
+                    if (goes_on) {
+                        const float n = next[q];
+#pragma unroll
+                        for (int i = 0; i < V; ++i) u.v[i] = fmaf(n, z.v[i], u.v[i]);
+                    }
                 }
-                store_vals<V>(xrow + (size_t)q * W + c, z);
-                if (goes_on) {
-                    const float n = next[q];
+            } else {
 #pragma unroll
-                    for (int i = 0; i < V; ++i) u.v[i] = fmaf(n, z.v[i], u.v[i]);
+                for (int q = 0; q < MAXS; ++q) {
+                    if (!EXACT && q >= S) break;
+                    if (a.fresh != nullptr) store_vals<V>(xrow + (size_t)q * W + c, x[q]);
+                    if (goes_on) {
+                        const float n = next[q];
+#pragma unroll
+                        for (int i = 0; i < V; ++i) u.v[i] = fmaf(n, x[q].v[i], u.v[i]);
+                    }
                 }
             }
-        } else {
+            if (!goes_on) continue;
+            if (a.alpha != nullptr) {
+                const Vals<V> g = have ? gain_early : load_vals<V>(a.gain + c), b = have ? offset_early : load_vals<V>(a.offset + c);
 #pragma unroll
-            for (int q = 0; q < MAXS; ++q) {
-                if (!EXACT && q >= S) break;
-                if (a.fresh != nullptr) store_vals<V>(xrow + (size_t)q * W + c, x[q]);
-                if (goes_on) {
-                    const float n = next[q];
-#pragma unroll
-                    for (int i = 0; i < V; ++i) u.v[i] = fmaf(n, x[q].v[i], u.v[i]);
-                }
+                for (int i = 0; i < V; ++i) u.v[i] = fmaf(tanhf(alpha * u.v[i]), g.v[i], b.v[i]);
             }
-        }
-        if (!goes_on) continue;
-        if (a.alpha != nullptr) {
-            const Vals<V> g = have ? gain_early : load_vals<V>(a.gain + c), b = have ? offset_early : load_vals<V>(a.offset + c);
+            store_vals<V>(static_cast<T*>(a.h) + (size_t)t * a.ldh + c, u);
+            if (ROUTES) {
 #pragma unroll
-            for (int i = 0; i < V; ++i) u.v[i] = fmaf(tanhf(alpha * u.v[i]), g.v[i], b.v[i]);
-        }
-        store_vals<V>(static_cast<T*>(a.h) + (size_t)t * a.ldh + c, u);
-        if (ROUTES) {
-#pragma unroll
-            for (int i = 0; i < V; ++i) smem[c + i] = lb_to_float(lb_from_float<T>(u.v[i]));        // the router reads what the experts read
+                for (int i = 0; i < V; ++i) smem[(t - t0) * W4 + c + i] = lb_to_float(lb_from_float<T>(u.v[i]));        // the router reads what the experts read
+            }
         }
     }
     if constexpr (ROUTES) {
         __syncthreads();
-        route_row<T>(r, smem, W, t, smem + (W + 3) / 4 * 4);
+        route_rows<ROWS, T>(r, smem, W4, W, t0, n_rows, smem + ROWS * W4);
     }
 }
 
@@ -384,17 +397,21 @@ int check_terms(const lb_output_terms& o) {
 template <int V, typename T>
 int launch_join(const lb_streams_args& a, const lb_output_terms& o, const lb_router& r, int n_rows, cudaStream_t s) {
     const int pieces = a.width / V;
+    // Steps of many rows route four rows a block: they share what the block reads of the router's matrix, and four warps choose at once.
+    const int rows = r.matrix != nullptr && n_rows > 148 && (size_t)4 * (a.width + router_floats(r)) * sizeof(float) <= 48 * 1024 ? 4 : 1;
     int threads = min(512, max(32, (pieces + 31) / 32 * 32));
-    if (r.matrix != nullptr) threads = max(threads, 32 * min(n_rows <= 148 ? 16 : 8, r.n_experts));
-    const size_t smem = r.matrix != nullptr ? ((size_t)(a.width + 3) / 4 * 4 + router_floats(r)) * sizeof(float) : 0;
+    if (r.matrix != nullptr) threads = max(threads, 32 * max(rows, min(n_rows <= 148 ? 16 : 8, r.n_experts)));
+    const size_t smem = r.matrix != nullptr ? rows * ((size_t)(a.width + 3) / 4 * 4 + router_floats(r)) * sizeof(float) : 0;
     LB_CHECK_ARG(smem <= 200 * 1024, "streams: rows of %d values with a router do not fit shared memory", a.width);
     auto launch = [&](auto kernel) -> int {
         if (smem > 40 * 1024) LB_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        LB_CHECK_CUDA(lb_launch_overlapped(kernel, dim3(n_rows), dim3(threads), smem, s, a, o, r));
+        LB_CHECK_CUDA(lb_launch_overlapped(kernel, dim3((n_rows + rows - 1) / rows), dim3(threads), smem, s, a, o, r, n_rows));
         return LB_OK;
     };
-#define LB_JOIN(MAXS, EXACT) \
-    return r.matrix != nullptr ? launch(streams_join_kernel<V, MAXS, EXACT, true, T>) : launch(streams_join_kernel<V, MAXS, EXACT, false, T>)
+#define LB_JOIN(MAXS, EXACT)                                                                    \
+    return r.matrix == nullptr ? launch(streams_join_kernel<V, MAXS, EXACT, 1, false, T>)       \
+           : rows == 1         ? launch(streams_join_kernel<V, MAXS, EXACT, 1, true, T>)        \
+                               : launch(streams_join_kernel<V, MAXS, EXACT, 4, true, T>)
     if constexpr (V == 1) {
         if (a.n_streams <= 4) LB_JOIN(4, false);
         LB_JOIN(kMaxStreams, false);
