@@ -233,21 +233,24 @@ __global__ void __launch_bounds__(256) channel_ring_kernel(lb_channel_memory m, 
 }
 
 // ---------------------------------------------------------------- pieces of 32 rows
+// Floats from the start of a (piece, head)'s scratch.  Under the delta rule U and the state lie in tiles of 16 value columns, as the scan's blocks read
+// and write them: [tile][32][16] and [tile][dim][16]; without it [32][vdim] and [dim][vdim].
+constexpr int kTileE = 16;
 struct PieceLayout {
-    int64_t p, q, keep, b, w, u, s, total;      // floats from the start of a (piece, head)'s scratch
+    int64_t p, q, keep, b, w, u, s, total;
 };
 __host__ __device__ inline PieceLayout piece_layout(int D, int E, int delta) {
-    auto up = [](int64_t n) { return (n + 3) / 4 * 4; };
     PieceLayout l{};
     int64_t at = 0;
-    auto take = [&](int64_t n) { const int64_t r = at; at += up(n); return r; };
+    auto take = [&](int64_t n) { const int64_t r = at; at += (n + 3) / 4 * 4; return r; };
+    const int64_t D4 = (D + 3) / 4 * 4, wide = delta ? (E + kTileE - 1) / kTileE * kTileE : E;
     l.p = take(kPiece * kPiece);                // P(t, j)
     l.q = take(kPiece * D);                     // exp(b_t) q_t
     l.keep = take(D);                           // exp(b_n)
-    l.b = take(delta ? kPiece * D : 0);         // exp(b_n - b_j) k_j
-    l.w = take(delta ? kPiece * D : 0);         // M K~, transposed: [D][32]
-    l.u = take(kPiece * E);                     // V, or under the delta rule M V and after the scan U
-    l.s = take((int64_t)D * E);                 // without the delta rule the piece's own sum; after the scan the state before the piece
+    l.b = take(delta ? kPiece * D4 : 0);        // exp(b_n - b_j) k_j, rows of D4
+    l.w = take(delta ? kPiece * D : 0);         // M K~, transposed: [dim][32]
+    l.u = take(kPiece * wide);                  // V, or under the delta rule M V and after the scan U
+    l.s = take(D * wide);                       // without the delta rule the piece's own sum; after the scan the state before the piece
     l.total = at;
     return l;
 }
@@ -520,16 +523,16 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
         }
     } else {
         for (int t = DELTA ? warp - 1 : warp; t < kPiece; t += DELTA ? 7 : 8)
-            for (int d = lane; d < D; d += 32) {
+            for (int d = lane; d < (DELTA ? D4 : D); d += 32) {
                 const float b = bs[t * LD + d], b_last = bs[(kPiece - 1) * LD + d], k = ks[t * LD + d], e = fast_exp2(b), kb = fast_exp2(b_last - b) * k;
-                out[l.q + t * D + d] = qs[t * LD + d] * m.q_scale * e;
+                if (d < D) out[l.q + t * D + d] = qs[t * LD + d] * m.q_scale * e;
                 if (DELTA) {
-                    out[l.b + t * D + d] = kb;
+                    out[l.b + t * D4 + d] = kb;
                     ks[t * LD + d] = k * e;        // K~
                 } else {
                     ks[t * LD + d] = kb;
                 }
-                if (t == 0) out[l.keep + d] = fast_exp2(b_last);
+                if (t == 0 && d < D) out[l.keep + d] = fast_exp2(b_last);
             }
     }
     __syncthreads();
@@ -547,9 +550,7 @@ __global__ void __launch_bounds__(256) channel_pieces_kernel(lb_channel_memory m
                     if (4 * x + k < D) *reinterpret_cast<float4*>(out + l.w + (4 * x + k) * kPiece + t0) = make_float4(y[0][k], y[1][k], y[2][k], y[3][k]);
                 } else {
                     const int c = 4 * (x - tiles_d);
-#pragma unroll
-                    for (int v = 0; v < 4; ++v)
-                        if (c + v < E) out[l.u + (t0 + k) * E + c + v] = y[k][v];
+                    *reinterpret_cast<float4*>(out + l.u + (c / kTileE * kPiece + t0 + k) * kTileE + c % kTileE) = make_float4(y[k][0], y[k][1], y[k][2], y[k][3]);
                 }
             }
         }
@@ -606,117 +607,103 @@ __global__ void __launch_bounds__(256) channel_scan_kernel(lb_channel_memory m, 
     *st = S;
 }
 
-// The scan under the delta rule: a block per (request, head, VT value columns) walks the request's pieces, U = M V - (M K~) S, then
-// S <- exp(b_n) S + sum_j (exp(b_n - b_j) k_j) u_j^T; the next piece's matrices travel while this one is added.  U: the eight warps share the channels,
-// a lane 4 x 4 results, the shares meet in shared memory in the warps' order.
-template <int VT>
+// The scan under the delta rule: a block per (request, head, tile of 16 value columns) walks the request's pieces, U = M V - (M K~) S, then
+// S <- exp(b_n) S + sum_j (exp(b_n - b_j) k_j) u_j^T; the next piece's matrices travel while this one is added.  Both products are made in 4 x 4 results a
+// thread (a 16-byte read of shared memory costs as much as four plain ones), the reduction cut over warps (over groups of threads for S) whose shares
+// meet in shared memory in a fixed order.
 __global__ void __launch_bounds__(256) delta_scan_kernel(lb_channel_memory m, StepArgs a, float* __restrict__ scratch) {
-    static_assert(VT == 16, "a warp's lanes are 8 x 4 tiles of 4 rows x 4 columns");
     extern __shared__ __align__(16) float smem[];
     lb_wait_for_predecessor();
     lb_dependents_may_launch();
+    constexpr int VT = kTileE;
     const int seq = blockIdx.x, h = blockIdx.y, D = m.dim, E = m.vdim, c0 = blockIdx.z * VT;
     const int pieces = (a.q_start[seq + 1] - a.q_start[seq] + kPiece - 1) / kPiece;
     if (pieces <= 0) return;
     int g0 = 0;
     for (int s = 0; s < seq; ++s) g0 += (a.q_start[s + 1] - a.q_start[s] + kPiece - 1) / kPiece;
     const PieceLayout l = piece_layout(D, E, 1);
-    const int matrix = kPiece * D, d4 = (D + 3) / 4 * 4;
-    float* S = smem;                           // [d4][VT]
-    float* U = S + d4 * VT;                    // [32][VT]
-    float* red = U + kPiece * VT;              // [8][32][VT]
-    float* buf = red + 8 * kPiece * VT;        // [2][W^T | B | keep | M V's columns]
-    const int buf_floats = 2 * matrix + d4 + kPiece * VT;
-    const size_t stride = (size_t)m.n_head * l.total;
+    const int D4 = (D + 3) / 4 * 4, matrices = D4 + kPiece * (D4 + D);        // keep, B and W lie one after the other
+    float* S = smem;                           // [D4][VT]
+    float* U = S + D4 * VT;                    // [32][VT]
+    float* red = U + kPiece * VT;              // [8][32][VT], or [groups][D4][VT]
+    float* buf = red + 8 * kPiece * VT;        // [2][keep | B | W^T | M V's columns]
+    const int buf_floats = matrices + kPiece * VT;
+    const size_t stride = (size_t)m.n_head * l.total, u_tile = l.u + (size_t)blockIdx.z * kPiece * VT, s_tile = l.s + (size_t)blockIdx.z * D * VT;
     float* first = scratch + ((size_t)g0 * m.n_head + h) * l.total;
     float* st = a.state + (size_t)a.slots[seq] * m.slot_stride + (size_t)h * D * E;
-    const bool whole = (E & 3) == 0 && c0 + VT <= E;      // the tile's columns travel in 16-byte pieces
     auto ask = [&](int p) {
         const float* src = first + (size_t)p * stride;
         float* dst = buf + (p & 1) * buf_floats;
-        cm_fetch(dst, src + l.w, matrix);
-        cm_fetch(dst + matrix, src + l.b, matrix);
-        cm_fetch(dst + 2 * matrix, src + l.keep, D);
-        float* mv = dst + 2 * matrix + d4;
-        if (whole) {
-            for (int i = threadIdx.x; i < kPiece * VT / 4; i += blockDim.x) cm_cp_async16(mv + 4 * i, src + l.u + (i / (VT / 4)) * E + c0 + 4 * (i % (VT / 4)));
-        } else {
-            for (int i = threadIdx.x; i < kPiece * VT; i += blockDim.x) {
-                const int t = i / VT, x = i - t * VT;
-                if (c0 + x < E) cm_cp_async4(mv + i, src + l.u + t * E + c0 + x);
-                else mv[i] = 0.0f;
-            }
-        }
+        for (int i = threadIdx.x; i < matrices / 4; i += 256) cm_cp_async16(dst + 4 * i, src + l.keep + 4 * i);
+        if (threadIdx.x < kPiece * VT / 4) cm_cp_async16(dst + matrices + 4 * threadIdx.x, src + u_tile + 4 * threadIdx.x);
         cm_cp_commit();
     };
     ask(0);
-    for (int i = threadIdx.x; i < d4 * VT; i += blockDim.x) {
+    for (int i = threadIdx.x; i < D4 * VT; i += blockDim.x) {
         const int d = i / VT, x = i - d * VT;
         S[i] = d < D && c0 + x < E ? st[(size_t)d * E + c0 + x] : 0.0f;
     }
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lt = 4 * (lane >> 2), lc = 4 * (lane & 3);
-    const int c = threadIdx.x % VT, tr = threadIdx.x / VT;
-    constexpr int TR = 256 / VT;               // thread rows
+    // S: tile (4 channels, 4 columns) of the thread, and its share of the rows.
+    const int tiles = D4, tile = threadIdx.x % tiles, group = threadIdx.x / tiles, d0 = 4 * (tile >> 2), x0 = 4 * (tile & 3);
+    int groups = 1;
+    while (2 * groups * tiles <= 256 && groups < 8) groups *= 2;
+    const int share = kPiece / groups;
     for (int p = 0; p < pieces; ++p) {
         cm_cp_wait_all();
         __syncthreads();                       // the piece has arrived; S is whole; the other buffer is free
         if (p + 1 < pieces) ask(p + 1);
-        const float* W = buf + (p & 1) * buf_floats;       // [D][32]
-        const float* B = W + matrix;
-        const float* keep = B + matrix;
-        const float* MV = keep + d4;
+        const float* keep = buf + (p & 1) * buf_floats;
+        const float* B = keep + D4;            // [32][D4]
+        const float* W = B + kPiece * D4;      // [D][32]
+        const float* MV = keep + matrices;
         float* at = first + (size_t)p * stride;
-        for (int i = threadIdx.x; i < D * VT; i += blockDim.x) {
-            const int d = i / VT, x = i - d * VT;
-            if (c0 + x < E) at[l.s + (size_t)d * E + c0 + x] = S[i];
-        }
+        for (int i = threadIdx.x; i < D * VT / 4; i += 256) *reinterpret_cast<float4*>(at + s_tile + 4 * i) = *reinterpret_cast<const float4*>(S + 4 * i);
         float y[4][4] = {};
 #pragma unroll 4
-        for (int d = warp; d < D; d += 8) {
-            const float4 w = *reinterpret_cast<const float4*>(W + d * kPiece + lt), s = *reinterpret_cast<const float4*>(S + d * VT + lc);
-            const float wv[4] = {w.x, w.y, w.z, w.w}, sv[4] = {s.x, s.y, s.z, s.w};
-#pragma unroll
-            for (int i = 0; i < 4; ++i)
-#pragma unroll
-                for (int j = 0; j < 4; ++j) y[i][j] = fmaf(wv[i], sv[j], y[i][j]);
-        }
+        for (int d = warp; d < D; d += 8) outer4(y, *reinterpret_cast<const float4*>(W + d * kPiece + lt), *reinterpret_cast<const float4*>(S + d * VT + lc));
 #pragma unroll
         for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(red + (warp * kPiece + lt + i) * VT + lc) = make_float4(y[i][0], y[i][1], y[i][2], y[i][3]);
         __syncthreads();
+        if (threadIdx.x < kPiece * VT / 4) {
+            float4 u = *reinterpret_cast<const float4*>(MV + 4 * threadIdx.x);
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int at_u = threadIdx.x + 256 * i;
-            float u = MV[at_u];
-#pragma unroll
-            for (int w = 0; w < 8; ++w) u -= red[w * kPiece * VT + at_u];
-            U[at_u] = u;
-            const int t = at_u / VT, x = at_u - t * VT;
-            if (c0 + x < E) at[l.u + (size_t)t * E + c0 + x] = u;
+            for (int w = 0; w < 8; ++w) {
+                const float4 r = *reinterpret_cast<const float4*>(red + w * kPiece * VT + 4 * threadIdx.x);
+                u.x -= r.x; u.y -= r.y; u.z -= r.z; u.w -= r.w;
+            }
+            *reinterpret_cast<float4*>(U + 4 * threadIdx.x) = u;
+            *reinterpret_cast<float4*>(at + u_tile + 4 * threadIdx.x) = u;
         }
         __syncthreads();
-        // S: thread (column, four channels at a time).
-        for (int d = 4 * tr; d < D; d += 4 * TR) {
-            float z[4] = {};
-            if ((D & 3) == 0) {
-#pragma unroll 16
-                for (int t = 0; t < kPiece; ++t) {
-                    const float u = U[t * VT + c];
-                    const float4 r = *reinterpret_cast<const float4*>(B + t * D + d);
-                    z[0] = fmaf(r.x, u, z[0]);
-                    z[1] = fmaf(r.y, u, z[1]);
-                    z[2] = fmaf(r.z, u, z[2]);
-                    z[3] = fmaf(r.w, u, z[3]);
-                }
-            } else {
-                for (int t = 0; t < kPiece; ++t) {
-                    const float u = U[t * VT + c];
+        float z[4][4] = {};
+        if (group < groups) {
+#pragma unroll 8
+            for (int t = group * share; t < (group + 1) * share; ++t)
+                outer4(z, *reinterpret_cast<const float4*>(B + t * D4 + d0), *reinterpret_cast<const float4*>(U + t * VT + x0));
+        }
+        if (groups > 1) {
+            if (group < groups) {
 #pragma unroll
-                    for (int k = 0; k < 4; ++k) z[k] = fmaf(B[t * D + min(d + k, D - 1)], u, z[k]);
-                }
+                for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(red + (group * D4 + d0 + i) * VT + x0) = make_float4(z[i][0], z[i][1], z[i][2], z[i][3]);
             }
+            __syncthreads();
+            for (int i = threadIdx.x; i < D4 * VT / 4; i += 256) {
+                const float k = keep[i >> 2];
+                float4 v = *reinterpret_cast<const float4*>(red + 4 * i), old = *reinterpret_cast<const float4*>(S + 4 * i);
+                for (int g = 1; g < groups; ++g) {
+                    const float4 r = *reinterpret_cast<const float4*>(red + g * D4 * VT + 4 * i);
+                    v.x += r.x; v.y += r.y; v.z += r.z; v.w += r.w;
+                }
+                *reinterpret_cast<float4*>(S + 4 * i) = make_float4(fmaf(k, old.x, v.x), fmaf(k, old.y, v.y), fmaf(k, old.z, v.z), fmaf(k, old.w, v.w));
+            }
+        } else {
 #pragma unroll
-            for (int k = 0; k < 4; ++k)
-                if (d + k < D) S[(d + k) * VT + c] = fmaf(keep[d + k], S[(d + k) * VT + c], z[k]);
+            for (int i = 0; i < 4; ++i) {
+                const float k = keep[d0 + i];
+                float4* dst = reinterpret_cast<float4*>(S + (d0 + i) * VT + x0);
+                *dst = make_float4(fmaf(k, dst->x, z[i][0]), fmaf(k, dst->y, z[i][1]), fmaf(k, dst->z, z[i][2]), fmaf(k, dst->w, z[i][3]));
+            }
         }
     }
     __syncthreads();
@@ -757,10 +744,11 @@ __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory 
             else qs[i] = 0.0f;
         }
     }
-    float* Us = Ss + (D * E + 3) / 4 * 4;      // [32][E]
+    const int wide = m.delta ? (E + kTileE - 1) / kTileE * kTileE : E;
+    float* Us = Ss + (D * wide + 3) / 4 * 4;   // [32][E], or in tiles
     if (staged) {
-        cm_fetch(Ss, in + l.s, D * E);
-        cm_fetch(Us, in + l.u, kPiece * E);
+        cm_fetch(Ss, in + l.s, D * wide);
+        cm_fetch(Us, in + l.u, kPiece * wide);
     }
     cm_cp_commit();
     const int c = threadIdx.x % EP, t0 = threadIdx.x / EP * R;
@@ -802,25 +790,27 @@ __global__ void __launch_bounds__(256) channel_outputs_kernel(lb_channel_memory 
 #pragma unroll
     for (int i = 0; i < R; ++i) y[i] = 0.0f;
     if (c < E) {
-        const float* S = (staged ? Ss : in + l.s) + c;
+        // Column c of the state and of U: in its tile under the delta rule.
+        const int ld = m.delta ? kTileE : E;
+        const float* S = (staged ? Ss : in + l.s) + (m.delta ? c / kTileE * D * kTileE + c % kTileE : c);
 #pragma unroll 2
         for (int d = 0; d < D; d += 4) {
             float s[4];
 #pragma unroll
-            for (int k = 0; k < 4; ++k) s[k] = d + k < D ? S[(size_t)(d + k) * E] : 0.0f;
+            for (int k = 0; k < 4; ++k) s[k] = d + k < D ? S[(d + k) * ld] : 0.0f;
 #pragma unroll
             for (int i = 0; i < R; ++i) {
                 const float4 q = *reinterpret_cast<const float4*>(qs + (t0 + i) * d4 + d);
                 y[i] = fmaf(q.x, s[0], fmaf(q.y, s[1], fmaf(q.z, s[2], fmaf(q.w, s[3], y[i]))));
             }
         }
-        const float* u = (staged ? Us : in + l.u) + c;
+        const float* u = (staged ? Us : in + l.u) + (m.delta ? c / kTileE * kPiece * kTileE + c % kTileE : c);
         const int last = min(n, t0 + R);       // rows after the last of this thread's are not seen
 #pragma unroll 2
         for (int j = 0; j < last; j += 4) {
             float s[4];
 #pragma unroll
-            for (int k = 0; k < 4; ++k) s[k] = j + k < n ? u[(j + k) * E] : 0.0f;
+            for (int k = 0; k < 4; ++k) s[k] = j + k < n ? u[(j + k) * ld] : 0.0f;
 #pragma unroll
             for (int i = 0; i < R; ++i) {
                 const float4 p = *reinterpret_cast<const float4*>(P + (t0 + i) * kPiece + j);
@@ -919,12 +909,11 @@ extern "C" int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memo
     };
     const dim3 grid(pieces, m.n_head);
     const size_t own = (2 * kPiece * 36 + kPiece + (3 * (size_t)kPiece + 48) * (d4 + 4) + (size_t)kPiece * ((E + 3) / 4 * 4 + 4)) * sizeof(float);
-    constexpr int VT = 16;
     if (m.delta) {
         if (int rc = dtype == LB_F32 ? launch(channel_pieces_kernel<float, true>, grid, own, m, a, scratch, n_seq)
                                      : launch(channel_pieces_kernel<__nv_bfloat16, true>, grid, own, m, a, scratch, n_seq)) return rc;
-        const size_t scan = ((size_t)d4 * VT + 9 * (size_t)kPiece * VT + 2 * (2 * (size_t)kPiece * D + d4 + kPiece * VT)) * sizeof(float);
-        if (int rc = launch(delta_scan_kernel<VT>, dim3(n_seq, m.n_head, (E + VT - 1) / VT), scan, m, a, scratch)) return rc;
+        const size_t scan = ((size_t)d4 * kTileE + 9 * (size_t)kPiece * kTileE + 2 * (d4 + (size_t)kPiece * (d4 + D) + kPiece * kTileE)) * sizeof(float);
+        if (int rc = launch(delta_scan_kernel, dim3(n_seq, m.n_head, (E + kTileE - 1) / kTileE), scan, m, a, scratch)) return rc;
     } else {
         if (int rc = dtype == LB_F32 ? launch(channel_pieces_kernel<float, false>, grid, own, m, a, scratch, n_seq)
                                      : launch(channel_pieces_kernel<__nv_bfloat16, false>, grid, own, m, a, scratch, n_seq)) return rc;
@@ -934,7 +923,8 @@ extern "C" int lb_channel_memory_pieces(int dtype, const lb_channel_memory* memo
     if (m.conv != nullptr)
         if (int rc = launch_ring(m, a, n_seq, s)) return rc;
     const size_t base = (kPiece * kPiece + (size_t)kPiece * d4 + 32 * 36 + ((E > 32 ? E : 32) * 33 + 35) / 4 * 4) * sizeof(float);
-    const size_t with_state = base + ((size_t)(D * E + 3) / 4 * 4 + (size_t)kPiece * E) * sizeof(float);
+    const int wide = m.delta ? (E + kTileE - 1) / kTileE * kTileE : E;
+    const size_t with_state = base + ((size_t)(D * wide + 3) / 4 * 4 + (size_t)kPiece * wide) * sizeof(float);
     const int staged = with_state <= 110 * 1024 ? 1 : 0;
     const size_t outs = staged ? with_state : base;
 #define LB_OUTPUTS(T)                                                                                 \

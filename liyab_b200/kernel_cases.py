@@ -6,6 +6,8 @@
     python -m liyab_b200.kernel_cases sample --rows 8 --vocab 50257 --temp 0.8 --top-k 40 --top-p 0.95
     python -m liyab_b200.kernel_cases decode-step --batch 8 --layers 12 --reps 20 [--eager]
     python -m liyab_b200.kernel_cases prefill-step --tokens 2048 --layers 12 --reps 3
+    python -m liyab_b200.kernel_cases channel-memory --batch 2 --new 1024 --heads 6 --dim 64 --vdim 128 --delta
+    python -m liyab_b200.kernel_cases streams --rows 2048 --streams 2 --width 768 --experts 18
 
 Each prints one line with the CUDA-event time per repetition and the achieved rate.  The cases are what the
 ncu summaries under profiles/ were captured on (one kernel, a few launches, inputs of a few hundred MB at most).
@@ -244,6 +246,52 @@ def case_prefill_step(args) -> None:
           f"median {r['wall_ms_per_step']:.3f} ms per step, {n_seq * per / r['ms_per_step'] * 1e3:.0f} tokens/s, {r['kernel_launches']} launches")
 
 
+def case_channel_memory(args) -> None:
+    """A memory with a decay per key channel: whole prompts in pieces (`--new` above 15) or rows of a few tokens, over random projections."""
+    from . import ops
+    dev, H, D, E, B, n = torch.device("cuda:0"), args.heads, args.dim, args.vdim, args.batch, args.new
+    gen = torch.Generator(device=dev).manual_seed(0)
+    r = lambda *shape: torch.randn(*shape, device=dev, generator=gen)
+    rank, taps = 16 if not args.delta else 32, 4 if args.delta else 0
+    cols = 2 * H * D + H * E + rank + (rank + H if args.delta else H * E)
+    m = dict(n_head=H, kv_head=H, dim=D, vdim=E, delta=args.delta, taps=taps, unit=args.delta, gate="sigmoid" if args.delta else "silu", z_bias=r(H * D),
+             a2=(r(H * D, rank) * rank ** -0.5).bfloat16(), g2=(r(H * E, rank) * rank ** -0.5).bfloat16() if args.delta else None,
+             conv=r(2 * H * D + H * E, taps) * 0.5 if args.delta else None, a_log=r(H) - 1 if args.delta else None, tau=16.0, norm=r(E), q_scale=D ** -0.5, eps=1e-5)
+    proj = r(B * n, (cols + 7) // 8 * 8)[:, :cols]
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    positions, tok_seq = i32(list(range(n)) * B), i32([s for s in range(B) for _ in range(n)])
+    q_start, slots = i32([s * n for s in range(B + 1)]), i32(list(range(B)))
+    state = torch.zeros(B, H * D * E + taps * (2 * H * D + H * E), device=dev)
+    heads = torch.empty(B * n, H * E, dtype=torch.bfloat16, device=dev)
+    scratch = torch.empty(ops.channel_memory_floats(B * n, B, H, D, E, args.delta), device=dev)
+    ms = _timed(lambda: ops.channel_memory(m, proj, positions, tok_seq, q_start, slots, state, heads, None, pieces=n >= 16, decode_only=n == 1, scratch=scratch),
+                args.reps)
+    moved = (proj.numel() * 4 + heads.numel() * 2 + 2 * state.numel() * 4) / 1e9
+    print(f"channel memory {B} x {n} rows, {H} heads of {D} x {E}{' delta' if args.delta else ''}: {1e3 * ms:.1f} us, {moved / ms * 1e3:.0f} GB/s of rows and state, "
+          f"{B * n * H * D * E * (6 if args.delta else 4) / ms / 1e9:.2f} TFLOP/s of the recurrence")
+
+
+def case_streams(args) -> None:
+    """The launch between two sublayers: routed results (or a row) into the streams, the next input, and a router on it with `--experts`."""
+    from . import ops
+    dev, T, S, W = torch.device("cuda:0"), args.rows, args.streams, args.width
+    gen = torch.Generator(device=dev).manual_seed(0)
+    r = lambda *shape: torch.randn(*shape, device=dev, generator=gen)
+    x, h = r(T, S * W), torch.empty(T, W, dtype=torch.bfloat16, device=dev)
+    mix, to, ls, norm = r(S, S) * 0.5 / S, r(S), r(W), (torch.full((1,), 0.5, device=dev), r(W), r(W))
+    router = None
+    if args.experts:
+        ids, weights = torch.empty(T, 2, dtype=torch.int32, device=dev), torch.empty(T, 2, device=dev)
+        router = ops.router_args(r(args.experts, W).bfloat16(), 2, ids, weights, correction=r(args.experts), groups=2, keep=1)
+        terms, read = ops.output_terms([r(T, W)], [1.0]), 4 * T * W
+    else:
+        ids = torch.randint(0, 16, (T, 2), dtype=torch.int32, device=dev, generator=gen)
+        place = torch.randperm(2 * T, device=dev, generator=gen).int()
+        terms, read = ops.output_terms((), (), r(2 * T, W), place, ids, r(T, 2), 16, h), 8 * T * W
+    ms = _timed(lambda: ops.streams_join(x, S, T, terms, mix, to, ls, next_in=to, norm=norm, h=h, router=router), args.reps)
+    print(f"streams {T} rows of {S} x {W}{', routed' if router else ''}: {1e3 * ms:.1f} us, {(8 * T * S * W + read + 2 * T * W) / ms / 1e6:.0f} GB/s")
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="python -m liyab_b200.kernel_cases")
     sub = ap.add_subparsers(dest="case", required=True)
@@ -300,6 +348,20 @@ def main(argv=None) -> int:
     sm.add_argument("--top-p", type=float, default=0.95)
     sm.add_argument("--spread", type=float, default=3.0, help="standard deviation of the random logits (8: peaked like a model's)")
     sm.add_argument("--reps", type=int, default=400)
+    cm = sub.add_parser("channel-memory")
+    cm.add_argument("--batch", type=int, default=2)
+    cm.add_argument("--new", type=int, default=1024, help="rows of each request in this step")
+    cm.add_argument("--heads", type=int, default=6)
+    cm.add_argument("--dim", type=int, default=64)
+    cm.add_argument("--vdim", type=int, default=128)
+    cm.add_argument("--delta", action="store_true", help="the delta rule with short convolutions (default: gated linear attention)")
+    cm.add_argument("--reps", type=int, default=20)
+    st = sub.add_parser("streams")
+    st.add_argument("--rows", type=int, default=2048)
+    st.add_argument("--streams", type=int, default=2)
+    st.add_argument("--width", type=int, default=768)
+    st.add_argument("--experts", type=int, default=0)
+    st.add_argument("--reps", type=int, default=20)
     for name in ("decode-step", "prefill-step"):
         p = sub.add_parser(name)
         p.add_argument("--batch", type=int, default=8)
@@ -315,7 +377,7 @@ def main(argv=None) -> int:
         p.add_argument("--stamps", action="store_true", help="decode-step: per-phase times from inside the one-kernel step")
     args = ap.parse_args(argv)
     {"gemm": case_gemm, "generic-attention": case_generic_attention, "gemm-f32": case_gemm_f32, "decode-attention": case_decode_attention, "prefill-attention": case_prefill_attention, "sample": case_sample, "decode-step": case_decode_step,
-     "prefill-step": case_prefill_step}[args.case](args)
+     "prefill-step": case_prefill_step, "channel-memory": case_channel_memory, "streams": case_streams}[args.case](args)
     return 0
 
 

@@ -990,8 +990,15 @@ def experts_direct(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, i
     return out
 
 
+def channel_memory_floats(n_tokens: int, n_seq: int, n_head: int, dim: int, vdim: int, delta: bool) -> int:
+    """How many floats of scratch channel_memory takes in pieces."""
+    fn = lib().lb_channel_memory_pieces_floats
+    fn.argtypes, fn.restype = [_i, _i, _i, _i, _i, _i], _l
+    return fn(n_tokens, n_seq, n_head, dim, vdim, int(delta))
+
+
 def channel_memory(m: dict, proj: torch.Tensor, positions: torch.Tensor, tok_seq: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, state: torch.Tensor,
-                   heads: torch.Tensor, o: Optional[torch.Tensor], pieces: bool, decode_only: bool = False) -> torch.Tensor:
+                   heads: torch.Tensor, o: Optional[torch.Tensor], pieces: bool, decode_only: bool = False, scratch: Optional[torch.Tensor] = None) -> torch.Tensor:
     """A memory per head with a decay per channel (csrc/channel_memory.cu) over the float projection rows [q | k | v | decays' rank | gate | rates].  m: n_head,
     kv_head, dim, vdim, delta, taps, unit, gate ("silu", "sigmoid"), a2, g2 (or None), conv (or None), z_bias, a_log (or None), tau, norm, q_scale, eps."""
     f32 = torch.float32
@@ -1011,8 +1018,7 @@ def channel_memory(m: dict, proj: torch.Tensor, positions: torch.Tensor, tok_seq
     if not pieces:
         check(lib().lb_channel_memory_rows(code, _c.byref(a), _c.byref(s), S, int(decode_only), stream_ptr()), "channel_memory_rows")
         return heads
-    fn = lib().lb_channel_memory_pieces_floats
-    fn.argtypes, fn.restype = [_i, _i, _i, _i, _i, _i], _l
-    scratch = torch.full((fn(T, S, H, D, E, int(m["delta"])),), float("nan"), device=proj.device)
+    if scratch is None:
+        scratch = torch.full((channel_memory_floats(T, S, H, D, E, m["delta"]),), float("nan"), device=proj.device)
     check(lib().lb_channel_memory_pieces(code, _c.byref(a), _c.byref(s), _dev(scratch, "scratch"), T, S, stream_ptr()), "channel_memory_pieces")
     return heads
