@@ -58,17 +58,35 @@ __device__ __forceinline__ void cm_fetch(float* dst, const float* src, int count
     }
 }
 
-// A row of a low-rank map: sum_r w[r] x[r] (+ bias).
+// A row of a low-rank map: sum_r w[r] x[r].  Ranks that split into 16-byte pieces are read in those, four pieces at a time in flight.
 template <typename T>
 __device__ __forceinline__ float low_rank(const T* __restrict__ w, const float* __restrict__ x, int rank) {
-    float acc0 = 0.0f, acc1 = 0.0f;
-    int r = 0;
-    for (; r + 1 < rank; r += 2) {
-        acc0 = fmaf(lb_to_float(w[r]), x[r], acc0);
-        acc1 = fmaf(lb_to_float(w[r + 1]), x[r + 1], acc1);
+    constexpr int N = 16 / sizeof(T);
+    float acc[2] = {0.0f, 0.0f};
+    if (rank % N == 0 && ((reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(x)) & 15) == 0) {
+        for (int r0 = 0; r0 < rank; r0 += 4 * N) {
+            uint4 wv[4];
+            float4 xv[4][N / 4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int r = min(r0 + u * N, rank - N);
+                wv[u] = *reinterpret_cast<const uint4*>(w + r);
+#pragma unroll
+                for (int k = 0; k < N / 4; ++k) xv[u][k] = *reinterpret_cast<const float4*>(x + r + 4 * k);
+            }
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                if (r0 + u * N >= rank) break;
+                const T* wt = reinterpret_cast<const T*>(&wv[u]);
+                const float* xt = reinterpret_cast<const float*>(xv[u]);
+#pragma unroll
+                for (int k = 0; k < N; ++k) acc[k & 1] = fmaf(lb_to_float(wt[k]), xt[k], acc[k & 1]);
+            }
+        }
+        return acc[0] + acc[1];
     }
-    if (r < rank) acc0 = fmaf(lb_to_float(w[r]), x[r], acc0);
-    return acc0 + acc1;
+    for (int r = 0; r < rank; ++r) acc[0] = fmaf(lb_to_float(w[r]), x[r], acc[0]);
+    return acc[0];
 }
 
 struct StepArgs {
@@ -92,13 +110,21 @@ __device__ __forceinline__ float conv_channel(const lb_channel_memory& m, const 
     if (m.conv == nullptr) return a.proj[(size_t)row * a.ld + c];
     const int K = m.taps;
     const float* w = m.conv + (size_t)c * K;
+    auto input = [&](int back) -> float {              // the input `back` tokens ago
+        if (row - back >= row0) return a.proj[(size_t)(row - back) * a.ld + c];
+        return pos - back >= 0 ? ring[(size_t)((pos - back) % K) * channels + c] : 0.0f;
+    };
     float acc = 0.0f;
-    for (int j = 0; j < K; ++j) {
-        const int back = K - 1 - j;                    // how many tokens ago
-        float u = 0.0f;
-        if (row - back >= row0) u = a.proj[(size_t)(row - back) * a.ld + c];
-        else if (pos - back >= 0) u = ring[(size_t)((pos - back) % K) * channels + c];
-        acc = fmaf(w[j], u, acc);
+    if (K <= 4) {                                      // all inputs and taps asked for together
+        float u[4], t[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            u[k] = k < K ? input(k) : 0.0f;
+            t[k] = k < K ? w[K - 1 - k] : 0.0f;
+        }
+        acc = fmaf(t[0], u[0], fmaf(t[1], u[1], fmaf(t[2], u[2], t[3] * u[3])));
+    } else {
+        for (int k = K - 1; k >= 0; --k) acc = fmaf(w[K - 1 - k], input(k), acc);
     }
     return acc * cm_sigmoid(acc);
 }
@@ -107,7 +133,7 @@ __device__ __forceinline__ float conv_channel(const lb_channel_memory& m, const 
 // Thread (c, ds) owns rows ds, ds + DS, .. of column c of the head's S (in shared memory where it fits, else where it lies).  The state travels
 // before this kernel waits for the one before it.
 template <typename T>
-__global__ void __launch_bounds__(256) channel_memory_rows_kernel(lb_channel_memory m, StepArgs a, int ep2, int staged, int write_ring) {
+__global__ void __launch_bounds__(512) channel_memory_rows_kernel(lb_channel_memory m, StepArgs a, int ep2, int staged, int write_ring) {
     extern __shared__ __align__(16) float smem[];
     const int seq = blockIdx.x, h = blockIdx.y, D = m.dim, E = m.vdim, share = m.n_head / m.kv_head;
     const int row0 = a.q_start[seq], row1 = a.q_start[seq + 1];
@@ -121,8 +147,8 @@ __global__ void __launch_bounds__(256) channel_memory_rows_kernel(lb_channel_mem
     float* vs = keep + D;                      // [E]
     float* gate = vs + E;                      // [E]
     float* os = gate + E;                      // [E]
-    float* red = os + E;                       // [256]
-    float* S = staged ? smem + (3 * (D + E) + 256 + 3) / 4 * 4 : st;
+    float* red = os + E;                       // [threads]
+    float* S = staged ? smem + (3 * (D + E) + blockDim.x + 3) / 4 * 4 : st;
     if (staged && row1 > row0) {
         cm_fetch(S, st, D * E);
         cm_cp_commit();
@@ -874,12 +900,13 @@ extern "C" int lb_channel_memory_rows(int dtype, const lb_channel_memory* memory
     auto s = static_cast<cudaStream_t>(stream);
     int ep2 = 1;
     while (ep2 < m.vdim) ep2 <<= 1;
-    const size_t base = (3 * ((size_t)m.dim + m.vdim) + 256 + 3) / 4 * 4 * sizeof(float), with_state = base + (size_t)m.dim * m.vdim * sizeof(float);
+    const int threads = 3 * m.dim + 2 * m.vdim > 256 ? 512 : 256;      // a thread a value of the row's queries, keys, decays, values and gates
+    const size_t base = (3 * ((size_t)m.dim + m.vdim) + threads + 3) / 4 * 4 * sizeof(float), with_state = base + (size_t)m.dim * m.vdim * sizeof(float);
     const int staged = with_state <= 160 * 1024 ? 1 : 0;
     const size_t smem = staged ? with_state : base;
     auto launch = [&](auto kernel) -> int {
         if (smem > 48 * 1024) LB_CHECK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        LB_CHECK_CUDA(lb_launch_overlapped(kernel, dim3(n_seq, m.n_head), dim3(256), smem, s, m, a, ep2, staged, decode_only));
+        LB_CHECK_CUDA(lb_launch_overlapped(kernel, dim3(n_seq, m.n_head), dim3(threads), smem, s, m, a, ep2, staged, decode_only));
         return LB_OK;
     };
     if (int rc = dtype == LB_F32 ? launch(channel_memory_rows_kernel<float>) : launch(channel_memory_rows_kernel<__nv_bfloat16>)) return rc;

@@ -196,19 +196,16 @@ __device__ __forceinline__ void route_rows(const lb_router& r, const float* h, i
         c[e] = r.correction != nullptr ? s + r.correction[e] : s;
     }
     __syncwarp();
-    // The largest of v[0 .. count), the lowest index among equals; every lane gets the index.
+    // The largest of v[0 .. count), the lowest index among equals; every lane gets the index.  Floats compare as unsigned numbers in this form.
     auto argmax = [&](const float* v, int count) {
-        float m = -CUDART_INF_F;
+        unsigned key = 0;
         int at = 0x7fffffff;
-        for (int i = lane; i < count; i += 32)
-            if (at == 0x7fffffff || v[i] > m) { m = v[i]; at = i; }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float m2 = __shfl_xor_sync(0xffffffffu, m, o);
-            const int at2 = __shfl_xor_sync(0xffffffffu, at, o);
-            if (at == 0x7fffffff || (at2 != 0x7fffffff && (m2 > m || (m2 == m && at2 < at)))) { m = m2; at = at2; }
+        for (int i = lane; i < count; i += 32) {
+            const unsigned bits = __float_as_uint(v[i]), k = bits & 0x80000000u ? ~bits : bits | 0x80000000u;
+            if (at == 0x7fffffff || k > key) { key = k; at = i; }
         }
-        return min(at, count - 1);
+        const unsigned top_key = __reduce_max_sync(0xffffffffu, key);
+        return min((int)__reduce_min_sync(0xffffffffu, key == top_key ? (unsigned)at : 0x7fffffffu), count - 1);
     };
     if (r.groups > 1 && r.keep < r.groups) {
         const int size = n / r.groups;
