@@ -606,16 +606,16 @@ def mokisun_config(size, layers=0):
     """Mokisun with the width, depth, head count, inner width and vocabulary of a GPT-2 size.  Of every four blocks the first is gated linear
     attention (heads of 64 x 64), the second attention under a window of 512 (heads of 64, a quarter as many key/value heads, half of a head rotated), the
     others a pair: attention over keys alone under a window of 512 (heads of 64, a quarter as many key/value heads) beside a gated delta rule (half as many
-    heads, 64 / 128 values, four taps); 16 experts of a quarter of the inner width and two identities in two groups, two a token of the better group; two
+    heads, 64 / 128 values, four taps); 16 experts of a quarter of the inner width and four identities in four groups, two a token of the two best groups; two
     streams."""
     g = SIZES[size]
     L, W, H = max(4, layers or g["n_layer"]), g["n_embd"], g["n_head"]
     kv, half = max(1, H // 4), max(1, H // 2)
-    gla = dict(heads=H, dim=64, vdim=64, tau=16.0, a_rank=16)
+    gla = dict(heads=H, dim=64, vdim=64, tau=8.0, a_rank=16)
     attn = dict(heads=H, kv_heads=kv, dim=64, vdim=64, scale=0.125, mask=dict(size=512), rot=dict(base=1e5, dims=32))
     pair = dict(left=dict(heads=H, kv_heads=kv, dim=64, vdim=64, scale=0.125, mask=dict(size=512)),
                 right=dict(heads=half, kv_heads=half, dim=64, vdim=128, conv=4, a_rank=32, g_rank=32), left_scale=1.0, right_scale=1.0)
-    moe = dict(kind="moe", expert=dict(ff=g["n_inner"] // 4), router=dict(experts=16, top=2, identity=2, scale=2.0, groups=dict(count=2, keep=1)))
+    moe = dict(kind="moe", expert=dict(ff=g["n_inner"] // 4), router=dict(experts=16, top=2, identity=4, scale=1.5, groups=dict(count=4, keep=2)))
     kinds = [("gla", gla), ("attention", attn), ("parallel", pair), ("parallel", pair)]
     return dict(architecture="Mokisun", vocab=g["vocab_size"], width=W, streams=2, norm=dict(eps=1e-5), max_positions=g["n_positions"],
                 layers=[dict(type=kinds[i % 4][0], mixer=kinds[i % 4][1], mlp=moe) for i in range(L)])
@@ -624,7 +624,7 @@ def mokisun_config(size, layers=0):
 def mokisun_bytes_and_flops(cfg, dtype_bytes, batch):
     """Bytes a decode step of `batch` requests must read (weights its rows touch, memories read and written, visible cache rows) and the FLOPs of a
     prefill (products with the weights a token uses, attention inside its window, the memories' updates and reads: 4 D E a token and head, and 2 D E more for
-    what the delta rule reads before it writes).  An even router sends top / 18 of the pairs to each of the 16 experts and two identities."""
+    what the delta rule reads before it writes).  An even router sends top / N of the pairs to each of the N experts and identities."""
     W, V = cfg["width"], cfg["vocab"]
     step_bytes, token_flops, attn, mem = 2 * V * W * dtype_bytes, 2 * V * W, [], []
     for l in cfg["layers"]:

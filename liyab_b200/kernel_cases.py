@@ -7,7 +7,7 @@
     python -m liyab_b200.kernel_cases decode-step --batch 8 --layers 12 --reps 20 [--eager]
     python -m liyab_b200.kernel_cases prefill-step --tokens 2048 --layers 12 --reps 3
     python -m liyab_b200.kernel_cases channel-memory --batch 2 --new 1024 --heads 6 --dim 64 --vdim 128 --delta
-    python -m liyab_b200.kernel_cases streams --rows 2048 --streams 2 --width 768 --experts 18
+    python -m liyab_b200.kernel_cases streams --rows 2048 --streams 2 --width 768 --experts 20
 
 Each prints one line with the CUDA-event time per repetition and the achieved rate.  The cases are what the
 ncu summaries under profiles/ were captured on (one kernel, a few launches, inputs of a few hundred MB at most).

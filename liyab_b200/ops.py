@@ -1022,3 +1022,12 @@ def channel_memory(m: dict, proj: torch.Tensor, positions: torch.Tensor, tok_seq
         scratch = torch.full((channel_memory_floats(T, S, H, D, E, m["delta"]),), float("nan"), device=proj.device)
     check(lib().lb_channel_memory_pieces(code, _c.byref(a), _c.byref(s), _dev(scratch, "scratch"), T, S, stream_ptr()), "channel_memory_pieces")
     return heads
+
+
+def expert_plan(ids: torch.Tensor, n_experts: int):
+    """(offsets [E + 1], place [pairs], pair_at [pairs]) of the pairs' experts; places that no pair with an expert below E takes stay -7."""
+    i32, n = torch.int32, ids.numel()
+    offsets = torch.full((n_experts + 1,), -7, dtype=i32, device=ids.device)
+    place, pair_at = (torch.full((n,), -7, dtype=i32, device=ids.device) for _ in range(2))
+    check(lib().lb_expert_plan(_dev(ids, "ids", i32), n, n_experts, _dev(offsets, "offsets"), _dev(place, "place"), _dev(pair_at, "pair_at"), stream_ptr()), "expert_plan")
+    return offsets, place, pair_at

@@ -190,7 +190,7 @@ def test_streams_between_two_sublayers(dev, dtype, S, W, top):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("N,W,top,groups,keep,softmax,renormalise", [(18, 96, 2, 2, 1, True, False), (6, 50, 3, 3, 2, True, True), (64, 768, 8, 8, 4, True, False),
+@pytest.mark.parametrize("N,W,top,groups,keep,softmax,renormalise", [(22, 96, 3, 2, 1, True, False), (6, 50, 3, 3, 2, True, True), (64, 768, 8, 8, 4, True, False),
                                                                      (1, 32, 1, 1, 1, True, False), (160, 132, 6, 5, 3, False, True), (33, 64, 4, 1, 1, False, False)])
 def test_router_with_corrections_and_groups(dev, dtype, N, W, top, groups, keep, softmax, renormalise):
     from liyab_b200 import ops
@@ -209,7 +209,7 @@ def test_router_with_corrections_and_groups(dev, dtype, N, W, top, groups, keep,
         assert ids[0].tolist() == list(range(top))
 
 
-@pytest.mark.parametrize("T,top,E,W,F", [(1, 2, 5, 64, 24), (8, 3, 6, 96, 40), (32, 2, 16, 320, 96), (13, 4, 3, 776, 8)])
+@pytest.mark.parametrize("T,top,E,W,F", [(1, 2, 5, 64, 24), (8, 3, 6, 96, 40), (32, 2, 14, 328, 88), (13, 4, 3, 776, 8)])
 def test_experts_without_a_plan(dev, T, top, E, W, F):
     from liyab_b200 import ops
     rng = np.random.default_rng(T)
@@ -323,3 +323,17 @@ def test_channel_memory(dev, dtype, strong, H, G, D, E, delta, taps, rank, gate_
                 at[s] += n
                 lo += n
         assert state[4].abs().max() == 0                                        # a slot that nobody holds
+
+
+@pytest.mark.parametrize("E", [1, 3, 16, 64, 256, 300])
+@pytest.mark.parametrize("n_pairs", [1, 31, 256, 257, 1000, 4096, 5003])
+def test_expert_plan(dev, n_pairs, E):
+    """Pairs sorted by expert, stably, whichever kernel makes the plan; pairs whose expert has no matrix stand nowhere in it."""
+    from liyab_b200 import ops
+    ids = torch.from_numpy(np.random.default_rng(n_pairs).integers(0, E + 2, n_pairs).astype(np.int32))
+    offsets, place, pair_at = ops.expert_plan(ids.to(dev), E)
+    real = [p for p in range(n_pairs) if ids[p] < E]
+    order = sorted(real, key=lambda p: int(ids[p]))
+    assert offsets.tolist() == [sum(int(ids[p]) < e for p in real) for e in range(E)] + [len(real)]
+    assert pair_at[:len(real)].tolist() == order and place[order].tolist() == list(range(len(real)))
+    assert bool((pair_at[len(real):] == -7).all()) and bool((place[[p for p in range(n_pairs) if ids[p] >= E]] == -7).all())
