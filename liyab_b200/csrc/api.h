@@ -352,7 +352,10 @@ int lb_matrix_memory_pieces(const float* q, const float* k, const float* v, cons
 int lb_router_topk(int dtype, const void* h, int64_t ldh, const void* router, int32_t* ids, float* weights, int n_rows, int n_experts, int width, int top,
                    int softmax, int renormalise, void* stream);
 int lb_expert_plan(const int32_t* ids, int n_pairs, int n_experts, int32_t* offsets, int32_t* place, int32_t* pair_at, void* stream);
-/* gated: mid[place, :n] = act(W_e[:n] . a) * (W_e[n:2n] . a) with a = weights[pair] * h[pair / top]; else y[place, :n] = W_e . mid[place] (float). */
+/* The halves of an expert's work: the argument `gated` of the products below (0 and 1 as the name says, or 2). */
+enum lb_expert_half { LB_EXPERT_SECOND = 0, LB_EXPERT_GATED = 1, LB_EXPERT_PLAIN = 2 };
+/* plain: mid[place, :n] = act(W_e . a), a as for gated and act one of sigmoid, silu, gelu_tanh, relu and relu2 (5: the square of relu; only here).
+ * gated: mid[place, :n] = act(W_e[:n] . a) * (W_e[n:2n] . a) with a = weights[pair] * h[pair / top]; else y[place, :n] = W_e . mid[place] (float). */
 int lb_expert_product(int dtype, int gated, const void* a, int64_t lda, const void* w, int64_t expert_stride, const int32_t* offsets,
                       const int32_t* pair_at, const float* weights, void* out, int64_t ldo, int n_pairs, int n_experts, int n, int k, int top, int act,
                       void* stream);
@@ -443,6 +446,30 @@ int lb_prefill_attention_tc_sink(const void* q, int64_t q_stride, int n_tokens, 
                                  int n_seq, int max_q_len, int n_head, int n_kv_head, int head_dim, int page_size, float scale, int window,
                                  const float* distance, const float* sink, void* stream);
 
+/* The attention kernels with a soft cap on the scores, s <- soft_cap tanh(s / soft_cap) before the softmax (0: none; not beside a penalty by
+ * distance).  bound: the largest |s| before the cap that can occur, 0 when unknown; where it is at most a quarter of the cap the bfloat16 kernels
+ * take the tangent's series instead of its exponential form (see lb_soft_cap in common.cuh). */
+int lb_paged_attention_generic_capped(int dtype, const void* q, int64_t q_stride, const void* cache, const int32_t* tok_seq, const int32_t* positions,
+                                      const int32_t* block_table, int table_stride, void* out, int64_t out_stride, int n_tokens, int n_head,
+                                      int n_kv_head, int head_dim, int page_size, float scale, int window, const float* distance, const float* sink,
+                                      float soft_cap, void* stream);
+int lb_decode_attention_capped(const void* q, int64_t q_stride, const void* cache, const int32_t* positions, const int32_t* block_table,
+                               int table_stride, void* out, int64_t out_stride, float* partial, int* counters, int n_seq, int n_head,
+                               int n_kv_head, int head_dim, int page_size, float scale, int window, int n_splits, const float* distance,
+                               const float* sink, float soft_cap, float bound, void* stream);
+int lb_decode_attention_mma_capped(const void* q, int64_t q_stride, const void* cache, int n_pages, const int32_t* positions,
+                                   const int32_t* block_table, int table_stride, void* out, int64_t out_stride, float* partial, int* counters,
+                                   int n_seq, int n_head, int n_kv_head, int head_dim, int page_size, float scale, int window, int n_splits,
+                                   const float* distance, const float* sink, float soft_cap, float bound, void* stream);
+int lb_prefill_attention_capped(const void* q, int64_t q_stride, const void* cache, const int32_t* q_start, const int32_t* n_past,
+                                const int32_t* block_table, int table_stride, void* out, int64_t out_stride, int n_seq, int max_q_len,
+                                int n_head, int n_kv_head, int head_dim, int page_size, float scale, int window, const float* distance,
+                                const float* sink, float soft_cap, float bound, void* stream);
+int lb_prefill_attention_tc_capped(const void* q, int64_t q_stride, int n_tokens, const void* cache, int n_pages, const int32_t* q_start,
+                                   const int32_t* n_past, const int32_t* block_table, int table_stride, void* out, int64_t out_stride,
+                                   int n_seq, int max_q_len, int n_head, int n_kv_head, int head_dim, int page_size, float scale, int window,
+                                   const float* distance, const float* sink, float soft_cap, float bound, void* stream);
+
 /* What attention over latent rows may have besides its sizes.  sink [n_head]: exp(sink[h]) joins the divisor of head h's softmax (no key, no
  * value, not scaled).  gate: one float a (token, head) at gate[t * ldg + h]; the head's result is multiplied by sigmoid of it.  interleaved:
  * the rotation pairs value 2i with 2i + 1 instead of i with i + rot_dims / 2.  latent (lb_latent_prepare_ext): the rows [latent | rotated key],
@@ -513,6 +540,11 @@ int lb_qkv_rotary_store_layout(int dtype, const float* proj, int64_t ld, int q_o
                                void* q_out, int64_t ldq, void* cache, const int32_t* slot_mapping, int n_tokens, int n_head, int n_kv_head, int dim, int vdim,
                                int padded, int page_size, int norm_mode, float eps, const int32_t* positions, const float* freq, int rot_dims,
                                const float* v_first_in, float* v_first_out, int64_t ldv, const float* lambda, int interleaved, void* stream);
+/* The same with a factor on cosine and sine, and with norm_mode 3: every head over its own root mean square after the rotation. */
+int lb_qkv_rotary_store_scaled(int dtype, const float* proj, int64_t ld, int q_off, int k_off, int v_off, const float* q_weight, const float* k_weight,
+                               void* q_out, int64_t ldq, void* cache, const int32_t* slot_mapping, int n_tokens, int n_head, int n_kv_head, int dim, int vdim,
+                               int padded, int page_size, int norm_mode, float eps, const int32_t* positions, const float* freq, int rot_dims,
+                               const float* v_first_in, float* v_first_out, int64_t ldv, const float* lambda, int interleaved, float rot_factor, void* stream);
 /* out[r, c] = o[r, c] / sqrt(mean(o[r, :]^2) + eps) * gain[c] * act(g[r, c]); gain and g may be null; act 0 sigmoid, 1 silu. */
 int lb_row_norm_gate(int out_dtype, const float* o, int64_t ldo, const float* g, int64_t ldg, const float* gain, void* out, int64_t ld_out, int n_rows,
                      int width, int act, float eps, void* stream);
@@ -537,6 +569,7 @@ typedef struct lb_output_terms {
     int top, n_real;
     const void* self;
     int64_t lds;
+    const float* factor[4];     /* row t of y[i] also times factor[i][t]; null: times one */
 } lb_output_terms;
 /* A router whose choice is corrected and restricted to the best groups (see streams.cu); matrix [n_experts, width] of the call's element type,
  * ids and weights [rows, top]. */
@@ -548,6 +581,7 @@ typedef struct lb_router {
     float scale;
     int32_t* ids;
     float* weights;
+    float* gate;                /* [rows] or null: the matrix has one more row, and gate[t] = sigmoid of its product with row t */
 } lb_router;
 /* The streams x [rows, n_streams * width] between two sublayers (see streams.cu).  mix [n_streams, n_streams] indexed [from, to], to [n_streams],
  * scale [width] or null: of the sublayer that ends; next_in [n_streams] (null: ones), alpha [1] (null: no norm), gain, offset [width]: of the one
@@ -571,6 +605,24 @@ typedef struct lb_streams_args {
     int64_t ldh;
 } lb_streams_args;
 int lb_streams_join(int dtype, const lb_streams_args* args, const lb_output_terms* terms, const lb_router* router, int n_rows, void* stream);
+/* Where one stream is joined by a normed sublayer output (see norm_join.cu): with y the sum of the terms,
+ *     x += scale * y / sqrt(mean(y^2) + eps) * (gain + gain_offset)
+ * over whole rows, then, with h, the next sublayer's input h = x / sqrt(mean(x^2) + next_eps) * (next_gain + next_offset), rows of the call's element
+ * type, and, with a router, the experts of h.  A null gain stands for ones (its offset is not looked at). */
+typedef struct lb_norm_join_args {
+    float* x;
+    int64_t ldx;
+    int width;
+    const float* gain;
+    float gain_offset, eps, scale;
+    const float* next_gain;
+    float next_offset, next_eps;
+    void* h;
+    int64_t ldh;
+} lb_norm_join_args;
+/* Bytes of the structs that callers in other languages lay out by hand: 0 lb_output_terms, 1 lb_router, 2 lb_streams_args, 3 lb_norm_join_args. */
+int lb_struct_bytes(int which);
+int lb_norm_join(int dtype, const lb_norm_join_args* args, const lb_output_terms* terms, const lb_router* router, int n_rows, void* stream);
 int lb_router_choice(int dtype, const lb_router* router, const void* h, int64_t ldh, int n_rows, int width, void* stream);
 int lb_terms_sum(int dtype, const lb_output_terms* terms, float* x, int64_t ldx, int n_rows, int width, int overwrite, void* stream);
 /* lb_expert_product_kind without a plan, for a few pairs (bfloat16): pair p = (row p / top, choice p % top) goes to expert ids[p]; a pair whose

@@ -59,7 +59,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, c
                         const int32_t* __restrict__ positions, const int32_t* __restrict__ block_table, int table_stride,
                         __nv_bfloat16* __restrict__ out, int64_t out_stride, float* __restrict__ partial,
                         int* __restrict__ counters, int n_kv_head, int page_shift, float scale, int window, int n_splits,
-                        const float* __restrict__ distance, const float* __restrict__ sink) {
+                        const float* __restrict__ distance, const float* __restrict__ sink, float soft_cap, float bound) {
     constexpr int TPK = HD / 8;                 // threads that share a key
     constexpr int KPW = 32 / TPK;               // keys a warp covers with one load
     constexpr int STATE = HD + 2;               // m, l, values
@@ -96,6 +96,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, c
         r1[g] = distance != nullptr ? distance[kvh * G + g] : 0.0f;
         r2[g] = distance != nullptr ? distance[n_kv_head * G + kvh * G + g] : 0.0f;
     }
+    const lb_soft_cap capped(soft_cap, bound);
     float m[G], l[G], acc[G][8];
 #pragma unroll
     for (int g = 0; g < G; ++g) {
@@ -140,6 +141,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, c
 #pragma unroll
                 for (int o = TPK / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
                 if (live) {
+                    if (capped.on) s = capped(s);
                     if (distance != nullptr) s -= lb_distance_penalty_log2(r1[g], r2[g], pos - j);
                     const float m_new = fmaxf(m[g], s);
                     const float corr = exp2f(m[g] - m_new);
@@ -238,11 +240,12 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, int64_t q_stride, c
 template <int HD, int G>
 int launch(const void* q, int64_t q_stride, const void* cache, const int32_t* positions, const int32_t* block_table,
            int table_stride, void* out, int64_t out_stride, float* partial, int* counters, int n_seq, int n_kv_head,
-           int page_shift, float scale, int window, int n_splits, const float* distance, const float* sink, cudaStream_t s) {
+           int page_shift, float scale, int window, int n_splits, const float* distance, const float* sink, float soft_cap, float bound,
+           cudaStream_t s) {
     dim3 grid(n_splits, n_kv_head, n_seq);
     LB_CHECK_CUDA(lb_launch_overlapped(decode_attention_kernel<HD, G>, dim3(grid), dim3(kThreads), 0, s, 
         (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)cache, positions, block_table, table_stride,
-        (__nv_bfloat16*)out, out_stride, partial, counters, n_kv_head, page_shift, scale, window, n_splits, distance, sink));
+        (__nv_bfloat16*)out, out_stride, partial, counters, n_kv_head, page_shift, scale, window, n_splits, distance, sink, soft_cap, bound));
     LB_CHECK_LAUNCH();
     return LB_OK;
 }
@@ -250,10 +253,11 @@ int launch(const void* q, int64_t q_stride, const void* cache, const int32_t* po
 template <int HD>
 int by_group(int group, const void* q, int64_t q_stride, const void* cache, const int32_t* positions,
              const int32_t* block_table, int table_stride, void* out, int64_t out_stride, float* partial, int* counters,
-             int n_seq, int n_kv_head, int page_shift, float scale, int window, int n_splits, const float* distance, const float* sink, cudaStream_t s) {
+             int n_seq, int n_kv_head, int page_shift, float scale, int window, int n_splits, const float* distance, const float* sink, float soft_cap, float bound,
+           cudaStream_t s) {
 #define LB_GO(G)                                                                                                   \
     return launch<HD, G>(q, q_stride, cache, positions, block_table, table_stride, out, out_stride, partial, counters, \
-                         n_seq, n_kv_head, page_shift, scale, window, n_splits, distance, sink, s)
+                         n_seq, n_kv_head, page_shift, scale, window, n_splits, distance, sink, soft_cap, bound, s)
     switch (group) {
         case 1: LB_GO(1);
         case 2: LB_GO(2);
@@ -300,6 +304,15 @@ extern "C" int lb_decode_attention_sink(const void* q, int64_t q_stride, const v
                                         int table_stride, void* out, int64_t out_stride, float* partial, int* counters, int n_seq, int n_head,
                                         int n_kv_head, int head_dim, int page_size, float scale, int window, int n_splits, const float* distance,
                                         const float* sink, void* stream) {
+    return lb_decode_attention_capped(q, q_stride, cache, positions, block_table, table_stride, out, out_stride, partial, counters, n_seq, n_head, n_kv_head,
+                                      head_dim, page_size, scale, window, n_splits, distance, sink, 0.0f, 0.0f, stream);
+}
+
+extern "C" int lb_decode_attention_capped(const void* q, int64_t q_stride, const void* cache, const int32_t* positions, const int32_t* block_table,
+                                          int table_stride, void* out, int64_t out_stride, float* partial, int* counters, int n_seq, int n_head,
+                                          int n_kv_head, int head_dim, int page_size, float scale, int window, int n_splits, const float* distance,
+                                          const float* sink, float soft_cap, float bound, void* stream) {
+    LB_CHECK_ARG(soft_cap >= 0.0f && (soft_cap == 0.0f || distance == nullptr), "decode attention: a soft cap is positive and goes without a penalty by distance");
     LB_CHECK_ARG(n_seq >= 0 && n_splits >= 1, "decode attention: bad sizes n_seq=%d n_splits=%d", n_seq, n_splits);
     if (!lb_decode_attention_supports(n_head, n_kv_head, head_dim, page_size))
         return lb_fail(LB_ERR_UNSUPPORTED, "decode attention: unsupported shape heads %d/%d head_dim %d page_size %d", n_head,
@@ -313,7 +326,7 @@ extern "C" int lb_decode_attention_sink(const void* q, int64_t q_stride, const v
     auto s = static_cast<cudaStream_t>(stream);
 #define LB_HD(HD)                                                                                                     \
     return by_group<HD>(group, q, q_stride, cache, positions, block_table, table_stride, out, out_stride, partial, counters, \
-                        n_seq, n_kv_head, page_shift, scale, window, n_splits, distance, sink, s)
+                        n_seq, n_kv_head, page_shift, scale, window, n_splits, distance, sink, soft_cap, bound, s)
     switch (head_dim) {
         case 16: LB_HD(16);
         case 32: LB_HD(32);

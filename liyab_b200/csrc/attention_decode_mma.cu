@@ -74,7 +74,8 @@ decode_attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, int kv_r
                             const int32_t* __restrict__ positions, const int32_t* __restrict__ block_table, int table_stride,
                             __nv_bfloat16* __restrict__ out, int64_t out_stride, float* __restrict__ partial,
                             int* __restrict__ counters, int n_head, int n_kv_head, int page_shift, float scale, int window,
-                            int n_splits, int cluster_merge, const float* __restrict__ distance, const float* __restrict__ sink) {
+                            int n_splits, int cluster_merge, const float* __restrict__ distance, const float* __restrict__ sink,
+                            float soft_cap, float bound) {
     constexpr int kThreads = kWarps * 32;
     constexpr int LD = HD;                      // a tile's row in shared memory; its 16-byte chunks are XOR-swizzled by the row
     constexpr int CH = HD / 8;                  // 16-byte chunks per row
@@ -168,6 +169,7 @@ decode_attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, int kv_r
     // The pairs (r1, r2) of the penalty by distance of this thread's two rows (query heads kvh G + g and + 8); in the scores' base-2
     // scale a key d positions back loses r1 log2(1 + r2 d) (or r1 d log2 e).  Weights: read before the wait for the kernel before this one.
     const bool biased = distance != nullptr;
+    const lb_soft_cap capped(soft_cap, bound);
     const float r1_lo = biased && g < G ? distance[kvh * G + g] : 0.0f, r2_lo = biased && g < G ? distance[n_head + kvh * G + g] : 0.0f;
     const float r1_hi = biased && g + 8 < G ? distance[kvh * G + g + 8] : 0.0f, r2_hi = biased && g + 8 < G ? distance[n_head + kvh * G + g + 8] : 0.0f;
 
@@ -244,6 +246,7 @@ decode_attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, int kv_r
             for (int e = 0; e < 4; ++e) {
                 const int j = j0 + nt * 8 + 2 * t + (e & 1);
                 float v = s[nt][e] * sc;
+                if (capped.on) v = capped(v);
                 if (biased) v -= lb_distance_penalty_log2(e >= 2 ? r1_hi : r1_lo, e >= 2 ? r2_hi : r2_lo, max(pos - j, 0));
                 s[nt][e] = (j >= begin && j < end) ? v : -CUDART_INF_F;
             }
@@ -434,7 +437,8 @@ struct Variant {
 
     static int launch(const CUtensorMap& map_kv, int kv_rows, int* status, const void* q, int64_t q_stride, const void* cache, const int32_t* positions, const int32_t* block_table,
                       int table_stride, void* out, int64_t out_stride, float* partial, int* counters, int n_seq, int n_head,
-                      int n_kv_head, int page_shift, float scale, int window, int n_splits, const float* distance, const float* sink, cudaStream_t s) {
+                      int n_kv_head, int page_shift, float scale, int window, int n_splits, const float* distance, const float* sink, float soft_cap,
+                      float bound, cudaStream_t s) {
         dim3 grid(n_splits, n_kv_head, n_seq);
         // Two to eight key ranges: the ranges of a request and head form a cluster and merge in shared memory.
         const int group = n_head / n_kv_head;
@@ -447,7 +451,7 @@ struct Variant {
                                                    dim3(kWarps * 32), smem + inbox, s, map_kv, kv_rows, status, (const __nv_bfloat16*)q,
                                                    q_stride, (const __nv_bfloat16*)cache, positions, block_table, table_stride,
                                                    (__nv_bfloat16*)out, out_stride, partial, counters, n_head, n_kv_head, page_shift,
-                                                   scale, window, n_splits, cluster ? 1 : 0, distance, sink));
+                                                   scale, window, n_splits, cluster ? 1 : 0, distance, sink, soft_cap, bound));
         return LB_OK;
     }
 };
@@ -459,7 +463,8 @@ struct Variant {
 template <int HD, bool TMA>
 int launch_for(const CUtensorMap& map_kv, int kv_rows, int* status, const void* q, int64_t q_stride, const void* cache, const int32_t* positions, const int32_t* block_table,
                int table_stride, void* out, int64_t out_stride, float* partial, int* counters, int n_seq, int n_head,
-               int n_kv_head, int page_shift, float scale, int window, int n_splits, const float* distance, const float* sink, cudaStream_t s) {
+               int n_kv_head, int page_shift, float scale, int window, int n_splits, const float* distance, const float* sink, float soft_cap,
+                      float bound, cudaStream_t s) {
     using Wide = Variant<HD, 4, 2, TMA>;
     using Narrow = Variant<HD, 2, 2, TMA>;
     static int n_sm = 0;
@@ -478,9 +483,9 @@ int launch_for(const CUtensorMap& map_kv, int kv_rows, int* status, const void* 
     const bool narrow = blocks > slots_wide && waves_wide * slots_wide >= waves_narrow * slots_narrow;
     if (narrow)
         return Narrow::launch(map_kv, kv_rows, status, q, q_stride, cache, positions, block_table, table_stride, out, out_stride, partial, counters,
-                              n_seq, n_head, n_kv_head, page_shift, scale, window, n_splits, distance, sink, s);
+                              n_seq, n_head, n_kv_head, page_shift, scale, window, n_splits, distance, sink, soft_cap, bound, s);
     return Wide::launch(map_kv, kv_rows, status, q, q_stride, cache, positions, block_table, table_stride, out, out_stride, partial, counters, n_seq,
-                        n_head, n_kv_head, page_shift, scale, window, n_splits, distance, sink, s);
+                        n_head, n_kv_head, page_shift, scale, window, n_splits, distance, sink, soft_cap, bound, s);
 }
 
 }  // namespace
@@ -515,6 +520,15 @@ extern "C" int lb_decode_attention_mma_sink(const void* q, int64_t q_stride, con
                                             const int32_t* block_table, int table_stride, void* out, int64_t out_stride, float* partial, int* counters,
                                             int n_seq, int n_head, int n_kv_head, int head_dim, int page_size, float scale, int window, int n_splits,
                                             const float* distance, const float* sink, void* stream) {
+    return lb_decode_attention_mma_capped(q, q_stride, cache, n_pages, positions, block_table, table_stride, out, out_stride, partial, counters, n_seq, n_head,
+                                          n_kv_head, head_dim, page_size, scale, window, n_splits, distance, sink, 0.0f, 0.0f, stream);
+}
+
+extern "C" int lb_decode_attention_mma_capped(const void* q, int64_t q_stride, const void* cache, int n_pages, const int32_t* positions,
+                                              const int32_t* block_table, int table_stride, void* out, int64_t out_stride, float* partial, int* counters,
+                                              int n_seq, int n_head, int n_kv_head, int head_dim, int page_size, float scale, int window, int n_splits,
+                                              const float* distance, const float* sink, float soft_cap, float bound, void* stream) {
+    LB_CHECK_ARG(soft_cap >= 0.0f && (soft_cap == 0.0f || distance == nullptr), "decode attention: a soft cap is positive and goes without a penalty by distance");
     LB_CHECK_ARG(n_seq >= 0 && n_splits >= 1, "decode attention: bad sizes n_seq=%d n_splits=%d", n_seq, n_splits);
     if (!lb_decode_attention_mma_supports(n_head, n_kv_head, head_dim, page_size))
         return lb_fail(LB_ERR_UNSUPPORTED, "decode attention (tensor cores): unsupported shape heads %d/%d head_dim %d page_size %d",
@@ -538,11 +552,11 @@ extern "C" int lb_decode_attention_mma_sink(const void* q, int64_t q_stride, con
             if (rc != LB_OK) return rc;
             return launch_for<64, true>(map_kv, (int)kv_rows, status, q, q_stride, cache, positions, block_table, table_stride,
                                         out, out_stride, partial, counters, n_seq, n_head, n_kv_head, page_shift, scale, window,
-                                        n_splits, distance, sink, s);
+                                        n_splits, distance, sink, soft_cap, bound, s);
         }
         return launch_for<64, false>(none, 0, nullptr, q, q_stride, cache, positions, block_table, table_stride, out, out_stride,
-                                     partial, counters, n_seq, n_head, n_kv_head, page_shift, scale, window, n_splits, distance, sink, s);
+                                     partial, counters, n_seq, n_head, n_kv_head, page_shift, scale, window, n_splits, distance, sink, soft_cap, bound, s);
     }
     return launch_for<128, false>(none, 0, nullptr, q, q_stride, cache, positions, block_table, table_stride, out, out_stride,
-                                  partial, counters, n_seq, n_head, n_kv_head, page_shift, scale, window, n_splits, distance, sink, s);
+                                  partial, counters, n_seq, n_head, n_kv_head, page_shift, scale, window, n_splits, distance, sink, soft_cap, bound, s);
 }

@@ -107,7 +107,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int32_t* __restrict__ q_start, const int32_t* __restrict__ n_past,
                             const int32_t* __restrict__ block_table, int table_stride, __nv_bfloat16* __restrict__ out,
                             int64_t out_stride, int n_head, int n_kv_head, int page_shift, int kv_rows, float scale, int window,
-                            const float* __restrict__ distance, const float* __restrict__ sink, int* status) {
+                            const float* __restrict__ distance, const float* __restrict__ sink,
+                            float soft_cap, float bound, int* status) {
     extern __shared__ uint8_t smem_raw[];
     uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     lb_wait_for_predecessor();            // queries, keys and values come from the kernel before this one
@@ -254,7 +255,9 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t t_row = tmem_base + ((uint32_t)(quarter * 32) << 16);
         const int pos = past + tile_q * kBM + min(r, rows_here - 1);    // rows past the end copy the last one; not stored
         const int first = lb_first_visible(pos, window);
-        const float sc = scale * kLog2e;
+        // With a soft cap the scores are brought to base 2 as they are capped, so nothing is left to multiply.
+        const lb_soft_cap capped(soft_cap, bound);
+        const float raw_sc = scale * kLog2e, sc = capped.on ? 1.0f : raw_sc;
         // The head's penalty by distance in the units of the raw scores (which are multiplied by sc later): a key d positions
         // back loses r1 ln(1 + r2 d) / scale = pen log2(1 + r2 d), or, with r2 < 0, r1 d / scale = pen d.
         const float r2 = distance != nullptr ? distance[n_head + head] : 0.0f;
@@ -277,7 +280,10 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             if (ok) {
                 tmem_ld32(s_row, v);
                 tmem_ld_wait();
-                if (distance != nullptr && r2 < 0.0f) {
+                if (capped.on) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(capped(__uint_as_float(v[i]) * raw_sc));
+                } else if (distance != nullptr && r2 < 0.0f) {
                     // pen (pos - j0 - i) = b0 - pen i.
                     const float b0 = pen * (float)(pos - j0);
 #pragma unroll
@@ -450,6 +456,15 @@ extern "C" int lb_prefill_attention_tc_sink(const void* q, int64_t q_stride, int
                                             const int32_t* n_past, const int32_t* block_table, int table_stride, void* out, int64_t out_stride,
                                             int n_seq, int max_q_len, int n_head, int n_kv_head, int head_dim, int page_size, float scale, int window,
                                             const float* distance, const float* sink, void* stream) {
+    return lb_prefill_attention_tc_capped(q, q_stride, n_tokens, cache, n_pages, q_start, n_past, block_table, table_stride, out, out_stride, n_seq, max_q_len,
+                                          n_head, n_kv_head, head_dim, page_size, scale, window, distance, sink, 0.0f, 0.0f, stream);
+}
+
+extern "C" int lb_prefill_attention_tc_capped(const void* q, int64_t q_stride, int n_tokens, const void* cache, int n_pages, const int32_t* q_start,
+                                              const int32_t* n_past, const int32_t* block_table, int table_stride, void* out, int64_t out_stride,
+                                              int n_seq, int max_q_len, int n_head, int n_kv_head, int head_dim, int page_size, float scale, int window,
+                                              const float* distance, const float* sink, float soft_cap, float bound, void* stream) {
+    LB_CHECK_ARG(soft_cap >= 0.0f && (soft_cap == 0.0f || distance == nullptr), "prefill attention (tcgen05): a soft cap is positive and goes without a penalty by distance");
     LB_CHECK_ARG(distance == nullptr || scale != 0.0f, "prefill attention (tcgen05): a penalty by distance needs a factor on the scores that is not zero");
     LB_CHECK_ARG(n_seq >= 0 && max_q_len >= 0 && n_tokens >= 0 && n_pages > 0, "prefill attention: bad sizes");
     if (!lb_prefill_attention_tc_supports(n_head, n_kv_head, head_dim, page_size))
@@ -480,7 +495,7 @@ extern "C" int lb_prefill_attention_tc_sink(const void* q, int64_t q_stride, int
     dim3 grid(n_head * n_seq, (max_q_len + kBM - 1) / kBM);
     LB_CHECK_CUDA(lb_launch_overlapped(prefill_attention_tc_kernel, dim3(grid), dim3(kThreads), smem, static_cast<cudaStream_t>(stream), 
         map_q, map_kv, q_start, n_past, block_table, table_stride, (__nv_bfloat16*)out, out_stride, n_head, n_kv_head, page_shift,
-        (int)kv_rows, scale, window, distance, sink, status));
+        (int)kv_rows, scale, window, distance, sink, soft_cap, bound, status));
     LB_CHECK_LAUNCH();
     return LB_OK;
 }

@@ -130,6 +130,31 @@ __device__ __forceinline__ float lb_sink_join_exp2(float sink, float m, float& l
 }
 constexpr float kLbLog2e = 1.4426950408889634f;
 
+// A soft cap on scores, cap tanh(s / cap).  Scores come in and leave in the scale of base-2 exponentials (both times log2 e).  Two forms:
+// where no score can be larger than a quarter of the cap (`bound`, 0 when unknown, is the largest |s| that can occur), the series of tanh around
+// zero up to the seventh power, whose next term is below 4e-7 of the value there and which needs no exponential; else 1 - 2 / (1 + exp(2z)).
+struct lb_soft_cap {
+    float in = 0.0f;         // series: 1 / (cap log2 e); else 2 / cap
+    float out = 0.0f;        // cap log2 e
+    bool on = false, series = false;
+    __device__ __forceinline__ lb_soft_cap(float cap, float bound) {
+        on = cap > 0.0f;
+        series = bound > 0.0f && bound <= 0.25f * cap;
+        if (!on) return;
+        out = cap * kLbLog2e;
+        in = series ? 1.0f / out : 2.0f / cap;
+    }
+    __device__ __forceinline__ float operator()(float s) const {
+        if (series) {
+            const float z = s * in, y = z * z;
+            float t = fmaf(y, -17.0f / 315.0f, 2.0f / 15.0f);
+            t = fmaf(y, t, -1.0f / 3.0f);
+            return fmaf(s, y * t, s);
+        }
+        return fmaf(-2.0f * out, __fdividef(1.0f, 1.0f + exp2f(s * in)), out);
+    }
+};
+
 __device__ __forceinline__ float lb_to_float(float v) { return v; }
 __device__ __forceinline__ float lb_to_float(__nv_bfloat16 v) { return __bfloat162float(v); }
 
@@ -211,7 +236,7 @@ __device__ __forceinline__ float lb_activate(float x, int act, const lb_act_pair
 
 // The two halves of a gated feed-forward meet: act(g) * u.  Kinds: 0 sigmoid, 1 silu, 2 GELU (tanh form), 3 relu, and 4, the capped
 // form with its two numbers (alpha, limit): g' = min(g, limit), u' = clamp(u, -limit, limit), g' sigmoid(alpha g') (u' + 1).
-enum lb_gate_kind : int { LB_GATE_SIGMOID = 0, LB_GATE_SILU = 1, LB_GATE_GELU_TANH = 2, LB_GATE_RELU = 3, LB_GATE_CAPPED = 4 };
+enum lb_gate_kind : int { LB_GATE_SIGMOID = 0, LB_GATE_SILU = 1, LB_GATE_GELU_TANH = 2, LB_GATE_RELU = 3, LB_GATE_CAPPED = 4, LB_GATE_RELU2 = 5 };
 __device__ __forceinline__ float lb_gated_pair(float g, float u, int kind, float alpha, float limit) {
     if (kind == LB_GATE_CAPPED) {
         g = fminf(g, limit);
@@ -221,6 +246,14 @@ __device__ __forceinline__ float lb_gated_pair(float g, float u, int kind, float
     const float sg = 1.0f / (1.0f + expf(-g));
     const float a = kind == LB_GATE_SILU ? g * sg : kind == LB_GATE_GELU_TANH ? lb_gelu_tanh(g) : kind == LB_GATE_RELU ? fmaxf(g, 0.0f) : sg;
     return a * u;
+}
+// The same activations on one value, without a second half; LB_GATE_RELU2, the square of relu, exists in this form only.
+__device__ __forceinline__ float lb_gate_alone(float z, int kind) {
+    if (kind == LB_GATE_RELU2) return z > 0.0f ? z * z : 0.0f;
+    if (kind == LB_GATE_RELU) return fmaxf(z, 0.0f);
+    if (kind == LB_GATE_GELU_TANH) return lb_gelu_tanh(z);
+    const float sg = 1.0f / (1.0f + expf(-z));
+    return kind == LB_GATE_SILU ? z * sg : sg;
 }
 
 template <typename... Params, typename... Args>

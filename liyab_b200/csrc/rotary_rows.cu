@@ -13,9 +13,10 @@ __device__ __forceinline__ float rr_sigmoid(float z) { return 1.0f / (1.0f + exp
 // ---------------------------------------------------------------- queries, keys and values: norm, rotation, blend, store
 // A block per token.  From the float row [.. q (H x D) .. k (G x D) .. v (G x E) ..]:
 //   norm_mode 0: queries and keys as they are; 1: every head over its own root mean square, gains [D] shared by the heads;
-//   2: all of q (and all of k) over one root mean square, gains [H x D] and [G x D];
+//   2: all of q (and all of k) over one root mean square, gains [H x D] and [G x D]; 3: every head over its own root mean square after the
+//   rotation (gains [D]), which the rotation changes only by its factor, so that the sum is made of the values before it;
 //   then the first rot_dims values of every query and key head are rotated, value i with value i + rot_dims / 2 (`interleaved`:
-//   value 2i with 2i + 1), by the angle position * freq[i];
+//   value 2i with 2i + 1), by the angle position * freq[i], cosine and sine times rot_factor;
 //   values: with v_first_in, v = (1 - lambda) v + lambda v_first_in[t]; with v_first_out, the row's own values are left there.
 // Queries go to q_out [H x P] (P >= D, E; the rest zeros), keys and values into the cache [page][K|V][G][slot][P].
 template <typename T>
@@ -24,7 +25,7 @@ __global__ void qkv_rotary_store_kernel(const float* __restrict__ proj, int64_t 
                                         const int32_t* __restrict__ slot_mapping, int H, int G, int D, int E, int P, int page_size, int norm_mode, float eps,
                                         const int32_t* __restrict__ positions, const float* __restrict__ freq, int rot_dims,
                                         const float* __restrict__ v_first_in, float* __restrict__ v_first_out, int64_t ldv, const float* __restrict__ lambda,
-                                        int interleaved) {
+                                        int interleaved, float rot_factor) {
     __shared__ float red[2][32];
     extern __shared__ float turn[];            // [rot_dims]: cosine then sine of every pair's angle, made once for all heads of the token
     lb_wait_for_predecessor();
@@ -41,7 +42,12 @@ __global__ void qkv_rotary_store_kernel(const float* __restrict__ proj, int64_t 
         for (int i = threadIdx.x; i < H * D; i += blockDim.x) sq = fmaf(row[q_off + i], row[q_off + i], sq);
         for (int i = threadIdx.x; i < G * D; i += blockDim.x) sk = fmaf(row[k_off + i], row[k_off + i], sk);
     }
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * freq[i], &turn[half + i], &turn[i]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float sn, cs;
+        sincosf((float)pos * freq[i], &sn, &cs);
+        turn[i] = cs * rot_factor;
+        turn[half + i] = sn * rot_factor;
+    }
     // Both sums of squares meet behind one barrier (which also makes the angles visible); every thread adds the warps' shares
     // in the same order.
     sq = lb_warp_sum(sq);
@@ -90,14 +96,15 @@ __global__ void qkv_rotary_store_kernel(const float* __restrict__ proj, int64_t 
             dst = cache + (size_t)page * 2 * plane + ((size_t)head * page_size + off) * P;
         }
         float inv = is_q ? inv_q : inv_k;
-        if (norm_mode == 1) {
+        if (norm_mode == 1 || norm_mode == 3) {
             float ss = 0.0f;
-            for (int d = lane; d < D; d += 32) ss = fmaf(src[d], src[d], ss);
+            const float turned = norm_mode == 3 ? rot_factor * rot_factor : 1.0f;
+            for (int d = lane; d < D; d += 32) ss = fmaf(d < rot_dims ? src[d] * turned : src[d], src[d], ss);
             inv = 1.0f / sqrtf(lb_warp_sum(ss) / (float)D + eps);
         }
         auto normed = [&](int d) {
             float v = src[d] * inv;
-            if (norm_mode != 0 && gain != nullptr) v *= gain[d];
+            if ((norm_mode == 1 || norm_mode == 2) && gain != nullptr) v *= gain[d];
             return v;
         };
         for (int d = lane; d < P; d += 32) {
@@ -112,6 +119,7 @@ __global__ void qkv_rotary_store_kernel(const float* __restrict__ proj, int64_t 
                 } else {
                     v = normed(d);
                 }
+                if (norm_mode == 3 && gain != nullptr) v *= gain[d];
             }
             dst[d] = lb_from_float<T>(v);
         }
@@ -281,9 +289,19 @@ extern "C" int lb_qkv_rotary_store_layout(int dtype, const float* proj, int64_t 
                                           int n_kv_head, int dim, int vdim, int padded, int page_size, int norm_mode, float eps, const int32_t* positions,
                                           const float* freq, int rot_dims, const float* v_first_in, float* v_first_out, int64_t ldv, const float* lambda,
                                           int interleaved, void* stream) {
+    return lb_qkv_rotary_store_scaled(dtype, proj, ld, q_off, k_off, v_off, q_weight, k_weight, q_out, ldq, cache, slot_mapping, n_tokens, n_head, n_kv_head, dim,
+                                      vdim, padded, page_size, norm_mode, eps, positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda, interleaved, 1.0f,
+                                      stream);
+}
+
+extern "C" int lb_qkv_rotary_store_scaled(int dtype, const float* proj, int64_t ld, int q_off, int k_off, int v_off, const float* q_weight,
+                                          const float* k_weight, void* q_out, int64_t ldq, void* cache, const int32_t* slot_mapping, int n_tokens, int n_head,
+                                          int n_kv_head, int dim, int vdim, int padded, int page_size, int norm_mode, float eps, const int32_t* positions,
+                                          const float* freq, int rot_dims, const float* v_first_in, float* v_first_out, int64_t ldv, const float* lambda,
+                                          int interleaved, float rot_factor, void* stream) {
     LB_CHECK_ARG(n_tokens >= 0 && n_head > 0 && n_kv_head > 0 && dim > 0 && vdim > 0 && padded >= dim && padded >= vdim && page_size > 0,
                  "qkv_rotary_store: bad sizes heads=%d/%d dim=%d vdim=%d padded=%d", n_head, n_kv_head, dim, vdim, padded);
-    LB_CHECK_ARG(norm_mode >= 0 && norm_mode <= 2, "qkv_rotary_store: norm mode %d (0 none, 1 a head, 2 the whole projection)", norm_mode);
+    LB_CHECK_ARG(norm_mode >= 0 && norm_mode <= 3, "qkv_rotary_store: norm mode %d (0 none, 1 a head, 2 the whole projection, 3 a head after its rotation)", norm_mode);
     LB_CHECK_ARG(rot_dims >= 0 && rot_dims <= dim && rot_dims % 2 == 0 && (rot_dims == 0 || (freq != nullptr && positions != nullptr)),
                  "qkv_rotary_store: %d of %d values cannot be rotated in pairs, or no frequencies and positions were given", rot_dims, dim);
     LB_CHECK_ARG(v_first_in == nullptr || lambda != nullptr, "qkv_rotary_store: a blend of values needs its weight");
@@ -295,11 +313,11 @@ extern "C" int lb_qkv_rotary_store_layout(int dtype, const float* proj, int64_t 
     if (dtype == LB_F32)
         LB_CHECK_CUDA(lb_launch_overlapped(qkv_rotary_store_kernel<float>, dim3(n_tokens), dim3(threads), smem, s, proj, ld, q_off, k_off, v_off, q_weight, k_weight,
                                            (float*)q_out, ldq, (float*)cache, slot_mapping, n_head, n_kv_head, dim, vdim, padded, page_size, norm_mode, eps,
-                                           positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda, interleaved));
+                                           positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda, interleaved, rot_factor));
     else if (dtype == LB_BF16)
         LB_CHECK_CUDA(lb_launch_overlapped(qkv_rotary_store_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), smem, s, proj, ld, q_off, k_off, v_off, q_weight,
                                            k_weight, (__nv_bfloat16*)q_out, ldq, (__nv_bfloat16*)cache, slot_mapping, n_head, n_kv_head, dim, vdim, padded,
-                                           page_size, norm_mode, eps, positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda, interleaved));
+                                           page_size, norm_mode, eps, positions, freq, rot_dims, v_first_in, v_first_out, ldv, lambda, interleaved, rot_factor));
     else return lb_fail(LB_ERR_INVALID_ARGUMENT, "qkv_rotary_store: unknown dtype %d", dtype);
     return LB_OK;
 }

@@ -6,7 +6,8 @@
 //                      pair and the pair at every place.  One block; nothing returns to the host.
 //   lb_expert_product  for every expert the product of its pairs' rows with its own matrix, in tiles of rows that never
 //                      span two experts.  Either the first half of an expert, mid = act(gate . a) * (up . a) with
-//                      a = weight * h[row] gathered through the plan, or the second, y = down . mid.  32-bit FMA sums with K
+//                      a = weight * h[row] gathered through the plan (or, for experts without a gate, mid = act(up . a)), or the
+//                      second, y = down . mid.  32-bit FMA sums with K
 //                      in ascending order, so a row's result does not depend on which other rows share its tile.
 //   lb_expert_combine  x[row] += the sum of its pairs' results, in the order of its choices.
 #include "api.h"
@@ -216,9 +217,16 @@ struct ProductArgs {
 
 constexpr int kBN = 64, kBK = 16;
 
+// What the first half makes of its sums: act(gate) * up, or, for experts without a gate, act(up) alone.
+template <bool GATED>
+__device__ __forceinline__ float first_half(const ProductArgs& p, float a, float b) {
+    return GATED ? lb_gated_pair(a, b, p.act, p.alpha, p.limit) : lb_gate_alone(a, p.act);
+}
+
 // 256 threads as 16 x 16; a thread makes TM x 4 results.  GATED: two matrices a tile (rows [0, N) gate, [N, 2N) up).
-template <typename T, int TM, bool GATED>
+template <typename T, int TM, int MODE>
 __global__ void __launch_bounds__(256) expert_product_kernel(ProductArgs p) {
+    constexpr bool GATED = MODE == LB_EXPERT_GATED, FIRST = MODE != LB_EXPERT_SECOND;
     constexpr int BM = 16 * TM;
     __shared__ float As[kBK][BM + 1];
     __shared__ float Bs[GATED ? 2 : 1][kBK][kBN + 1];
@@ -266,7 +274,7 @@ __global__ void __launch_bounds__(256) expert_product_kernel(ProductArgs p) {
         a_src[i] = nullptr;
         a_scale[i] = 1.0f;
         if (r < r_end) {
-            if (GATED) {
+            if (FIRST) {
                 const int pair = p.pair_at[r];
                 a_src[i] = A + (size_t)(pair / p.top) * p.lda;
                 if (p.weights != nullptr) a_scale[i] = p.weights[pair];
@@ -317,8 +325,8 @@ __global__ void __launch_bounds__(256) expert_product_kernel(ProductArgs p) {
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
             if (n >= p.N) continue;
-            if (GATED) {
-                static_cast<T*>(p.out)[(size_t)r * p.ldo + n] = lb_from_float<T>(lb_gated_pair(acc[i][j], acc2[i][j], p.act, p.alpha, p.limit));
+            if (FIRST) {
+                static_cast<T*>(p.out)[(size_t)r * p.ldo + n] = lb_from_float<T>(first_half<GATED>(p, acc[i][j], acc2[GATED ? i : 0][j]));
             } else {
                 static_cast<float*>(p.out)[(size_t)r * p.ldo + n] = acc[i][j];
             }
@@ -351,8 +359,9 @@ constexpr int kMM = 64, kMN = 64, kMK = 32, kMLD = kMK + 8, kMStages = 3;
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-template <bool GATED>
+template <int MODE>
 __global__ void __launch_bounds__(128) expert_product_mma_kernel(ProductArgs p) {
+    constexpr bool GATED = MODE == LB_EXPERT_GATED, FIRST = MODE != LB_EXPERT_SECOND;
     using B16 = __nv_bfloat16;
     __shared__ __align__(16) B16 As[kMStages][kMM][kMLD];
     __shared__ __align__(16) B16 Bs[kMStages][GATED ? 2 : 1][kMN][kMLD];
@@ -394,7 +403,7 @@ __global__ void __launch_bounds__(128) expert_product_mma_kernel(ProductArgs p) 
         piece_k[i] = (v & 3) * 8;
         const int r = r0 + piece_row[i];
         a_src[i] = nullptr;
-        if (r < r_end) a_src[i] = GATED ? A + (size_t)(p.pair_at[r] / p.top) * p.lda : A + (size_t)r * p.lda;
+        if (r < r_end) a_src[i] = FIRST ? A + (size_t)(p.pair_at[r] / p.top) * p.lda : A + (size_t)r * p.lda;
         const int n = n0 + piece_row[i];
         b_src[i] = n < p.N ? W + (size_t)n * p.K : nullptr;
     }
@@ -451,7 +460,7 @@ __global__ void __launch_bounds__(128) expert_product_mma_kernel(ProductArgs p) 
     }
     // The rows' weights (first half), then the gate.
     float w_lo = 1.0f, w_hi = 1.0f;
-    if (GATED && p.weights != nullptr) {
+    if (FIRST && p.weights != nullptr) {
         const int lo = r0 + warp * 16 + g, hi = lo + 8;
         if (lo < r_end) w_lo = p.weights[p.pair_at[lo]];
         if (hi < r_end) w_hi = p.weights[p.pair_at[hi]];
@@ -462,20 +471,20 @@ __global__ void __launch_bounds__(128) expert_product_mma_kernel(ProductArgs p) 
         for (int e4 = 0; e4 < 4; ++e4) {
             const int row = r0 + warp * 16 + g + (e4 >= 2 ? 8 : 0), n = n0 + nt * 8 + 2 * t + (e4 & 1);
             if (row >= r_end || n >= p.N) continue;
-            if (GATED) {
+            if (FIRST) {
                 const float w = e4 >= 2 ? w_hi : w_lo;
-                static_cast<B16*>(p.out)[(size_t)row * p.ldo + n] = __float2bfloat16_rn(lb_gated_pair(w * acc[nt][e4], w * acc2[nt][e4], p.act, p.alpha, p.limit));
+                static_cast<B16*>(p.out)[(size_t)row * p.ldo + n] = __float2bfloat16_rn(first_half<GATED>(p, w * acc[nt][e4], w * acc2[GATED ? nt : 0][e4]));
             } else {
                 static_cast<float*>(p.out)[(size_t)row * p.ldo + n] = acc[nt][e4];
             }
         }
 }
 
-template <bool GATED>
+template <int MODE>
 int launch_product_mma(const ProductArgs& p, int n_pairs, cudaStream_t s) {
     const int tiles = (n_pairs + kMM - 1) / kMM + min(p.E, n_pairs);
     const dim3 grid((unsigned)tiles, (unsigned)((p.N + kMN - 1) / kMN)), block(128);
-    LB_CHECK_CUDA(lb_launch_overlapped(expert_product_mma_kernel<GATED>, grid, block, 0, s, p));
+    LB_CHECK_CUDA(lb_launch_overlapped(expert_product_mma_kernel<MODE>, grid, block, 0, s, p));
     return LB_OK;
 }
 
@@ -490,8 +499,9 @@ bool mma_takes(const ProductArgs& p) {
 // is read by the lanes themselves, and 1,024 values of K of every row a warp reads travel together (cp.async, 20 pieces of 16 bytes a
 // lane in flight, whatever the compiler makes of the loop), so a launch is two round trips to memory and the stream of the experts'
 // matrices, with every SM taking part.  Sums are 32-bit in a fixed order; alignment as the tensor-core form's.
-template <bool GATED>
+template <int MODE>
 __global__ void __launch_bounds__(128) expert_product_rows_kernel(ProductArgs p) {
+    constexpr bool GATED = MODE == LB_EXPERT_GATED, FIRST = MODE != LB_EXPERT_SECOND;
     using B16 = __nv_bfloat16;
     constexpr int F = GATED ? 2 : 4, kAhead = 4;
     lb_wait_for_predecessor();
@@ -512,7 +522,7 @@ __global__ void __launch_bounds__(128) expert_product_rows_kernel(ProductArgs p)
         }
         pair = p.pair_at[r];
     }
-    const uint4* a_row = reinterpret_cast<const uint4*>(static_cast<const B16*>(p.a) + (size_t)(GATED ? pair / p.top : r) * p.lda);
+    const uint4* a_row = reinterpret_cast<const uint4*>(static_cast<const B16*>(p.a) + (size_t)(FIRST ? pair / p.top : r) * p.lda);
     const B16* W = static_cast<const B16*>(p.w) + (size_t)e * p.expert_stride;
     const int k8 = p.K / 8;
     const uint4* w[GATED ? 2 * F : F];
@@ -562,23 +572,23 @@ __global__ void __launch_bounds__(128) expert_product_rows_kernel(ProductArgs p)
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) acc[m] += __shfl_xor_sync(0xffffffffu, acc[m], o);
     if (lane != 0) return;
-    const float scale = GATED && p.weights != nullptr ? p.weights[pair] : 1.0f;
+    const float scale = FIRST && p.weights != nullptr ? p.weights[pair] : 1.0f;
 #pragma unroll
     for (int f = 0; f < F; ++f) {
         const int n = n0 + f;
         if (n >= p.N) break;
-        if (GATED) static_cast<B16*>(p.out)[(size_t)r * p.ldo + n] = __float2bfloat16_rn(lb_gated_pair(scale * acc[f], scale * acc[F + f], p.act, p.alpha, p.limit));
+        if (FIRST) static_cast<B16*>(p.out)[(size_t)r * p.ldo + n] = __float2bfloat16_rn(first_half<GATED>(p, scale * acc[f], scale * acc[GATED ? F + f : 0]));
         else static_cast<float*>(p.out)[(size_t)r * p.ldo + n] = acc[f];
     }
 }
 
 constexpr int kFewPairs = 64;
 
-template <bool GATED>
+template <int MODE>
 int launch_product_rows(const ProductArgs& p, int n_pairs, cudaStream_t s) {
-    const int features = 4 * (GATED ? 2 : 4);       // a block's four warps, F features each
+    const int features = 4 * (MODE == LB_EXPERT_GATED ? 2 : 4);       // a block's four warps, F features each
     const dim3 grid((unsigned)n_pairs, (unsigned)((p.N + features - 1) / features)), block(128);
-    LB_CHECK_CUDA(lb_launch_overlapped(expert_product_rows_kernel<GATED>, grid, block, 0, s, p));
+    LB_CHECK_CUDA(lb_launch_overlapped(expert_product_rows_kernel<MODE>, grid, block, 0, s, p));
     return LB_OK;
 }
 
@@ -600,15 +610,15 @@ __global__ void expert_combine_kernel(float* __restrict__ x, int64_t ldx, const 
     }
 }
 
-template <typename T, bool GATED>
+template <typename T, int MODE>
 int launch_product(const ProductArgs& p, int n_pairs, cudaStream_t s) {
     // Row tiles of 16 where the pairs are few (a decode step), of 64 otherwise; no more tiles than pairs / tile + experts.
     const bool small = n_pairs <= 16 * p.E;
     const int BM = small ? 16 : 64;
     const int tiles = (n_pairs + BM - 1) / BM + min(p.E, n_pairs);
     const dim3 grid((unsigned)tiles, (unsigned)((p.N + kBN - 1) / kBN)), block(256);
-    if (small) LB_CHECK_CUDA(lb_launch_overlapped(expert_product_kernel<T, 1, GATED>, grid, block, 0, s, p));
-    else LB_CHECK_CUDA(lb_launch_overlapped(expert_product_kernel<T, 4, GATED>, grid, block, 0, s, p));
+    if (small) LB_CHECK_CUDA(lb_launch_overlapped(expert_product_kernel<T, 1, MODE>, grid, block, 0, s, p));
+    else LB_CHECK_CUDA(lb_launch_overlapped(expert_product_kernel<T, 4, MODE>, grid, block, 0, s, p));
     return LB_OK;
 }
 
@@ -670,26 +680,30 @@ extern "C" int lb_expert_product_set_plain(int on) {
     return LB_OK;
 }
 
-extern "C" int lb_expert_product(int dtype, int gated, const void* a, int64_t lda, const void* w, int64_t expert_stride, const int32_t* offsets,
+extern "C" int lb_expert_product(int dtype, int mode, const void* a, int64_t lda, const void* w, int64_t expert_stride, const int32_t* offsets,
                                  const int32_t* pair_at, const float* weights, void* out, int64_t ldo, int n_pairs, int n_experts, int n, int k, int top,
                                  int act, void* stream) {
-    return lb_expert_product_kind(dtype, gated, a, lda, w, expert_stride, offsets, pair_at, weights, out, ldo, n_pairs, n_experts, n, k, top, act, 0.0f, 0.0f,
+    return lb_expert_product_kind(dtype, mode, a, lda, w, expert_stride, offsets, pair_at, weights, out, ldo, n_pairs, n_experts, n, k, top, act, 0.0f, 0.0f,
                                   stream);
 }
 
-extern "C" int lb_expert_product_kind(int dtype, int gated, const void* a, int64_t lda, const void* w, int64_t expert_stride, const int32_t* offsets,
+extern "C" int lb_expert_product_kind(int dtype, int mode, const void* a, int64_t lda, const void* w, int64_t expert_stride, const int32_t* offsets,
                                       const int32_t* pair_at, const float* weights, void* out, int64_t ldo, int n_pairs, int n_experts, int n, int k, int top,
                                       int act, float alpha, float limit, void* stream) {
-    LB_CHECK_ARG(n_pairs >= 0 && n_experts > 0 && n > 0 && k > 0 && top > 0 && act >= 0 && act <= LB_GATE_CAPPED, "expert product: bad sizes");
+    LB_CHECK_ARG(n_pairs >= 0 && n_experts > 0 && n > 0 && k > 0 && top > 0 && act >= 0 && act <= LB_GATE_RELU2 && mode >= 0 && mode <= LB_EXPERT_PLAIN && (act != LB_GATE_RELU2 || mode != LB_EXPERT_GATED) &&
+                     (act != LB_GATE_CAPPED || mode != LB_EXPERT_PLAIN), "expert product: bad sizes");
     if (n_pairs == 0) return LB_OK;
     ProductArgs p{a, lda, w, expert_stride, offsets, pair_at, weights, out, ldo, n_experts, n, k, top, act, alpha, limit, nullptr};
     auto s = static_cast<cudaStream_t>(stream);
-    if (dtype == LB_F32) return gated ? launch_product<float, true>(p, n_pairs, s) : launch_product<float, false>(p, n_pairs, s);
-    if (dtype == LB_BF16 && mma_takes(p) && !lb_expert_product_plain_only && n_pairs <= kFewPairs)
-        return gated ? launch_product_rows<true>(p, n_pairs, s) : launch_product_rows<false>(p, n_pairs, s);
-    if (dtype == LB_BF16 && mma_takes(p) && !lb_expert_product_plain_only)
-        return gated ? launch_product_mma<true>(p, n_pairs, s) : launch_product_mma<false>(p, n_pairs, s);
-    if (dtype == LB_BF16) return gated ? launch_product<__nv_bfloat16, true>(p, n_pairs, s) : launch_product<__nv_bfloat16, false>(p, n_pairs, s);
+#define LB_BY_MODE(LAUNCH, ...)                                                                                           \
+    return mode == LB_EXPERT_GATED   ? LAUNCH<__VA_ARGS__ LB_EXPERT_GATED>(p, n_pairs, s)                                 \
+           : mode == LB_EXPERT_PLAIN ? LAUNCH<__VA_ARGS__ LB_EXPERT_PLAIN>(p, n_pairs, s)                                 \
+                                     : LAUNCH<__VA_ARGS__ LB_EXPERT_SECOND>(p, n_pairs, s)
+#define LB_COMMA ,
+    if (dtype == LB_F32) LB_BY_MODE(launch_product, float LB_COMMA);
+    if (dtype == LB_BF16 && mma_takes(p) && !lb_expert_product_plain_only && n_pairs <= kFewPairs) LB_BY_MODE(launch_product_rows, );
+    if (dtype == LB_BF16 && mma_takes(p) && !lb_expert_product_plain_only) LB_BY_MODE(launch_product_mma, );
+    if (dtype == LB_BF16) LB_BY_MODE(launch_product, __nv_bfloat16 LB_COMMA);
     return lb_fail(LB_ERR_INVALID_ARGUMENT, "expert product: unknown dtype %d", dtype);
 }
 
@@ -699,15 +713,18 @@ extern "C" int lb_expert_product_direct_supports(int dtype, const void* a, int64
     return dtype == LB_BF16 && n_pairs <= kFewPairs && mma_takes(p) && !lb_expert_product_plain_only ? 1 : 0;
 }
 
-extern "C" int lb_expert_product_direct(int dtype, int gated, const void* a, int64_t lda, const void* w, int64_t expert_stride, const int32_t* ids,
+extern "C" int lb_expert_product_direct(int dtype, int mode, const void* a, int64_t lda, const void* w, int64_t expert_stride, const int32_t* ids,
                                         const float* weights, void* out, int64_t ldo, int n_pairs, int n_experts, int n, int k, int top, int act, float alpha,
                                         float limit, void* stream) {
-    LB_CHECK_ARG(n_pairs >= 0 && n_experts > 0 && n > 0 && k > 0 && top > 0 && act >= 0 && act <= LB_GATE_CAPPED && ids != nullptr, "expert product: bad sizes");
+    LB_CHECK_ARG(n_pairs >= 0 && n_experts > 0 && n > 0 && k > 0 && top > 0 && act >= 0 && act <= LB_GATE_RELU2 && mode >= 0 && mode <= LB_EXPERT_PLAIN && (act != LB_GATE_RELU2 || mode != LB_EXPERT_GATED) &&
+                     (act != LB_GATE_CAPPED || mode != LB_EXPERT_PLAIN) && ids != nullptr, "expert product: bad sizes");
     LB_CHECK_ARG(lb_expert_product_direct_supports(dtype, a, lda, w, expert_stride, n_pairs, k), "expert product without a plan: %d pairs, K = %d are not taken", n_pairs, k);
     if (n_pairs == 0) return LB_OK;
     ProductArgs p{a, lda, w, expert_stride, nullptr, nullptr, weights, out, ldo, n_experts, n, k, top, act, alpha, limit, ids};
     auto s = static_cast<cudaStream_t>(stream);
-    return gated ? launch_product_rows<true>(p, n_pairs, s) : launch_product_rows<false>(p, n_pairs, s);
+    LB_BY_MODE(launch_product_rows, );
+#undef LB_COMMA
+#undef LB_BY_MODE
 }
 
 extern "C" int lb_expert_combine(float* x, int64_t ldx, const float* y, int64_t ldy, const int32_t* place, int n_rows, int width, int top, void* stream) {

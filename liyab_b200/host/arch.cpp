@@ -60,6 +60,7 @@ void register_vosurax();   // vosurax.cpp
 void register_viresun();   // viresun.cpp
 void register_revudra();   // revudra.cpp
 void register_mokisun();   // mokisun.cpp
+void register_gekitar();   // gekitar.cpp
 
 void register_architecture(Architecture arch) { table()[arch.name] = std::move(arch); }
 
@@ -72,6 +73,7 @@ void register_builtin_architectures() {
         register_viresun();
         register_revudra();
         register_mokisun();
+        register_gekitar();
         register_architecture({"liyab_spec", {}, [](const Json& raw) { return std::make_unique<SpecConfig>(raw); }});
     });
     // Plug-ins named by the environment (paths separated by ':') are loaded once, so that the programs can run

@@ -78,6 +78,9 @@ void register_builtin_parts() {
         arrangements().add("sublayer_norm", {[](const LayerSpec& l, const LayerParts& parts, const Runtime&) {
                                return std::make_shared<SublayerNormBlock>(l, parts);
                            }});
+        arrangements().add("sandwich_norm", {[](const LayerSpec& l, const LayerParts& parts, const Runtime&) {
+                               return std::make_shared<SandwichBlock>(l, parts);
+                           }});
         arrangements().add("pre_norm", {[](const LayerSpec& l, const LayerParts& parts, const Runtime&) {
                                return std::make_shared<PreNormBlock>(l, parts);
                            }});

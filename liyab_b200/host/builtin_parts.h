@@ -445,5 +445,87 @@ private:
     LayerParts keep_;
 };
 
+// The sum of a sublayer's output terms, for whoever watches the parts.
+inline void show_terms(StepContext& ctx, const char* name, const OutputTerms& terms, int64_t width) {
+    if (ctx.tap_fn == nullptr) return;
+    const Rows sum = ctx.workspace->get("block.shown", ctx.n_tokens, width, DType::F32);
+    kernels::terms_sum(ctx.stream(), ctx.runtime.dtype, terms, sum, ctx.n_tokens, true);
+    ctx.tap(name, sum);
+}
+
+// `sandwich_norm`: a norm before and a norm after every sublayer: x += m norm_b(mixer(norm_a(x))); x += m norm_d(feed_forward(norm_c(x))), with m the
+// option `residual_scale` (default 1).  Slots: mixer_norm, mixer, mixer_out_norm, and, unless the block has no feed-forward, ff_norm, feed_forward and
+// ff_out_norm.  The norms after the sublayers are RMS norms over the whole row.  The launch that ends a sublayer sums its output terms, norms the sum,
+// adds it to the stream and makes the next sublayer's input (the next block's as well, where that starts with such a norm), with the choice
+// of its experts where it has some.
+
+class SandwichBlock final : public Arrangement {
+public:
+    SandwichBlock(const LayerSpec& spec, const LayerParts& parts)
+        : mixer_norm(parts.get<Norm>("mixer_norm")), mixer(parts.get<Mixer>("mixer")), mixer_out_norm(parts.get<Norm>("mixer_out_norm")),
+          scale(static_cast<float>(spec.options.get_number("residual_scale", 1.0))), keep_(parts) {
+        const bool with_ff = spec.find("feed_forward") != nullptr;
+        if (with_ff) {
+            ff_norm = &parts.get<Norm>("ff_norm");
+            feed_forward = &parts.get<FeedForward>("feed_forward");
+            ff_out_norm = &parts.get<Norm>("ff_out_norm");
+        }
+        if (spec.slots.size() != (with_ff ? 6u : 3u))
+            throw invalid_model("arrangement 'sandwich_norm' takes the slots mixer_norm, mixer and mixer_out_norm, and ff_norm and ff_out_norm with feed_forward, only");
+        if (!whole_row(mixer_out_norm) || (with_ff && !whole_row(*ff_out_norm)))
+            throw unsupported("arrangement 'sandwich_norm' takes RMS norms over the whole row (gain only) on its sublayers' outputs");
+    }
+    bool capturable() const override {
+        return mixer_norm.capturable() && mixer.capturable() && (feed_forward == nullptr || (ff_norm->capturable() && feed_forward->capturable()));
+    }
+    std::vector<Mixer*> mixers() const override { return {&mixer}; }
+    std::optional<NormRecipe> input_norm() const override { return whole_row(mixer_norm); }
+    void forward(StepContext& ctx, const Rows& x, CacheUnit unit) override {
+        const int T = ctx.n_tokens;
+        const DType dt = ctx.runtime.dtype;
+        const Rows h = ctx.workspace->get("block.normed", T, x.cols, dt), y = ctx.workspace->get("block.sublayer", T, x.cols, DType::F32);
+        if (ctx.next_input_entry != unit.entry || ctx.next_input.data != h.data) {
+            ctx.phase(Phase::Norm);
+            mixer_norm.forward(ctx, x, h, T, nullptr);
+        }
+        ctx.tap("mixer_norm", h);
+        ctx.phase(Phase::Mixer);
+        OutputTerms terms = mixer.forward_terms(ctx, h, y, unit);
+        show_terms(ctx, "mixer.out", terms, x.cols);
+        NormRecipe out = *whole_row(mixer_out_norm);
+        if (feed_forward != nullptr) {
+            const std::optional<NormRecipe> next = whole_row(*ff_norm);
+            const std::optional<RowRouter> router = next ? feed_forward->row_router(ctx) : std::nullopt;
+            kernels::norm_join(ctx.stream(), dt, x, out, scale, terms, T, next ? &*next : nullptr, next ? &h : nullptr, router ? &*router : nullptr);
+            ctx.tap("mixer", x);
+            ctx.phase(Phase::FeedForward);
+            if (!next) ff_norm->forward(ctx, x, h, T, nullptr);
+            ctx.tap("ff_norm", h);
+            terms = feed_forward->forward_terms(ctx, h, y, router.has_value());
+            show_terms(ctx, "feed_forward.out", terms, x.cols);
+            out = *whole_row(*ff_out_norm);
+        }
+        const NormRecipe* last = ctx.next_norm;
+        kernels::norm_join(ctx.stream(), dt, x, out, scale, terms, T, last, last != nullptr ? &h : nullptr, nullptr);
+        ctx.next_input = h;
+        ctx.next_input_entry = last != nullptr ? unit.entry + 1 : -1;
+        ctx.tap(feed_forward != nullptr ? "feed_forward" : "mixer", x);
+    }
+    Norm& mixer_norm;
+    Mixer& mixer;
+    Norm& mixer_out_norm;
+    Norm* ff_norm = nullptr;
+    FeedForward* feed_forward = nullptr;
+    Norm* ff_out_norm = nullptr;
+    float scale;
+
+private:
+    // The recipe of an RMS norm over the whole row, where the norm is one.
+    static std::optional<NormRecipe> whole_row(const Norm& n) {
+        std::optional<NormRecipe> r = n.recipe();
+        return r && r->rms && r->offset == nullptr ? r : std::nullopt;
+    }
+    LayerParts keep_;
+};
 
 }  // namespace liyab::builtin

@@ -173,8 +173,14 @@ Rows DecoderModel::forward(StepContext& ctx) {
             ctx.tap("pass_offset", x);
             ctx.stream_rounded_entry = -1;
         }
+        // The block after this one may take its input from this one's last launch, unless something is added to the stream between them.
+        std::optional<NormRecipe> next;
+        if (i + 1 < spec.run_order.size() && spec.run_order[i + 1].offset_row < 0) next = layers[static_cast<size_t>(spec.run_order[i + 1].layer)].block->input_norm();
+        ctx.next_norm = next ? &*next : nullptr;
         layers[static_cast<size_t>(e.layer)].block->forward(ctx, x, CacheUnit{e.cache, e.cache == static_cast<int>(i), static_cast<int>(i)});
     }
+    ctx.next_norm = nullptr;
+    ctx.next_input_entry = -1;
     const int R = ctx.n_logit_rows;
     if (R == 0) return no_logits();
     // The head's buffers are sized by the rows whose logits are wanted, not by the step's tokens.

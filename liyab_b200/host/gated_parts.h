@@ -50,9 +50,35 @@ private:
     DeviceBuffer joined_;
 };
 
-inline std::vector<float> rotation_frequencies(int dims, double base) {
+// A rotation stretched over more positions than it was made for (an option {factor, original, fast, slow}): a pair that turns `fast` times or more
+// over `original` positions keeps its frequency, one that turns `slow` times or fewer has it divided by `factor`, pairs between the two blend along
+// a straight line over their numbers; cosine and sine are multiplied by 0.1 ln(factor) + 1.
+struct RotationScaling {
+    double factor = 1.0, original = 0.0, fast = 0.0, slow = 0.0;
+    static std::optional<RotationScaling> from(const PartSpec& s) {
+        const Json* j = s.options.find("rot_scaling");
+        if (j == nullptr || j->is_null()) return std::nullopt;
+        RotationScaling r{j->get_number("factor", 0.0), j->get_number("original", 0.0), j->get_number("fast", 0.0), j->get_number("slow", 0.0)};
+        if (!(r.factor > 0 && r.original > 0 && r.fast > 0 && r.slow > 0)) throw invalid_model("{}: rot_scaling needs positive factor, original, fast and slow", s.kind);
+        return r;
+    }
+    double magnitude() const { return 0.1 * std::log(factor) + 1.0; }
+};
+
+inline std::vector<float> rotation_frequencies(int dims, double base, const std::optional<RotationScaling>& scaling = std::nullopt) {
     std::vector<float> f;
-    for (int i = 0; i < dims / 2; ++i) f.push_back(static_cast<float>(std::pow(base, -2.0 * i / dims)));
+    double lo = 0.0, hi = 0.0;
+    if (scaling && dims > 0) {
+        // The pair (as a real number) that turns so many times over the original length.
+        auto pair_of = [&](double turns) { return dims * std::log(scaling->original / (2.0 * M_PI * turns)) / (2.0 * std::log(base)); };
+        lo = std::max(std::floor(pair_of(scaling->fast)), 0.0);
+        hi = std::min(std::ceil(pair_of(scaling->slow)), static_cast<double>(dims - 1));
+    }
+    for (int i = 0; i < dims / 2; ++i) {
+        const double plain = std::pow(base, -2.0 * i / dims);
+        const double ramp = scaling ? std::clamp((i - lo) / std::max(hi - lo, 0.001), 0.0, 1.0) : 0.0;
+        f.push_back(static_cast<float>(scaling ? plain / scaling->factor * ramp + plain * (1.0 - ramp) : plain));
+    }
     return f;
 }
 
@@ -77,6 +103,8 @@ inline std::vector<float> rotation_frequencies(int dims, double base) {
 // `rot_layout` "interleaved": the rotation pairs value 2i with 2i + 1.  `values` "keys": the values are the keys as projected (no rows for v in the
 // projection; vdim = dim, and no rotation or norm may come between).  `slopes`: the score of the key d positions back loses
 // slope_h d with slope_h = 2^(-8 (h + 1) / n_head) for head h counted from 0.  `unit_sink`: one is added to every softmax's divisor.
+// `soft_cap` c > 0: a score s becomes c tanh(s / c).  `qk_norm_at` "rotated": the norm of every query and key head comes after the rotation instead of
+// before it.  `rot_scaling`: see RotationScaling.  `out_bias`: the output projection has a bias.
 
 class GatedAttention final : public Mixer {
 public:
@@ -115,7 +143,18 @@ public:
         norm_projection = qk_norm && over == "projection";
         rot_dims = static_cast<int>(s.options.get_int("rot_dims", 0));
         if (rot_dims < 0 || rot_dims > D || rot_dims % 2 != 0) throw invalid_model("gated_attention: {} of {} values cannot be rotated in pairs", rot_dims, D);
-        freq.host = rotation_frequencies(rot_dims, s.options.get_number("rot_base", 10000.0));
+        const std::optional<RotationScaling> scaling = RotationScaling::from(s);
+        freq.host = rotation_frequencies(rot_dims, s.options.get_number("rot_base", 10000.0), scaling);
+        if (scaling) rot_factor = static_cast<float>(scaling->magnitude());
+        const std::string at = s.options.get_string("qk_norm_at", "projected");
+        if (at != "projected" && at != "rotated") throw unsupported("gated_attention: qk_norm_at '{}' is not supported; supported: projected, rotated", at);
+        norm_rotated = qk_norm && at == "rotated" && rot_dims > 0;
+        if (norm_rotated && norm_projection) throw unsupported("gated_attention: a norm after the rotation is one a head");
+        shape.soft_cap = static_cast<float>(s.options.get_number("soft_cap", 0.0));
+        if (!(shape.soft_cap >= 0.0f)) throw invalid_model("gated_attention: soft_cap {} is negative", shape.soft_cap);
+        // Normed queries and keys without gains have length sqrt(dim) at most, but for the rounding of their values, which bounds the scores.
+        if (qk_norm && !norm_projection && q_gain == nullptr && k_gain == nullptr)
+            shape.score_bound = 1.02f * static_cast<float>(D) * std::abs(shape.scale) * (norm_rotated ? 1.0f : rot_factor * rot_factor);
         if (s.options.get_bool("sink", false)) shape.sink = f32_or_null(&p.at("sink"));
         const std::string layout = s.options.get_string("rot_layout", "half");
         if (layout != "half" && layout != "interleaved") throw unsupported("gated_attention: rot_layout '{}' is not supported; supported: half, interleaved", layout);
@@ -123,6 +162,8 @@ public:
         values_are_keys = values_from_keys(s);
         if (values_are_keys && (E != D || qk_norm || rot_dims > 0))
             throw unsupported("gated_attention: values that are the keys as projected take vdim = dim, no norm of the keys and no rotation");
+        if (shape.soft_cap > 0.0f && (shape.distance != nullptr || s.options.get_bool("slopes", false)))
+            throw unsupported("gated_attention: capped scores go without a penalty by distance");
         if (s.options.get_bool("slopes", false)) {
             if (shape.distance != nullptr) throw unsupported("gated_attention: slopes or a learned penalty by distance, not both");
             for (int h = 0; h < H; ++h) slopes.host.push_back(static_cast<float>(std::exp2(-8.0 * (h + 1) / H)));
@@ -160,7 +201,7 @@ public:
         if (s.options.get_bool("sink", false)) out.push_back({"sink", {H}, ParamKind::Vector});
         if (s.options.get_string("value_blend", "none") == "blend") out.push_back({"blend", {1}, ParamKind::Vector});
         if (s.options.get_bool("distance_bias", false)) out.push_back({"distance", {2 * H}, ParamKind::Vector});
-        Linear::declare(out, "out.", hidden, H * E, false);
+        Linear::declare(out, "out.", hidden, H * E, s.options.get_bool("out_bias", false));
         return out;
     }
     // The head size the cache and the kernels work on: in bfloat16 the next size every tensor-core kernel takes, else a multiple of four.
@@ -193,7 +234,9 @@ public:
     int64_t hidden = 0;
     int H = 0, G = 0, D = 0, E = 0, gate = -1;
     bool qk_norm = false, norm_projection = false, blend_source = false, rotary_store = false, interleaved = false, values_are_keys = false;
+    bool norm_rotated = false;
     int rot_dims = 0;
+    float rot_factor = 1.0f;
     const float* blend = nullptr;
     float eps = 1e-6f, temp_coef = 0.0f;
     int temp_every = 0;
@@ -225,9 +268,9 @@ private:
             // The values that layers blend with travel from the source layer to the others in a buffer of the step.
             Rows shared;
             if (blend_source || blend != nullptr) shared = ws.get("gated_attention.value_source", T, static_cast<int64_t>(G) * E, DType::F32);
-            kernels::qkv_rotary_store(s, pr, cols, q_gain, k_gain, q, unit.write ? cache : nullptr, view->slot_mapping, T, !qk_norm ? 0 : norm_projection ? 2 : 1, eps,
+            kernels::qkv_rotary_store(s, pr, cols, q_gain, k_gain, q, unit.write ? cache : nullptr, view->slot_mapping, T, !qk_norm ? 0 : norm_projection ? 2 : norm_rotated ? 3 : 1, eps,
                                       ctx.positions, rot_dims > 0 ? freq.get(s) : nullptr, rot_dims, blend != nullptr ? &shared : nullptr,
-                                      blend_source ? &shared : nullptr, blend, interleaved);
+                                      blend_source ? &shared : nullptr, blend, interleaved, rot_factor);
         } else {
             kernels::qk_norm_store(s, pr, cols, q_gain, k_gain, q, unit.write ? cache : nullptr, view->slot_mapping, T, qk_norm, eps, ctx.positions, temp_coef,
                                    temp_every);
@@ -244,7 +287,7 @@ private:
             kernels::head_gate(s, att, P, g, nullptr, heads, T, H, E, false, std::max(gate, 0), eps);
         }
         ctx.tap("attention", heads);
-        kernels::linear(ctx.runtime, &ws, heads, out.weight, nullptr, y, T, kernels::kNone, residual);
+        kernels::linear(ctx.runtime, &ws, heads, out.weight, out.bias, y, T, kernels::kNone, residual);
     }
     PartialBias bias;
     DeviceFloats freq, slopes, unit_sinks;
@@ -503,6 +546,7 @@ public:
     GatedFeedForward(const PartSpec& s, const Params& p)
         : inner(need_int(s, "inner")), gate(kernels::gate_from_name(s.options.get_string("activation", "silu"))),
           alpha(static_cast<float>(s.options.get_number("gate_alpha", 1.0))), limit(static_cast<float>(s.options.get_number("gate_limit", 0.0))) {
+        if (gate == kernels::kRelu2Gate) throw unsupported("gated: the activation relu2 has no gated form");
         gate_up = Linear(p, "gate_up.", "gated.gate_up");
         down = Linear(p, "down.", "gated.down");
     }
@@ -565,6 +609,9 @@ private:
 // input itself (times the weight; with weight_on output).  `correction`: a learned number an expert that is added to its score for the choice only.
 // `groups` g and `keep_groups` k: the outputs form g equal groups of neighbours, a group counts as its best choice score, and only experts of
 // the k best groups can be chosen.  `route_scale`: a factor on the weights.
+// `expert` "plain": experts without a gate, down(act(W_up a)), activations relu2 (the square of relu), relu, silu, gelu_tanh, sigmoid; the parameter
+// is `experts.up.weight` [experts x inner, hidden] then, and the shared expert has that form too.  `shared_gate`: the shared expert's result is
+// multiplied by the sigmoid of one number a row, which is the last row of the router's matrix.
 
 class RoutedExperts final : public FeedForward {
 public:
@@ -590,16 +637,30 @@ public:
         keep_groups = static_cast<int>(s.options.get_int("keep_groups", groups));
         route_scale = static_cast<float>(s.options.get_number("route_scale", 1.0));
         if (s.options.get_bool("correction", false)) correction = f32_or_null(&p.at("router.correction"));
-        corrected = identity > 0 || groups > 1 || correction != nullptr || route_scale != 1.0f;
-        if (corrected && by_table) throw unsupported("routed: a table of experts has no router to correct");
+        plain = plain_experts(s);
+        shared_gate = s.options.get_bool("shared_gate", false);
+        if (!plain && gate == kernels::kRelu2Gate) throw unsupported("routed: the activation relu2 goes with experts without a gate");
+        if (shared_gate && s.options.get_int("shared_inner", 0) <= 0) throw invalid_model("routed: a gate on a shared expert needs one (shared_inner)");
+        by_terms = identity > 0 || groups > 1 || correction != nullptr || route_scale != 1.0f || plain || shared_gate;
+        if (by_terms && by_table) throw unsupported("routed: a table of experts has no router to correct");
         if (identity < 0 || groups < 1 || (experts + identity) % groups != 0 || keep_groups < 1 || keep_groups > groups || top > (experts + identity) / groups * keep_groups)
             throw invalid_model("routed: top {} of {} experts and {} identities in {} groups of which {} count", top, experts, identity, groups, keep_groups);
         if (identity > 0 && !weight_on_output) throw unsupported("routed: identity experts take the weight on the output");
-        gate_up = p.at("experts.gate_up.weight");
+        gate_up = p.at(plain ? "experts.up.weight" : "experts.gate_up.weight");
         down = p.at("experts.down.weight");
-        if (s.options.get_int("shared_inner", 0) > 0) shared = std::make_unique<GatedFeedForward>(shared_spec(s), p.sub("shared."));
+        if (s.options.get_int("shared_inner", 0) <= 0) return;
+        if (plain) shared = std::make_unique<DenseFeedForward>(shared_spec(s), p.sub("shared."));
+        else shared = std::make_unique<GatedFeedForward>(shared_spec(s), p.sub("shared."));
+    }
+    static bool plain_experts(const PartSpec& s) {
+        const std::string form = s.options.get_string("expert", "gated");
+        if (form != "gated" && form != "plain") throw unsupported("routed: expert '{}' is not supported; supported: gated, plain", form);
+        return form == "plain";
     }
     static PartSpec shared_spec(const PartSpec& s) {
+        if (plain_experts(s))
+            return {"dense", Json::object().set("hidden", need_int(s, "hidden")).set("inner", s.options.get_int("shared_inner", 0)).set("bias", false)
+                                 .set("activation", s.options.get_string("shared_activation", s.options.get_string("activation", "relu2")))};
         return {"gated", Json::object().set("hidden", need_int(s, "hidden")).set("inner", s.options.get_int("shared_inner", 0))
                              .set("activation", s.options.get_string("shared_activation", s.options.get_string("activation", "silu")))};
     }
@@ -610,15 +671,15 @@ public:
             out.push_back({"table", {need_int(s, "vocab"), need_int(s, "top")}, ParamKind::Index});
         } else {
             const int64_t N = E + s.options.get_int("identity", 0);
-            out.push_back({"router.weight", {N, hidden}, ParamKind::Matrix});
+            out.push_back({"router.weight", {N + (s.options.get_bool("shared_gate", false) ? 1 : 0), hidden}, ParamKind::Matrix});
             if (s.options.get_bool("router_bias", false)) out.push_back({"router.bias", {N}, ParamKind::Vector});
             if (s.options.get_bool("correction", false)) out.push_back({"router.correction", {N}, ParamKind::Vector});
         }
-        for (ParamDecl d : std::vector<ParamDecl>{{"experts.gate_up.weight", {E * 2 * inner, hidden}, ParamKind::Matrix},
+        for (ParamDecl d : std::vector<ParamDecl>{{plain_experts(s) ? "experts.up.weight" : "experts.gate_up.weight", {E * (plain_experts(s) ? 1 : 2) * inner, hidden}, ParamKind::Matrix},
                                    {"experts.down.weight", {E * hidden, inner}, ParamKind::Matrix}})
             out.push_back(std::move(d));
         if (s.options.get_int("shared_inner", 0) > 0)
-            for (const auto& d : GatedFeedForward::parameters(shared_spec(s))) out.push_back({"shared." + d.name, d.shape, d.kind});
+            for (const auto& d : plain_experts(s) ? DenseFeedForward::parameters(shared_spec(s)) : GatedFeedForward::parameters(shared_spec(s))) out.push_back({"shared." + d.name, d.shape, d.kind});
         return out;
     }
     bool capturable() const override { return true; }
@@ -627,7 +688,7 @@ public:
     void forward_into(StepContext& ctx, const Rows& h, const Rows& y) override { run(ctx, h, y, true); }
     // The rows' sums are left to the launch that joins them to the streams; the experts may have been chosen by the launch that made h.
     OutputTerms forward_terms(StepContext& ctx, const Rows& h, const Rows& y, bool routed) override {
-        if (!corrected) return FeedForward::forward_terms(ctx, h, y, routed);
+        if (!by_terms) return FeedForward::forward_terms(ctx, h, y, routed);
         const int T = ctx.n_tokens, pairs = T * top;
         Workspace& ws = *ctx.workspace;
         cudaStream_t s = ctx.stream();
@@ -640,17 +701,18 @@ public:
         const float* on_input = weight_on_output ? nullptr : r.weights;
         OutputTerms t;
         const int N1 = static_cast<int>(inner), N2 = static_cast<int>(hidden);
-        if (kernels::expert_product_direct_supports(h, gate_up, pairs, N1, N2, true) && kernels::expert_product_direct_supports(mid, down, pairs, N2, N1, false)) {
+        const kernels::ExpertHalf first = plain ? kernels::kPlainHalf : kernels::kGatedHalf, second = kernels::kSecondHalf;
+        if (kernels::expert_product_direct_supports(h, gate_up, pairs, N1, N2, first) && kernels::expert_product_direct_supports(mid, down, pairs, N2, N1, second)) {
             // A few pairs: every pair finds its expert by itself, no plan.
-            kernels::expert_product_direct(s, true, h, gate_up, experts, r.ids, on_input, mid, pairs, N1, N2, top, gate, alpha, limit);
-            kernels::expert_product_direct(s, false, mid, down, experts, r.ids, nullptr, out, pairs, N2, N1, top, gate);
+            kernels::expert_product_direct(s, first, h, gate_up, experts, r.ids, on_input, mid, pairs, N1, N2, top, gate, alpha, limit);
+            kernels::expert_product_direct(s, second, mid, down, experts, r.ids, nullptr, out, pairs, N2, N1, top, gate);
         } else {
             int32_t* place = static_cast<int32_t*>(ws.get("routed.place", T, top, DType::I32).data);
             int32_t* pair_at = static_cast<int32_t*>(ws.get("routed.pair_at", T, top, DType::I32).data);
             int32_t* offsets = static_cast<int32_t*>(ws.flat("routed.offsets", experts + 1, DType::I32));
             kernels::expert_plan(s, r.ids, pairs, experts, offsets, place, pair_at);
-            kernels::expert_product(s, true, h, gate_up, experts, offsets, pair_at, on_input, mid, pairs, N1, N2, top, gate, alpha, limit);
-            kernels::expert_product(s, false, mid, down, experts, offsets, pair_at, nullptr, out, pairs, N2, N1, top, gate);
+            kernels::expert_product(s, first, h, gate_up, experts, offsets, pair_at, on_input, mid, pairs, N1, N2, top, gate, alpha, limit);
+            kernels::expert_product(s, second, mid, down, experts, offsets, pair_at, nullptr, out, pairs, N2, N1, top, gate);
             t.place = place;
         }
         t.pairs = out;
@@ -663,11 +725,12 @@ public:
             shared->forward_into(ctx, h, y);
             t.rows = {y};
             t.scale = {1.0f};
+            if (shared_gate) t.factor = {r.gate};
         }
         return t;
     }
     std::optional<RowRouter> row_router(StepContext& ctx) override {
-        if (!corrected) return std::nullopt;
+        if (!by_terms) return std::nullopt;
         const int T = ctx.n_tokens;
         RowRouter r;
         r.matrix = router.data;
@@ -682,10 +745,11 @@ public:
         r.scale = route_scale;
         r.ids = static_cast<int32_t*>(ctx.workspace->get("routed.ids", T, top, DType::I32).data);
         r.weights = ctx.workspace->get("routed.weights", T, top, DType::F32).f32();
+        if (shared_gate) r.gate = ctx.workspace->get("routed.shared_gate", T, 1, DType::F32).f32();
         return r;
     }
     void run(StepContext& ctx, const Rows& h, const Rows& x, bool overwrite) {
-        if (corrected) {
+        if (by_terms) {
             const Rows y = ctx.workspace->get("routed.shared", ctx.n_tokens, hidden, DType::F32);
             kernels::terms_sum(ctx.stream(), ctx.runtime.dtype, forward_terms(ctx, h, y, false), x, ctx.n_tokens, overwrite);
             ctx.tap("routed", x);
@@ -713,9 +777,9 @@ public:
         mid = Rows{mid.data, mid.dtype, static_cast<int64_t>(pairs), inner, inner};
         Rows y = ws.get("routed.out", T, static_cast<int64_t>(top) * hidden, DType::F32);
         y = Rows{y.data, y.dtype, static_cast<int64_t>(pairs), hidden, hidden};
-        kernels::expert_product(s, true, h, gate_up, experts, offsets, pair_at, weight_on_output ? nullptr : weights, mid, pairs, static_cast<int>(inner),
+        kernels::expert_product(s, kernels::kGatedHalf, h, gate_up, experts, offsets, pair_at, weight_on_output ? nullptr : weights, mid, pairs, static_cast<int>(inner),
                                 static_cast<int>(hidden), top, gate, alpha, limit);
-        kernels::expert_product(s, false, mid, down, experts, offsets, pair_at, weights, y, pairs, static_cast<int>(hidden), static_cast<int>(inner), top, gate);
+        kernels::expert_product(s, kernels::kSecondHalf, mid, down, experts, offsets, pair_at, weights, y, pairs, static_cast<int>(hidden), static_cast<int>(inner), top, gate);
         kernels::expert_combine(s, x, y, place, T, top, weight_on_output ? weights : nullptr, overwrite);
         ctx.tap("routed", x);
         if (shared) shared->forward(ctx, h, x);
@@ -725,14 +789,14 @@ public:
     static constexpr int kLookupInPlan = 1024;
     int64_t hidden, inner;
     int experts, top, gate;
-    bool renormalise, softmax = false, weight_on_output = false, by_table = false, corrected = false;
+    bool renormalise, softmax = false, weight_on_output = false, by_table = false, by_terms = false, plain = false, shared_gate = false;
     int identity = 0, groups = 1, keep_groups = 1;
     float route_scale = 1.0f;
     const float* correction = nullptr;
     float alpha, limit;
     const float* router_bias = nullptr;
     Tensor router, table, gate_up, down;
-    std::unique_ptr<GatedFeedForward> shared;
+    std::unique_ptr<FeedForward> shared;
 };
 
 }  // namespace liyab::builtin

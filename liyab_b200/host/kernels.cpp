@@ -260,9 +260,9 @@ void attention_generic(cudaStream_t s, DType dtype, const Rows& q, const void* c
                        const int32_t* positions, const int32_t* block_table, int table_width, const Rows& out, int n_tokens,
                        const AttentionShape& a) {
     if (q.dtype != dtype || out.dtype != dtype) throw invalid_argument("attention: q, cache and out must have one element type");
-    check(lb_paged_attention_generic_sink(code(dtype, "cache"), q.data, q.stride, cache, tok_seq, positions, block_table, table_width,
+    check(lb_paged_attention_generic_capped(code(dtype, "cache"), q.data, q.stride, cache, tok_seq, positions, block_table, table_width,
                                           out.data, out.stride, n_tokens, a.n_head, a.n_kv_head, a.head_dim, a.page_size, a.scale,
-                                          a.mask(), a.distance, a.sink, s), "paged_attention_generic");
+                                          a.mask(), a.distance, a.sink, a.soft_cap, s), "paged_attention_generic");
 }
 
 void decode_attention(cudaStream_t s, bool tensor_cores, const Rows& q, const void* cache, int n_pages, const int32_t* positions,
@@ -274,12 +274,12 @@ void decode_attention(cudaStream_t s, bool tensor_cores, const Rows& q, const vo
     if (n_splits > 1 && (partial == nullptr || counters == nullptr))
         throw invalid_argument("decode attention: scratch buffers are missing");
     if (tensor_cores)
-        check(lb_decode_attention_mma_sink(q.data, q.stride, cache, n_pages, positions, block_table, table_width, out.data, out.stride,
+        check(lb_decode_attention_mma_capped(q.data, q.stride, cache, n_pages, positions, block_table, table_width, out.data, out.stride,
                                            partial, counters, n_seq, a.n_head, a.n_kv_head, a.head_dim, a.page_size, a.scale, a.mask(),
-                                           n_splits, a.distance, a.sink, s), "decode_attention_mma");
+                                           n_splits, a.distance, a.sink, a.soft_cap, a.score_bound, s), "decode_attention_mma");
     else
-        check(lb_decode_attention_sink(q.data, q.stride, cache, positions, block_table, table_width, out.data, out.stride, partial,
-                                       counters, n_seq, a.n_head, a.n_kv_head, a.head_dim, a.page_size, a.scale, a.mask(), n_splits, a.distance, a.sink, s),
+        check(lb_decode_attention_capped(q.data, q.stride, cache, positions, block_table, table_width, out.data, out.stride, partial,
+                                       counters, n_seq, a.n_head, a.n_kv_head, a.head_dim, a.page_size, a.scale, a.mask(), n_splits, a.distance, a.sink, a.soft_cap, a.score_bound, s),
               "decode_attention");
 }
 
@@ -294,12 +294,12 @@ void prefill_attention(const Runtime& rt, const Rows& q, int n_tokens, const voi
     const bool tc = prefill_tc_supports(a) && q.stride % 8 == 0 && out.stride % 8 == 0 && aligned16(q.data) &&
                     aligned16(out.data) && blocks <= 4 * static_cast<int64_t>(rt.sm_count) && a.scale > 0;     // it takes the maximum of the raw scores
     if (tc)
-        check(lb_prefill_attention_tc_sink(q.data, q.stride, n_tokens, cache, n_pages, q_start, n_past, block_table, table_width,
+        check(lb_prefill_attention_tc_capped(q.data, q.stride, n_tokens, cache, n_pages, q_start, n_past, block_table, table_width,
                                            out.data, out.stride, n_seq, max_q_len, a.n_head, a.n_kv_head, a.head_dim, a.page_size,
-                                           a.scale, a.mask(), a.distance, a.sink, rt.stream), "prefill_attention_tc");
+                                           a.scale, a.mask(), a.distance, a.sink, a.soft_cap, a.score_bound, rt.stream), "prefill_attention_tc");
     else
-        check(lb_prefill_attention_sink(q.data, q.stride, cache, q_start, n_past, block_table, table_width, out.data, out.stride, n_seq,
-                                        max_q_len, a.n_head, a.n_kv_head, a.head_dim, a.page_size, a.scale, a.mask(), a.distance, a.sink, rt.stream),
+        check(lb_prefill_attention_capped(q.data, q.stride, cache, q_start, n_past, block_table, table_width, out.data, out.stride, n_seq,
+                                        max_q_len, a.n_head, a.n_kv_head, a.head_dim, a.page_size, a.scale, a.mask(), a.distance, a.sink, a.soft_cap, a.score_bound, rt.stream),
               "prefill_attention");
 }
 
@@ -343,7 +343,8 @@ int gate_from_name(const std::string& name) {
     if (name == "gelu_tanh") return kGeluGate;
     if (name == "relu") return kRelu;
     if (name == "capped") return kCapped;
-    throw unsupported("gate '{}' is not supported; supported: sigmoid, silu, gelu_tanh, relu, capped", name);
+    if (name == "relu2") return kRelu2Gate;
+    throw unsupported("gate '{}' is not supported; supported: sigmoid, silu, gelu_tanh, relu, capped, relu2", name);
 }
 
 void head_gate(cudaStream_t s, const Rows& o, int o_head, const Rows& g, const float* gain, const Rows& out, int n_tokens, int n_head, int vdim, bool norm,
@@ -360,16 +361,16 @@ void gated_act(cudaStream_t s, const Rows& gu, const Rows& mid, int n_rows, int 
 
 void qkv_rotary_store(cudaStream_t s, const Rows& proj, const QkvColumns& c, const float* q_weight, const float* k_weight, const Rows& q_out, void* cache,
                       const int32_t* slot_mapping, int n_tokens, int norm_mode, float eps, const int32_t* positions, const float* freq, int rot_dims,
-                      const Rows* v_first_in, const Rows* v_first_out, const float* lambda, bool interleaved) {
+                      const Rows* v_first_in, const Rows* v_first_out, const float* lambda, bool interleaved, float rot_factor) {
     if (proj.dtype != DType::F32 || q_out.cols != static_cast<int64_t>(c.n_head) * c.padded) throw invalid_argument("qkv_rotary_store: buffers do not fit");
     const int64_t vcols = static_cast<int64_t>(c.n_kv_head) * c.vdim;
     const Rows* shared = v_first_in != nullptr ? v_first_in : v_first_out;
     if (shared != nullptr && (shared->dtype != DType::F32 || shared->cols != vcols || shared->rows < n_tokens))
         throw invalid_argument("qkv_rotary_store: the shared values are float32 [tokens, {}]", vcols);
-    check(lb_qkv_rotary_store_layout(code(q_out.dtype, "q_out"), proj.f32(), proj.stride, c.q_off, c.k_off, c.v_off, q_weight, k_weight, q_out.data, q_out.stride, cache,
+    check(lb_qkv_rotary_store_scaled(code(q_out.dtype, "q_out"), proj.f32(), proj.stride, c.q_off, c.k_off, c.v_off, q_weight, k_weight, q_out.data, q_out.stride, cache,
                               slot_mapping, n_tokens, c.n_head, c.n_kv_head, c.dim, c.vdim, c.padded, c.page_size, norm_mode, eps, positions, freq, rot_dims,
                               v_first_in != nullptr ? v_first_in->f32() : nullptr, v_first_out != nullptr ? v_first_out->f32() : nullptr,
-                              shared != nullptr ? shared->stride : 0, lambda, interleaved ? 1 : 0, s), "qkv_rotary_store");
+                              shared != nullptr ? shared->stride : 0, lambda, interleaved ? 1 : 0, rot_factor, s), "qkv_rotary_store");
 }
 
 void row_norm_gate(cudaStream_t s, const Rows& o, const Rows& g, const float* gain, const Rows& out, int n_rows, int gate, float eps) {
@@ -447,12 +448,12 @@ void expert_plan(cudaStream_t s, const int32_t* ids, int n_pairs, int n_experts,
     check(lb_expert_plan(ids, n_pairs, n_experts, offsets, place, pair_at, s), "expert_plan");
 }
 
-void expert_product(cudaStream_t s, bool gated, const Rows& a, const Tensor& w, int n_experts, const int32_t* offsets, const int32_t* pair_at,
+void expert_product(cudaStream_t s, ExpertHalf half, const Rows& a, const Tensor& w, int n_experts, const int32_t* offsets, const int32_t* pair_at,
                     const float* weights, const Rows& out, int n_pairs, int n, int k, int top, int gate, float alpha, float limit) {
-    if (a.dtype != w.dtype || w.numel() != static_cast<int64_t>(n_experts) * (gated ? 2 : 1) * n * k || a.cols != k || out.cols != n)
+    if (a.dtype != w.dtype || w.numel() != static_cast<int64_t>(n_experts) * (half == kGatedHalf ? 2 : 1) * n * k || a.cols != k || out.cols != n)
         throw invalid_argument("expert product: shapes do not fit");
-    if (out.dtype != (gated ? a.dtype : DType::F32)) throw invalid_argument("expert product: the output has the wrong type");
-    check(lb_expert_product_kind(code(a.dtype, "a"), gated ? 1 : 0, a.data, a.stride, w.data, static_cast<int64_t>(gated ? 2 : 1) * n * k, offsets, pair_at,
+    if (out.dtype != (half != kSecondHalf ? a.dtype : DType::F32)) throw invalid_argument("expert product: the output has the wrong type");
+    check(lb_expert_product_kind(code(a.dtype, "a"), half, a.data, a.stride, w.data, static_cast<int64_t>(half == kGatedHalf ? 2 : 1) * n * k, offsets, pair_at,
                                  weights, out.data, out.stride, n_pairs, n_experts, n, k, top, gate, alpha, limit, s), "expert_product");
 }
 
@@ -615,6 +616,7 @@ lb_output_terms terms_of(const OutputTerms& t, DType dtype, int64_t width) {
         o.y[i] = t.rows[i].f32();
         o.ldy[i] = t.rows[i].stride;
         o.scale[i] = t.scale[i];
+        o.factor[i] = i < t.factor.size() ? t.factor[i] : nullptr;
     }
     o.n_rows = static_cast<int>(t.rows.size());
     if (t.pairs.data != nullptr) {
@@ -633,7 +635,7 @@ lb_output_terms terms_of(const OutputTerms& t, DType dtype, int64_t width) {
     return o;
 }
 lb_router router_of(const RowRouter& r) {
-    return lb_router{r.matrix, r.bias, r.correction, r.n_experts, r.top, r.groups, r.keep, r.softmax ? 1 : 0, r.renormalise ? 1 : 0, r.scale, r.ids, r.weights};
+    return lb_router{r.matrix, r.bias, r.correction, r.n_experts, r.top, r.groups, r.keep, r.softmax ? 1 : 0, r.renormalise ? 1 : 0, r.scale, r.ids, r.weights, r.gate};
 }
 lb_streams_args streams_of(const Rows& x, int n_streams, const StreamReader* reader, const Rows* h, DType dtype) {
     if (x.dtype != DType::F32 || n_streams < 1 || x.cols % n_streams != 0) throw invalid_argument("streams: float32 rows of {} equal parts", n_streams);
@@ -681,6 +683,31 @@ void streams_join(cudaStream_t s, DType dtype, const Rows& x, const Join& join, 
     check(lb_streams_join(code(dtype, "h"), &a, &o, router != nullptr ? &r : nullptr, n_rows, s), "streams_join");
 }
 
+void norm_join(cudaStream_t s, DType dtype, const Rows& x, const NormRecipe& norm, float scale, const OutputTerms& terms, int n_rows, const NormRecipe* next,
+               const Rows* h, const RowRouter* router) {
+    if (x.dtype != DType::F32 || !norm.rms || norm.offset != nullptr) throw invalid_argument("norm join: float32 rows and an RMS norm over the whole row");
+    lb_norm_join_args a{};
+    a.x = x.f32();
+    a.ldx = x.stride;
+    a.width = static_cast<int>(x.cols);
+    a.gain = norm.gain;
+    a.gain_offset = norm.gain_offset;
+    a.eps = norm.eps;
+    a.scale = scale;
+    if (next != nullptr) {
+        if (h == nullptr || h->dtype != dtype || h->cols != x.cols || !next->rms || next->offset != nullptr) throw invalid_argument("norm join: the next input does not fit");
+        a.next_gain = next->gain;
+        a.next_offset = next->gain_offset;
+        a.next_eps = next->eps;
+        a.h = h->data;
+        a.ldh = h->stride;
+    }
+    const lb_output_terms o = terms_of(terms, dtype, x.cols);
+    lb_router r{};
+    if (router != nullptr) r = router_of(*router);
+    check(lb_norm_join(code(dtype, "h"), &a, &o, router != nullptr ? &r : nullptr, n_rows, s), "norm_join");
+}
+
 void router_choice(cudaStream_t s, const Rows& h, const RowRouter& router, int n_rows) {
     const lb_router r = router_of(router);
     check(lb_router_choice(code(h.dtype, "h"), &r, h.data, h.stride, n_rows, static_cast<int>(h.cols), s), "router_choice");
@@ -692,16 +719,16 @@ void terms_sum(cudaStream_t s, DType dtype, const OutputTerms& terms, const Rows
     check(lb_terms_sum(code(dtype, "self"), &o, x.f32(), x.stride, n_rows, static_cast<int>(x.cols), overwrite ? 1 : 0, s), "terms_sum");
 }
 
-bool expert_product_direct_supports(const Rows& a, const Tensor& w, int n_pairs, int n, int k, bool gated) {
-    return a.dtype == w.dtype && lb_expert_product_direct_supports(code(a.dtype, "a"), a.data, a.stride, w.data, static_cast<int64_t>(gated ? 2 : 1) * n * k, n_pairs, k) != 0;
+bool expert_product_direct_supports(const Rows& a, const Tensor& w, int n_pairs, int n, int k, ExpertHalf half) {
+    return a.dtype == w.dtype && lb_expert_product_direct_supports(code(a.dtype, "a"), a.data, a.stride, w.data, static_cast<int64_t>(half == kGatedHalf ? 2 : 1) * n * k, n_pairs, k) != 0;
 }
 
-void expert_product_direct(cudaStream_t s, bool gated, const Rows& a, const Tensor& w, int n_experts, const int32_t* ids, const float* weights, const Rows& out,
+void expert_product_direct(cudaStream_t s, ExpertHalf half, const Rows& a, const Tensor& w, int n_experts, const int32_t* ids, const float* weights, const Rows& out,
                            int n_pairs, int n, int k, int top, int gate, float alpha, float limit) {
-    if (a.dtype != w.dtype || w.numel() != static_cast<int64_t>(n_experts) * (gated ? 2 : 1) * n * k || a.cols != k || out.cols != n)
+    if (a.dtype != w.dtype || w.numel() != static_cast<int64_t>(n_experts) * (half == kGatedHalf ? 2 : 1) * n * k || a.cols != k || out.cols != n)
         throw invalid_argument("expert product: shapes do not fit");
-    if (out.dtype != (gated ? a.dtype : DType::F32)) throw invalid_argument("expert product: the output has the wrong type");
-    check(lb_expert_product_direct(code(a.dtype, "a"), gated ? 1 : 0, a.data, a.stride, w.data, static_cast<int64_t>(gated ? 2 : 1) * n * k, ids, weights, out.data,
+    if (out.dtype != (half != kSecondHalf ? a.dtype : DType::F32)) throw invalid_argument("expert product: the output has the wrong type");
+    check(lb_expert_product_direct(code(a.dtype, "a"), half, a.data, a.stride, w.data, static_cast<int64_t>(half == kGatedHalf ? 2 : 1) * n * k, ids, weights, out.data,
                                    out.stride, n_pairs, n_experts, n, k, top, gate, alpha, limit, s), "expert_product_direct");
 }
 

@@ -94,6 +94,8 @@ struct AttentionShape {
     const float* distance = nullptr;
     // A sink a head: device floats [n_head]; exp(sink[h]) joins the divisor of the head's softmax as it is, with no key and no value.
     const float* sink = nullptr;
+    // A soft cap on the scores, s <- soft_cap tanh(s / soft_cap) (0: none), and the largest |s| before it that can occur (0: unknown).
+    float soft_cap = 0.0f, score_bound = 0.0f;
     // One number for the kernels: 0 all earlier keys, w > 0 a window, -c a chunk (a shape has one of the two at most).
     int mask() const { return chunk > 0 ? -chunk : window; }
 };
@@ -190,12 +192,13 @@ void qk_norm_store(cudaStream_t s, const Rows& proj, const QkvColumns& c, const 
                    const int32_t* slot_mapping, int n_tokens, bool norm, float eps, const int32_t* positions = nullptr, float temp_coef = 0.0f,
                    int temp_every = 0);
 // The same for queries and keys that are normed over the whole projection and rotated, and for values that blend with an earlier layer's:
-// norm_mode 0 none, 1 a head (gains [dim]), 2 all of q and all of k each over one root mean square (gains [n_head * dim], [n_kv_head * dim]);
+// norm_mode 0 none, 1 a head (gains [dim]), 2 all of q and all of k each over one root mean square (gains [n_head * dim], [n_kv_head * dim]),
+// 3 a head, after its rotation (gains [dim]); rot_factor multiplies cosine and sine;
 // the first rot_dims values of a head rotated in pairs (i, i + rot_dims / 2), or, `interleaved`, (2i, 2i + 1), by positions[t] * freq[i]; with v_first_in the values become
 // (1 - lambda) v + lambda v_first_in[t], with v_first_out the row's own values are left there (float [T, n_kv_head * vdim]).
 void qkv_rotary_store(cudaStream_t s, const Rows& proj, const QkvColumns& c, const float* q_weight, const float* k_weight, const Rows& q_out, void* cache,
                       const int32_t* slot_mapping, int n_tokens, int norm_mode, float eps, const int32_t* positions, const float* freq, int rot_dims,
-                      const Rows* v_first_in, const Rows* v_first_out, const float* lambda, bool interleaved = false);
+                      const Rows* v_first_in, const Rows* v_first_out, const float* lambda, bool interleaved = false, float rot_factor = 1.0f);
 // out = o over the root mean square of the whole row, times gain (or null), times gate(g) (rows g without data: no gate).
 void row_norm_gate(cudaStream_t s, const Rows& o, const Rows& g, const float* gain, const Rows& out, int n_rows, int gate, float eps);
 // In place over the float rows x[:n_rows]: sigmoid, silu, gelu_tanh or relu (a Gate code).
@@ -207,7 +210,7 @@ void expert_plan_table(cudaStream_t s, const int32_t* tokens, const Tensor& tabl
                        int32_t* offsets, int32_t* place, int32_t* pair_at);
 void rows_to_bf16(cudaStream_t s, const Rows& x, const Rows& y, int n_rows);
 // kCapped has two numbers (alpha, limit): g' = min(g, limit), u' = clamp(u, -limit, limit), g' sigmoid(alpha g') (u' + 1).
-enum Gate : int { kSigmoid = 0, kSilu = 1, kGeluGate = 2, kRelu = 3, kCapped = 4 };
+enum Gate : int { kSigmoid = 0, kSilu = 1, kGeluGate = 2, kRelu = 3, kCapped = 4, kRelu2Gate = 5 };
 int gate_from_name(const std::string& name);
 // out[t, h * vdim + c] = f(o[t, h * o_head + c]) * gain * gate(g[t, h * vdim + c]); f: over the head's root mean square when `norm`;
 // rows g without data: no gate.
@@ -244,7 +247,9 @@ void matrix_memory_pieces(cudaStream_t s, const Rows& q, const Rows& k, const Ro
 void router_topk(cudaStream_t s, const Rows& h, const Tensor& router, int32_t* ids, float* weights, int n_rows, int top, bool softmax, bool renormalise,
                  const float* bias = nullptr);
 void expert_plan(cudaStream_t s, const int32_t* ids, int n_pairs, int n_experts, int32_t* offsets, int32_t* place, int32_t* pair_at);
-void expert_product(cudaStream_t s, bool gated, const Rows& a, const Tensor& w, int n_experts, const int32_t* offsets, const int32_t* pair_at,
+// What a product of an expert makes: y = down . mid, mid = act(gate . a) * (up . a), or mid = act(up . a).
+enum ExpertHalf : int { kSecondHalf = 0, kGatedHalf = 1, kPlainHalf = 2 };
+void expert_product(cudaStream_t s, ExpertHalf half, const Rows& a, const Tensor& w, int n_experts, const int32_t* offsets, const int32_t* pair_at,
                     const float* weights, const Rows& out, int n_pairs, int n, int k, int top, int gate, float alpha = 0.0f, float limit = 0.0f);
 // With `weights` [rows, top] every result is multiplied by its weight as it is added.
 // `overwrite`: the sums are written to x instead of added.
@@ -275,12 +280,16 @@ void streams_read(cudaStream_t s, DType dtype, const Rows& x, int n_streams, con
 // The streams take a sublayer's output; with `reader` the next sublayer's input goes to h, and with `router` its rows are routed.
 void streams_join(cudaStream_t s, DType dtype, const Rows& x, const Join& join, const OutputTerms& terms, int n_rows, const StreamReader* reader, const Rows* h,
                   const RowRouter* router);
+// x += scale * norm(sum of the terms), then h = next(x) in the compute type and, with a router, the experts of h: one launch (csrc/norm_join.cu).
+// Both norms are RMS norms over the whole row.
+void norm_join(cudaStream_t s, DType dtype, const Rows& x, const NormRecipe& norm, float scale, const OutputTerms& terms, int n_rows, const NormRecipe* next,
+               const Rows* h, const RowRouter* router);
 void router_choice(cudaStream_t s, const Rows& h, const RowRouter& router, int n_rows);
 // x (+)= the terms' sum; `dtype`: the type of the terms' own rows (`self`).
 void terms_sum(cudaStream_t s, DType dtype, const OutputTerms& terms, const Rows& x, int n_rows, bool overwrite);
 // The experts' products of a few pairs without a plan (pairs in their own order; a pair whose expert has no matrix is left alone).
-bool expert_product_direct_supports(const Rows& a, const Tensor& w, int n_pairs, int n, int k, bool gated);
-void expert_product_direct(cudaStream_t s, bool gated, const Rows& a, const Tensor& w, int n_experts, const int32_t* ids, const float* weights, const Rows& out,
+bool expert_product_direct_supports(const Rows& a, const Tensor& w, int n_pairs, int n, int k, ExpertHalf half);
+void expert_product_direct(cudaStream_t s, ExpertHalf half, const Rows& a, const Tensor& w, int n_experts, const int32_t* ids, const float* weights, const Rows& out,
                            int n_pairs, int n, int k, int top, int gate, float alpha = 0.0f, float limit = 0.0f);
 
 // ---- a matrix memory per head with a decay per key channel (gated linear attention; the delta rule) ----

@@ -83,8 +83,9 @@ private:
 // Further options.  `q_rank` r > 0: the queries come through a latent of their own, q = q_up (rms_norm(q_down h) * q_norm.weight); the down
 // map is part of the one projection.  `rot_layout` "interleaved": the rotation pairs value 2i with 2i + 1 instead of i with i + rot_dims/2.
 // `sink`: a learned number a head (the parameter `sink`) whose exponential joins the divisor of the head's softmax; no key, no value, not
-// scaled.  `head_gate`: the projection also makes one number a head, and the head's result is multiplied by its sigmoid.
-// The projection's rows: [queries or their latent | latent row (with own_latent) | gates (with head_gate)].
+// scaled.  `head_gate`: the projection also makes one number a head, and the head's result is multiplied by its sigmoid.  `value_gate`: it makes
+// one number for every value of every head instead, and the values are multiplied by the sigmoids one by one.
+// The projection's rows: [queries or their latent | latent row (with own_latent) | gates (with head_gate or value_gate)].
 
 class LatentAttention final : public Mixer {
 public:
@@ -106,6 +107,8 @@ public:
         if (layout != "half" && layout != "interleaved") throw unsupported("latent_attention: rot_layout '{}' is not supported; supported: half, interleaved", layout);
         a.interleaved = layout == "interleaved";
         head_gate = s.options.get_bool("head_gate", false);
+        value_gate = s.options.get_bool("value_gate", false);
+        if (head_gate && value_gate) throw unsupported("latent_attention: a gate a head or a gate a value, not both");
         if (a.rot_dims < 0 || a.rot_dims > a.rot || a.rot_dims % 2 != 0)
             throw invalid_model("latent_attention: {} of {} rotated values cannot be rotated in pairs", a.rot_dims, a.rot);
         if (a.window < 0) throw invalid_model("latent_attention: window {} is negative", a.window);
@@ -128,11 +131,11 @@ public:
         const int64_t hidden = need_int(s, "hidden"), H = need_int(s, "n_head"), dim = need_int(s, "dim", 0), rot = need_int(s, "rot_dim", 0);
         const int64_t vdim = need_int(s, "vdim"), rank = need_int(s, "kv_rank");
         const bool own = s.options.get_bool("own_latent", true), gated = s.options.get_bool("head_gate", false);
-        const int64_t q_rank = s.options.get_int("q_rank", 0);
+        const int64_t q_rank = s.options.get_int("q_rank", 0), gates = gated ? H : s.options.get_bool("value_gate", false) ? H * vdim : 0;
         std::vector<ParamDecl> out;
         // One projection makes the queries (or their latent) and, where the part has a latent of its own, the row [latent | rotated key] behind
         // them, then the heads' gates.
-        Linear::declare(out, "proj.", (q_rank > 0 ? q_rank : H * (dim + rot)) + (own ? rank + rot : 0) + (gated ? H : 0), hidden, false);
+        Linear::declare(out, "proj.", (q_rank > 0 ? q_rank : H * (dim + rot)) + (own ? rank + rot : 0) + gates, hidden, false);
         if (q_rank > 0) {
             out.push_back({"q_norm.weight", {q_rank}, ParamKind::Vector});
             Linear::declare(out, "q_up.", H * (dim + rot), q_rank, false);
@@ -168,6 +171,7 @@ public:
         const Rows qd = ws.get(own_latent ? "latent.qd" : "latent.q", T, proj.weight.dim(0), DType::F32);
         proj.forward(ctx, h, qd, T);
         const Rows row = own_latent ? qd.columns(first_cols, D) : Rows{};
+        const Rows value_gates = value_gate ? qd.columns(first_cols + (own_latent ? D : 0), static_cast<int64_t>(a.n_head) * a.vdim) : Rows{};
         const Rows gates = head_gate ? qd.columns(first_cols + (own_latent ? D : 0), a.n_head) : Rows{};
         const Rows* gate = head_gate ? &gates : nullptr;
         Rows q = qd.columns(0, q_cols);
@@ -230,14 +234,20 @@ public:
         }
         if (!few) kernels::head_matmul(s, attended, a.rank, uv, static_cast<int64_t>(a.vdim) * a.rank, 1, a.rank, values, a.vdim, T, a.vdim, a.rank, a.n_head);
         ctx.tap("attention", values);
-        out.forward(ctx, values, y, T, kernels::kNone, residual);
+        Rows heads = values;
+        if (value_gate) {
+            heads = ws.get("latent.heads", T, static_cast<int64_t>(a.n_head) * a.vdim, dt);
+            kernels::head_gate(s, values, a.vdim, value_gates, nullptr, heads, T, a.n_head, a.vdim, false, kernels::kSigmoid, eps);
+            ctx.tap("attention.gated", heads);
+        }
+        out.forward(ctx, heads, y, T, kernels::kNone, residual);
     }
 
     static constexpr int kFewTokens = 64;
     kernels::LatentShape a;
     int64_t hidden = 0, q_cols = 0, q_rank = 0;
     float eps = 1e-6f;
-    bool own_latent = true, head_gate = false;
+    bool own_latent = true, head_gate = false, value_gate = false;
     Linear proj, out, q_up;
     const float* q_gain = nullptr;
     Tensor uk, uv;

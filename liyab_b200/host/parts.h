@@ -83,6 +83,7 @@ struct StreamReader {
 struct OutputTerms {
     std::vector<Rows> rows;
     std::vector<float> scale;
+    std::vector<const float*> factor;      // one float a token (device) that also multiplies the row, or null; may be shorter than `rows`
     Rows pairs, self;
     const int32_t* place = nullptr;
     const int32_t* ids = nullptr;
@@ -101,6 +102,7 @@ struct RowRouter {
     float scale = 1.0f;
     int32_t* ids = nullptr;
     float* weights = nullptr;
+    float* gate = nullptr;      // where set, the matrix has one more row and gate[t] becomes the sigmoid of its product with row t
 };
 
 using TapFn = std::function<void(std::string_view name, const Rows& rows)>;
@@ -153,6 +155,9 @@ struct StepContext {
     // else changes the stream.
     Rows stream_rounded;
     int stream_rounded_entry = -1;
+    // Where the block after this one starts with an RMS norm over the whole row: that norm, so that the launch which ends a block can make the next
+    // one's input as well (null: it cannot).  The input it made is found at `next_input` below.
+    const struct NormRecipe* next_norm = nullptr;
     // Models with several residual streams: what the run after this one makes its input from (null for the last run), and that input where the
     // run before has made it already (for the run numbered `next_input_entry`; -1: nobody did), with the sublayer's last move of the streams.
     const StreamReader* next_reader = nullptr;
@@ -312,6 +317,8 @@ public:
     virtual std::vector<StateNeed> extra_states() const { return {}; }
     // How many residual streams the block works on; its `x` then holds them one after the other in a row.
     virtual int streams() const { return 1; }
+    // The norm that makes the block's first input, where the run before may apply it (a block with one stream).
+    virtual std::optional<NormRecipe> input_norm() const { return std::nullopt; }
     // What the block's first sublayer makes its input from, where the run before may do that for it.
     virtual std::optional<StreamReader> reader() const { return std::nullopt; }
 };

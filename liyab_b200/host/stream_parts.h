@@ -101,7 +101,7 @@ public:
         if (ctx.next_input_entry != unit.entry || ctx.next_input.data != h.data) make_input(ctx, x, mixer_join, mixer_norm, h);
         ctx.tap("mixer_norm", h);
         OutputTerms terms = mixer.forward_terms(ctx, h, y, unit);
-        show(ctx, "mixer.out", terms, width);
+        show_terms(ctx, "mixer.out", terms, width);
         if (feed_forward != nullptr) {
             const std::optional<StreamReader> next = reader_of(*ff_join, *ff_norm);
             const std::optional<RowRouter> router = next ? feed_forward->row_router(ctx) : std::nullopt;
@@ -111,7 +111,7 @@ public:
             if (!next) make_input(ctx, x, *ff_join, *ff_norm, h);
             ctx.tap("ff_norm", h);
             terms = feed_forward->forward_terms(ctx, h, y, router.has_value());
-            show(ctx, "feed_forward.out", terms, width);
+            show_terms(ctx, "feed_forward.out", terms, width);
         }
         // The last launch of the block makes the next block's input as well.
         kernels::streams_join(s, dt, x, feed_forward != nullptr ? *ff_join : mixer_join, terms, T, ctx.next_reader, ctx.next_reader != nullptr ? &h : nullptr, nullptr);
@@ -143,12 +143,6 @@ private:
         plain.in = j.in();
         kernels::streams_read(ctx.stream(), DType::F32, x, j.streams(), nullptr, ctx.n_tokens, plain, u);
         n.forward(ctx, u, h, ctx.n_tokens, nullptr);
-    }
-    static void show(StepContext& ctx, const char* name, const OutputTerms& terms, int64_t width) {
-        if (ctx.tap_fn == nullptr) return;
-        const Rows sum = ctx.workspace->get("block.shown", ctx.n_tokens, width, DType::F32);
-        kernels::terms_sum(ctx.stream(), ctx.runtime.dtype, terms, sum, ctx.n_tokens, true);
-        ctx.tap(name, sum);
     }
     LayerParts keep_;
 };

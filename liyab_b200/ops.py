@@ -54,12 +54,12 @@ _SIGNATURES = {
     "lb_decode_attention_mma_biased": [_p, _l, _p, _i, _p, _p, _i, _p, _l, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p],
     "lb_prefill_attention_biased": [_p, _l, _p, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p],
     "lb_prefill_attention_tc_biased": [_p, _l, _i, _p, _i, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p],
-    "lb_paged_attention_generic_sink": [_i, _p, _l, _p, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _f, _i, _p, _p, _p],
-    "lb_decode_attention_sink": [_p, _l, _p, _p, _p, _i, _p, _l, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _p],
-    "lb_decode_attention_mma_sink": [_p, _l, _p, _i, _p, _p, _i, _p, _l, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _p],
-    "lb_prefill_attention_sink": [_p, _l, _p, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p, _p],
-    "lb_prefill_attention_tc_sink": [_p, _l, _i, _p, _i, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p, _p],
-    "lb_qkv_rotary_store_layout": [_i, _p, _l, _i, _i, _i, _p, _p, _p, _l, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _p, _p, _l, _p, _i, _p],
+    "lb_paged_attention_generic_capped": [_i, _p, _l, _p, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _f, _i, _p, _p, _f, _p],
+    "lb_decode_attention_capped": [_p, _l, _p, _p, _p, _i, _p, _l, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _f, _f, _p],
+    "lb_decode_attention_mma_capped": [_p, _l, _p, _i, _p, _p, _i, _p, _l, _p, _p, _i, _i, _i, _i, _i, _f, _i, _i, _p, _p, _f, _f, _p],
+    "lb_prefill_attention_capped": [_p, _l, _p, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p, _f, _f, _p],
+    "lb_prefill_attention_tc_capped": [_p, _l, _i, _p, _i, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _i, _f, _i, _p, _p, _f, _f, _p],
+    "lb_qkv_rotary_store_scaled": [_i, _p, _l, _i, _i, _i, _p, _p, _p, _l, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _p, _p, _l, _p, _i, _f, _p],
     "lb_row_norm_gate": [_i, _p, _l, _p, _l, _p, _p, _l, _i, _i, _i, _f, _p],
     "lb_activate_columns": [_p, _l, _i, _i, _i, _p],
     "lb_router_table": [_p, _p, _p, _p, _i, _i, _i, _i, _p],
@@ -79,6 +79,10 @@ def lib():
             fn = getattr(l, name)
             fn.argtypes = args
             fn.restype = _i
+        # A struct that is shorter here than in the library would have the kernels read past its end.
+        for which, args in enumerate((OutputTerms, Router, StreamsArgs, NormJoinArgs)):
+            if l.lb_struct_bytes(which) != _c.sizeof(args):
+                raise RuntimeError(f"{args.__name__} has {_c.sizeof(args)} bytes here and {l.lb_struct_bytes(which)} in the library")
         _lib = l
     return _lib
 
@@ -355,19 +359,19 @@ def linear(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: 
 def paged_attention_generic(q: torch.Tensor, cache: torch.Tensor, tok_seq: torch.Tensor, positions: torch.Tensor,
                             block_table: torch.Tensor, out: torch.Tensor, n_tokens: int, n_head: int, n_kv_head: int,
                             head_dim: int, page_size: int, scale: float, window: int = 0, distance: Optional[torch.Tensor] = None,
-                            sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                            sink: Optional[torch.Tensor] = None, soft_cap: float = 0.0) -> torch.Tensor:
     """Causal attention of the step's tokens over their requests' pages, 32-bit arithmetic.  `distance` (float32, r1 [n_head] then
     r2 [n_head]): the score of the key d positions back loses r1 ln(1 + r2 d).  `sink` (float32 [n_head]): exp(sink[h]) joins the divisor
-    of head h's softmax, with no key and no value."""
+    of head h's softmax, with no key and no value.  `soft_cap` c > 0: a score s becomes c tanh(s / c)."""
     if q.dtype != cache.dtype or out.dtype != cache.dtype:
         raise invalid_argument("attention: q, cache and out must have one element type")
     if q.stride(1) != 1 or out.stride(1) != 1:
         raise invalid_argument("attention: q and out must be dense within a row")
-    check(lib().lb_paged_attention_generic_sink(
+    check(lib().lb_paged_attention_generic_capped(
         _code(cache.dtype, "cache"), _dev(q, "q"), q.stride(0), _dev(cache, "cache"),
         _dev(tok_seq, "tok_seq", torch.int32), _dev(positions, "positions", torch.int32),
         _dev(block_table, "block_table", torch.int32), block_table.stride(0), _dev(out, "out"), out.stride(0),
-        n_tokens, n_head, n_kv_head, head_dim, page_size, float(scale), int(window), _distance(distance, n_head), _sink(sink, n_head), stream_ptr()),
+        n_tokens, n_head, n_kv_head, head_dim, page_size, float(scale), int(window), _distance(distance, n_head), _sink(sink, n_head), float(soft_cap), stream_ptr()),
         "paged_attention_generic")
     return out
 
@@ -412,10 +416,10 @@ def decode_attention(q: torch.Tensor, cache: torch.Tensor, positions: torch.Tens
                      out: torch.Tensor, partial: Optional[torch.Tensor], counters: Optional[torch.Tensor], n_seq: int,
                      n_head: int, n_kv_head: int, head_dim: int, page_size: int, scale: float, window: int,
                      n_splits: int, tensor_cores: Optional[bool] = None, distance: Optional[torch.Tensor] = None,
-                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     sink: Optional[torch.Tensor] = None, soft_cap: float = 0.0, score_bound: float = 0.0) -> torch.Tensor:
     """Attention of one new token per request over its pages (bfloat16), keys split `n_splits` ways.
     `tensor_cores`: None picks the tensor-core kernel where it takes the shape, else the scalar one.  `distance`: as for
-    paged_attention_generic."""
+    paged_attention_generic.  `score_bound`: the largest |score| before the cap that can occur, 0 when unknown."""
     if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise invalid_argument("decode attention takes bfloat16 only")
     if q.stride(1) != 1 or out.stride(1) != 1 or q.stride(0) % 8 != 0 or q.data_ptr() % 16 != 0:
@@ -427,12 +431,13 @@ def decode_attention(q: torch.Tensor, cache: torch.Tensor, positions: torch.Tens
     if tensor_cores is None:
         tensor_cores = decode_attention_kernels(n_head, n_kv_head, head_dim, page_size)[1]
     cache_args = (_dev(cache, "cache"), cache.shape[0]) if tensor_cores else (_dev(cache, "cache"),)
-    fn = lib().lb_decode_attention_mma_sink if tensor_cores else lib().lb_decode_attention_sink
+    fn = lib().lb_decode_attention_mma_capped if tensor_cores else lib().lb_decode_attention_capped
     check(fn(
         _dev(q, "q"), q.stride(0), *cache_args, _dev(positions, "positions", torch.int32),
         _dev(block_table, "block_table", torch.int32), block_table.stride(0), _dev(out, "out"), out.stride(0),
         _opt(partial, "partial", torch.float32), _opt(counters, "counters", torch.int32), n_seq, n_head, n_kv_head,
-        head_dim, page_size, float(scale), int(window), int(n_splits), _distance(distance, n_head), _sink(sink, n_head), stream_ptr()), "decode_attention")
+        head_dim, page_size, float(scale), int(window), int(n_splits), _distance(distance, n_head), _sink(sink, n_head), float(soft_cap), float(score_bound),
+        stream_ptr()), "decode_attention")
     return out
 
 
@@ -457,10 +462,11 @@ def prefill_attention_tc_supports(n_head: int, n_kv_head: int, head_dim: int, pa
 def prefill_attention(q: torch.Tensor, cache: torch.Tensor, q_start: torch.Tensor, n_past: torch.Tensor,
                       block_table: torch.Tensor, out: torch.Tensor, n_seq: int, max_q_len: int, n_head: int,
                       n_kv_head: int, head_dim: int, page_size: int, scale: float, window: int = 0,
-                      tcgen05: Optional[bool] = None, distance: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      tcgen05: Optional[bool] = None, distance: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
+                      soft_cap: float = 0.0, score_bound: float = 0.0) -> torch.Tensor:
     """Attention of the step's prompt portions over their pages (bfloat16, tensor cores).  `tcgen05`: None picks
     the tcgen05 kernel where it takes the shape and the rows are 16-byte aligned, else the mma.sync one.  `distance`: as for
-    paged_attention_generic."""
+    paged_attention_generic; `score_bound`: as for decode_attention."""
     if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
         raise invalid_argument("prefill attention takes bfloat16 only")
     if q.stride(1) != 1 or out.stride(1) != 1:
@@ -474,18 +480,19 @@ def prefill_attention(q: torch.Tensor, cache: torch.Tensor, q_start: torch.Tenso
                    and out.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0
                    and blocks <= 4 * _sm_count(q.device))
     if tcgen05:
-        check(lib().lb_prefill_attention_tc_sink(
+        check(lib().lb_prefill_attention_tc_capped(
             _dev(q, "q"), q.stride(0), q.shape[0], _dev(cache, "cache"), cache.shape[0],
             _dev(q_start, "q_start", torch.int32), _dev(n_past, "n_past", torch.int32),
             _dev(block_table, "block_table", torch.int32), block_table.stride(0), _dev(out, "out"), out.stride(0), n_seq,
-            max_q_len, n_head, n_kv_head, head_dim, page_size, float(scale), int(window), _distance(distance, n_head), _sink(sink, n_head), stream_ptr()),
-            "prefill_attention_tc")
+            max_q_len, n_head, n_kv_head, head_dim, page_size, float(scale), int(window), _distance(distance, n_head), _sink(sink, n_head), float(soft_cap), float(score_bound),
+            stream_ptr()), "prefill_attention_tc")
         return out
-    check(lib().lb_prefill_attention_sink(
+    check(lib().lb_prefill_attention_capped(
         _dev(q, "q"), q.stride(0), _dev(cache, "cache"), _dev(q_start, "q_start", torch.int32),
         _dev(n_past, "n_past", torch.int32), _dev(block_table, "block_table", torch.int32), block_table.stride(0),
         _dev(out, "out"), out.stride(0), n_seq, max_q_len, n_head, n_kv_head, head_dim, page_size, float(scale),
-        int(window), _distance(distance, n_head), _sink(sink, n_head), stream_ptr()), "prefill_attention")
+        int(window), _distance(distance, n_head), _sink(sink, n_head), float(soft_cap), float(score_bound), stream_ptr()),
+        "prefill_attention")
     return out
 
 
@@ -859,16 +866,16 @@ def qkv_rotary_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w
                      q_out: torch.Tensor, cache: Optional[torch.Tensor], slot_mapping: torch.Tensor, n_head: int, n_kv_head: int, dim: int, vdim: int,
                      padded: int, page_size: int, norm_mode: int, eps: float, positions: torch.Tensor, freq: Optional[torch.Tensor], rot_dims: int,
                      v_first_in: Optional[torch.Tensor] = None, v_first_out: Optional[torch.Tensor] = None, blend: Optional[torch.Tensor] = None,
-                     interleaved: bool = False) -> torch.Tensor:
-    """Queries, keys and values of a float projection on their way to attention: norm_mode 0 none, 1 a head, 2 the whole projection; the first
-    rot_dims values of every head rotated by positions[t] * freq[i] (pairs (i, i + rot_dims / 2), or `interleaved` (2i, 2i + 1)); values blended with v_first_in by blend[0], or left in v_first_out."""
+                     interleaved: bool = False, rot_factor: float = 1.0) -> torch.Tensor:
+    """Queries, keys and values of a float projection on their way to attention: norm_mode 0 none, 1 a head, 2 the whole projection, 3 a head after its rotation; the first
+    rot_dims values of every head rotated by positions[t] * freq[i] (pairs (i, i + rot_dims / 2), or `interleaved` (2i, 2i + 1)), cosine and sine times rot_factor; values blended with v_first_in by blend[0], or left in v_first_out."""
     shared = v_first_in if v_first_in is not None else v_first_out
-    check(lib().lb_qkv_rotary_store_layout(_code(q_out.dtype, "q_out"), _dev(proj, "proj", torch.float32), proj.stride(0), q_off, k_off, v_off,
+    check(lib().lb_qkv_rotary_store_scaled(_code(q_out.dtype, "q_out"), _dev(proj, "proj", torch.float32), proj.stride(0), q_off, k_off, v_off,
                                     _opt(q_weight, "q_weight", torch.float32), _opt(k_weight, "k_weight", torch.float32), _dev(q_out, "q_out"), q_out.stride(0),
                                     _opt(cache, "cache", q_out.dtype), _dev(slot_mapping, "slot_mapping", torch.int32), proj.shape[0], n_head, n_kv_head, dim, vdim,
                                     padded, page_size, norm_mode, float(eps), _dev(positions, "positions", torch.int32), _opt(freq, "freq", torch.float32), rot_dims,
                                     _opt(v_first_in, "v_first_in", torch.float32), _opt(v_first_out, "v_first_out", torch.float32),
-                                    shared.stride(0) if shared is not None else 0, _opt(blend, "blend", torch.float32), int(interleaved), stream_ptr()), "qkv_rotary_store")
+                                    shared.stride(0) if shared is not None else 0, _opt(blend, "blend", torch.float32), int(interleaved), float(rot_factor), stream_ptr()), "qkv_rotary_store")
     return q_out
 
 
@@ -901,12 +908,12 @@ def router_table(tokens: torch.Tensor, table: torch.Tensor, n_experts: int):
 
 class OutputTerms(ctypes.Structure):
     _fields_ = [("n_rows", _i), ("y", _p * 4), ("ldy", _l * 4), ("scale", _f * 4), ("pairs", _p), ("ldp", _l), ("place", _p), ("ids", _p), ("weights", _p),
-                ("top", _i), ("n_real", _i), ("self_rows", _p), ("lds", _l)]
+                ("top", _i), ("n_real", _i), ("self_rows", _p), ("lds", _l), ("factor", _p * 4)]
 
 
 class Router(ctypes.Structure):
     _fields_ = [("matrix", _p), ("bias", _p), ("correction", _p), ("n_experts", _i), ("top", _i), ("groups", _i), ("keep", _i), ("softmax", _i), ("renormalise", _i),
-                ("scale", _f), ("ids", _p), ("weights", _p)]
+                ("scale", _f), ("ids", _p), ("weights", _p), ("gate", _p)]
 
 
 class StreamsArgs(ctypes.Structure):
@@ -934,12 +941,15 @@ declare("lb_channel_memory_pieces", [_i, _p, _p, _p, _i, _i, _p])
 
 
 def output_terms(rows=(), scale=(), pairs: Optional[torch.Tensor] = None, place: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
-                 weights: Optional[torch.Tensor] = None, n_real: int = 0, self_rows: Optional[torch.Tensor] = None) -> OutputTerms:
-    """A sublayer's output as the launch that joins it reads it: rows times numbers, and routed experts' results gathered row by row."""
+                 weights: Optional[torch.Tensor] = None, n_real: int = 0, self_rows: Optional[torch.Tensor] = None, factor=()) -> OutputTerms:
+    """A sublayer's output as the launch that joins it reads it: rows times numbers (and, with `factor`, times one float a row), and routed experts'
+    results gathered row by row."""
     o = OutputTerms()
     o.n_rows = len(rows)
     for k, (y, s) in enumerate(zip(rows, scale)):
         o.y[k], o.ldy[k], o.scale[k] = _dev(y, "y", torch.float32), y.stride(0), float(s)
+    for k, f in enumerate(factor):
+        o.factor[k] = _opt(f, "factor", torch.float32)
     if pairs is not None:
         o.pairs, o.ldp, o.place, o.ids = _dev(pairs, "pairs", torch.float32), pairs.stride(0), _opt(place, "place", torch.int32), _dev(ids, "ids", torch.int32)
         o.weights, o.top, o.n_real = _opt(weights, "weights", torch.float32), ids.shape[1], n_real
@@ -949,9 +959,11 @@ def output_terms(rows=(), scale=(), pairs: Optional[torch.Tensor] = None, place:
 
 
 def router_args(matrix: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.Tensor, bias: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None,
-           groups: int = 1, keep: int = 1, softmax: bool = True, renormalise: bool = False, scale: float = 1.0) -> Router:
-    return Router(_dev(matrix, "matrix"), _opt(bias, "bias", torch.float32), _opt(correction, "correction", torch.float32), matrix.shape[0], top, groups, keep,
-                  int(softmax), int(renormalise), float(scale), _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32))
+           groups: int = 1, keep: int = 1, softmax: bool = True, renormalise: bool = False, scale: float = 1.0, gate: Optional[torch.Tensor] = None) -> Router:
+    """gate: one float a row, the sigmoid of the product with the matrix's last row, which is no expert then."""
+    return Router(_dev(matrix, "matrix"), _opt(bias, "bias", torch.float32), _opt(correction, "correction", torch.float32),
+                  matrix.shape[0] - (1 if gate is not None else 0), top, groups, keep, int(softmax), int(renormalise), float(scale),
+                  _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32), _opt(gate, "gate", torch.float32))
 
 
 def streams_join(x: torch.Tensor, n_streams: int, n_rows: int, terms: Optional[OutputTerms] = None, mix: Optional[torch.Tensor] = None,
@@ -967,6 +979,28 @@ def streams_join(x: torch.Tensor, n_streams: int, n_rows: int, terms: Optional[O
                                 _c.byref(router) if router is not None else None, n_rows, stream_ptr()), "streams_join")
 
 
+class NormJoinArgs(ctypes.Structure):
+    _fields_ = [("x", _p), ("ldx", _l), ("width", _i), ("gain", _p), ("gain_offset", _f), ("eps", _f), ("scale", _f), ("next_gain", _p), ("next_offset", _f),
+                ("next_eps", _f), ("h", _p), ("ldh", _l)]
+
+
+declare("lb_norm_join", [_i, _p, _p, _p, _i, _p])
+declare("lb_struct_bytes", [_i])
+
+
+def norm_join(x: torch.Tensor, terms: OutputTerms, norm, n_rows: int, scale: float = 1.0, next_norm=None, h: Optional[torch.Tensor] = None,
+              router: Optional[Router] = None) -> None:
+    """x += scale * norm(sum of the terms), h = next_norm(x), both RMS norms over whole rows given as (gain or None, offset on the gain, eps); with a router
+    the experts of h (csrc/norm_join.cu)."""
+    f32 = torch.float32
+    gain, off, eps = norm
+    ngain, noff, neps = next_norm if next_norm is not None else (None, 0.0, 0.0)
+    a = NormJoinArgs(_dev(x, "x", f32), x.stride(0), x.shape[1], _opt(gain, "gain", f32), float(off), float(eps), float(scale), _opt(ngain, "next_gain", f32),
+                     float(noff), float(neps), _opt(h, "h"), h.stride(0) if h is not None else 0)
+    check(lib().lb_norm_join(_code(h.dtype, "h") if h is not None else F32, _c.byref(a), _c.byref(terms), _c.byref(router) if router is not None else None, n_rows,
+                             stream_ptr()), "norm_join")
+
+
 def router_choice(r: Router, h: torch.Tensor) -> None:
     check(lib().lb_router_choice(_code(h.dtype, "h"), _c.byref(r), _dev(h, "h"), h.stride(0), h.shape[0], h.shape[1], stream_ptr()), "router_choice")
 
@@ -977,14 +1011,15 @@ def terms_sum(terms: OutputTerms, x: torch.Tensor, dtype: torch.dtype, overwrite
     return x
 
 
-def experts_direct(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, gate: str = "silu") -> torch.Tensor:
-    """Every pair's result [T * top, width] without a plan (a few pairs, bfloat16); gate_up [E, 2 F, width], down [E, width, F].  Pairs whose expert is not
-    one of the E stay NaN."""
+def experts_direct(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, gate: str = "silu", plain: bool = False) -> torch.Tensor:
+    """Every pair's result [T * top, width] without a plan (a few pairs, bfloat16); gate_up [E, 2 F, width] (plain: [E, F, width], experts without a gate),
+    down [E, width, F].  Pairs whose expert is not one of the E stay NaN."""
     T, top = ids.shape
-    E, F2, width = gate_up.shape
-    mid = torch.full((T * top, F2 // 2), float("nan"), dtype=h.dtype, device=h.device)
+    E, rows, width = gate_up.shape
+    F = rows if plain else rows // 2
+    mid = torch.full((T * top, F), float("nan"), dtype=h.dtype, device=h.device)
     out = torch.full((T * top, width), float("nan"), dtype=torch.float32, device=h.device)
-    for gated, a, w, o, n, k in ((1, h, gate_up, mid, F2 // 2, width), (0, mid, down, out, width, F2 // 2)):
+    for gated, a, w, o, n, k in ((2 if plain else 1, h, gate_up, mid, F, width), (0, mid, down, out, width, F)):
         check(lib().lb_expert_product_direct(_code(h.dtype, "h"), gated, _dev(a, "a"), a.stride(0), _dev(w, "w", h.dtype), w.stride(0), _dev(ids, "ids", torch.int32), None,
                                              _dev(o, "o"), o.stride(0), T * top, E, n, k, top, GATE_KINDS[gate], 0.0, 0.0, stream_ptr()), "expert_product_direct")
     return out
