@@ -8,6 +8,7 @@
     python bench.py --design viresun [--size small]   # Viresun beside Vosurax and GPT-2 (see viresun_line)
     python bench.py --design revudra [--size small]   # Revudra beside Vosurax and GPT-2 (see revudra_line)
     python bench.py --design mokisun [--size small]   # Mokisun beside Vosurax and GPT-2 (see mokisun_line)
+    python bench.py --design gekitar [--size small]   # Gekitar beside Revudra and GPT-2 (see gekitar_line)
 
 A step is one decode step of the whole batch.  The default run has the layer
 sizes of GPT-2 small (12 layers, width 768, 12 heads) with random weights, a batch of
@@ -689,6 +690,94 @@ def mokisun_line(args) -> int:
     return 0
 
 
+def gekitar_config(size, layers=0):
+    """Gekitar with the width, depth, head count, inner width and vocabulary of a GPT-2 size.  Of every four blocks the first is attention over all
+    earlier positions (heads of 64, a quarter as many key/value heads, all of a head rotated at stretched frequencies, scores capped at 50) with the dense
+    feed-forward; the second attention over latent rows (heads of 48 + 16 rotated values, a latent of 256, queries through a latent of half the
+    width, a gate a value); the third the same under a window of 512 without the gate; the fourth reads the third's rows.  The second and
+    fourth have 16 experts of a quarter of the inner width, two a token, beside a shared one of that size, the third the dense feed-forward."""
+    g = SIZES[size]
+    L, W, H = max(4, layers or g["n_layer"]), g["n_embd"], g["n_head"]
+    attn = dict(heads=H, kv_heads=max(1, H // 4), dim=64, vdim=64, scale=0.125, softcap=50.0,
+                rot=dict(base=5e5, dims=64, scaling=dict(factor=4.0, original=512, fast=32.0, slow=1.0)))
+    latent = dict(heads=H, dim=48, rot_dim=16, vdim=64, kv_rank=256, q_rank=W // 2, scale=0.125, rot=dict(base=1e4, dims=16))
+    windowed = dict(latent, mask=dict(size=512))
+    dense = dict(kind="dense", ff=g["n_inner"], limit=7.0)
+    moe = dict(kind="moe", expert=dict(ff=g["n_inner"] // 4), router=dict(experts=16, top=2), shared=dict(ff=g["n_inner"] // 4))
+    blocks = []
+    for i in range(L):
+        kind, mixer, mlp = [("attention", attn, dense), ("latent_attention", latent, moe), ("latent_attention_2", windowed, dense),
+                            ("latent_attention_2", dict(windowed, kv_from=i - 1), moe)][i % 4]
+        blocks.append(dict(type=kind, mixer=mixer, mlp=mlp))
+    return dict(architecture="Gekitar", vocab=g["vocab_size"], width=W, norm=dict(eps=1e-6), embedding=dict(scale=float(W) ** 0.5), max_positions=g["n_positions"],
+                layers=blocks)
+
+
+def gekitar_bytes_and_flops(cfg, dtype_bytes, batch):
+    """Bytes a decode step of `batch` requests must read (weights its rows touch, visible cache rows) and the FLOPs of a prefill (products with the
+    weights a token uses, attention over the keys or the latent rows that a position sees, as it is computed)."""
+    W, V = cfg["width"], cfg["vocab"]
+    step_bytes, token_flops, attn, lat = 2 * V * W * dtype_bytes, 2 * V * W, [], []
+    for l in cfg["layers"]:
+        m, mlp = l["mixer"], l["mlp"]
+        H, D, E = m["heads"], m["dim"], m["vdim"]
+        if l["type"] == "attention":
+            mats = W * (H * D + m["kv_heads"] * (D + E)) + W * H * E
+            attn.append((H, m["kv_heads"], D, E))
+        else:
+            C, R = m["kv_rank"], m["rot_dim"]
+            mats = W * (m["q_rank"] + (0 if "kv_from" in m else C + R) + (H * E if l["type"] == "latent_attention" else 0))
+            mats += m["q_rank"] * H * (D + R) + H * C * (D + E) + W * H * E
+            lat.append((H, C, R, m["mask"]["size"] if "mask" in m else 1 << 30))
+        used = touched = mats
+        if mlp and mlp["kind"] == "dense":
+            used += 3 * W * mlp["ff"]
+            touched += 3 * W * mlp["ff"]
+        elif mlp:
+            X, top, F, S = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"], mlp["shared"]["ff"]
+            used += W * (X + 1) + 2 * W * (top * F + S)
+            touched += W * (X + 1) + 2 * W * (F * X * (1.0 - (1.0 - top / X) ** batch) + S)      # the experts a batch is expected to touch
+        token_flops += 2 * used
+        step_bytes += touched * dtype_bytes
+    def decode_bytes(mean_context):
+        return step_bytes + batch * dtype_bytes * (sum(2 * G * max(D, E) * mean_context for _, G, D, E in attn) +
+                                                   sum((C + R) * min(mean_context, c) for _, C, R, c in lat))
+
+    def prefill_flops(seq_lens, rows):
+        total = sum(seq_lens) * (token_flops - 2 * V * W) + 2 * rows * V * W
+        for H, G, D, E in attn:
+            total += sum(2 * H * (D + E) * s * (s + 1) // 2 for s in seq_lens)
+        for H, C, R, c in lat:
+            total += sum(2 * H * (2 * C + R) * sum(min(i + 1, c) for i in range(s)) for s in seq_lens)
+        return total
+
+    return decode_bytes, prefill_flops
+
+
+def gekitar_line(args) -> int:
+    """--design gekitar: decode (batch 1 / 8 / 64, 512-token prompts) and prefill (2 x 1024 tokens) of Gekitar at the layer sizes of GPT-2 `--size`, and
+    the same four figures of Revudra (the engine's closest design: rotated attention with sinks, attention over latent rows, small experts) and of GPT-2 at
+    that size."""
+    from liyab_b200.weights import write_random_model
+    pk = peaks()
+    dtype_bytes = 2 if args.dtype == "bfloat16" else 4
+    cfg = gekitar_config(args.size, args.layers)
+    steps = min(args.steps, 128)
+    out = {"design": "gekitar", "size": args.size, "dtype": args.dtype, "peaks": pk["source"],
+           "config": {k: cfg[k] for k in ("width", "vocab")} | {"layers": len(cfg["layers"]), "mixers": [l["mixer"] for l in cfg["layers"][:4]],
+                                                                "dense": cfg["layers"][0]["mlp"], "experts": cfg["layers"][1]["mlp"]}}
+    with tempfile.TemporaryDirectory(prefix="liyab_b200_bench_") as tmp:
+        folder = write_random_model(os.path.join(tmp, "gekitar"), cfg, seed=0, dtype=args.dtype)
+        out["gekitar"] = design_block(folder, args.dtype, steps, pk, lambda b: gekitar_bytes_and_flops(cfg, dtype_bytes, b))
+        other = revudra_config(args.size, args.layers)
+        folder = write_random_model(os.path.join(tmp, "revudra"), other, seed=0, dtype=args.dtype)
+        out["revudra"] = design_block(folder, args.dtype, steps, pk, lambda b: revudra_bytes_and_flops(other, dtype_bytes, b))
+        if not args.layers:
+            out["gpt2"], _ = size_block(tmp, args.size, args.dtype, steps, pk)
+    print(json.dumps(out))
+    return 0
+
+
 def reference_arm(args) -> int:
     from baseline.reference_arm import run
     return run(args)
@@ -706,8 +795,8 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-points", action="store_true", help="the headline figure only")
     ap.add_argument("--no-extra", action="store_true", help="skip the 32-bit engine, the other sizes and the mixed workload")
-    ap.add_argument("--design", default="gpt2", choices=["gpt2", "puzutar", "vosurax", "viresun", "revudra", "mokisun"],
-                    help="puzutar, vosurax, viresun, revudra, mokisun: that design at the layer sizes of GPT-2 --size beside GPT-2 itself (its own JSON line; the default run is unchanged)")
+    ap.add_argument("--design", default="gpt2", choices=["gpt2", "puzutar", "vosurax", "viresun", "revudra", "mokisun", "gekitar"],
+                    help="puzutar, vosurax, viresun, revudra, mokisun, gekitar: that design at the layer sizes of GPT-2 --size beside GPT-2 itself (its own JSON line; the default run is unchanged)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
@@ -721,6 +810,8 @@ def main() -> int:
         return revudra_line(args)
     if args.design == "mokisun":
         return mokisun_line(args)
+    if args.design == "gekitar":
+        return gekitar_line(args)
     if args.gpus != 1:
         print(f"bench.py measures a single-GPU engine; --gpus {args.gpus} is not supported (run with --gpus 1)")
         return 2
