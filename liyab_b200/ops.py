@@ -800,7 +800,7 @@ for _name, _args in {
 }.items():
     _SIGNATURES[_name] = _args
 
-GATE_KINDS = {"sigmoid": 0, "silu": 1, "gelu_tanh": 2, "relu": 3, "capped": 4}
+GATE_KINDS = {"sigmoid": 0, "silu": 1, "gelu_tanh": 2, "relu": 3, "capped": 4, "relu2": 5}      # relu2: experts without a gate only
 
 
 def embed_sinusoid(tokens: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, base: float, gain: Optional[torch.Tensor], x: torch.Tensor,
@@ -986,6 +986,7 @@ class NormJoinArgs(ctypes.Structure):
 
 declare("lb_norm_join", [_i, _p, _p, _p, _i, _p])
 declare("lb_struct_bytes", [_i])
+declare("lb_expert_product_kind", [_i, _i, _p, _l, _p, _l, _p, _p, _p, _p, _l, _i, _i, _i, _i, _i, _i, _f, _f, _p])
 
 
 def norm_join(x: torch.Tensor, terms: OutputTerms, norm, n_rows: int, scale: float = 1.0, next_norm=None, h: Optional[torch.Tensor] = None,
@@ -1009,6 +1010,27 @@ def terms_sum(terms: OutputTerms, x: torch.Tensor, dtype: torch.dtype, overwrite
     check(lib().lb_terms_sum(_code(dtype, "self"), _c.byref(terms), _dev(x, "x", torch.float32), x.stride(0), x.shape[0], x.shape[1], int(overwrite), stream_ptr()),
           "terms_sum")
     return x
+
+
+def experts_planned(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: Optional[torch.Tensor], gate: str = "silu",
+                    plain: bool = False, plain_units: bool = False) -> torch.Tensor:
+    """Every pair's result [T * top, width] through a plan, in the pairs' order; arguments as for experts_direct, `weights` [T, top] multiply the experts'
+    inputs.  `plain_units`: bfloat16 products on the 32-bit units."""
+    T, top = ids.shape
+    E, rows, width = gate_up.shape
+    F = rows if plain else rows // 2
+    offsets, place, pair_at = expert_plan(ids.flatten(), E)
+    mid = torch.full((T * top, F), float("nan"), dtype=h.dtype, device=h.device)
+    out = torch.full((T * top, width), float("nan"), dtype=torch.float32, device=h.device)
+    lib().lb_expert_product_set_plain(int(plain_units))
+    try:
+        for half, a, w, o, n, k in ((2 if plain else 1, h, gate_up, mid, F, width), (0, mid, down, out, width, F)):
+            check(lib().lb_expert_product_kind(_code(h.dtype, "h"), half, _dev(a, "a"), a.stride(0), _dev(w, "w", h.dtype), w.stride(0), _dev(offsets, "offsets"),
+                                               _dev(pair_at, "pair_at"), _opt(weights, "weights", torch.float32), _dev(o, "o"), o.stride(0), T * top, E, n, k, top,
+                                               GATE_KINDS[gate] if half else 0, 0.0, 0.0, stream_ptr()), "expert_product")
+    finally:
+        lib().lb_expert_product_set_plain(0)
+    return out[place.long()]
 
 
 def experts_direct(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, gate: str = "silu", plain: bool = False) -> torch.Tensor:
