@@ -221,6 +221,10 @@ int lb_rope_heads(int q_dtype, int wide_dtype, const void* q, int64_t ldq, const
  * 32-bit FMA whatever the element types (built: f32 f32 f32; bf16 bf16 f32; f32 bf16 bf16; f32 bf16 f32). */
 int lb_head_matmul(int a_dtype, int b_dtype, int c_dtype, const void* A, int64_t lda, int64_t a_head, const void* B, int64_t b_head,
                    int64_t b_k, int64_t b_n, void* C, int64_t ldc, int64_t c_head, int M, int N, int K, int n_head, void* stream);
+/* The same with C[t, h * c_head + n] multiplied by sigmoid(gate[t * ldg + h * N + n]). */
+int lb_head_matmul_gated(int a_dtype, int b_dtype, int c_dtype, const void* A, int64_t lda, int64_t a_head, const void* B, int64_t b_head,
+                         int64_t b_k, int64_t b_n, void* C, int64_t ldc, int64_t c_head, int M, int N, int K, int n_head, const float* gate, int64_t ldg,
+                         void* stream);
 /* out[t, h * rank + :] = sum_j p_j c_j with p = softmax_j((wide[t, h, :] . row_j) * scale) over the rows j of the token's
  * request with 0 <= position - j < window (window 0: all j <= position). */
 int lb_latent_attention(int cache_dtype, const float* wide, int64_t ldw, const void* cache, const int32_t* tok_seq,
@@ -241,6 +245,8 @@ int lb_latent_finish(const float* attended, int64_t lda, const float* part_o, co
 int lb_head_matmul_mma_supports(int64_t lda, int64_t a_head, int64_t b_head, int64_t b_k, int64_t b_n, int64_t ldc, int64_t c_head, int N, int K);
 int lb_head_matmul_mma(int a_dtype, const void* A, int64_t lda, int64_t a_head, const void* B, int64_t b_head, int64_t b_k, int64_t b_n, void* C, int64_t ldc,
                        int64_t c_head, int M, int N, int K, int n_head, void* stream);
+int lb_head_matmul_mma_gated(int a_dtype, const void* A, int64_t lda, int64_t a_head, const void* B, int64_t b_head, int64_t b_k, int64_t b_n, void* C,
+                             int64_t ldc, int64_t c_head, int M, int N, int K, int n_head, const float* gate, int64_t ldg, void* stream);
 /* The same attention on the tensor cores for bfloat16 wide queries and cache rows (lb_latent_attention_mma_supports: rank one of
  * 32, 64, 96, 128, 192, 256, 384, 512; rot a multiple of 16).  Request i brings rows q_start[i] .. q_start[i + 1] - 1, the first at
  * position n_past[i]; max_q_len is the longest such run.  n_splits > 1 cuts every request's keys over that many blocks; it needs
@@ -473,7 +479,8 @@ int lb_prefill_attention_tc_capped(const void* q, int64_t q_stride, int n_tokens
 /* What attention over latent rows may have besides its sizes.  sink [n_head]: exp(sink[h]) joins the divisor of head h's softmax (no key, no
  * value, not scaled).  gate: one float a (token, head) at gate[t * ldg + h]; the head's result is multiplied by sigmoid of it.  interleaved:
  * the rotation pairs value 2i with 2i + 1 instead of i with i + rot_dims / 2.  latent (lb_latent_prepare_ext): the rows [latent | rotated key],
- * ldl floats apart, where they do not follow the queries in qd.  A null pointer to the struct means none of it. */
+ * ldl floats apart, where they do not follow the queries in qd.  value_gate (lb_latent_finish_ext): one float for every value of every head,
+ * value_gate[t * ldvg + h * vdim + v], whose sigmoid multiplies it.  A null pointer to the struct means none of it. */
 typedef struct lb_latent_extras {
     const float* sink;
     const float* gate;
@@ -481,6 +488,8 @@ typedef struct lb_latent_extras {
     int interleaved;
     const float* latent;
     int64_t ldl;
+    const float* value_gate;
+    int64_t ldvg;
 } lb_latent_extras;
 int lb_latent_store_ext(int cache_dtype, const float* d, int64_t ldd, const float* gain, const float* freq, const int32_t* positions,
                         const int32_t* slot_mapping, void* cache, int n_tokens, int rank, int rot, int rot_dims, float eps, const lb_latent_extras* extras,

@@ -248,6 +248,28 @@ __global__ void gated_act_kernel(const float* __restrict__ gu, int64_t ld, TO* _
     }
 }
 
+// The same where rows split into 16-byte pieces: blocks over pieces and rows, four values a thread and trip.
+template <typename TO>
+__global__ void __launch_bounds__(256) gated_act_vec_kernel(const float* __restrict__ gu, int64_t ld, TO* __restrict__ mid, int64_t ldm, int n_rows, int F, int act,
+                                                            float alpha, float limit) {
+    lb_wait_for_predecessor();
+    lb_dependents_may_launch();
+    const int c = 4 * (blockIdx.x * blockDim.x + threadIdx.x);
+    if (c >= F) return;
+    for (int r = blockIdx.y; r < n_rows; r += gridDim.y) {
+        const float4 a = *reinterpret_cast<const float4*>(gu + (size_t)r * ld + c), u = *reinterpret_cast<const float4*>(gu + (size_t)r * ld + F + c);
+        const float x = lb_gated_pair(a.x, u.x, act, alpha, limit), y = lb_gated_pair(a.y, u.y, act, alpha, limit);
+        const float z = lb_gated_pair(a.z, u.z, act, alpha, limit), w = lb_gated_pair(a.w, u.w, act, alpha, limit);
+        TO* dst = mid + (size_t)r * ldm + c;
+        if constexpr (sizeof(TO) == 4) {
+            *reinterpret_cast<float4*>(dst) = make_float4(x, y, z, w);
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(x, y), hi = __floats2bfloat162_rn(z, w);
+            *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+        }
+    }
+}
+
 int grid_for(long total, int threads) { return (int)min((total + threads - 1) / threads, (long)148 * 16); }
 
 }  // namespace
@@ -359,6 +381,17 @@ extern "C" int lb_gated_act_kind(int out_dtype, const float* gu, int64_t ld, voi
     if (n_rows == 0) return LB_OK;
     auto s = static_cast<cudaStream_t>(stream);
     const dim3 grid(grid_for((long)n_rows * inner, 256)), block(256);
+    if (inner % 4 == 0 && ld % 4 == 0 && ldm % 4 == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(mid)) & 15) == 0) {
+        const int threads = min(256, (inner / 4 + 31) / 32 * 32);
+        const dim3 pieces((unsigned)((inner / 4 + threads - 1) / threads), (unsigned)min(n_rows, 4096));
+        if (out_dtype == LB_F32)
+            LB_CHECK_CUDA(lb_launch_overlapped(gated_act_vec_kernel<float>, pieces, dim3(threads), 0, s, gu, ld, (float*)mid, ldm, n_rows, inner, act, alpha, limit));
+        else if (out_dtype == LB_BF16)
+            LB_CHECK_CUDA(lb_launch_overlapped(gated_act_vec_kernel<__nv_bfloat16>, pieces, dim3(threads), 0, s, gu, ld, (__nv_bfloat16*)mid, ldm, n_rows, inner, act,
+                                               alpha, limit));
+        else return lb_fail(LB_ERR_INVALID_ARGUMENT, "gated_act: unknown dtype %d", out_dtype);
+        return LB_OK;
+    }
     if (out_dtype == LB_F32)
         LB_CHECK_CUDA(lb_launch_overlapped(gated_act_kernel<float>, grid, block, 0, s, gu, ld, (float*)mid, ldm, n_rows, inner, act, alpha, limit));
     else if (out_dtype == LB_BF16)

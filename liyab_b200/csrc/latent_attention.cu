@@ -151,12 +151,27 @@ latent_prepare_kernel(const float* __restrict__ qd, int64_t ldq, const __nv_bflo
 __global__ void __launch_bounds__(128)
 latent_finish_kernel(const float* __restrict__ attended, int64_t lda, const float* __restrict__ part_o, const float* __restrict__ part_ml,
                      const __nv_bfloat16* __restrict__ uv, __nv_bfloat16* __restrict__ values, int64_t ldv, int n_tokens, int n_head, int rank, int vdim,
-                     int n_splits, const float* __restrict__ sink, const float* __restrict__ gate, int64_t ldg) {
+                     int n_splits, const float* __restrict__ sink, const float* __restrict__ gate, int64_t ldg, const float* __restrict__ value_gate,
+                     int64_t ldvg) {
     extern __shared__ float osm[];             // the attended latent [rank], then the parts' factors [n_splits]
     float* factor = osm + rank;
+    const int t = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int pieces = rank / 8;
+    // A warp's values in batches of eight (v0, v0 + 4, ..); a batch's first pieces of the map are all asked for before any is used, the first batch's
+    // before the wait for the attention.  Lane b holds the gate of the batch's value b.
+    uint4 ahead_uv[8];
+    float gate_of = 1.0f;
+    auto fetch = [&](int v0) {
+#pragma unroll
+        for (int b = 0; b < 8; ++b) {
+            const int v = v0 + 4 * b;
+            ahead_uv[b] = make_uint4(0u, 0u, 0u, 0u);
+            if (v < vdim && lane < pieces) ahead_uv[b] = *reinterpret_cast<const uint4*>(uv + ((size_t)h * vdim + v) * rank + lane * 8);
+        }
+    };
+    fetch(warp);
     lb_wait_for_predecessor();
     lb_dependents_may_launch();
-    const int t = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (n_splits > 1) {
         // The parts' sums for this thread's first two latent values are asked for before the factors are made (up to 16 parts).
         constexpr int kParts = 16;
@@ -213,15 +228,11 @@ latent_finish_kernel(const float* __restrict__ attended, int64_t lda, const floa
     }
     __syncthreads();
     const float times = head_factor(gate, ldg, t, h);
-    const int pieces = rank / 8;
-    // A warp's values in batches of eight; a batch's first pieces are all asked for before any is used.
     for (int v0 = warp; v0 < vdim; v0 += 32) {
-        uint4 ahead[8];
-#pragma unroll
-        for (int b = 0; b < 8; ++b) {
-            const int v = v0 + 4 * b;
-            ahead[b] = make_uint4(0u, 0u, 0u, 0u);
-            if (v < vdim && lane < pieces) ahead[b] = *reinterpret_cast<const uint4*>(uv + ((size_t)h * vdim + v) * rank + lane * 8);
+        if (v0 != warp) fetch(v0);
+        if (value_gate != nullptr && lane < 8 && v0 + 4 * lane < vdim) {
+            const float z = value_gate[(size_t)t * ldvg + (size_t)h * vdim + v0 + 4 * lane];
+            gate_of = 1.0f / (1.0f + expf(-z));
         }
 #pragma unroll
         for (int b = 0; b < 8; ++b) {
@@ -230,7 +241,7 @@ latent_finish_kernel(const float* __restrict__ attended, int64_t lda, const floa
             const __nv_bfloat16* row = uv + ((size_t)h * vdim + v) * rank;
             float acc = 0.0f;
             for (int c = lane; c < pieces; c += 32) {
-                const uint4 raw = c == lane ? ahead[b] : *reinterpret_cast<const uint4*>(row + c * 8);
+                const uint4 raw = c == lane ? ahead_uv[b] : *reinterpret_cast<const uint4*>(row + c * 8);
                 const __nv_bfloat162* w = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {
@@ -239,7 +250,7 @@ latent_finish_kernel(const float* __restrict__ attended, int64_t lda, const floa
                     acc = fmaf(f.y, osm[c * 8 + 2 * k + 1], acc);
                 }
             }
-            acc = lb_warp_sum(acc);
+            acc = lb_warp_sum(acc) * __shfl_sync(0xffffffffu, gate_of, b);
             if (lane == 0) values[(size_t)t * ldv + (size_t)h * vdim + v] = __float2bfloat16_rn(acc * times);
         }
     }
@@ -250,7 +261,7 @@ latent_finish_kernel(const float* __restrict__ attended, int64_t lda, const floa
 template <typename TA, typename TB, typename TC>
 __global__ void __launch_bounds__(256)
 head_matmul_kernel(const TA* __restrict__ A, int64_t lda, int64_t a_head, const TB* __restrict__ B, int64_t b_head, int64_t b_k, int64_t b_n,
-                   TC* __restrict__ C, int64_t ldc, int64_t c_head, int M, int N, int K) {
+                   TC* __restrict__ C, int64_t ldc, int64_t c_head, int M, int N, int K, const float* __restrict__ gate, int64_t ldg) {
     __shared__ float As[32][33];
     __shared__ float Bs[32][65];
     lb_wait_for_predecessor();
@@ -296,7 +307,9 @@ head_matmul_kernel(const TA* __restrict__ A, int64_t lda, int64_t a_head, const 
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx + 16 * j;
-            if (n < N) C[(size_t)r * ldc + (size_t)h * c_head + n] = lb_from_float<TC>(acc[i][j]);
+            if (n >= N) continue;
+            const float f = gate != nullptr ? 1.0f / (1.0f + expf(-gate[(size_t)r * ldg + (size_t)h * N + n])) : 1.0f;
+            C[(size_t)r * ldc + (size_t)h * c_head + n] = lb_from_float<TC>(acc[i][j] * f);
         }
     }
 }
@@ -414,10 +427,10 @@ int pick_latent_attention(const float* wide, int64_t ldw, const void* cache, con
 
 template <typename TA, typename TB, typename TC>
 int launch_head_matmul(const void* A, int64_t lda, int64_t a_head, const void* B, int64_t b_head, int64_t b_k, int64_t b_n, void* C, int64_t ldc,
-                       int64_t c_head, int M, int N, int K, int n_head, cudaStream_t s) {
+                       int64_t c_head, int M, int N, int K, int n_head, const float* gate, int64_t ldg, cudaStream_t s) {
     const dim3 grid((N + 63) / 64, (M + 31) / 32, n_head);
     LB_CHECK_CUDA(lb_launch_overlapped(head_matmul_kernel<TA, TB, TC>, grid, dim3(256), 0, s, (const TA*)A, lda, a_head, (const TB*)B, b_head, b_k, b_n,
-                                       (TC*)C, ldc, c_head, M, N, K));
+                                       (TC*)C, ldc, c_head, M, N, K, gate, ldg));
     return LB_OK;
 }
 
@@ -491,7 +504,7 @@ extern "C" int lb_latent_finish_ext(const float* attended, int64_t lda, const fl
     if (n_tokens == 0) return LB_OK;
     LB_CHECK_CUDA(lb_launch_overlapped(latent_finish_kernel, dim3(n_tokens, n_head), dim3(128), (size_t)(rank + 32) * sizeof(float), static_cast<cudaStream_t>(stream),
                                        attended, lda, part_o, part_ml, (const __nv_bfloat16*)uv, (__nv_bfloat16*)values, ldv, n_tokens, n_head, rank, vdim,
-                                       n_splits, x.sink, x.gate, x.ldg));
+                                       n_splits, x.sink, x.gate, x.ldg, x.value_gate, x.ldvg));
     return LB_OK;
 }
 
@@ -518,11 +531,17 @@ extern "C" int lb_rope_heads_ext(int q_dtype, int wide_dtype, const void* q, int
 
 extern "C" int lb_head_matmul(int a_dtype, int b_dtype, int c_dtype, const void* A, int64_t lda, int64_t a_head, const void* B, int64_t b_head,
                               int64_t b_k, int64_t b_n, void* C, int64_t ldc, int64_t c_head, int M, int N, int K, int n_head, void* stream) {
+    return lb_head_matmul_gated(a_dtype, b_dtype, c_dtype, A, lda, a_head, B, b_head, b_k, b_n, C, ldc, c_head, M, N, K, n_head, nullptr, 0, stream);
+}
+
+extern "C" int lb_head_matmul_gated(int a_dtype, int b_dtype, int c_dtype, const void* A, int64_t lda, int64_t a_head, const void* B, int64_t b_head,
+                                    int64_t b_k, int64_t b_n, void* C, int64_t ldc, int64_t c_head, int M, int N, int K, int n_head, const float* gate,
+                                    int64_t ldg, void* stream) {
     LB_CHECK_ARG(M >= 0 && N > 0 && K > 0 && n_head > 0 && n_head <= 65535, "product per head: bad sizes M=%d N=%d K=%d heads=%d", M, N, K, n_head);
     if (M == 0) return LB_OK;
     auto s = static_cast<cudaStream_t>(stream);
     using B16 = __nv_bfloat16;
-#define LB_HEADS(TA, TB, TC) return launch_head_matmul<TA, TB, TC>(A, lda, a_head, B, b_head, b_k, b_n, C, ldc, c_head, M, N, K, n_head, s)
+#define LB_HEADS(TA, TB, TC) return launch_head_matmul<TA, TB, TC>(A, lda, a_head, B, b_head, b_k, b_n, C, ldc, c_head, M, N, K, n_head, gate, ldg, s)
     if (a_dtype == LB_F32 && b_dtype == LB_F32 && c_dtype == LB_F32) LB_HEADS(float, float, float);
     if (a_dtype == LB_BF16 && b_dtype == LB_BF16 && c_dtype == LB_F32) LB_HEADS(B16, B16, float);
     if (a_dtype == LB_F32 && b_dtype == LB_BF16 && c_dtype == LB_BF16) LB_HEADS(float, B16, B16);

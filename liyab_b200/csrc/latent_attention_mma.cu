@@ -474,7 +474,7 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_o, const floa
 template <bool KN, int KC, typename TA>
 __global__ void __launch_bounds__(128)
 head_matmul_mma_kernel(const TA* __restrict__ A, int64_t lda, int64_t a_head, const bf16* __restrict__ B, int64_t b_head, int64_t b_k, int64_t b_n,
-                       bf16* __restrict__ C, int64_t ldc, int64_t c_head, int M, int N, int K) {
+                       bf16* __restrict__ C, int64_t ldc, int64_t c_head, int M, int N, int K, const float* __restrict__ gate, int64_t ldg) {
     __shared__ __align__(16) bf16 As[64][KC + 8];
     __shared__ __align__(16) bf16 Bs[KN ? KC : 64][KN ? 72 : KC + 8];
     lb_wait_for_predecessor();
@@ -536,7 +536,14 @@ head_matmul_mma_kernel(const TA* __restrict__ A, int64_t lda, int64_t a_head, co
 #pragma unroll
         for (int nt = 0; nt < 8; ++nt) {
             const int n = n0 + nt * 8 + 2 * t4;
-            if (n < N) *reinterpret_cast<__nv_bfloat162*>(C + (size_t)r * ldc + (size_t)h * c_head + n) = __floats2bfloat162_rn(acc[nt][2 * half], acc[nt][2 * half + 1]);
+            if (n >= N) continue;
+            float a = acc[nt][2 * half], b2 = acc[nt][2 * half + 1];
+            if (gate != nullptr) {
+                const float* z = gate + (size_t)r * ldg + (size_t)h * N + n;
+                a *= 1.0f / (1.0f + expf(-z[0]));
+                b2 *= 1.0f / (1.0f + expf(-z[1]));
+            }
+            *reinterpret_cast<__nv_bfloat162*>(C + (size_t)r * ldc + (size_t)h * c_head + n) = __floats2bfloat162_rn(a, b2);
         }
     }
 }
@@ -582,6 +589,11 @@ extern "C" int lb_head_matmul_mma_supports(int64_t lda, int64_t a_head, int64_t 
 
 extern "C" int lb_head_matmul_mma(int a_dtype, const void* A, int64_t lda, int64_t a_head, const void* B, int64_t b_head, int64_t b_k, int64_t b_n, void* C, int64_t ldc,
                                   int64_t c_head, int M, int N, int K, int n_head, void* stream) {
+    return lb_head_matmul_mma_gated(a_dtype, A, lda, a_head, B, b_head, b_k, b_n, C, ldc, c_head, M, N, K, n_head, nullptr, 0, stream);
+}
+
+extern "C" int lb_head_matmul_mma_gated(int a_dtype, const void* A, int64_t lda, int64_t a_head, const void* B, int64_t b_head, int64_t b_k, int64_t b_n, void* C,
+                                        int64_t ldc, int64_t c_head, int M, int N, int K, int n_head, const float* gate, int64_t ldg, void* stream) {
     if (!lb_head_matmul_mma_supports(lda, a_head, b_head, b_k, b_n, ldc, c_head, N, K))
         return lb_fail(LB_ERR_UNSUPPORTED, "product per head on tensor cores: strides or sizes off its 16-byte pieces");
     LB_CHECK_ARG(M >= 0 && N > 0 && K > 0 && n_head > 0 && n_head <= 65535, "product per head: bad sizes M=%d N=%d K=%d heads=%d", M, N, K, n_head);
@@ -592,10 +604,10 @@ extern "C" int lb_head_matmul_mma(int a_dtype, const void* A, int64_t lda, int64
 #define LB_HEADS(KN, KC)                                                                                                                                    \
     if (a_dtype == LB_F32)                                                                                                                                  \
         LB_CHECK_CUDA(lb_launch_overlapped(head_matmul_mma_kernel<KN, KC, float>, grid, dim3(128), 0, s, (const float*)A, lda, a_head, (const bf16*)B, b_head, b_k, \
-                                           b_n, (bf16*)C, ldc, c_head, M, N, K));                                                                           \
+                                           b_n, (bf16*)C, ldc, c_head, M, N, K, gate, ldg));                                                                           \
     else                                                                                                                                                    \
         LB_CHECK_CUDA(lb_launch_overlapped(head_matmul_mma_kernel<KN, KC, bf16>, grid, dim3(128), 0, s, (const bf16*)A, lda, a_head, (const bf16*)B, b_head, b_k,  \
-                                           b_n, (bf16*)C, ldc, c_head, M, N, K))
+                                           b_n, (bf16*)C, ldc, c_head, M, N, K, gate, ldg))
     if (b_n == 1) {
         if (M <= 64) { LB_HEADS(true, 128); }
         else { LB_HEADS(true, 64); }

@@ -111,10 +111,78 @@ __global__ void __launch_bounds__(512) norm_join_kernel(lb_norm_join_args a, lb_
     }
 }
 
+// Many rows of a single term without a router: a warp a row of up to 128 NV values, everything it reads asked for at once (which the choices inside a
+// sum of terms do not let the compiler do), sums by shuffles, no block-wide barrier; the gains are read as they are used (the four rows of a block share
+// them in the first-level cache).
+template <int NV, typename T>
+__global__ void __launch_bounds__(128) norm_join_warp_kernel(lb_norm_join_args a, lb_output_terms o, int n_rows) {
+    const int lane = threadIdx.x & 31, t = blockIdx.x * 4 + (threadIdx.x >> 5), W = a.width;
+    lb_wait_for_predecessor();
+    lb_dependents_may_launch();
+    if (t >= n_rows) return;
+    Vals<4> x[NV], y[NV];
+    float* xrow = a.x + (size_t)t * a.ldx;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = 4 * (lane + 32 * i);
+        if (c >= W) break;
+        x[i] = load_vals<4>(xrow + c);
+        y[i] = load_vals<4>(o.y[0] + (size_t)t * o.ldy[0] + c);
+    }
+    const float times = o.factor[0] != nullptr ? o.scale[0] * o.factor[0][t] : o.scale[0];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        if (4 * (lane + 32 * i) >= W) break;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            y[i].v[k] *= times;
+            ss = fmaf(y[i].v[k], y[i].v[k], ss);
+        }
+    }
+    const float inv_w = 1.0f / (float)W, f = a.scale / sqrtf(lb_warp_sum(ss) * inv_w + a.eps);
+    ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = 4 * (lane + 32 * i);
+        if (c >= W) break;
+        Vals<4> g;
+        if (a.gain != nullptr) g = load_vals<4>(a.gain + c);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            x[i].v[k] = fmaf(y[i].v[k] * f, a.gain != nullptr ? g.v[k] + a.gain_offset : 1.0f, x[i].v[k]);
+            ss = fmaf(x[i].v[k], x[i].v[k], ss);
+        }
+        store_vals<4>(xrow + c, x[i]);
+    }
+    if (a.h == nullptr) return;
+    const float n = 1.0f / sqrtf(lb_warp_sum(ss) * inv_w + a.next_eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = 4 * (lane + 32 * i);
+        if (c >= W) break;
+        Vals<4> g, h;
+        if (a.next_gain != nullptr) g = load_vals<4>(a.next_gain + c);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) h.v[k] = x[i].v[k] * n * (a.next_gain != nullptr ? g.v[k] + a.next_offset : 1.0f);
+        store_vals<4>(static_cast<T*>(a.h) + (size_t)t * a.ldh + c, h);
+    }
+}
+
 template <int V, typename T>
 int launch_norm_join(const lb_norm_join_args& a, const lb_output_terms& o, const lb_router& r, int n_rows, cudaStream_t s) {
     const bool routes = r.matrix != nullptr;
     const int pieces = a.width / V;
+    if constexpr (V == 4) {
+        if (!routes && o.n_rows == 1 && o.pairs == nullptr && n_rows > 296 && a.width <= 1024) {
+            const dim3 grid((unsigned)((n_rows + 3) / 4)), block(128);
+            if (a.width <= 256) LB_CHECK_CUDA(lb_launch_overlapped(norm_join_warp_kernel<2, T>, grid, block, 0, s, a, o, n_rows));
+            else if (a.width <= 512) LB_CHECK_CUDA(lb_launch_overlapped(norm_join_warp_kernel<4, T>, grid, block, 0, s, a, o, n_rows));
+            else if (a.width <= 768) LB_CHECK_CUDA(lb_launch_overlapped(norm_join_warp_kernel<6, T>, grid, block, 0, s, a, o, n_rows));
+            else LB_CHECK_CUDA(lb_launch_overlapped(norm_join_warp_kernel<8, T>, grid, block, 0, s, a, o, n_rows));
+            return LB_OK;
+        }
+    }
     const int rows = routes && n_rows > 148 && (size_t)4 * (a.width + 4 + router_floats(r)) * sizeof(float) <= 48 * 1024 ? 4 : 1;
     // Many rows: two pieces a thread, so that more rows are under way on an SM.
     int nv = n_rows > 296 && pieces > 64 ? 2 : 1;

@@ -126,6 +126,87 @@ __global__ void qkv_rotary_store_kernel(const float* __restrict__ proj, int64_t 
     }
 }
 
+// The same where neighbouring values are paired, heads are normed one by one or not at all and no values blend: a warp a head, a pair of values a lane (NP
+// pairs where heads are larger), so that a head is one load, one sum, one rotation in registers and one store.  A warp asks for up to four heads at
+// once, and every lane makes the angles of its own pairs before the wait for the projection.
+template <typename T, int NP>
+__global__ void __launch_bounds__(512) qkv_pairs_store_kernel(const float* __restrict__ proj, int64_t ld, int q_off, int k_off, int v_off, const float* __restrict__ qw,
+                                                              const float* __restrict__ kw, T* __restrict__ q_out, int64_t ldq, T* __restrict__ cache,
+                                                              const int32_t* __restrict__ slot_mapping, int H, int G, int D, int E, int P, int page_size,
+                                                              int norm_mode, float eps, const int32_t* __restrict__ positions, const float* __restrict__ freq,
+                                                              int rot_dims, float rot_factor) {
+    constexpr int kAhead = 4;
+    const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5, jobs = H + 2 * G;
+    const int slot = cache != nullptr ? slot_mapping[t] : -1;
+    const int page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot - page * page_size : 0;
+    float cs[NP], sn[NP];
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+        const int pair = lane + 32 * i;
+        cs[i] = 1.0f;
+        sn[i] = 0.0f;
+        if (2 * pair < rot_dims) {
+            sincosf((float)positions[t] * freq[pair], &sn[i], &cs[i]);
+            cs[i] *= rot_factor;
+            sn[i] *= rot_factor;
+        }
+    }
+    lb_wait_for_predecessor();
+    lb_dependents_may_launch();
+    const float* row = proj + (size_t)t * ld;
+    const size_t plane = (size_t)G * page_size * P;
+    for (int job0 = warp; job0 < jobs; job0 += kAhead * n_warps) {
+        float2 v[kAhead][NP];
+#pragma unroll
+        for (int j = 0; j < kAhead; ++j) {
+            const int job = job0 + j * n_warps;
+            const bool is_v = job >= H + G;
+            const float* src = row + (job < H ? q_off + job * D : is_v ? v_off + (job - H - G) * E : k_off + (job - H) * D);
+#pragma unroll
+            for (int i = 0; i < NP; ++i) {
+                const int d = 2 * (lane + 32 * i);
+                v[j][i] = job < jobs && d < (is_v ? E : D) ? *reinterpret_cast<const float2*>(src + d) : make_float2(0.0f, 0.0f);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < kAhead; ++j) {
+            const int job = job0 + j * n_warps;
+            if (job >= jobs) break;
+            const bool is_q = job < H, is_v = job >= H + G;
+            if (!is_v) {
+                float ss = 0.0f;
+#pragma unroll
+                for (int i = 0; i < NP; ++i) {
+                    const float a = v[j][i].x, b = v[j][i].y;
+                    const float2 turned = make_float2(a * cs[i] - b * sn[i], b * cs[i] + a * sn[i]);
+                    ss += norm_mode == 3 ? fmaf(turned.x, turned.x, turned.y * turned.y) : fmaf(a, a, b * b);
+                    v[j][i] = turned;
+                }
+                if (norm_mode != 0) {
+                    const float inv = 1.0f / sqrtf(lb_warp_sum(ss) / (float)D + eps);
+                    const float* gain = is_q ? qw : kw;
+#pragma unroll
+                    for (int i = 0; i < NP; ++i) {
+                        const int d = 2 * (lane + 32 * i);
+                        v[j][i].x *= gain != nullptr && d < D ? inv * gain[d] : inv;
+                        v[j][i].y *= gain != nullptr && d < D ? inv * gain[d + 1] : inv;
+                    }
+                }
+            }
+            if (!is_q && slot < 0) continue;
+            T* dst = is_q ? q_out + (size_t)t * ldq + (size_t)job * P
+                          : cache + (size_t)page * 2 * plane + (is_v ? plane : 0) + ((size_t)(job - H - (is_v ? G : 0)) * page_size + off) * P;
+#pragma unroll
+            for (int i = 0; i < NP; ++i) {
+                const int d = 2 * (lane + 32 * i);
+                if (d >= P) break;
+                if constexpr (sizeof(T) == 4) *reinterpret_cast<float2*>(dst + d) = v[j][i];
+                else *reinterpret_cast<__nv_bfloat162*>(dst + d) = __floats2bfloat162_rn(v[j][i].x, v[j][i].y);
+            }
+        }
+    }
+}
+
 // ---------------------------------------------------------------- out = rms(o over the whole row) * gain * gate(g)
 // A block per row; rows of up to four values a thread stay in registers between the sum of squares and the write.
 template <typename TO>
@@ -309,6 +390,21 @@ extern "C" int lb_qkv_rotary_store_scaled(int dtype, const float* proj, int64_t 
     auto s = static_cast<cudaStream_t>(stream);
     // A warp a head where a block holds them all (a step of few tokens is then one pass); eight warps in turn for steps of many tokens.
     const int jobs = n_head + 2 * n_kv_head, threads = 32 * min(n_tokens <= 64 ? 16 : 8, jobs);
+    // Neighbouring pairs, heads one by one, nothing blended, everything on whole pairs: a pair a lane.
+    const uintptr_t places = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(cache);
+    if ((interleaved || rot_dims == 0) && v_first_in == nullptr && v_first_out == nullptr && padded <= 128 && (norm_mode == 0 || norm_mode == 3 ||
+        (norm_mode == 1 && q_weight == nullptr && k_weight == nullptr)) && (dim | vdim | padded | q_off | k_off | v_off) % 2 == 0 && ld % 2 == 0 && ldq % 2 == 0 &&
+        (places & 7) == 0 && (dtype == LB_F32 || dtype == LB_BF16)) {
+#define LB_PAIRS(T, NP) LB_CHECK_CUDA(lb_launch_overlapped(qkv_pairs_store_kernel<T, NP>, dim3(n_tokens), dim3(threads), 0, s, proj, ld, q_off, k_off, v_off, q_weight, \
+                                                           k_weight, (T*)q_out, ldq, (T*)cache, slot_mapping, n_head, n_kv_head, dim, vdim, padded, page_size,     \
+                                                           norm_mode, eps, positions, freq, rot_dims, rot_factor))
+        if (dtype == LB_F32 && padded <= 64) LB_PAIRS(float, 1);
+        else if (dtype == LB_F32) LB_PAIRS(float, 2);
+        else if (padded <= 64) LB_PAIRS(__nv_bfloat16, 1);
+        else LB_PAIRS(__nv_bfloat16, 2);
+#undef LB_PAIRS
+        return LB_OK;
+    }
     const size_t smem = (size_t)max(rot_dims, 1) * sizeof(float);
     if (dtype == LB_F32)
         LB_CHECK_CUDA(lb_launch_overlapped(qkv_rotary_store_kernel<float>, dim3(n_tokens), dim3(threads), smem, s, proj, ld, q_off, k_off, v_off, q_weight, k_weight,

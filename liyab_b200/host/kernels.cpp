@@ -543,13 +543,17 @@ void rope_heads(cudaStream_t s, const Rows& q, const float* freq, const int32_t*
 }
 
 void head_matmul(cudaStream_t s, const Rows& a, int64_t a_head, const Tensor& b, int64_t b_head, int64_t b_k, int64_t b_n, const Rows& c,
-                 int64_t c_head, int m, int n, int k, int n_head) {
+                 int64_t c_head, int m, int n, int k, int n_head, const Rows* gate) {
+    if (gate != nullptr && (gate->dtype != DType::F32 || gate->cols != static_cast<int64_t>(n_head) * n)) throw invalid_argument("product per head: the gate is one float a result");
+    const float* g = gate != nullptr ? gate->f32() : nullptr;
+    const int64_t ldg = gate != nullptr ? gate->stride : 0;
     if (b.dtype == DType::BF16 && c.dtype == DType::BF16 && lb_head_matmul_mma_supports(a.stride, a_head, b_head, b_k, b_n, c.stride, c_head, n, k)) {
-        check(lb_head_matmul_mma(code(a.dtype, "a"), a.data, a.stride, a_head, b.data, b_head, b_k, b_n, c.data, c.stride, c_head, m, n, k, n_head, s), "head_matmul_mma");
+        check(lb_head_matmul_mma_gated(code(a.dtype, "a"), a.data, a.stride, a_head, b.data, b_head, b_k, b_n, c.data, c.stride, c_head, m, n, k, n_head, g, ldg, s),
+              "head_matmul_mma");
         return;
     }
-    check(lb_head_matmul(code(a.dtype, "a"), code(b.dtype, "b"), code(c.dtype, "c"), a.data, a.stride, a_head, b.data, b_head, b_k, b_n, c.data, c.stride,
-                         c_head, m, n, k, n_head, s), "head_matmul");
+    check(lb_head_matmul_gated(code(a.dtype, "a"), code(b.dtype, "b"), code(c.dtype, "c"), a.data, a.stride, a_head, b.data, b_head, b_k, b_n, c.data, c.stride,
+                               c_head, m, n, k, n_head, g, ldg, s), "head_matmul");
 }
 
 bool latent_few_supports(const LatentShape& a) { return lb_latent_few_supports(a.dim, a.rot, a.rank, a.vdim, 1) != 0; }
@@ -563,9 +567,14 @@ void latent_prepare(cudaStream_t s, const Rows& qd, const Tensor& uk, const floa
 }
 
 void latent_finish(cudaStream_t s, const Rows& attended, const float* part_o, const float* part_ml, const Tensor& uv, const Rows& values, int n_tokens,
-                   const LatentShape& a, int n_splits, const Rows* gate) {
+                   const LatentShape& a, int n_splits, const Rows* gate, const Rows* value_gate) {
     if (attended.dtype != DType::F32 || uv.dtype != DType::BF16 || values.dtype != DType::BF16) throw invalid_argument("latent values: float32 latents, bfloat16 map and values");
-    const lb_latent_extras x = latent_extras(a, gate);
+    lb_latent_extras x = latent_extras(a, gate);
+    if (value_gate != nullptr) {
+        if (value_gate->dtype != DType::F32 || value_gate->cols != values.cols) throw invalid_argument("latent values: the gate is one float a value");
+        x.value_gate = value_gate->f32();
+        x.ldvg = value_gate->stride;
+    }
     check(lb_latent_finish_ext(attended.f32(), attended.stride, part_o, part_ml, uv.data, values.data, values.stride, n_tokens, a.n_head, a.rank, a.vdim, n_splits,
                                &x, s), "latent_finish");
 }

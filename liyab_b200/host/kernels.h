@@ -153,14 +153,15 @@ void rope_heads(cudaStream_t s, const Rows& q, const float* freq, const int32_t*
 // C[t, h * c_head + n] = sum_k A[t, h * a_head + k] * B[h * b_head + k * b_k + n * b_n].
 // Float rows, bfloat16 maps and output whose strides fit 16-byte pieces go to the tensor cores; everything else to the 32-bit units.
 void head_matmul(cudaStream_t s, const Rows& a, int64_t a_head, const Tensor& b, int64_t b_head, int64_t b_k, int64_t b_n, const Rows& c,
-                 int64_t c_head, int m, int n, int k, int n_head);
+                 int64_t c_head, int m, int n, int k, int n_head, const Rows* gate = nullptr);      // gate: float [m, n_head * n], C times its sigmoid
 // Steps of few tokens in bfloat16: rotation, keys' map and cache row in one launch; merge of the attention's parts and values' map in one.
 bool latent_few_supports(const LatentShape& a);
 void latent_prepare(cudaStream_t s, const Rows& qd, const Tensor& uk, const float* gain, const float* freq, const int32_t* positions,
                     const int32_t* slot_mapping, void* cache, const Rows& wide, int n_tokens, const LatentShape& a, float eps,
                     const Rows* latent = nullptr);      // latent: the rows [latent | rotated key] where they do not follow the queries in qd
 void latent_finish(cudaStream_t s, const Rows& attended, const float* part_o, const float* part_ml, const Tensor& uv, const Rows& values, int n_tokens,
-                   const LatentShape& a, int n_splits, const Rows* gate = nullptr);      // gate: one float a (token, head); the head's values times its sigmoid
+                   const LatentShape& a, int n_splits, const Rows* gate = nullptr,       // gate: one float a (token, head); the head's values times its sigmoid
+                   const Rows* value_gate = nullptr);                                  // value_gate: one float for every value of every head
 // The tensor-core kernel (bfloat16 wide queries and cache): whether it takes the shape, into how many parts a decode step's keys are cut
 // (a function of the step's shape and the longest span a query can see, so a recorded step and an eager one cut alike), and the launch.
 bool latent_mma_supports(const LatentShape& a);

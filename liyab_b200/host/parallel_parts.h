@@ -228,19 +228,14 @@ public:
             // the attention itself when the keys are not split.
             kernels::latent_attention_mma(s, wide, cache, ctx.q_start, ctx.n_past, view->block_table, view->table_width, attended, part_o, part_ml, T,
                                           ctx.n_seq, ctx.max_q_len, shape, splits, !few, few ? nullptr : gate);
-            if (few) kernels::latent_finish(s, attended, part_o, part_ml, uv, values, T, shape, splits, gate);
+            if (few) kernels::latent_finish(s, attended, part_o, part_ml, uv, values, T, shape, splits, gate, value_gate ? &value_gates : nullptr);
         } else {
             kernels::latent_attention(s, dt, wide, cache, ctx.tok_seq, ctx.positions, view->block_table, view->table_width, attended, T, shape, gate);
         }
-        if (!few) kernels::head_matmul(s, attended, a.rank, uv, static_cast<int64_t>(a.vdim) * a.rank, 1, a.rank, values, a.vdim, T, a.vdim, a.rank, a.n_head);
+        if (!few) kernels::head_matmul(s, attended, a.rank, uv, static_cast<int64_t>(a.vdim) * a.rank, 1, a.rank, values, a.vdim, T, a.vdim, a.rank, a.n_head,
+                                       value_gate ? &value_gates : nullptr);
         ctx.tap("attention", values);
-        Rows heads = values;
-        if (value_gate) {
-            heads = ws.get("latent.heads", T, static_cast<int64_t>(a.n_head) * a.vdim, dt);
-            kernels::head_gate(s, values, a.vdim, value_gates, nullptr, heads, T, a.n_head, a.vdim, false, kernels::kSigmoid, eps);
-            ctx.tap("attention.gated", heads);
-        }
-        out.forward(ctx, heads, y, T, kernels::kNone, residual);
+        out.forward(ctx, values, y, T, kernels::kNone, residual);
     }
 
     static constexpr int kFewTokens = 64;

@@ -524,9 +524,9 @@ for _name, _args in {
     "lb_token_side": [_i, _p, _l, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f, _p],
     "lb_latent_store": [_i, _p, _l, _p, _p, _p, _p, _p, _i, _i, _i, _i, _f, _p],
     "lb_rope_heads": [_i, _i, _p, _l, _p, _p, _p, _l, _i, _i, _i, _i, _i, _i, _p],
-    "lb_head_matmul": [_i, _i, _i, _p, _l, _l, _p, _l, _l, _l, _p, _l, _l, _i, _i, _i, _i, _p],
+    "lb_head_matmul_gated": [_i, _i, _i, _p, _l, _l, _p, _l, _l, _l, _p, _l, _l, _i, _i, _i, _i, _p, _l, _p],
     "lb_head_matmul_mma_supports": [_l, _l, _l, _l, _l, _l, _l, _i, _i],
-    "lb_head_matmul_mma": [_i, _p, _l, _l, _p, _l, _l, _l, _p, _l, _l, _i, _i, _i, _i, _p],
+    "lb_head_matmul_mma_gated": [_i, _p, _l, _l, _p, _l, _l, _l, _p, _l, _l, _i, _i, _i, _i, _p, _l, _p],
     "lb_latent_attention": [_i, _p, _l, _p, _p, _p, _p, _i, _p, _l, _i, _i, _i, _i, _i, _f, _i, _p],
     "lb_latent_attention_mma_supports": [_i, _i, _i, _i],
     "lb_latent_attention_mma": [_p, _l, _p, _p, _p, _p, _i, _p, _l, _p, _p, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _p],
@@ -598,17 +598,19 @@ def rope_heads(q: torch.Tensor, freq: torch.Tensor, positions: torch.Tensor, wid
 
 
 def head_matmul(a: torch.Tensor, a_head: int, b: torch.Tensor, b_head: int, b_k: int, b_n: int, c: torch.Tensor, c_head: int, n: int, k: int,
-                n_head: int, tensor_cores: bool = False) -> torch.Tensor:
-    """c[t, h * c_head + j] = sum_i a[t, h * a_head + i] * b.flat[h * b_head + i * b_k + j * b_n] for j < n, i < k, every head h."""
+                n_head: int, tensor_cores: bool = False, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """c[t, h * c_head + j] = sum_i a[t, h * a_head + i] * b.flat[h * b_head + i * b_k + j * b_n] for j < n, i < k, every head h; with `gate` (float32
+    [m, n_head * n]) times its sigmoid."""
     m = a.shape[0]
+    g, ldg = _opt(gate, "gate", torch.float32), gate.stride(0) if gate is not None else 0
     if tensor_cores:
         if not lib().lb_head_matmul_mma_supports(a.stride(0), a_head, b_head, b_k, b_n, c.stride(0), c_head, n, k):
             raise invalid_argument("head_matmul: the tensor-core kernel does not take these strides")
-        check(lib().lb_head_matmul_mma(_code(a.dtype, "a"), _dev(a, "a"), a.stride(0), a_head, _dev(b, "b", torch.bfloat16), b_head, b_k, b_n,
-                                       _dev(c, "c", torch.bfloat16), c.stride(0), c_head, m, n, k, n_head, stream_ptr()), "head_matmul_mma")
+        check(lib().lb_head_matmul_mma_gated(_code(a.dtype, "a"), _dev(a, "a"), a.stride(0), a_head, _dev(b, "b", torch.bfloat16), b_head, b_k, b_n,
+                                       _dev(c, "c", torch.bfloat16), c.stride(0), c_head, m, n, k, n_head, g, ldg, stream_ptr()), "head_matmul_mma")
     else:
-        check(lib().lb_head_matmul(_code(a.dtype, "a"), _code(b.dtype, "b"), _code(c.dtype, "c"), _dev(a, "a"), a.stride(0), a_head, _dev(b, "b"),
-                                   b_head, b_k, b_n, _dev(c, "c"), c.stride(0), c_head, m, n, k, n_head, stream_ptr()), "head_matmul")
+        check(lib().lb_head_matmul_gated(_code(a.dtype, "a"), _code(b.dtype, "b"), _code(c.dtype, "c"), _dev(a, "a"), a.stride(0), a_head, _dev(b, "b"),
+                                   b_head, b_k, b_n, _dev(c, "c"), c.stride(0), c_head, m, n, k, n_head, g, ldg, stream_ptr()), "head_matmul")
     return c
 
 

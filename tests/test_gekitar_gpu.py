@@ -72,14 +72,14 @@ def check(got, want, dtype, rel_tol=REL_TOL, median=1.5e-2, worst=6e-2, apart=0.
 
 
 # What the plain model calls a part's output -> the name of the engine's tap.
-TAPS = {"mixer_in": "mixer_norm", "attention": "attention", "heads": "attention.gated", "mixer_out": "mixer.out", "feed_forward_in": "ff_norm",
+TAPS = {"mixer_in": "mixer_norm", "attention": "attention", "heads": "attention", "mixer_out": "mixer.out", "feed_forward_in": "ff_norm",
         "feed_forward_out": "feed_forward.out", "out": "block"}
 
 
 @pytest.mark.parametrize("name", sorted(CONFIGS))
 def test_every_mechanism_by_itself(name, models):
-    """The parts' outputs, layer by layer, against the plain functions in float32: the embedded rows, both sublayers' inputs, the attention's heads before
-    their gate and after, both sublayers' outputs before their norm, and the stream after the block.  A whole prompt, then the same prompt cut in two
+    """The parts' outputs, layer by layer, against the plain functions in float32: the embedded rows, both sublayers' inputs, the attention's heads
+    (behind their gate where they have one), both sublayers' outputs before their norm, and the stream after the block.  A whole prompt, then the same prompt cut in two
     and in three."""
     from liyab_b200.engine import StepEntry
     path, config, weights = models[name]
@@ -111,7 +111,7 @@ def test_every_mechanism_by_itself(name, models):
         for i, ref_run in enumerate(want):
             runs[i]["block"] = runs[i]["feed_forward" if "feed_forward" in runs[i] else "mixer"]      # the stream as the block leaves it
             for plain_name, tap_name in TAPS.items():
-                if plain_name not in ref_run or (plain_name == "heads" and config["layers"][i]["type"] != "latent_attention"):
+                if plain_name not in ref_run or plain_name == ("attention" if "heads" in ref_run else "heads"):        # latent attention: behind its gate
                     continue
                 ref = ref_run[plain_name]
                 rows = np.concatenate(runs[i][tap_name], axis=0)

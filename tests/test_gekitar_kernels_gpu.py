@@ -180,7 +180,7 @@ def choice(z, top):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("W,T,N,top", [(96, 13, 6, 2), (768, 9, 16, 2), (100, 300, 5, 3), (98, 7, 4, 4), (33, 301, 3, 1), (2052, 5, 40, 6), (1, 4, 1, 1), (2500, 150, 8, 2), (4100, 310, 2, 1),
+@pytest.mark.parametrize("W,T,N,top", [(96, 13, 6, 2), (768, 9, 16, 2), (100, 300, 5, 3), (98, 7, 4, 4), (33, 301, 3, 1), (2052, 5, 40, 6), (200, 310, 4, 2), (512, 300, 4, 1), (768, 301, 4, 2), (1024, 299, 2, 1), (1, 4, 1, 1), (2500, 150, 8, 2), (4100, 310, 2, 1),
                                        (2051, 2, 2, 1), (9000, 3, 2, 1)])
 def test_launch_between_two_norms(dev, dtype, W, T, N, top):
     """Terms of both kinds (rows times numbers and times one float a row; routed results through a plan's places and without one), norm, sum into the stream, the next
@@ -223,6 +223,16 @@ def test_launch_between_two_norms(dev, dtype, W, T, N, top):
             assert (rid.cpu() == wid).float().mean() > 0.99
             same = (rid.cpu() == wid).all(1)
             assert (d(rw) - ww)[same].abs().max() < 1e-4 and (d(gate) - torch.sigmoid(z[:, N])).abs().max() < 1e-5
+    # A single term (hundreds of rows take a warp a row), with a factor a row.
+    for last in (True, False):
+        x = torch.empty(T, W + 4, device=dev)[:, :W]
+        x.copy_(x0)
+        h = None if last else torch.full((T, W), float("nan"), dtype=dtype, device=dev)
+        ops.norm_join(x, ops.output_terms([y1], [0.5], factor=(f2,)), (gain, 1.0, eps), T, scale, next_norm=None if last else (gain2, 0.5, eps2), h=h)
+        want = d(x0) + scale * rms(0.5 * d(f2)[:, None] * d(y1), eps) * (1.0 + d(gain))
+        assert (d(x) - want).abs().max() < 2e-5 * max(1.0, float(want.abs().max()))
+        hw = rms(want, eps2) * (0.5 + d(gain2))
+        assert last or (d(h) - hw).abs().max() < (2e-5 if dtype == torch.float32 else 1e-2) * max(1.0, float(hw.abs().max()))
     # Without gains: ones.
     x = x0.clone()
     ops.norm_join(x, ops.output_terms([y1], [1.0]), (None, 1.0, eps), T)
@@ -283,3 +293,40 @@ def test_activations_that_have_no_such_form_are_refused(dev):
     gu = torch.zeros(2, 8, device=dev)
     with pytest.raises(LiyabError):
         ops.gated_act_kind(gu, torch.zeros(2, 4, device=dev), "relu2")
+
+
+# ---------------------------------------------------------------- the gate on every value
+
+@pytest.mark.parametrize("M,H,E,C", [(5, 3, 14, 24), (70, 4, 32, 64), (64, 12, 64, 256), (200, 2, 70, 10), (1, 1, 1, 1), (33, 5, 8, 40)])
+def test_gate_on_every_value_of_the_values_product(dev, M, H, E, C):
+    """The product per head with a gate a result on the 32-bit units (both types) and on the tensor cores, with and without the gate, gates that lie in columns of
+    a wider buffer."""
+    from liyab_b200 import ops
+    rng = np.random.default_rng(M * E)
+    r = lambda *s: torch.from_numpy(rng.standard_normal(s)).float().to(dev)
+    att, uv, wide = r(M, H * C), r(H * E, C) * C ** -0.5, r(M, 7 + H * E)
+    gate = wide[:, 7:]
+    d = lambda t: t.double().cpu()
+    for tb, tc, tensor in ((torch.float32, torch.float32, False), (torch.bfloat16, torch.bfloat16, False), (torch.bfloat16, torch.bfloat16, True)):
+        w = uv.to(tb)
+        want = torch.einsum("mhc,hec->mhe", d(att).reshape(M, H, C), d(w).reshape(H, E, C)).reshape(M, H * E)
+        if tensor and not (C % 8 == 0 and E % 2 == 0):
+            continue
+        for g in (gate, None):
+            out = torch.full((M, H * E), float("nan"), dtype=tc, device=dev)
+            ops.head_matmul(att, C, w, E * C, 1, C, out, E, E, C, H, tensor_cores=tensor, gate=g)
+            ref = want * torch.sigmoid(d(gate)) if g is not None else want
+            assert (d(out) - ref).abs().max() < (1e-5 if tc == torch.float32 else 2e-2) * max(1.0, float(ref.abs().max()))
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("rows,F", [(3, 48), (70, 3072), (5, 50), (9, 4), (1, 1), (5000, 8)])
+def test_capped_gate_in_pieces_and_value_by_value(dev, dtype, rows, F):
+    from liyab_b200 import ops
+    rng = np.random.default_rng(rows + F)
+    gu = torch.from_numpy(rng.standard_normal((rows, 2 * F)) * 3).float().to(dev)
+    out = torch.full((rows, F), float("nan"), dtype=dtype, device=dev)
+    ops.gated_act_kind(gu, out, "capped", 1.702, 2.0)
+    g, u = gu[:, :F].double().cpu().clamp(max=2.0), gu[:, F:].double().cpu().clamp(-2.0, 2.0)
+    want = g * torch.sigmoid(1.702 * g) * (u + 1)
+    assert (out.double().cpu() - want).abs().max() < (1e-5 if dtype == torch.float32 else 3e-2)
