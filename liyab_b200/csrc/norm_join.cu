@@ -111,62 +111,105 @@ __global__ void __launch_bounds__(512) norm_join_kernel(lb_norm_join_args a, lb_
     }
 }
 
-// Many rows of a single term without a router: a warp a row of up to 128 NV values, everything it reads asked for at once (which the choices inside a
-// sum of terms do not let the compiler do), sums by shuffles, no block-wide barrier; the gains are read as they are used (the four rows of a block share
-// them in the first-level cache).
-template <int NV, typename T>
-__global__ void __launch_bounds__(128) norm_join_warp_kernel(lb_norm_join_args a, lb_output_terms o, int n_rows) {
-    const int lane = threadIdx.x & 31, t = blockIdx.x * 4 + (threadIdx.x >> 5), W = a.width;
-    lb_wait_for_predecessor();
-    lb_dependents_may_launch();
-    if (t >= n_rows) return;
-    Vals<4> x[NV], y[NV];
+// Many rows of a single term: LANES threads a row of up to 4 LANES NV values, everything they read asked for at once (which the choices inside a sum of
+// terms do not let the compiler do); `sum` adds up over them.  The rows of a block share the gains in the first-level cache.  A row that is not `live`
+// takes part in the sums and writes nothing.  `kept` (or null): where the row h goes as floats for the router.
+template <int NV, int LANES, typename T, typename Sum>
+__device__ __forceinline__ void join_row(const lb_norm_join_args& a, const lb_output_terms& o, int t, int lane, bool live, float* kept, Sum sum) {
+    const int W = a.width;
+    Vals<4> x[NV], y[NV], g[NV];
     float* xrow = a.x + (size_t)t * a.ldx;
+    const float* yrow = o.y[0] + (size_t)t * o.ldy[0];
+    // Predicated, not skipped: a branch a piece would make every load wait for the one before.
+    auto piece = [&](const float* p, int i, float otherwise) {
+        Vals<4> v;
+        const int c = 4 * (lane + LANES * i);
+        const float4 q = c < W ? *reinterpret_cast<const float4*>(p + c) : make_float4(otherwise, otherwise, otherwise, otherwise);
+        v.v[0] = q.x; v.v[1] = q.y; v.v[2] = q.z; v.v[3] = q.w;
+        return v;
+    };
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-        const int c = 4 * (lane + 32 * i);
-        if (c >= W) break;
-        x[i] = load_vals<4>(xrow + c);
-        y[i] = load_vals<4>(o.y[0] + (size_t)t * o.ldy[0] + c);
-    }
+    for (int i = 0; i < NV; ++i) y[i] = piece(yrow, i, 0.0f);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) x[i] = piece(xrow, i, 0.0f);
     const float times = o.factor[0] != nullptr ? o.scale[0] * o.factor[0][t] : o.scale[0];
+    const float gain_offset = a.gain != nullptr ? a.gain_offset : 1.0f, next_offset = a.next_gain != nullptr ? a.next_offset : 1.0f;
+    auto gains = [&](const float* p) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            if (p != nullptr) g[i] = piece(p, i, 0.0f);
+            else g[i].v[0] = g[i].v[1] = g[i].v[2] = g[i].v[3] = 0.0f;
+        }
+    };
+    gains(a.gain);
     float ss = 0.0f;
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-        if (4 * (lane + 32 * i) >= W) break;
+    for (int i = 0; i < NV; ++i)
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
             y[i].v[k] *= times;
             ss = fmaf(y[i].v[k], y[i].v[k], ss);
         }
-    }
-    const float inv_w = 1.0f / (float)W, f = a.scale / sqrtf(lb_warp_sum(ss) * inv_w + a.eps);
+    const float inv_w = 1.0f / (float)W, f = a.scale / sqrtf(sum(ss) * inv_w + a.eps);
     ss = 0.0f;
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-        const int c = 4 * (lane + 32 * i);
-        if (c >= W) break;
-        Vals<4> g;
-        if (a.gain != nullptr) g = load_vals<4>(a.gain + c);
+    for (int i = 0; i < NV; ++i)
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
-            x[i].v[k] = fmaf(y[i].v[k] * f, a.gain != nullptr ? g.v[k] + a.gain_offset : 1.0f, x[i].v[k]);
+            x[i].v[k] = fmaf(y[i].v[k] * f, g[i].v[k] + gain_offset, x[i].v[k]);
             ss = fmaf(x[i].v[k], x[i].v[k], ss);
         }
-        store_vals<4>(xrow + c, x[i]);
-    }
-    if (a.h == nullptr) return;
-    const float n = 1.0f / sqrtf(lb_warp_sum(ss) * inv_w + a.next_eps);
+    if (a.h != nullptr) gains(a.next_gain);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-        const int c = 4 * (lane + 32 * i);
-        if (c >= W) break;
-        Vals<4> g, h;
-        if (a.next_gain != nullptr) g = load_vals<4>(a.next_gain + c);
+        const int c = 4 * (lane + LANES * i);
+        if (live && c < W) store_vals<4>(xrow + c, x[i]);
+    }
+    if (a.h == nullptr) return;
+    const float n = 1.0f / sqrtf(sum(ss) * inv_w + a.next_eps);
 #pragma unroll
-        for (int k = 0; k < 4; ++k) h.v[k] = x[i].v[k] * n * (a.next_gain != nullptr ? g.v[k] + a.next_offset : 1.0f);
+    for (int i = 0; i < NV; ++i) {
+        const int c = 4 * (lane + LANES * i);
+        Vals<4> h;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) h.v[k] = x[i].v[k] * n * (g[i].v[k] + next_offset);
+        if (!live || c >= W) continue;
+        if (kept != nullptr) {
+            Vals<4> read;                   // the router reads what the experts read
+#pragma unroll
+            for (int k = 0; k < 4; ++k) read.v[k] = lb_to_float(lb_from_float<T>(h.v[k]));
+            store_vals<4>(kept + c, read);
+        }
         store_vals<4>(static_cast<T*>(a.h) + (size_t)t * a.ldh + c, h);
     }
+}
+
+template <int NV, typename T>
+__global__ void __launch_bounds__(128) norm_join_warp_kernel(lb_norm_join_args a, lb_output_terms o, int n_rows) {
+    const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
+    lb_wait_for_predecessor();
+    lb_dependents_may_launch();
+    if (t < n_rows) join_row<NV, 32, T>(a, o, t, threadIdx.x & 31, true, nullptr, [](float v) { return lb_warp_sum(v); });
+}
+
+// The same with a router: 64 threads a row, four rows a block, then all of the block routes the four.
+template <int NV, typename T>
+__global__ void __launch_bounds__(256, 4) norm_join_routed_kernel(lb_norm_join_args a, lb_output_terms o, lb_router r, int n_rows) {
+    extern __shared__ __align__(16) float smem[];
+    __shared__ float halves[2][8];
+    const int warp = threadIdx.x >> 5, row = threadIdx.x >> 6, t0 = blockIdx.x * 4;
+    lb_wait_for_predecessor();
+    lb_dependents_may_launch();
+    int turn = 0;
+    join_row<NV, 64, T>(a, o, min(t0 + row, n_rows - 1), threadIdx.x & 63, t0 + row < n_rows, smem + row * a.width, [&](float v) {
+        v = lb_warp_sum(v);
+        float* both = halves[turn++];
+        if ((threadIdx.x & 31) == 0) both[warp] = v;
+        __syncthreads();
+        return both[2 * row] + both[2 * row + 1];
+    });
+    __syncthreads();
+    route_rows<4, T>(r, smem, a.width, a.width, t0, n_rows, smem + 4 * a.width);
 }
 
 template <int V, typename T>
@@ -174,12 +217,17 @@ int launch_norm_join(const lb_norm_join_args& a, const lb_output_terms& o, const
     const bool routes = r.matrix != nullptr;
     const int pieces = a.width / V;
     if constexpr (V == 4) {
-        if (!routes && o.n_rows == 1 && o.pairs == nullptr && n_rows > 296 && a.width <= 1024) {
-            const dim3 grid((unsigned)((n_rows + 3) / 4)), block(128);
-            if (a.width <= 256) LB_CHECK_CUDA(lb_launch_overlapped(norm_join_warp_kernel<2, T>, grid, block, 0, s, a, o, n_rows));
-            else if (a.width <= 512) LB_CHECK_CUDA(lb_launch_overlapped(norm_join_warp_kernel<4, T>, grid, block, 0, s, a, o, n_rows));
-            else if (a.width <= 768) LB_CHECK_CUDA(lb_launch_overlapped(norm_join_warp_kernel<6, T>, grid, block, 0, s, a, o, n_rows));
-            else LB_CHECK_CUDA(lb_launch_overlapped(norm_join_warp_kernel<8, T>, grid, block, 0, s, a, o, n_rows));
+        const size_t scratch = routes ? 4 * (a.width + router_floats(r)) * sizeof(float) : 0;
+        if (o.n_rows == 1 && o.pairs == nullptr && n_rows > 296 && a.width <= 1024 && scratch <= 48 * 1024) {
+            const dim3 grid((unsigned)((n_rows + 3) / 4));
+#define LB_JOIN_ROWS(NV)                                                                                                                   \
+    if (routes) LB_CHECK_CUDA(lb_launch_overlapped(norm_join_routed_kernel<(NV + 1) / 2, T>, grid, dim3(256), scratch, s, a, o, r, n_rows)); \
+    else LB_CHECK_CUDA(lb_launch_overlapped(norm_join_warp_kernel<NV, T>, grid, dim3(128), 0, s, a, o, n_rows))
+            if (a.width <= 256) { LB_JOIN_ROWS(2); }
+            else if (a.width <= 512) { LB_JOIN_ROWS(4); }
+            else if (a.width <= 768) { LB_JOIN_ROWS(6); }
+            else { LB_JOIN_ROWS(8); }
+#undef LB_JOIN_ROWS
             return LB_OK;
         }
     }

@@ -233,6 +233,17 @@ def test_launch_between_two_norms(dev, dtype, W, T, N, top):
         assert (d(x) - want).abs().max() < 2e-5 * max(1.0, float(want.abs().max()))
         hw = rms(want, eps2) * (0.5 + d(gain2))
         assert last or (d(h) - hw).abs().max() < (2e-5 if dtype == torch.float32 else 1e-2) * max(1.0, float(hw.abs().max()))
+    x = torch.empty(T, W + 4, device=dev)[:, :W]
+    x.copy_(x0)
+    h, gate = torch.full((T, W), float("nan"), dtype=dtype, device=dev), torch.full((T,), float("nan"), device=dev)
+    rid, rw = torch.full((T, top), -1, dtype=torch.int32, device=dev), torch.full((T, top), float("nan"), device=dev)
+    ops.norm_join(x, ops.output_terms([y1], [0.5], factor=(f2,)), (gain, 1.0, eps), T, scale, next_norm=(gain2, 0.5, eps2), h=h,
+                  router=ops.router_args(matrix, top, rid, rw, renormalise=True, gate=gate))
+    z = d(h) @ d(matrix).t()
+    wid, ww = choice(z[:, :N], top)
+    same = (rid.cpu() == wid).all(1)
+    assert (d(x) - want).abs().max() < 2e-5 * max(1.0, float(want.abs().max())) and same.float().mean() > 0.99
+    assert (d(rw) - ww)[same].abs().max() < 1e-4 and (d(gate) - torch.sigmoid(z[:, N])).abs().max() < 1e-5
     # Without gains: ones.
     x = x0.clone()
     ops.norm_join(x, ops.output_terms([y1], [1.0]), (None, 1.0, eps), T)
