@@ -228,6 +228,10 @@ latent_finish_kernel(const float* __restrict__ attended, int64_t lda, const floa
     }
     __syncthreads();
     const float times = head_factor(gate, ldg, t, h);
+    // A lane meets the same eight latent values in every row of the map: they stay in registers.
+    float mine[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) mine[k] = lane < pieces ? osm[lane * 8 + k] : 0.0f;
     for (int v0 = warp; v0 < vdim; v0 += 32) {
         if (v0 != warp) fetch(v0);
         if (value_gate != nullptr && lane < 8 && v0 + 4 * lane < vdim) {
@@ -240,8 +244,15 @@ latent_finish_kernel(const float* __restrict__ attended, int64_t lda, const floa
             if (v >= vdim) break;                                  // uniform across the warp
             const __nv_bfloat16* row = uv + ((size_t)h * vdim + v) * rank;
             float acc = 0.0f;
-            for (int c = lane; c < pieces; c += 32) {
-                const uint4 raw = c == lane ? ahead_uv[b] : *reinterpret_cast<const uint4*>(row + c * 8);
+            const __nv_bfloat162* first = reinterpret_cast<const __nv_bfloat162*>(&ahead_uv[b]);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const float2 f = __bfloat1622float2(first[k]);
+                acc = fmaf(f.x, mine[2 * k], acc);
+                acc = fmaf(f.y, mine[2 * k + 1], acc);
+            }
+            for (int c = lane + 32; c < pieces; c += 32) {
+                const uint4 raw = *reinterpret_cast<const uint4*>(row + c * 8);
                 const __nv_bfloat162* w = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
                 for (int k = 0; k < 4; ++k) {

@@ -42,8 +42,9 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst)), "l"(src));
+// 16 bytes, or zeros (nothing is read then).
+__device__ __forceinline__ void cp_async16_or_zero(void* dst, const void* src, bool there) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(there ? 16 : 0));
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
@@ -100,31 +101,36 @@ latent_attention_mma_kernel(const bf16* __restrict__ wide, int64_t ldw, const bf
     const int per = (tile_hi - tile_lo + n_splits) / n_splits;
     const int my_lo = tile_lo + split * per, my_hi = min(tile_hi, my_lo + per - 1);
 
-    auto load_tile = [&](int tile, int buf) {
+    // Lane k knows where the row of key k of a tile lies (-1: no such key): one look-up a tile, made a tile ahead, instead of one a row.
+    auto row_of = [&](int tile) -> int {
+        const int j = tile * kKeys + lane;
+        if (j < lo_min || j > p_last) return -1;
+        const int page = j / page_size;
+        return table[page] * page_size + (j - page * page_size);
+    };
+    auto load_tile = [&](int rows, int buf) {
         bf16* dst0 = ks + (size_t)buf * kKeys * DS;
-        for (int key = warp; key < kKeys; key += 4) {
-            const int j = tile * kKeys + key;
+#pragma unroll
+        for (int i = 0; i < kKeys / 4; ++i) {
+            const int key = warp + 4 * i, at = __shfl_sync(0xffffffffu, rows, key);
             bf16* dst = dst0 + (size_t)key * DS;
-            if (j >= lo_min && j <= p_last) {
-                const bf16* src = cache + ((size_t)table[j / page_size] * page_size + (j % page_size)) * D;
-                for (int c = lane; c < chunks; c += 32) cp_async16(dst + c * 8, src + c * 8);
-            } else {
-                for (int c = lane; c < chunks; c += 32) *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(0u, 0u, 0u, 0u);
-            }
+            const bf16* src = cache + (size_t)max(at, 0) * D;
+            for (int c = lane; c < chunks; c += 32) cp_async16_or_zero(dst + c * 8, src + c * 8, at >= 0);
         }
         cp_async_commit();
     };
-    if (my_lo <= my_hi) load_tile(my_lo, 0);                     // on its way while the queries are staged
+    int rows_next = my_lo <= my_hi ? row_of(my_lo) : -1;
     // Queries: row r is token first + r / HB, head hg * HB + r % HB.
-    for (int r = warp; r < M; r += 4) {
+    for (int r = warp; r < M && my_lo <= my_hi; r += 4) {
         const int tok = r / HB, head = hg * HB + r % HB;
         const bool valid = tok < n_here && head < n_head;
         const bf16* src = wide + (size_t)(first + min(tok, n_here - 1)) * ldw + (size_t)min(head, n_head - 1) * D;
-        for (int c = lane; c < chunks; c += 32) {
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (valid) v = *reinterpret_cast<const uint4*>(src + c * 8);
-            *reinterpret_cast<uint4*>(qs + (size_t)r * DS + c * 8) = v;
-        }
+        for (int c = lane; c < chunks; c += 32) cp_async16_or_zero(qs + (size_t)r * DS + c * 8, src + c * 8, valid);
+    }
+
+    if (my_lo <= my_hi) {
+        load_tile(rows_next, 0);                                 // with the queries in one group
+        rows_next = my_lo < my_hi ? row_of(my_lo + 1) : -1;
     }
 
     float o[MT][RT][4];
@@ -143,7 +149,10 @@ latent_attention_mma_kernel(const bf16* __restrict__ wide, int64_t ldw, const bf
         const int buf = (tile - my_lo) & 1;
         cp_async_wait_all();
         __syncthreads();                                        // the tile (and, first time, the queries) is there; the step before is over
-        if (tile < my_hi) load_tile(tile + 1, buf ^ 1);
+        if (tile < my_hi) {
+            load_tile(rows_next, buf ^ 1);
+            rows_next = tile + 1 < my_hi ? row_of(tile + 2) : -1;
+        }
         const bf16* kt = ks + (size_t)buf * kKeys * DS;
 
         // ---- scores of keys 8w .. 8w + 7 for all rows
@@ -290,31 +299,34 @@ latent_attention_rows_kernel(const bf16* __restrict__ wide, int64_t ldw, const b
     const int32_t* table = block_table + (size_t)s * table_stride;
     const int tile_lo = lo_min / kKeys, tile_hi = p_last / kKeys;
 
-    auto load_tile = [&](int tile, int buf) {
+    // Lane k knows where the row of key k of a tile lies (-1: no such key): one look-up a tile, made a tile ahead, instead of one a row.
+    auto row_of = [&](int tile) -> int {
+        const int j = tile * kKeys + lane;
+        if (j < lo_min || j > p_last) return -1;
+        const int page = j / page_size;
+        return table[page] * page_size + (j - page * page_size);
+    };
+    auto load_tile = [&](int rows, int buf) {
         bf16* dst0 = ks + (size_t)buf * kKeys * DS;
-        for (int key = warp; key < kKeys; key += 4) {
-            const int j = tile * kKeys + key;
+#pragma unroll
+        for (int i = 0; i < kKeys / 4; ++i) {
+            const int key = warp + 4 * i, at = __shfl_sync(0xffffffffu, rows, key);
             bf16* dst = dst0 + (size_t)key * DS;
-            if (j >= lo_min && j <= p_last) {
-                const bf16* src = cache + ((size_t)table[j / page_size] * page_size + (j % page_size)) * D;
-                for (int c = lane; c < chunks; c += 32) cp_async16(dst + c * 8, src + c * 8);
-            } else {
-                for (int c = lane; c < chunks; c += 32) *reinterpret_cast<uint4*>(dst + c * 8) = make_uint4(0u, 0u, 0u, 0u);
-            }
+            const bf16* src = cache + (size_t)max(at, 0) * D;
+            for (int c = lane; c < chunks; c += 32) cp_async16_or_zero(dst + c * 8, src + c * 8, at >= 0);
         }
         cp_async_commit();
     };
-    load_tile(tile_lo, 0);                                        // on its way while the queries are staged
+    int rows_next = row_of(tile_lo);
     for (int r = warp; r < M; r += 4) {
         const int tok = r / HB, head = hg * HB + r % HB;
         const bool valid = tok < n_here && head < n_head;
         const bf16* src = wide + (size_t)(first + min(tok, n_here - 1)) * ldw + (size_t)min(head, n_head - 1) * D;
-        for (int c = lane; c < chunks; c += 32) {
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (valid) v = *reinterpret_cast<const uint4*>(src + c * 8);
-            *reinterpret_cast<uint4*>(qs + (size_t)r * DS + c * 8) = v;
-        }
+        for (int c = lane; c < chunks; c += 32) cp_async16_or_zero(qs + (size_t)r * DS + c * 8, src + c * 8, valid);
     }
+
+    load_tile(rows_next, 0);                                      // with the queries in one group
+    rows_next = tile_lo < tile_hi ? row_of(tile_lo + 1) : -1;
 
     // This thread's two rows (g and g + 8 of the warp's sixteen): their tokens' positions and first visible keys.
     int p_row[2], lo_row[2];
@@ -337,7 +349,10 @@ latent_attention_rows_kernel(const bf16* __restrict__ wide, int64_t ldw, const b
         const int buf = (tile - tile_lo) & 1;
         cp_async_wait_all();
         __syncthreads();
-        if (tile < tile_hi) load_tile(tile + 1, buf ^ 1);
+        if (tile < tile_hi) {
+            load_tile(rows_next, buf ^ 1);
+            rows_next = tile + 1 < tile_hi ? row_of(tile + 2) : -1;
+        }
         const bf16* kt = ks + (size_t)buf * kKeys * DS;
 
         float sc[4][4];
