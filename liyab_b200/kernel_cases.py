@@ -7,6 +7,8 @@
     python -m liyab_b200.kernel_cases decode-step --batch 8 --layers 12 --reps 20 [--eager]
     python -m liyab_b200.kernel_cases prefill-step --tokens 2048 --layers 12 --reps 3
     python -m liyab_b200.kernel_cases channel-memory --batch 2 --new 1024 --heads 6 --dim 64 --vdim 128 --delta
+    python -m liyab_b200.kernel_cases prefill-attention --soft-cap 50 --score-bound 8.2
+    python -m liyab_b200.kernel_cases norm-join --rows 2048 --width 768 --experts 16
     python -m liyab_b200.kernel_cases streams --rows 2048 --streams 2 --width 768 --experts 20
 
 Each prints one line with the CUDA-event time per repetition and the achieved rate.  The cases are what the
@@ -175,11 +177,11 @@ def case_prefill_attention(args) -> None:
 
     def launch():
         ops.prefill_attention(q, cache, q_start, n_past, table, out, S, L, H, H, hd, ps, hd ** -0.5, 0,
-                              tcgen05=False if args.mma_sync else None)
+                              tcgen05=False if args.mma_sync else None, soft_cap=args.soft_cap, score_bound=args.score_bound)
 
     ms = _graph_timed(launch, args.reps) if args.graph else _timed(launch, args.reps)
     flop = S * H * (L * L / 2) * hd * 4
-    print(f"prefill-attention seqs={S} length={L} heads={H} head_dim={hd}: {ms * 1e3:.1f} us, {flop / ms / 1e9:.1f} TFLOP/s "
+    print(f"prefill-attention seqs={S} length={L} heads={H} head_dim={hd}{f" soft cap {args.soft_cap:g}" if args.soft_cap else ""}: {ms * 1e3:.1f} us, {flop / ms / 1e9:.1f} TFLOP/s "
           f"(causal half of the square)")
 
 
@@ -292,6 +294,28 @@ def case_streams(args) -> None:
     print(f"streams {T} rows of {S} x {W}{', routed' if router else ''}: {1e3 * ms:.1f} us, {(8 * T * S * W + read + 2 * T * W) / ms / 1e6:.0f} GB/s")
 
 
+def case_norm_join(args) -> None:
+    """The launch between two norms: a row (or, with `--routed`, routed results and a gated row) through its norm into the stream, the next input, and a
+    router with a gate on it with `--experts`."""
+    from . import ops
+    dev, T, W = torch.device("cuda:0"), args.rows, args.width
+    gen = torch.Generator(device=dev).manual_seed(0)
+    r = lambda *shape: torch.randn(*shape, device=dev, generator=gen)
+    x, y, h, gain, factor = r(T, W), r(T, W), torch.empty(T, W, dtype=torch.bfloat16, device=dev), r(W) * 0.1, r(T)
+    terms, read = ops.output_terms([y], [1.0]), 4 * T * W
+    if args.routed:
+        ids = torch.randint(0, 16, (T, 2), dtype=torch.int32, device=dev, generator=gen)
+        place, pairs, weights = torch.randperm(2 * T, device=dev, generator=gen).int(), r(2 * T, W), r(T, 2)
+        terms, read = ops.output_terms([y], [1.0], pairs, place, ids, weights, 16, None, factor=(factor,)), 12 * T * W
+    router = None
+    if args.experts:
+        chosen, shares, gate = torch.empty(T, 2, dtype=torch.int32, device=dev), torch.empty(T, 2, device=dev), torch.empty(T, device=dev)
+        router = ops.router_args(r(args.experts + 1, W).bfloat16(), 2, chosen, shares, renormalise=True, gate=gate)
+    launch = lambda: ops.norm_join(x, terms, (gain, 1.0, 1e-6), T, next_norm=(gain, 1.0, 1e-6), h=h, router=router)
+    ms = _graph_timed(launch, args.reps)
+    print(f"norm-join {T} rows of {W}{', routed results' if args.routed else ''}{', with a router' if router else ''}: {1e3 * ms:.1f} us, {(10 * T * W + read) / ms / 1e6:.0f} GB/s")
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="python -m liyab_b200.kernel_cases")
     sub = ap.add_subparsers(dest="case", required=True)
@@ -339,6 +363,8 @@ def main(argv=None) -> int:
     a.add_argument("--head-dim", type=int, default=64)
     a.add_argument("--reps", type=int, default=20)
     a.add_argument("--graph", action="store_true", help="time 20 launches captured in a CUDA graph")
+    a.add_argument("--soft-cap", type=float, default=0.0, help="cap on the scores, c tanh(s / c)")
+    a.add_argument("--score-bound", type=float, default=0.0, help="the largest |score| that can occur (0: unknown)")
     a.add_argument("--mma-sync", action="store_true", help="the mma.sync kernel even where the tcgen05 one takes the shape")
     sm = sub.add_parser("sample")
     sm.add_argument("--rows", type=int, default=8)
@@ -356,6 +382,12 @@ def main(argv=None) -> int:
     cm.add_argument("--vdim", type=int, default=128)
     cm.add_argument("--delta", action="store_true", help="the delta rule with short convolutions (default: gated linear attention)")
     cm.add_argument("--reps", type=int, default=20)
+    nj = sub.add_parser("norm-join")
+    nj.add_argument("--rows", type=int, default=2048)
+    nj.add_argument("--width", type=int, default=768)
+    nj.add_argument("--experts", type=int, default=0)
+    nj.add_argument("--routed", action="store_true", help="the sublayer's output is routed experts' results and a gated shared one")
+    nj.add_argument("--reps", type=int, default=20)
     st = sub.add_parser("streams")
     st.add_argument("--rows", type=int, default=2048)
     st.add_argument("--streams", type=int, default=2)
@@ -377,7 +409,7 @@ def main(argv=None) -> int:
         p.add_argument("--stamps", action="store_true", help="decode-step: per-phase times from inside the one-kernel step")
     args = ap.parse_args(argv)
     {"gemm": case_gemm, "generic-attention": case_generic_attention, "gemm-f32": case_gemm_f32, "decode-attention": case_decode_attention, "prefill-attention": case_prefill_attention, "sample": case_sample, "decode-step": case_decode_step,
-     "prefill-step": case_prefill_step, "channel-memory": case_channel_memory, "streams": case_streams}[args.case](args)
+     "prefill-step": case_prefill_step, "channel-memory": case_channel_memory, "streams": case_streams, "norm-join": case_norm_join}[args.case](args)
     return 0
 
 
